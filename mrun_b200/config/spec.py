@@ -53,13 +53,15 @@ class RMSNormSpec:
 
 @dataclass(frozen=True)
 class LayerNormSpec:
-    """Layer norm with a weight and no bias: (x - mean) / sqrt(variance + eps) * w, the variance
-    the mean of the squared deviations.  ``bare`` as for :class:`RMSNormSpec`."""
+    """Layer norm with a weight: (x - mean) / sqrt(variance + eps) * w, the variance the mean of the
+    squared deviations.  ``bare`` as for :class:`RMSNormSpec`.  ``bias``: a vector is added
+    after the weight (``<name>.b`` for a bare weight, ``<name>.bias`` else)."""
 
     kind: ClassVar[str] = "layernorm"
     size: int
     eps: float
     bare: bool = False
+    bias: bool = False
 
 
 # --------------------------------------------------------------------------- position encodings
@@ -182,7 +184,16 @@ class GatedAttentionSpec:
     they come out of their projection, before norm and rotation (``vdim`` = ``dim``).  Which keys a
     token at position i sees: all up to itself; with ``window`` = W the last W, itself included;
     with ``chunk`` = C those of its own chunk, floor(j / C) = floor(i / C), chunks counted from
-    position 0 of the sequence."""
+    position 0 of the sequence.
+
+    ``qk_norm`` = ``"unit"``: as ``"head"`` without a weight.  What may be done to a score s = (q . k)
+    * ``softmax_scale`` before the softmax, in this order: ``temperature`` = (coef, every): q at
+    position p counts 1 + coef * ln(floor((p + 1) / every) + 1) times; ``soft_cap`` = c: s <- c *
+    tanh(s / c); ``distance_bias`` = (rows, reach): s <- s + rel[bucket(i - j), head] with a table
+    ``rel`` of ``rows`` rows; bucket(n) = n for n < rows / 2, else min(rows - 1, rows / 2 +
+    floor(ln(n / (rows / 2)) / ln(reach / (rows / 2)) * (rows - rows / 2))).  ``element_gate``: the
+    heads' outputs together are multiplied element by element by sigmoid(g x), ``g`` with a row a
+    feature (in place of ``head_gate``)."""
 
     kind: ClassVar[str] = "gated_attention"
     hidden: int
@@ -200,6 +211,10 @@ class GatedAttentionSpec:
     window: Optional[int] = None
     chunk: Optional[int] = None
     values: str = "projection"
+    temperature: Optional[Tuple[float, float]] = None
+    soft_cap: Optional[float] = None
+    distance_bias: Optional[Tuple[int, float]] = None
+    element_gate: bool = False
 
 
 @dataclass(frozen=True)
@@ -262,11 +277,53 @@ class ChannelDeltaSpec:
 
 
 @dataclass(frozen=True)
+class TimeMixingSpec:
+    """Linear attention over shifted rows, with a decay per head and key channel made from the
+    input, a bonus for the current token and a state of fixed size.  With x' the previous token's
+    x (zeros for the first), each of r, k, v, g, w reads its own blend x + (x' - x) * mu.  r, k, v
+    (``heads`` x ``dim``) are projections of their blends, the gate is SiLU of one; the decay is
+    exp(-exp(w2 tanh(w1 .) + w0)), w1 with ``rank`` rows.  Per head o_t = (S_(t-1) + diag(u) k_t
+    v_t^T)^T r_t, then S_t = diag(decay_t) S_(t-1) + k_t v_t^T.  Every head's o is divided by its
+    root mean square (``eps`` inside the root), the heads together are multiplied by a weight and
+    the gate and projected out.  The previous token's x is part of the state."""
+
+    kind: ClassVar[str] = "time_mixing"
+    hidden: int
+    heads: int
+    dim: int
+    rank: int
+    eps: float
+
+
+@dataclass(frozen=True)
+class StateSpaceSpec:
+    """A selective state-space mixer with a scalar decay per head (Mamba-2).  One projection makes
+    [z: inner | x: inner | B: groups * state | C: groups * state | dt: heads], inner = ``heads`` *
+    ``vdim``; x, B and C pass a causal convolution of ``conv`` taps per channel with a bias, and
+    SiLU.  dt <- softplus(dt + dt_bias); per head (head h reads group floor(h / (heads / groups)))
+    S_t = exp(-exp(A_log) dt) S_(t-1) + dt B_t x_t^T (``state`` x ``vdim``), y_t = S_t^T C_t + D x_t.
+    The heads' y together are multiplied by SiLU(z), divided by the root mean square of each of
+    ``norm_groups`` equal parts (``eps`` inside the root), multiplied by a weight and projected
+    out.  The convolution's last inputs are part of the state."""
+
+    kind: ClassVar[str] = "state_space"
+    hidden: int
+    heads: int
+    vdim: int
+    state: int
+    groups: int
+    conv: int
+    norm_groups: int
+    eps: float
+
+
+@dataclass(frozen=True)
 class ParallelMixerSpec:
-    """Two mixers side by side that read the same input: the result is ``share`` times the sum of
-    their outputs, each first divided by its root mean square over the model width (``eps``
-    inside the root) and multiplied by a weight of its own, ``<left_prefix>.<out_name>`` and
-    ``<right_prefix>.<out_name>``.  The two may keep a cache each, at most one of them paged."""
+    """Two mixers side by side that read the same input.  ``combine`` = ``"norm_mean"``: the result
+    is ``share`` times the sum of their outputs, each first divided by its root mean square over
+    the model width (``eps`` inside the root) and multiplied by a weight of its own,
+    ``<left_prefix>.<out_name>`` and ``<right_prefix>.<out_name>``; ``"sum"``: it is ``scales[0]`` *
+    left + ``scales[1]`` * right.  The two may keep a cache each, at most one of them paged."""
 
     kind: ClassVar[str] = "parallel"
     hidden: int
@@ -277,6 +334,8 @@ class ParallelMixerSpec:
     left_prefix: str = "left"
     right_prefix: str = "right"
     out_name: str = "out"
+    combine: str = "norm_mean"
+    scales: Tuple[float, float] = (1.0, 1.0)
 
 
 # --------------------------------------------------------------------------- feed-forwards
@@ -292,6 +351,18 @@ class GatedMLPSpec:
     # the checkpoint's names of the gate, up and down matrices under the part's prefix; a name
     # that ends in ``.weight`` may have a ``.bias`` beside it
     tensor_names: Tuple[str, str, str] = ("gate_proj.weight", "up_proj.weight", "down_proj.weight")
+
+
+@dataclass(frozen=True)
+class DenseMLPSpec:
+    """``down(act(up(x)))`` without a gate and without biases; ``activation``: ``"relu2"``, the square
+    of the positive part."""
+
+    kind: ClassVar[str] = "dense_mlp"
+    hidden: int
+    intermediate: int
+    activation: str = "relu2"
+    tensor_names: Tuple[str, str] = ("up", "down")
 
 
 @dataclass(frozen=True)
@@ -415,7 +486,8 @@ class LayerSpec:
     """One block: norm → mixer → residual → norm → feed-forward → residual (``pre_norm``).  The
     ``sandwich`` arrangement also norms each branch's output (``*_post_norm``) and multiplies it
     by ``residual_scale`` before the sum; its ``feed_forward`` may be None (a layer of a mixer
-    only)."""
+    only).  The ``post_norm`` arrangement norms a branch's output only: x += norm(mixer(x)), x +=
+    norm(ff(x)), with the norms in ``mixer_norm`` and ``feed_forward_norm``."""
 
     prefix: str
     mixer: Any

@@ -15,7 +15,7 @@
 //                32-bit; the four warps' results meet in a small buffer of their own, so the
 //                ring is never drained.
 //
-// A stage is 2 x 64 x D x 2 bytes without padding (the swizzle keeps ldmatrix free of bank
+// A stage is 64 x (D + DV) x 2 bytes without padding (the swizzle keeps ldmatrix free of bank
 // conflicts), so two blocks with three stages each fit a multiprocessor at D = 128 and up to five
 // tiles a multiprocessor are in flight.  Head sizes 64 and 128, page sizes that are powers of
 // two, at most 16 query heads per kv head.  Every mbarrier wait is bounded; a wait that runs out
@@ -32,7 +32,7 @@
 #include "attention_frag.cuh"
 #include "tcgen05.cuh"
 
-#if MRUN_HEAD_DIM % 64 == 0 && MRUN_HEAD_DIM <= 128
+#if MRUN_HEAD_DIM % 64 == 0 && MRUN_HEAD_DIM <= 128 && MRUN_VALUE_DIM % 64 == 0 && MRUN_VALUE_DIM <= 128
 #define MRUN_DECODE_TMA 1
 #else
 #define MRUN_DECODE_TMA 0
@@ -44,21 +44,24 @@ namespace {
 
 using namespace tc5;
 
-constexpr int SPANS = D / 64;                        // 64-wide spans of the head dimension
+constexpr int SPANS = D / 64, SPANS_V = DV / 64;     // 64-wide spans of the head dimensions
 constexpr int SPAN_BYTES = BLOCK_N * 128;            // 64 rows x 128 bytes
-constexpr int TILE_BYTES = SPANS * SPAN_BYTES;       // one K (or V) tile
-constexpr int STAGE_BYTES = 2 * TILE_BYTES;          // K then V
+constexpr int TILE_BYTES = SPANS * SPAN_BYTES;       // one K tile
+constexpr int TILE_V_BYTES = SPANS_V * SPAN_BYTES;   // one V tile
+constexpr int STAGE_BYTES = TILE_BYTES + TILE_V_BYTES;      // K then V
 constexpr int CONSUMERS = 128, TMA_THREADS = CONSUMERS + 32;
-constexpr int MS = D + 2;                            // a merged row: D values, maximum, sum
+constexpr int MS = DV + 2;                           // a merged row: DV values, maximum, sum
+// the queries, whose place a block's piece of a pair takes in the cluster kernel (8 rows of DV + 4 floats)
+constexpr int Q_REGION = 16 * LD * 2 > 8 * (DV + 4) * 4 ? 16 * LD * 2 : 8 * (DV + 4) * 4;
 constexpr long long WAIT_CYCLES = 3000000000LL;      // about 1.5 s at 2 GHz
 
 enum : int { STATUS_PRODUCER = 1, STATUS_CONSUMER = 2 };
 
 __host__ __device__ constexpr size_t tma_smem_bytes(int ring, int group) {
     return (size_t)ring * STAGE_BYTES + 1024                           // the ring, 1024-byte aligned
-           + (size_t)16 * LD * sizeof(bf16)                             // q rows
+           + (size_t)Q_REGION                                           // q rows
            + (size_t)4 * group * MS * sizeof(float)                     // the four warps' results
-           + (size_t)4 * D * sizeof(float) + 2 * D * sizeof(bf16);      // head staging, the step's own k and v
+           + (size_t)4 * D * sizeof(float) + (D + DV) * sizeof(bf16);   // head staging, the step's own k and v
 }
 
 // Address of the 16-byte chunk `chunk` (0 .. D/8 - 1) of row `row` of a swizzled tile.
@@ -72,7 +75,8 @@ __device__ __forceinline__ void consumer_sync() { asm volatile("bar.sync 1, 128;
 // arithmetic as attend_tile<16>, with the fragments fetched through the swizzle.
 __device__ __forceinline__ void attend_slice(const bf16* q_tile, const unsigned char* k_tile, const unsigned char* v_tile,
                                              int krow0, int key_base, float scale_log2, const int (&row_pos)[2],
-                                             const int (&row_lo)[2], float (&m)[2], float (&l)[2], float (&o)[D / 8][4]) {
+                                             const int (&row_lo)[2], const mrun::ScoreRow (&form_row)[2], bool near_keys,
+                                             float (&m)[2], float (&l)[2], float (&o)[DV / 8][4]) {
     const int lane = threadIdx.x & 31;
     float s[2][4];
 #pragma unroll
@@ -91,8 +95,9 @@ __device__ __forceinline__ void attend_slice(const bf16* q_tile, const unsigned 
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
             const int r = e >> 1;
-            float v = s[nt][e] * scale_log2;
             const int key = key_base + krow0 + nt * 8 + (lane & 3) * 2 + (e & 1);
+            float v = s[nt][e] * scale_log2;
+            if constexpr (SCORED) v = scored(form_row[r], s[nt][e], near_keys, row_pos[r] - key);
             if (key > row_pos[r] || key < row_lo[r]) v = -INFINITY;
             s[nt][e] = v;
             mx[r] = fmaxf(mx[r], v);
@@ -119,7 +124,7 @@ __device__ __forceinline__ void attend_slice(const bf16* q_tile, const unsigned 
 #pragma unroll
     for (int r = 0; r < 2; ++r) l[r] = l[r] * corr[r] + sum[r];       // per-thread partial; reduced at the end
 #pragma unroll
-    for (int dt = 0; dt < D / 8; ++dt) {
+    for (int dt = 0; dt < DV / 8; ++dt) {
         o[dt][0] *= corr[0]; o[dt][1] *= corr[0];
         o[dt][2] *= corr[1]; o[dt][3] *= corr[1];
     }
@@ -129,7 +134,7 @@ __device__ __forceinline__ void attend_slice(const bf16* q_tile, const unsigned 
     a[2] = pack_bf16(s[1][0], s[1][1]);
     a[3] = pack_bf16(s[1][2], s[1][3]);
 #pragma unroll
-    for (int dt = 0; dt < D / 8; dt += 2) {
+    for (int dt = 0; dt < DV / 8; dt += 2) {
         unsigned b[4];
         ldmatrix_x4_trans(b, swz(v_tile, krow0 + (lane & 7) + ((lane >> 3) & 1) * 8, dt + (lane >> 4)));
         mma_bf16(o[dt], a, b[0], b[1]);
@@ -180,18 +185,20 @@ decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_consta
                   const int* __restrict__ positions, const int* __restrict__ tile_prefix,
                   const int4* __restrict__ assignment, int tokens, float* __restrict__ part_o,
                   float* __restrict__ part_ml, int* __restrict__ counters, int heads, int kv_heads, int page_size,
-                  int page_shift, float scale_log2, int window, float sink_log2, const FusedInput fused, int* __restrict__ status) {
+                  int page_shift, float scale_log2, int window, float sink_log2, const FusedInput fused,
+                  const mrun_score_form form, int* __restrict__ status) {
     extern __shared__ __align__(1024) unsigned char smem_raw[];
     unsigned char* ring = reinterpret_cast<unsigned char*>(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
     const int group = heads / kv_heads;
-    bf16* q_tile = reinterpret_cast<bf16*>(ring + RING * STAGE_BYTES);                   // [16][LD]
-    float* merge = reinterpret_cast<float*>(q_tile + 16 * LD);                            // [4][group][MS]
+    bf16* q_tile = reinterpret_cast<bf16*>(ring + RING * STAGE_BYTES);                   // [16][LD], Q_REGION bytes
+    float* merge = reinterpret_cast<float*>(ring + RING * STAGE_BYTES + Q_REGION);                            // [4][group][MS]
     float (*head_vec)[D] = reinterpret_cast<float (*)[D]>(merge + 4 * group * MS);        // [4][D]
     bf16* new_k = reinterpret_cast<bf16*>(head_vec + 4);                                  // this step's own key, value
     bf16* new_v = new_k + D;
     __shared__ unsigned long long full_bar[RING], empty_bar[RING];
     __shared__ int ticket_shared, aborted;
 
+    const long out_stride = output_stride(form, heads);
     const int block_id = blockIdx.x, n_blocks_grid = gridDim.x;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int4 mine = assignment[2 * block_id], shape = assignment[2 * block_id + 1];
@@ -215,7 +222,7 @@ decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_consta
         first_sg = next_segment(0, u_begin, u_end, first_kvh, first_tok, tiles_per_head, tile_prefix, positions, window);
     // rows of a V tile that no copy fills must not hold NaN patterns: 0 * NaN is NaN
     for (int s = 0; s < RING; ++s)
-        for (int i = threadIdx.x; i < TILE_BYTES / 16; i += TMA_THREADS)
+        for (int i = threadIdx.x; i < TILE_V_BYTES / 16; i += TMA_THREADS)
             reinterpret_cast<uint4*>(ring + s * STAGE_BYTES + TILE_BYTES)[i] = make_uint4(0, 0, 0, 0);
     fence_async_smem();
     __syncthreads();
@@ -241,7 +248,7 @@ decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_consta
                 for (int b = lane; b < boxes; b += 32) {
                     const int first_key = key0 + b * box_rows;
                     if (first_key <= sg.pos && first_key + box_rows - 1 >= sg.lo && table[first_key >> page_shift] >= 0)
-                        bytes += (unsigned)(2 * box_rows * D * 2);
+                        bytes += (unsigned)(box_rows * (D + DV) * 2);
                 }
                 if (bytes) mbar_expect_tx(&full_bar[s], bytes);
                 else mbar_arrive(&full_bar[s]);
@@ -251,11 +258,13 @@ decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_consta
                     const int page = table[first_key >> page_shift];
                     if (page < 0) continue;
 #pragma unroll
-                    for (int h = 0; h < SPANS; ++h) {
-                        tma_load_4d(stage + h * SPAN_BYTES + b * box_rows * 128, &map_k, h * 64,
-                                    first_key & (page_size - 1), sg.kvh, page, &full_bar[s]);
-                        tma_load_4d(stage + TILE_BYTES + h * SPAN_BYTES + b * box_rows * 128, &map_v, h * 64,
-                                    first_key & (page_size - 1), sg.kvh, page, &full_bar[s]);
+                    for (int h = 0; h < (SPANS > SPANS_V ? SPANS : SPANS_V); ++h) {
+                        if (h < SPANS)
+                            tma_load_4d(stage + h * SPAN_BYTES + b * box_rows * 128, &map_k, h * 64,
+                                        first_key & (page_size - 1), sg.kvh, page, &full_bar[s]);
+                        if (h < SPANS_V)
+                            tma_load_4d(stage + TILE_BYTES + h * SPAN_BYTES + b * box_rows * 128, &map_v, h * 64,
+                                        first_key & (page_size - 1), sg.kvh, page, &full_bar[s]);
                     }
                 }
             }
@@ -270,8 +279,8 @@ decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_consta
         // padding rows come out as zeros
         for (int t = block_id; t < tokens; t += n_blocks_grid)
             if (positions[t] < 0)
-                for (int i = threadIdx.x; i < heads * D; i += CONSUMERS)
-                    out[(size_t)(fused.rows ? fused.rows[t] : t) * heads * D + i] = __float2bfloat16_rn(0.f);
+                for (int i = threadIdx.x; i < heads * DV; i += CONSUMERS)
+                    out[(size_t)(fused.rows ? fused.rows[t] : t) * out_stride + i] = __float2bfloat16_rn(0.f);
 
         // A warp whose wait ran out sets the flag and keeps walking (its later waits return at once,
         // its numbers are void), so that every barrier of the four warps is still met by all.
@@ -282,9 +291,9 @@ decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_consta
             const int pos = sg.pos, lo = sg.lo;
             const int b1 = pos / BLOCK_N;
             float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
-            float o[D / 8][4];
+            float o[DV / 8][4];
 #pragma unroll
-            for (int dt = 0; dt < D / 8; ++dt) o[dt][0] = o[dt][1] = o[dt][2] = o[dt][3] = 0.f;
+            for (int dt = 0; dt < DV / 8; ++dt) o[dt][0] = o[dt][1] = o[dt][2] = o[dt][3] = 0.f;
 
             const bool owns_new_token = fused.enabled && sg.last_block == b1;
             const int q_row = fused.rows ? fused.rows[sg.tok] : sg.tok;        // the row of q and out
@@ -297,7 +306,7 @@ decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_consta
                     *reinterpret_cast<uint4*>(q_tile + row * LD + chunk * 8) = value;
                 }
             } else {
-                // q, k and v arrive raw: [q heads | k heads | v heads] of D elements each in the token's row
+                // q, k and v arrive raw: [q heads | k heads | v heads] in the token's row
                 const bf16* token_row = q + (size_t)sg.tok * q_stride;
                 const float2* cs = fused.rot ? fused.rot + (size_t)sg.tok * (fused.rotary_dim >> 1) : nullptr;
                 // where the token's own key and value go: asked for now, used after the heads are made
@@ -316,15 +325,15 @@ decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_consta
                         norm_rotate_head(token_row + (size_t)(heads + sg.kvh) * D, fused.k_weight, fused.eps, cs,
                                          fused.rotary_dim, head_vec[0], new_k);
                     if (warp == 1)
-                        for (int e = lane; e < D; e += 32) new_v[e] = token_row[(size_t)(heads + kv_heads + sg.kvh) * D + e];
+                        for (int e = lane; e < DV; e += 32) new_v[e] = token_row[(size_t)(heads + kv_heads) * D + (size_t)sg.kvh * DV + e];
                     consumer_sync();
                     if (slot >= 0) {
                         const int page = slot / page_size, off = slot - page * page_size;
-                        const size_t at = (((size_t)page * kv_heads + sg.kvh) * page_size + off) * D;
-                        for (int c = threadIdx.x; c < 2 * CHUNKS; c += CONSUMERS) {
+                        const size_t cache_at = ((size_t)page * kv_heads + sg.kvh) * page_size + off;
+                        for (int c = threadIdx.x; c < CHUNKS + CHUNKS_V; c += CONSUMERS) {
                             const bool is_v = c >= CHUNKS;
                             const int chunk = is_v ? c - CHUNKS : c;
-                            *reinterpret_cast<uint4*>((is_v ? fused.v_cache : fused.k_cache) + at + chunk * 8) =
+                            *reinterpret_cast<uint4*>((is_v ? fused.v_cache + cache_at * DV : fused.k_cache + cache_at * D) + chunk * 8) =
                                 *reinterpret_cast<const uint4*>((is_v ? new_v : new_k) + chunk * 8);
                         }
                     }
@@ -339,6 +348,10 @@ decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_consta
                 row_pos[rr] = row < group ? pos : -1;
                 row_lo[rr] = lo;
             }
+            mrun::ScoreRow form_row[2];
+#pragma unroll
+            for (int rr = 0; rr < 2; ++rr)
+                form_row[rr] = make_score_row(form, scale_log2, pos, sg.kvh * group + min((lane >> 2) + rr * 8, group - 1));
             for (int block = sg.first_block; block <= sg.last_block; ++block, ++it) {
                 const int s = it % RING, use = it / RING;
                 if (!__all_sync(0xffffffffu, mbar_wait(&full_bar[s], use & 1, WAIT_CYCLES, &aborted)) && alive) {
@@ -354,7 +367,7 @@ decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_consta
                 if (owns_new_token && block == b1) {
                     // the page row of this step's token was not written when the tile was requested
                     const int row = pos - key_base;
-                    for (int c = threadIdx.x; c < 2 * CHUNKS; c += CONSUMERS) {
+                    for (int c = threadIdx.x; c < CHUNKS + CHUNKS_V; c += CONSUMERS) {
                         const bool is_v = c >= CHUNKS;
                         const int chunk = is_v ? c - CHUNKS : c;
                         *reinterpret_cast<uint4*>(const_cast<unsigned char*>(swz(is_v ? v_tile : k_tile, row, chunk))) =
@@ -364,7 +377,8 @@ decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_consta
                 }
                 // warp w takes keys 16w .. 16w+15 of the tile
                 if (key_base + warp * 16 <= pos && key_base + warp * 16 + 15 >= lo)
-                    attend_slice(q_tile, k_tile, v_tile, warp * 16, key_base, scale_log2, row_pos, row_lo, m, l, o);
+                    attend_slice(q_tile, k_tile, v_tile, warp * 16, key_base, scale_log2, row_pos, row_lo, form_row,
+                                 SCORED && pos - (key_base + warp * 16 + 15) < form.bias_len - 1, m, l, o);
                 __syncwarp();
                 if (lane == 0) mbar_arrive(&empty_bar[s]);
             }
@@ -373,52 +387,50 @@ decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_consta
                 l[rr] += __shfl_xor_sync(0xffffffffu, l[rr], 1);
                 l[rr] += __shfl_xor_sync(0xffffffffu, l[rr], 2);
             }
-            // the four warps meet: merge[warp][row < group][D + 2]
+            // the four warps meet: merge[warp][row < group][DV + 2]
 #pragma unroll
             for (int rr = 0; rr < 2; ++rr) {
                 const int row = (lane >> 2) + rr * 8;
                 if (row < group) {
                     float* dst = merge + (warp * group + row) * MS;
 #pragma unroll
-                    for (int dt = 0; dt < D / 8; ++dt) {
+                    for (int dt = 0; dt < DV / 8; ++dt) {
                         dst[dt * 8 + (lane & 3) * 2] = o[dt][2 * rr];
                         dst[dt * 8 + (lane & 3) * 2 + 1] = o[dt][2 * rr + 1];
                     }
                     if ((lane & 3) == 0) {
-                        dst[D] = m[rr];
-                        dst[D + 1] = l[rr];
+                        dst[DV] = m[rr];
+                        dst[DV + 1] = l[rr];
                     }
                 }
             }
             consumer_sync();
             const size_t my_slot = (size_t)block_id * 2 + (seg == 0 ? 0 : 1);
             // a thread takes four values of a row: the warps' maxima and sums are read once for them
-            for (int i = threadIdx.x; i < group * (D / 4); i += CONSUMERS) {
-                const int row = i / (D / 4), d = (i - row * (D / 4)) * 4;
+            for (int i = threadIdx.x; i < group * (DV / 4); i += CONSUMERS) {
+                const int row = i / (DV / 4), d = (i - row * (DV / 4)) * 4;
                 float mm = -INFINITY;
 #pragma unroll
-                for (int w = 0; w < 4; ++w) mm = fmaxf(mm, merge[(w * group + row) * MS + D]);
+                for (int w = 0; w < 4; ++w) mm = fmaxf(mm, merge[(w * group + row) * MS + DV]);
                 float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
                 float ll = 0.f;
 #pragma unroll
                 for (int w = 0; w < 4; ++w) {
                     const float* src = merge + (w * group + row) * MS;
-                    const float c = (src[D] == -INFINITY) ? 0.f : exp2f(src[D] - mm);
+                    const float c = (src[DV] == -INFINITY) ? 0.f : exp2f(src[DV] - mm);
                     const float2 lo2 = *reinterpret_cast<const float2*>(src + d), hi2 = *reinterpret_cast<const float2*>(src + d + 2);
                     acc.x += lo2.x * c; acc.y += lo2.y * c; acc.z += hi2.x * c; acc.w += hi2.y * c;
-                    ll += src[D + 1] * c;
+                    ll += src[DV + 1] * c;
                 }
                 if (sg.complete) {
                     ll = with_sink(ll, mm, sink_log2);
                     const float inv = ll > 0.f ? 1.f / ll : 0.f;
-                    __nv_bfloat162 lo2 = __floats2bfloat162_rn(acc.x * inv, acc.y * inv);
-                    __nv_bfloat162 hi2 = __floats2bfloat162_rn(acc.z * inv, acc.w * inv);
-                    uint2 packed;
-                    packed.x = *reinterpret_cast<unsigned*>(&lo2);
-                    packed.y = *reinterpret_cast<unsigned*>(&hi2);
-                    *reinterpret_cast<uint2*>(out + ((size_t)q_row * heads + sg.kvh * group + row) * D + d) = packed;
+                    float v[4] = {acc.x * inv, acc.y * inv, acc.z * inv, acc.w * inv};
+                    finish_outputs<4>(form, q_row, (sg.kvh * group + row) * DV + d, v);
+                    *reinterpret_cast<uint2*>(out + (size_t)q_row * out_stride + (sg.kvh * group + row) * DV + d) =
+                        make_uint2(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]));
                 } else {
-                    *reinterpret_cast<float4*>(part_o + (my_slot * 16 + row) * D + d) = acc;
+                    *reinterpret_cast<float4*>(part_o + (my_slot * 16 + row) * DV + d) = acc;
                     if (d == 0) *reinterpret_cast<float2*>(part_ml + (my_slot * 16 + row) * 2) = make_float2(mm, ll);
                 }
             }
@@ -442,8 +454,8 @@ decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_consta
                     // A thread takes four values of a row.  The pieces are read four at a time, all
                     // loads of a round requested before any is used (one piece after the other the
                     // merge took a third of a block's time).
-                    for (int i = threadIdx.x; i < group * (D / 4); i += CONSUMERS) {
-                        const int row = i / (D / 4), d = (i - row * (D / 4)) * 4;
+                    for (int i = threadIdx.x; i < group * (DV / 4); i += CONSUMERS) {
+                        const int row = i / (DV / 4), d = (i - row * (DV / 4)) * 4;
                         // block p's piece of this pair is its first segment iff its range starts inside the pair
                         auto slot_of = [&](int p) -> size_t {
                             return (size_t)p * 2 + ((splits > 0 || p * per >= sg.pair_start) ? 0 : 1);
@@ -469,7 +481,7 @@ decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_consta
                                 if (p0 + k <= p_last) {
                                     const size_t at = slot_of(p0 + k) * 16 + row;
                                     ml[k] = __ldcg(reinterpret_cast<const float2*>(part_ml + at * 2));
-                                    po[k] = __ldcg(reinterpret_cast<const float4*>(part_o + at * D + d));
+                                    po[k] = __ldcg(reinterpret_cast<const float4*>(part_o + at * DV + d));
                                 }
                             }
 #pragma unroll
@@ -481,12 +493,10 @@ decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_consta
                         }
                         ll = with_sink(ll, mm, sink_log2);
                         const float inv = ll > 0.f ? 1.f / ll : 0.f;
-                        __nv_bfloat162 lo2 = __floats2bfloat162_rn(acc.x * inv, acc.y * inv);
-                        __nv_bfloat162 hi2 = __floats2bfloat162_rn(acc.z * inv, acc.w * inv);
-                        uint2 packed;
-                        packed.x = *reinterpret_cast<unsigned*>(&lo2);
-                        packed.y = *reinterpret_cast<unsigned*>(&hi2);
-                        *reinterpret_cast<uint2*>(out + ((size_t)q_row * heads + sg.kvh * group + row) * D + d) = packed;
+                        float v[4] = {acc.x * inv, acc.y * inv, acc.z * inv, acc.w * inv};
+                        finish_outputs<4>(form, q_row, (sg.kvh * group + row) * DV + d, v);
+                        *reinterpret_cast<uint2*>(out + (size_t)q_row * out_stride + (sg.kvh * group + row) * DV + d) =
+                            make_uint2(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]));
                     }
                     if (threadIdx.x == 0) counters[sg.tok * kv_heads + sg.kvh] = 0;
                 }
@@ -539,22 +549,24 @@ decode_cluster_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_co
                       const bf16* __restrict__ q, long q_stride, bf16* __restrict__ out,
                       const int* __restrict__ block_tables, int max_blocks, const int* __restrict__ token_slot,
                       const int* __restrict__ positions, int heads, int kv_heads, int page_size, int page_shift,
-                      float scale_log2, int window, float sink_log2, const FusedInput fused, int* __restrict__ status) {
+                      float scale_log2, int window, float sink_log2, const FusedInput fused,
+                  const mrun_score_form form, int* __restrict__ status) {
     extern __shared__ __align__(1024) unsigned char smem_raw[];
     unsigned char* ring = reinterpret_cast<unsigned char*>(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
     const int group = heads / kv_heads;
-    bf16* q_tile = reinterpret_cast<bf16*>(ring + RING * STAGE_BYTES);                   // [16][LD]
-    float* merge = reinterpret_cast<float*>(q_tile + 16 * LD);                            // [4][group][MS]
+    bf16* q_tile = reinterpret_cast<bf16*>(ring + RING * STAGE_BYTES);                   // [16][LD], Q_REGION bytes
+    float* merge = reinterpret_cast<float*>(ring + RING * STAGE_BYTES + Q_REGION);                            // [4][group][MS]
     float (*head_vec)[D] = reinterpret_cast<float (*)[D]>(merge + 4 * group * MS);        // [4][D]
     bf16* new_k = reinterpret_cast<bf16*>(head_vec + 4);
     bf16* new_v = new_k + D;
     // the block's piece takes the place of the queries once the tiles are done: [group][PS],
-    // PS = D + 4 so that a row starts on 16 bytes (group <= 8: 8 x 132 floats fit 16 x LD bf16)
-    constexpr int PS = D + 4;
+    // PS = DV + 4 so that a row starts on 16 bytes (group <= 8: Q_REGION holds 8 such rows)
+    constexpr int PS = DV + 4;
     float* piece = reinterpret_cast<float*>(q_tile);
     __shared__ unsigned long long full_bar[RING], empty_bar[RING];
     __shared__ int aborted;
 
+    const long out_stride = output_stride(form, heads);
     const unsigned rank = blockIdx.x, pieces = gridDim.x;
     const int pair = blockIdx.y, tok = pair / kv_heads, kvh = pair - tok * kv_heads;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -562,8 +574,8 @@ decode_cluster_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_co
     const int q_row = fused.rows ? fused.rows[tok] : tok;
     if (pos < 0) {                                   // a padding row: zeros, and the whole cluster leaves
         if (rank == 0)
-            for (int i = threadIdx.x; i < group * D; i += TMA_THREADS)
-                out[((size_t)q_row * heads + kvh * group) * D + i] = __float2bfloat16_rn(0.f);
+            for (int i = threadIdx.x; i < group * DV; i += TMA_THREADS)
+                out[(size_t)q_row * out_stride + kvh * group * DV + i] = __float2bfloat16_rn(0.f);
         return;
     }
     const int lo = mrun::first_visible(pos, window);
@@ -615,13 +627,13 @@ decode_cluster_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_co
                 const bool wanted = first_key <= pos && first_key + box_rows - 1 >= lo;
                 const int page = !wanted ? -1 : windowed ? my_page : table[first_key >> page_shift];
                 if (page >= 0) {
-                    bytes += (unsigned)(2 * box_rows * D * 2);
+                    bytes += (unsigned)(box_rows * (D + DV) * 2);
                     continue;
                 }
                 // Rows of a V tile that no copy fills must not hold NaN patterns (0 * NaN is NaN): the
                 // lane that leaves a box out clears the box's V rows itself, before it arrives.
 #pragma unroll
-                for (int h = 0; h < SPANS; ++h) {
+                for (int h = 0; h < SPANS_V; ++h) {
                     uint4* rows = reinterpret_cast<uint4*>(stage + TILE_BYTES + h * SPAN_BYTES + b * box_rows * 128);
                     for (int i = 0; i < box_rows * 8; ++i) rows[i] = make_uint4(0, 0, 0, 0);
                 }
@@ -634,11 +646,13 @@ decode_cluster_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_co
                 const int page = windowed ? my_page : table[first_key >> page_shift];
                 if (page < 0) continue;
 #pragma unroll
-                for (int h = 0; h < SPANS; ++h) {
-                    tma_load_4d(stage + h * SPAN_BYTES + b * box_rows * 128, &map_k, h * 64,
-                                first_key & (page_size - 1), kvh, page, &full_bar[s]);
-                    tma_load_4d(stage + TILE_BYTES + h * SPAN_BYTES + b * box_rows * 128, &map_v, h * 64,
-                                first_key & (page_size - 1), kvh, page, &full_bar[s]);
+                for (int h = 0; h < (SPANS > SPANS_V ? SPANS : SPANS_V); ++h) {
+                    if (h < SPANS)
+                        tma_load_4d(stage + h * SPAN_BYTES + b * box_rows * 128, &map_k, h * 64,
+                                    first_key & (page_size - 1), kvh, page, &full_bar[s]);
+                    if (h < SPANS_V)
+                        tma_load_4d(stage + TILE_BYTES + h * SPAN_BYTES + b * box_rows * 128, &map_v, h * 64,
+                                    first_key & (page_size - 1), kvh, page, &full_bar[s]);
                 }
             }
         }
@@ -649,9 +663,9 @@ decode_cluster_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_co
     } else {
         // ----------------------------------------------------------------------------- consumers
         float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
-        float o[D / 8][4];
+        float o[DV / 8][4];
 #pragma unroll
-        for (int dt = 0; dt < D / 8; ++dt) o[dt][0] = o[dt][1] = o[dt][2] = o[dt][3] = 0.f;
+        for (int dt = 0; dt < DV / 8; ++dt) o[dt][0] = o[dt][1] = o[dt][2] = o[dt][3] = 0.f;
         if (len > 0) {
             const bool owns_new_token = fused.enabled && last_block == b1;
             if (!fused.enabled) {
@@ -678,15 +692,15 @@ decode_cluster_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_co
                         norm_rotate_head(token_row + (size_t)(heads + kvh) * D, fused.k_weight, fused.eps, cs,
                                          fused.rotary_dim, head_vec[0], new_k);
                     if (warp == 1)
-                        for (int e = lane; e < D; e += 32) new_v[e] = token_row[(size_t)(heads + kv_heads + kvh) * D + e];
+                        for (int e = lane; e < DV; e += 32) new_v[e] = token_row[(size_t)(heads + kv_heads) * D + (size_t)kvh * DV + e];
                     consumer_sync();
                     if (slot >= 0) {
                         const int page = slot / page_size, off = slot - page * page_size;
-                        const size_t at = (((size_t)page * kv_heads + kvh) * page_size + off) * D;
-                        for (int c = threadIdx.x; c < 2 * CHUNKS; c += CONSUMERS) {
+                        const size_t cache_at = ((size_t)page * kv_heads + kvh) * page_size + off;
+                        for (int c = threadIdx.x; c < CHUNKS + CHUNKS_V; c += CONSUMERS) {
                             const bool is_v = c >= CHUNKS;
                             const int chunk = is_v ? c - CHUNKS : c;
-                            *reinterpret_cast<uint4*>((is_v ? fused.v_cache : fused.k_cache) + at + chunk * 8) =
+                            *reinterpret_cast<uint4*>((is_v ? fused.v_cache + cache_at * DV : fused.k_cache + cache_at * D) + chunk * 8) =
                                 *reinterpret_cast<const uint4*>((is_v ? new_v : new_k) + chunk * 8);
                         }
                     }
@@ -701,6 +715,10 @@ decode_cluster_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_co
                 row_pos[rr] = row < group ? pos : -1;
                 row_lo[rr] = lo;
             }
+            mrun::ScoreRow form_row[2];
+#pragma unroll
+            for (int rr = 0; rr < 2; ++rr)
+                form_row[rr] = make_score_row(form, scale_log2, pos, kvh * group + min((lane >> 2) + rr * 8, group - 1));
             bool alive = true;
             int it = 0;
             for (int block = first_block; block <= last_block; ++block, ++it) {
@@ -717,7 +735,7 @@ decode_cluster_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_co
                 const int key_base = block * BLOCK_N;
                 if (owns_new_token && block == b1) {
                     const int row = pos - key_base;
-                    for (int c = threadIdx.x; c < 2 * CHUNKS; c += CONSUMERS) {
+                    for (int c = threadIdx.x; c < CHUNKS + CHUNKS_V; c += CONSUMERS) {
                         const bool is_v = c >= CHUNKS;
                         const int chunk = is_v ? c - CHUNKS : c;
                         *reinterpret_cast<uint4*>(const_cast<unsigned char*>(swz(is_v ? v_tile : k_tile, row, chunk))) =
@@ -726,7 +744,8 @@ decode_cluster_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_co
                     consumer_sync();
                 }
                 if (key_base + warp * 16 <= pos && key_base + warp * 16 + 15 >= lo)
-                    attend_slice(q_tile, k_tile, v_tile, warp * 16, key_base, scale_log2, row_pos, row_lo, m, l, o);
+                    attend_slice(q_tile, k_tile, v_tile, warp * 16, key_base, scale_log2, row_pos, row_lo, form_row,
+                                 SCORED && pos - (key_base + warp * 16 + 15) < form.bias_len - 1, m, l, o);
                 __syncwarp();
                 if (lane == 0) mbar_arrive(&empty_bar[s]);
             }
@@ -736,59 +755,57 @@ decode_cluster_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_co
                 l[rr] += __shfl_xor_sync(0xffffffffu, l[rr], 2);
             }
         }
-        // the four warps meet: merge[warp][row < group][D + 2] (a block without tiles brings nothing)
+        // the four warps meet: merge[warp][row < group][DV + 2] (a block without tiles brings nothing)
 #pragma unroll
         for (int rr = 0; rr < 2; ++rr) {
             const int row = (lane >> 2) + rr * 8;
             if (row < group) {
                 float* dst = merge + (warp * group + row) * MS;
 #pragma unroll
-                for (int dt = 0; dt < D / 8; ++dt) {
+                for (int dt = 0; dt < DV / 8; ++dt) {
                     dst[dt * 8 + (lane & 3) * 2] = o[dt][2 * rr];
                     dst[dt * 8 + (lane & 3) * 2 + 1] = o[dt][2 * rr + 1];
                 }
                 if ((lane & 3) == 0) {
-                    dst[D] = m[rr];
-                    dst[D + 1] = l[rr];
+                    dst[DV] = m[rr];
+                    dst[DV + 1] = l[rr];
                 }
             }
         }
         consumer_sync();                                        // also: nobody reads the queries any more
-        for (int i = threadIdx.x; i < group * (D / 4); i += CONSUMERS) {
-            const int row = i / (D / 4), d = (i - row * (D / 4)) * 4;
+        for (int i = threadIdx.x; i < group * (DV / 4); i += CONSUMERS) {
+            const int row = i / (DV / 4), d = (i - row * (DV / 4)) * 4;
             float mm = -INFINITY;
 #pragma unroll
-            for (int w = 0; w < 4; ++w) mm = fmaxf(mm, merge[(w * group + row) * MS + D]);
+            for (int w = 0; w < 4; ++w) mm = fmaxf(mm, merge[(w * group + row) * MS + DV]);
             float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
             float ll = 0.f;
 #pragma unroll
             for (int w = 0; w < 4; ++w) {
                 const float* src = merge + (w * group + row) * MS;
-                const float c = (src[D] == -INFINITY) ? 0.f : exp2f(src[D] - mm);
+                const float c = (src[DV] == -INFINITY) ? 0.f : exp2f(src[DV] - mm);
                 const float2 lo2 = *reinterpret_cast<const float2*>(src + d), hi2 = *reinterpret_cast<const float2*>(src + d + 2);
                 acc.x += lo2.x * c; acc.y += lo2.y * c; acc.z += hi2.x * c; acc.w += hi2.y * c;
-                ll += src[D + 1] * c;
+                ll += src[DV + 1] * c;
             }
             if (pieces == 1) {
                 ll = with_sink(ll, mm, sink_log2);
                 const float inv = ll > 0.f ? 1.f / ll : 0.f;
-                __nv_bfloat162 lo2 = __floats2bfloat162_rn(acc.x * inv, acc.y * inv);
-                __nv_bfloat162 hi2 = __floats2bfloat162_rn(acc.z * inv, acc.w * inv);
-                uint2 packed;
-                packed.x = *reinterpret_cast<unsigned*>(&lo2);
-                packed.y = *reinterpret_cast<unsigned*>(&hi2);
-                *reinterpret_cast<uint2*>(out + ((size_t)q_row * heads + kvh * group + row) * D + d) = packed;
+                float v[4] = {acc.x * inv, acc.y * inv, acc.z * inv, acc.w * inv};
+                finish_outputs<4>(form, q_row, (kvh * group + row) * DV + d, v);
+                *reinterpret_cast<uint2*>(out + (size_t)q_row * out_stride + (kvh * group + row) * DV + d) =
+                    make_uint2(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]));
             } else {
                 *reinterpret_cast<float4*>(piece + row * PS + d) = acc;
-                if (d == 0) *reinterpret_cast<float2*>(piece + row * PS + D) = make_float2(mm, ll);
+                if (d == 0) *reinterpret_cast<float2*>(piece + row * PS + DV) = make_float2(mm, ll);
             }
         }
     }
     if (pieces > 1) {
         cluster_sync_all();                                     // every block's piece is in its shared memory
         if (rank == 0 && warp < 4) {
-            for (int i = threadIdx.x; i < group * (D / 4); i += CONSUMERS) {
-                const int row = i / (D / 4), d = (i - row * (D / 4)) * 4;
+            for (int i = threadIdx.x; i < group * (DV / 4); i += CONSUMERS) {
+                const int row = i / (DV / 4), d = (i - row * (DV / 4)) * 4;
                 // four pieces a round, all of a round's loads requested before any is used; the
                 // running maximum rescales what the rounds before have added
                 float mm = -INFINITY, ll = 0.f;
@@ -801,7 +818,7 @@ decode_cluster_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_co
                         ml[k] = make_float2(-INFINITY, 0.f);
                         po[k] = make_float4(0.f, 0.f, 0.f, 0.f);
                         if (p0 + k < pieces) {
-                            ml[k] = cluster_load2(cluster_address(piece + row * PS + D, p0 + k));
+                            ml[k] = cluster_load2(cluster_address(piece + row * PS + DV, p0 + k));
                             po[k] = cluster_load4(cluster_address(piece + row * PS + d, p0 + k));
                         }
                     }
@@ -821,12 +838,10 @@ decode_cluster_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_co
                 }
                 ll = with_sink(ll, mm, sink_log2);
                 const float inv = ll > 0.f ? 1.f / ll : 0.f;
-                __nv_bfloat162 lo2 = __floats2bfloat162_rn(acc.x * inv, acc.y * inv);
-                __nv_bfloat162 hi2 = __floats2bfloat162_rn(acc.z * inv, acc.w * inv);
-                uint2 packed;
-                packed.x = *reinterpret_cast<unsigned*>(&lo2);
-                packed.y = *reinterpret_cast<unsigned*>(&hi2);
-                *reinterpret_cast<uint2*>(out + ((size_t)q_row * heads + kvh * group + row) * D + d) = packed;
+                float v[4] = {acc.x * inv, acc.y * inv, acc.z * inv, acc.w * inv};
+                finish_outputs<4>(form, q_row, (kvh * group + row) * DV + d, v);
+                *reinterpret_cast<uint2*>(out + (size_t)q_row * out_stride + (kvh * group + row) * DV + d) =
+                    make_uint2(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]));
             }
         }
         cluster_sync_all();                                     // the pieces may go: the first block has read them
@@ -882,7 +897,7 @@ template <int RING>
 int launch_cluster(const CUtensorMap& map_k, const CUtensorMap& map_v, const void* q, long q_stride, void* out,
                    const int* block_tables, int max_blocks, const int* token_slot, const int* positions, int tokens,
                    int cluster, int heads, int kv_heads, int page_size, float scale, int window, float sink, const FusedInput& in,
-                   int* status, cudaStream_t stream) {
+                   const mrun_score_form& form, int* status, cudaStream_t stream) {
     const int group = heads / kv_heads;
     const size_t smem = tma_smem_bytes(RING, group);
     static size_t allowed = 0;
@@ -907,7 +922,7 @@ int launch_cluster(const CUtensorMap& map_k, const CUtensorMap& map_v, const voi
     config.numAttrs = 1;
     MRUN_CHECK_CUDA(cudaLaunchKernelEx(&config, decode_cluster_kernel<RING>, map_k, map_v, (const bf16*)q, q_stride, (bf16*)out,
                                        block_tables, max_blocks, token_slot, positions, heads, kv_heads, page_size,
-                                       page_shift_of(page_size), scale * LOG2E, window, sink * LOG2E, in, status),
+                                       page_shift_of(page_size), scale * LOG2E, window, sink * LOG2E, in, form, status),
                     "attn_decode_cluster");
     return 0;
 }
@@ -935,9 +950,10 @@ MRUN_API int mrun_attn_decode_cluster(const void* q, long q_stride, void* out, v
                                       const int* positions, int tokens, int cluster, int heads, int kv_heads,
                                       int head_dim, int page_size, float scale, int window, float sink, int fused,
                                       const float* q_weight, const float* k_weight, float eps, const float* rot,
-                                      int rotary_dim, const int* slots, const int* rows, long pages, int* status,
-                                      cudaStream_t stream) {
+                                      int rotary_dim, const int* slots, const int* rows, long pages,
+                                      const mrun_score_form* form, int* status, cudaStream_t stream) {
 #if MRUN_DECODE_TMA
+    if (int rc = check_form("attn_decode_cluster", form, heads)) return rc;
     if (int rc = check_common("attn_decode_cluster", heads, kv_heads, head_dim, page_size, max_blocks, window, 8)) return rc;
     MRUN_REQUIRE(tokens >= 0 && (long)tokens * kv_heads <= 65535, "attn_decode_cluster: tokens=%d kv_heads=%d", tokens, kv_heads);
     MRUN_REQUIRE(cluster == 1 || cluster == 2 || cluster == 4 || cluster == 8 || cluster == 16,
@@ -951,7 +967,7 @@ MRUN_API int mrun_attn_decode_cluster(const void* q, long q_stride, void* out, v
                  "attn_decode_cluster: rotary_dim=%d must be even and at most head_dim=%d", rotary_dim, head_dim);
     MRUN_REQUIRE(!fused || (q_weight == nullptr) == (k_weight == nullptr),
                  "attn_decode_cluster: q and k norm weights come together");
-    MRUN_REQUIRE(!fused || q_stride >= (long)(heads + 2 * kv_heads) * head_dim,
+    MRUN_REQUIRE(!fused || q_stride >= (long)(heads + kv_heads) * head_dim + (long)kv_heads * DV,
                  "attn_decode_cluster: the raw rows must hold q, k and v (stride %ld)", q_stride);
     MRUN_REQUIRE(!(fused && rows), "attn_decode_cluster: a selection of rows does not go with raw q, k, v input");
     if (tokens == 0) return 0;
@@ -959,7 +975,7 @@ MRUN_API int mrun_attn_decode_cluster(const void* q, long q_stride, void* out, v
     CUtensorMap map_k, map_v;
     const int box_rows = page_size < BLOCK_N ? page_size : BLOCK_N;
     if (int rc = paged_cache_map(&map_k, k_cache, pages, kv_heads, page_size, D, box_rows, "attn_decode_cluster")) return rc;
-    if (int rc = paged_cache_map(&map_v, v_cache, pages, kv_heads, page_size, D, box_rows, "attn_decode_cluster")) return rc;
+    if (int rc = paged_cache_map(&map_v, v_cache, pages, kv_heads, page_size, DV, box_rows, "attn_decode_cluster")) return rc;
     FusedInput in = {};
     if (fused) {
         in.enabled = 1;
@@ -975,9 +991,9 @@ MRUN_API int mrun_attn_decode_cluster(const void* q, long q_stride, void* out, v
     in.rows = rows;
     if (ring_for(group) == 3)
         return launch_cluster<3>(map_k, map_v, q, q_stride, out, block_tables, max_blocks, token_slot, positions, tokens,
-                                 cluster, heads, kv_heads, page_size, scale, window, sink, in, status, stream);
+                                 cluster, heads, kv_heads, page_size, scale, window, sink, in, form_or_none(form), status, stream);
     return launch_cluster<2>(map_k, map_v, q, q_stride, out, block_tables, max_blocks, token_slot, positions, tokens, cluster,
-                             heads, kv_heads, page_size, scale, window, sink, in, status, stream);
+                             heads, kv_heads, page_size, scale, window, sink, in, form_or_none(form), status, stream);
 #else
     return mrun_set_error("attn_decode_cluster: not built for head_dim=%d (head sizes 64 and 128 only)", MRUN_HEAD_DIM);
 #endif
@@ -994,9 +1010,10 @@ MRUN_API int mrun_attn_decode_tma(const void* q, long q_stride, void* out, void*
                                   float* part_o, float* part_ml, int* counters, int blocks, int heads, int kv_heads,
                                   int head_dim, int page_size, float scale, int window, float sink, int fused,
                                   const float* q_weight, const float* k_weight, float eps, const float* rot,
-                                  int rotary_dim, const int* slots, const int* rows, long pages, int* status,
-                                  cudaStream_t stream) {
+                                  int rotary_dim, const int* slots, const int* rows, long pages,
+                                  const mrun_score_form* form, int* status, cudaStream_t stream) {
 #if MRUN_DECODE_TMA
+    if (int rc = check_form("attn_decode_tma", form, heads)) return rc;
     if (int rc = check_common("attn_decode_tma", heads, kv_heads, head_dim, page_size, max_blocks, window, 16)) return rc;
     MRUN_REQUIRE(tokens >= 0 && blocks >= 1 && blocks <= 65535, "attn_decode_tma: tokens=%d blocks=%d", tokens, blocks);
     MRUN_REQUIRE(tile_prefix && assignment && part_o && part_ml && counters && status,
@@ -1009,7 +1026,7 @@ MRUN_API int mrun_attn_decode_tma(const void* q, long q_stride, void* out, void*
                  "attn_decode_tma: rotary_dim=%d must be even and at most head_dim=%d", rotary_dim, head_dim);
     MRUN_REQUIRE(!fused || (q_weight == nullptr) == (k_weight == nullptr),
                  "attn_decode_tma: q and k norm weights come together");
-    MRUN_REQUIRE(!fused || q_stride >= (long)(heads + 2 * kv_heads) * head_dim,
+    MRUN_REQUIRE(!fused || q_stride >= (long)(heads + kv_heads) * head_dim + (long)kv_heads * DV,
                  "attn_decode_tma: the raw rows must hold q, k and v (stride %ld)", q_stride);
     MRUN_REQUIRE(!(fused && rows), "attn_decode_tma: a selection of rows does not go with raw q, k, v input");
     if (tokens == 0) return 0;
@@ -1019,7 +1036,7 @@ MRUN_API int mrun_attn_decode_tma(const void* q, long q_stride, void* out, void*
     CUtensorMap map_k, map_v;
     const int box_rows = page_size < BLOCK_N ? page_size : BLOCK_N;
     if (int rc = paged_cache_map(&map_k, k_cache, pages, kv_heads, page_size, D, box_rows, "attn_decode_tma")) return rc;
-    if (int rc = paged_cache_map(&map_v, v_cache, pages, kv_heads, page_size, D, box_rows, "attn_decode_tma")) return rc;
+    if (int rc = paged_cache_map(&map_v, v_cache, pages, kv_heads, page_size, DV, box_rows, "attn_decode_tma")) return rc;
     FusedInput in = {};
     if (fused) {
         in.enabled = 1;
@@ -1038,12 +1055,12 @@ MRUN_API int mrun_attn_decode_tma(const void* q, long q_stride, void* out, void*
         decode_tma_kernel<3><<<dim3(blocks), TMA_THREADS, smem, stream>>>(
             map_k, map_v, (const bf16*)q, q_stride, (bf16*)out, block_tables, max_blocks, token_slot, positions,
             tile_prefix, (const int4*)assignment, tokens, part_o, part_ml, counters, heads, kv_heads, page_size,
-            page_shift_of(page_size), scale * LOG2E, window, sink * LOG2E, in, status);
+            page_shift_of(page_size), scale * LOG2E, window, sink * LOG2E, in, form_or_none(form), status);
     else
         decode_tma_kernel<2><<<dim3(blocks), TMA_THREADS, smem, stream>>>(
             map_k, map_v, (const bf16*)q, q_stride, (bf16*)out, block_tables, max_blocks, token_slot, positions,
             tile_prefix, (const int4*)assignment, tokens, part_o, part_ml, counters, heads, kv_heads, page_size,
-            page_shift_of(page_size), scale * LOG2E, window, sink * LOG2E, in, status);
+            page_shift_of(page_size), scale * LOG2E, window, sink * LOG2E, in, form_or_none(form), status);
     MRUN_CHECK_LAUNCH("attn_decode_tma");
     return 0;
 #else

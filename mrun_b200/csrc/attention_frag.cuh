@@ -1,23 +1,34 @@
 // What the mma.sync attention kernels of one head size share: the fragment loads and products,
 // the description of raw q, k, v input that the decode kernels norm, rotate and store themselves,
-// and the argument checks.  Compiled with -DMRUN_HEAD_DIM=<multiple of 16, at most 256>.
+// and the argument checks.  Compiled with -DMRUN_HEAD_DIM=<multiple of 16, at most 256>; values of
+// another size than the keys with -DMRUN_VALUE_DIM=<the same>, scores that are worked on before the
+// softmax and a gated output (attention_score.cuh) with -DMRUN_SCORED=1.
 #pragma once
 
 #include "attention_paging.cuh"
+#include "attention_score.cuh"
 #include "common.cuh"
 
 #ifndef MRUN_HEAD_DIM
 #error "compile with -DMRUN_HEAD_DIM=<head size>"
 #endif
+#ifndef MRUN_VALUE_DIM
+#define MRUN_VALUE_DIM MRUN_HEAD_DIM
+#endif
+#ifndef MRUN_SCORED
+#define MRUN_SCORED 0
+#endif
 
 namespace {
 
-constexpr int D = MRUN_HEAD_DIM;
+constexpr int D = MRUN_HEAD_DIM, DV = MRUN_VALUE_DIM;
+constexpr bool SCORED = MRUN_SCORED;
 static_assert(D % 16 == 0 && D >= 16 && D <= 256, "head size must be a multiple of 16, at most 256");
-constexpr int LD = D + 8;            // smem row stride in elements: odd number of 16-byte chunks
+static_assert(DV % 16 == 0 && DV >= 16 && DV <= 256, "value size must be a multiple of 16, at most 256");
+constexpr int LD = D + 8, LDV = DV + 8;      // smem row strides in elements: odd numbers of 16-byte chunks
 constexpr int BLOCK_N = 64;          // keys per tile
 constexpr int THREADS = 128;
-constexpr int CHUNKS = D / 8;        // 16-byte chunks per row
+constexpr int CHUNKS = D / 8, CHUNKS_V = DV / 8;     // 16-byte chunks per row
 constexpr float LOG2E = 1.4426950408889634f;
 
 using bf16 = __nv_bfloat16;
@@ -156,5 +167,40 @@ inline int check_common(const char* name, int heads, int kv_heads, int head_dim,
     return 0;
 }
 
+// The score form of a call: required where the library was compiled for it, refused elsewhere.
+inline int check_form(const char* name, const mrun_score_form* form, int heads) {
+    MRUN_REQUIRE(SCORED == (form != nullptr), "%s: this library was built %s a score form", name, SCORED ? "for" : "without");
+    if (form == nullptr) return 0;
+    MRUN_REQUIRE(form->cap >= 0.f && (form->temp_coef == 0.f || form->temp_every > 0.f), "%s: bad cap or temperature", name);
+    MRUN_REQUIRE(form->bias == nullptr || form->bias_len > 0, "%s: an empty bias table", name);
+    MRUN_REQUIRE(form->out_stride >= (long)heads * DV && form->out_stride % 8 == 0,
+                 "%s: output rows %ld apart, expected a multiple of 8 and at least %d", name, form->out_stride, heads * DV);
+    MRUN_REQUIRE(form->gate == nullptr || (form->gate_stride >= (long)heads * DV && form->gate_stride % 8 == 0 &&
+                                           ((uintptr_t)form->gate & 15) == 0),
+                 "%s: the gate's rows must start on 16 bytes and hold %d features", name, heads * DV);
+    return 0;
+}
+inline mrun_score_form form_or_none(const mrun_score_form* form) { return form ? *form : mrun_score_form{}; }
+
+// What a row of scores is worked on with, for the two rows of a thread (query head `head0` + row of a
+// token at `pos`); nothing in libraries without a score form.
+__device__ __forceinline__ mrun::ScoreRow make_score_row(const mrun_score_form& form, float scale_log2, int pos, int head) {
+    if constexpr (SCORED) return mrun::score_row(form, scale_log2 / LOG2E, pos, head);
+    else return mrun::ScoreRow{};
+}
+// One raw product as a score in base-2 units.  `near`: some key of the tile is close enough for an entry
+// of the bias table of its own.
+__device__ __forceinline__ float scored(const mrun::ScoreRow& row, float dot, bool near, int distance) {
+    return mrun::capped_score(row, dot) + (near ? mrun::distance_bias(row, distance) : row.far_bias);
+}
+
+__device__ __forceinline__ long output_stride(const mrun_score_form& form, int heads) {
+    return SCORED ? form.out_stride : (long)heads * DV;
+}
+// N finished features of an output row, gated where the library does that.
+template <int N>
+__device__ __forceinline__ void finish_outputs(const mrun_score_form& form, size_t token, int col, float (&v)[N]) {
+    if constexpr (SCORED) mrun::gate_outputs<N>(form, token, col, v);
+}
 
 }  // namespace

@@ -1,5 +1,6 @@
 // Paged grouped-query attention on the tensor cores (bf16 operands, 32-bit accumulation and
-// softmax), compiled for one head size: -DMRUN_HEAD_DIM=<multiple of 16, at most 256>.
+// softmax), compiled for one head size: -DMRUN_HEAD_DIM=<multiple of 16, at most 256> (values of
+// another size and worked-on scores as in attention_frag.cuh).
 //
 // Two kernels share the tile loader and the fragment code:
 //
@@ -27,14 +28,29 @@
 
 namespace {
 
-// Loads keys key0 .. key0+63 of one kv head into a key tile and a value tile, both [64][LD].
+// Loads keys key0 .. key0+63 of one kv head into a key tile [64][LD] and a value tile [64][LDV].
 // Rows whose key lies outside [lo, hi] or whose page is not held are zero-filled.  A row's place
 // in the cache is worked out once and used for both tensors.  `page_shift` is log2(page_size)
 // when the page size is a power of two (shift and mask instead of a division), else -1.
 __device__ __forceinline__ void load_kv_tiles(bf16* k_tile, bf16* v_tile, const bf16* __restrict__ k_cache,
                                               const bf16* __restrict__ v_cache, const Paging& pg, int key0,
                                               int lo, int hi) {
-    if constexpr (THREADS % CHUNKS == 0) {
+    if constexpr (D != DV) {
+        for (int c = threadIdx.x; c < BLOCK_N * CHUNKS; c += THREADS) {
+            const int row = c / CHUNKS, chunk = c - row * CHUNKS;
+            const int key = key0 + row;
+            bool valid = key >= lo && key <= hi;
+            const long at = cache_row<D>(pg, key, valid) + chunk * 8;
+            cp_async_16(k_tile + row * LD + chunk * 8, valid ? k_cache + at : k_cache, valid);
+        }
+        for (int c = threadIdx.x; c < BLOCK_N * CHUNKS_V; c += THREADS) {
+            const int row = c / CHUNKS_V, chunk = c - row * CHUNKS_V;
+            const int key = key0 + row;
+            bool valid = key >= lo && key <= hi;
+            const long at = cache_row<DV>(pg, key, valid) + chunk * 8;
+            cp_async_16(v_tile + row * LDV + chunk * 8, valid ? v_cache + at : v_cache, valid);
+        }
+    } else if constexpr (THREADS % CHUNKS == 0) {
         // a thread keeps its 16-byte column and walks down the rows
         constexpr int STEP = THREADS / CHUNKS;
         const int chunk = threadIdx.x % CHUNKS, r0 = threadIdx.x / CHUNKS;
@@ -66,7 +82,8 @@ template <int N_KEYS>
 __device__ __forceinline__ void attend_tile(const bf16* q_tile, const bf16* k_tile, const bf16* v_tile,
                                             int krow0, int key_base, float scale_log2, bool need_mask,
                                             const int (&row_pos)[2], const int (&row_lo)[2],
-                                            float (&m)[2], float (&l)[2], float (&o)[D / 8][4]) {
+                                            const mrun::ScoreRow (&form_row)[2], bool near_keys,
+                                            float (&m)[2], float (&l)[2], float (&o)[DV / 8][4]) {
     constexpr int NT = N_KEYS / 8;     // score n-tiles
     const int lane = threadIdx.x & 31;
     float s[NT][4];
@@ -94,6 +111,8 @@ __device__ __forceinline__ void attend_tile(const bf16* q_tile, const bf16* k_ti
         for (int e = 0; e < 4; ++e) {
             const int r = e >> 1;
             float v = s[nt][e] * scale_log2;
+            if constexpr (SCORED)
+                v = scored(form_row[r], s[nt][e], near_keys, row_pos[r] - (key_base + krow0 + nt * 8 + (lane & 3) * 2 + (e & 1)));
             if (need_mask) {
                 const int key = key_base + krow0 + nt * 8 + (lane & 3) * 2 + (e & 1);
                 if (key > row_pos[r] || key < row_lo[r]) v = -INFINITY;
@@ -125,7 +144,7 @@ __device__ __forceinline__ void attend_tile(const bf16* q_tile, const bf16* k_ti
 #pragma unroll
     for (int r = 0; r < 2; ++r) l[r] = l[r] * corr[r] + sum[r];   // per-thread partial; reduced at the end
 #pragma unroll
-    for (int dt = 0; dt < D / 8; ++dt) {
+    for (int dt = 0; dt < DV / 8; ++dt) {
         o[dt][0] *= corr[0]; o[dt][1] *= corr[0];
         o[dt][2] *= corr[1]; o[dt][3] *= corr[1];
     }
@@ -139,9 +158,9 @@ __device__ __forceinline__ void attend_tile(const bf16* q_tile, const bf16* k_ti
         a[2] = pack_bf16(s[2 * kk + 1][0], s[2 * kk + 1][1]);
         a[3] = pack_bf16(s[2 * kk + 1][2], s[2 * kk + 1][3]);
 #pragma unroll
-        for (int dt = 0; dt < D / 8; dt += 2) {
+        for (int dt = 0; dt < DV / 8; dt += 2) {
             unsigned b[4];
-            ldmatrix_x4_trans(b, v_tile + (krow0 + kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * LD + dt * 8 + (lane >> 4) * 8);
+            ldmatrix_x4_trans(b, v_tile + (krow0 + kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * LDV + dt * 8 + (lane >> 4) * 8);
             mma_bf16(o[dt], a, b[0], b[1]);
             mma_bf16(o[dt + 1], a, b[2], b[3]);
         }
@@ -157,11 +176,11 @@ prefill_kernel(const bf16* __restrict__ q, long q_stride, bf16* __restrict__ out
                const int* __restrict__ block_tables, int max_blocks, const int* __restrict__ token_slot,
                const int* __restrict__ positions, const int* __restrict__ tile_tok0,
                const int* __restrict__ tile_ntok, int heads, int kv_heads, int page_size, int page_shift,
-               float scale_log2, int window, float sink_log2) {
+               float scale_log2, int window, float sink_log2, const mrun_score_form form) {
     extern __shared__ __align__(16) unsigned char smem_raw[];
     bf16* q_tile = reinterpret_cast<bf16*>(smem_raw);           // [64][LD]
     bf16* k_tiles = q_tile + 64 * LD;                           // [2][64][LD]
-    bf16* v_tiles = k_tiles + 2 * BLOCK_N * LD;                 // [2][64][LD]
+    bf16* v_tiles = k_tiles + 2 * BLOCK_N * LD;                 // [2][64][LDV]
 
     const int tile = blockIdx.y, kvh = blockIdx.x;      // the list's first tile (the longest, the host sorts) for every kv head first
     const int group = heads / kv_heads;
@@ -202,14 +221,18 @@ prefill_kernel(const bf16* __restrict__ q, long q_stride, bf16* __restrict__ out
     const int w_pos_first = pos_first + w_row0 / group;
 
     float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
-    float o[D / 8][4];
+    float o[DV / 8][4];
 #pragma unroll
-    for (int dt = 0; dt < D / 8; ++dt) o[dt][0] = o[dt][1] = o[dt][2] = o[dt][3] = 0.f;
+    for (int dt = 0; dt < DV / 8; ++dt) o[dt][0] = o[dt][1] = o[dt][2] = o[dt][3] = 0.f;
+    mrun::ScoreRow form_row[2];
+#pragma unroll
+    for (int r = 0; r < 2; ++r)
+        form_row[r] = make_score_row(form, scale_log2, row_pos[r], kvh * group + (warp * 16 + (lane >> 2) + r * 8) % group);
 
     for (int block = first_block; block <= last_block; ++block) {
         const int stage = (block - first_block) & 1;
         if (block < last_block) {
-            load_kv_tiles(k_tiles + (stage ^ 1) * BLOCK_N * LD, v_tiles + (stage ^ 1) * BLOCK_N * LD, k_cache, v_cache,
+            load_kv_tiles(k_tiles + (stage ^ 1) * BLOCK_N * LD, v_tiles + (stage ^ 1) * BLOCK_N * LDV, k_cache, v_cache,
                           pg, (block + 1) * BLOCK_N, lo_tile, pos_last);
             cp_async_commit();
             cp_async_wait<1>();
@@ -225,14 +248,16 @@ prefill_kernel(const bf16* __restrict__ q, long q_stride, bf16* __restrict__ out
                 const int w_lo_last = mrun::first_visible(w_pos_last, window);
                 const bool need_mask = key_base + BLOCK_N - 1 > w_pos_first || key_base < w_lo_last;
                 attend_tile<BLOCK_N>(q_tile + w_row0 * LD, k_tiles + stage * BLOCK_N * LD,
-                                     v_tiles + stage * BLOCK_N * LD, 0, key_base, scale_log2, need_mask, row_pos,
-                                     row_lo, m, l, o);
+                                     v_tiles + stage * BLOCK_N * LDV, 0, key_base, scale_log2, need_mask, row_pos,
+                                     row_lo, form_row, SCORED && w_pos_first - (key_base + BLOCK_N - 1) < form.bias_len - 1,
+                                     m, l, o);
             }
         }
         __syncthreads();
     }
 
-    // finish the row sums over the quad, normalise, stage through q_tile, write coalesced
+    // finish the row sums over the quad, normalise, stage from the start of shared memory (every warp
+    // is done with its queries and tiles), write coalesced
 #pragma unroll
     for (int r = 0; r < 2; ++r) {
         l[r] += __shfl_xor_sync(0xffffffffu, l[r], 1);
@@ -240,19 +265,25 @@ prefill_kernel(const bf16* __restrict__ q, long q_stride, bf16* __restrict__ out
     }
     l[0] = with_sink(l[0], m[0], sink_log2);
     l[1] = with_sink(l[1], m[1], sink_log2);
-    const float inv0 = l[0] > 0.f ? 1.f / l[0] : 0.f, inv1 = l[1] > 0.f ? 1.f / l[1] : 0.f;
-    bf16* stage_rows = q_tile + w_row0 * LD;
+    bf16* stage_rows = q_tile + w_row0 * LDV;
 #pragma unroll
-    for (int dt = 0; dt < D / 8; ++dt) {
-        const int col = dt * 8 + (lane & 3) * 2;
-        *reinterpret_cast<unsigned*>(stage_rows + (lane >> 2) * LD + col) = pack_bf16(o[dt][0] * inv0, o[dt][1] * inv0);
-        *reinterpret_cast<unsigned*>(stage_rows + ((lane >> 2) + 8) * LD + col) = pack_bf16(o[dt][2] * inv1, o[dt][3] * inv1);
+    for (int r = 0; r < 2; ++r) {
+        const int row = w_row0 + (lane >> 2) + r * 8;
+        const float inv = l[r] > 0.f ? 1.f / l[r] : 0.f;
+#pragma unroll
+        for (int dt = 0; dt < DV / 8; ++dt) {
+            const int col = dt * 8 + (lane & 3) * 2;
+            float v[2] = {o[dt][2 * r] * inv, o[dt][2 * r + 1] * inv};
+            if (row < n_rows) finish_outputs<2>(form, tok0 + row / group, (kvh * group + row % group) * DV + col, v);
+            *reinterpret_cast<unsigned*>(stage_rows + ((lane >> 2) + r * 8) * LDV + col) = pack_bf16(v[0], v[1]);
+        }
     }
     __syncthreads();
-    for (int c = threadIdx.x; c < n_rows * CHUNKS; c += THREADS) {
-        const int row = c / CHUNKS, chunk = c - row * CHUNKS;
-        bf16* dst = out + ((size_t)(tok0 + row / group) * heads + kvh * group + row % group) * D + chunk * 8;
-        *reinterpret_cast<uint4*>(dst) = *reinterpret_cast<const uint4*>(q_tile + row * LD + chunk * 8);
+    const long out_stride = output_stride(form, heads);
+    for (int c = threadIdx.x; c < n_rows * CHUNKS_V; c += THREADS) {
+        const int row = c / CHUNKS_V, chunk = c - row * CHUNKS_V;
+        bf16* dst = out + (size_t)(tok0 + row / group) * out_stride + (kvh * group + row % group) * DV + chunk * 8;
+        *reinterpret_cast<uint4*>(dst) = *reinterpret_cast<const uint4*>(q_tile + row * LDV + chunk * 8);
     }
 }
 
@@ -266,7 +297,7 @@ prefill_kernel(const bf16* __restrict__ q, long q_stride, bf16* __restrict__ out
 // block's range is a sequence of segments, each a run of tiles of one pair; only its first and
 // its last segment can be part of a pair.  A partial segment writes its unnormalised 32-bit
 // result and its running (max, sum) to scratch (slot 0 if it is the block's first segment, else
-// slot 1): part_o [blocks, 2, 16, D], part_ml [blocks, 2, 16, 2].  The block that arrives last at
+// slot 1): part_o [blocks, 2, 16, DV], part_ml [blocks, 2, 16, 2].  The block that arrives last at
 // the pair's counter merges the pair's pieces in block order and sets the counter back to zero,
 // so no second kernel runs and the result does not depend on which block came last.
 // ------------------------------------------------------------------------------------------
@@ -415,7 +446,7 @@ __global__ void decode_assign_kernel(const int* __restrict__ tile_prefix, int to
 }
 
 // grid: `blocks` blocks, the number the plan was made for.
-// part_o: [blocks][2][16][D] floats, part_ml: [blocks][2][16][2] floats, counters: [tokens * kv_heads]
+// part_o: [blocks][2][16][DV] floats, part_ml: [blocks][2][16][2] floats, counters: [tokens * kv_heads]
 // ints, zero before the call and zero again after it.
 __global__ void __launch_bounds__(THREADS)
 decode_kernel(const bf16* __restrict__ q, long q_stride, bf16* __restrict__ out,
@@ -424,19 +455,21 @@ decode_kernel(const bf16* __restrict__ q, long q_stride, bf16* __restrict__ out,
               const int* __restrict__ positions, const int* __restrict__ tile_prefix,
               const int4* __restrict__ assignment, int tokens, float* __restrict__ part_o,
               float* __restrict__ part_ml, int* __restrict__ counters, int heads, int kv_heads, int page_size,
-              int page_shift, float scale_log2, int window, float sink_log2, const FusedInput fused) {
+              int page_shift, float scale_log2, int window, float sink_log2, const FusedInput fused,
+              const mrun_score_form form) {
     extern __shared__ __align__(16) unsigned char smem_raw[];
     bf16* q_tile = reinterpret_cast<bf16*>(smem_raw);           // [16][LD]
     bf16* k_tiles = q_tile + 16 * LD;                           // [STAGES][64][LD]
-    bf16* v_tiles = k_tiles + STAGES * BLOCK_N * LD;            // [STAGES][64][LD]
+    bf16* v_tiles = k_tiles + STAGES * BLOCK_N * LD;            // [STAGES][64][LDV]
     float* merge = reinterpret_cast<float*>(k_tiles);           // reused after a segment's loop
     __shared__ int ticket_shared;
-    __shared__ __align__(16) bf16 new_k[D], new_v[D];           // this step's own key and value (fused input)
-    // Staging of a head vector per warp (fused input).  It lives in the value tile of the last
+    __shared__ __align__(16) bf16 new_k[D], new_v[DV];          // this step's own key and value (fused input)
+    // Staging of a head vector per warp (fused input).  It lives in the key tile of the last
     // stage, which no copy targets before the first tile of a segment has been consumed; shared
     // memory is what limits the blocks per SM, and a static array here costs one of three.
-    float (*head_vec)[D] = reinterpret_cast<float (*)[D]>(v_tiles + (STAGES - 1) * BLOCK_N * LD);
-    constexpr int MS = D + 2;
+    float (*head_vec)[D] = reinterpret_cast<float (*)[D]>(k_tiles + (STAGES - 1) * BLOCK_N * LD);
+    constexpr int MS = DV + 2;
+    const long out_stride = output_stride(form, heads);
 
     const int block_id = blockIdx.x, n_blocks_grid = gridDim.x;
     const int group = heads / kv_heads;
@@ -451,7 +484,7 @@ decode_kernel(const bf16* __restrict__ q, long q_stride, bf16* __restrict__ out,
     // padding rows come out as zeros
     for (int t = block_id; t < tokens; t += n_blocks_grid)
         if (positions[t] < 0)
-            for (int i = threadIdx.x; i < heads * D; i += THREADS) out[(size_t)t * heads * D + i] = __float2bfloat16_rn(0.f);
+            for (int i = threadIdx.x; i < heads * DV; i += THREADS) out[(size_t)t * out_stride + i] = __float2bfloat16_rn(0.f);
 
     for (int seg = 0; u < u_end; ++seg) {
         // ---------------------------------------------------------------- which pair, which tiles
@@ -480,15 +513,15 @@ decode_kernel(const bf16* __restrict__ q, long q_stride, bf16* __restrict__ out,
         const int last_block = first_block + len - 1;
 
         float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
-        float o[D / 8][4];
+        float o[DV / 8][4];
 #pragma unroll
-        for (int dt = 0; dt < D / 8; ++dt) o[dt][0] = o[dt][1] = o[dt][2] = o[dt][3] = 0.f;
+        for (int dt = 0; dt < DV / 8; ++dt) o[dt][0] = o[dt][1] = o[dt][2] = o[dt][3] = 0.f;
 
         // prologue: STAGES - 1 tiles in flight (an empty group keeps the counting uniform)
 #pragma unroll
         for (int s = 0; s < STAGES - 1; ++s) {
             if (first_block + s <= last_block)
-                load_kv_tiles(k_tiles + s * BLOCK_N * LD, v_tiles + s * BLOCK_N * LD, k_cache, v_cache, pg,
+                load_kv_tiles(k_tiles + s * BLOCK_N * LD, v_tiles + s * BLOCK_N * LDV, k_cache, v_cache, pg,
                               (first_block + s) * BLOCK_N, lo, pos);
             cp_async_commit();
         }
@@ -504,7 +537,7 @@ decode_kernel(const bf16* __restrict__ q, long q_stride, bf16* __restrict__ out,
                 *reinterpret_cast<uint4*>(q_tile + row * LD + chunk * 8) = value;
             }
         } else {
-            // q, k and v arrive raw: [q heads | k heads | v heads] of D elements each in the token's row
+            // q, k and v arrive raw: [q heads | k heads | v heads] in the token's row
             const bf16* token_row = q + (size_t)tok * q_stride;
             const float2* cs = fused.rot ? fused.rot + (size_t)tok * (fused.rotary_dim >> 1) : nullptr;
             for (int row = warp; row < 16; row += THREADS / 32) {
@@ -521,16 +554,16 @@ decode_kernel(const bf16* __restrict__ q, long q_stride, bf16* __restrict__ out,
                     norm_rotate_head(token_row + (size_t)(heads + kvh) * D, fused.k_weight, fused.eps, cs,
                                      fused.rotary_dim, head_vec[0], new_k);
                 if (warp == 1)
-                    for (int e = lane; e < D; e += 32) new_v[e] = token_row[(size_t)(heads + kv_heads + kvh) * D + e];
+                    for (int e = lane; e < DV; e += 32) new_v[e] = token_row[(size_t)(heads + kv_heads) * D + (size_t)kvh * DV + e];
                 __syncthreads();
                 const int slot = fused.slots ? fused.slots[tok] : -1;
                 if (slot >= 0) {
                     const int page = slot / page_size, off = slot - page * page_size;
-                    const size_t at = (((size_t)page * kv_heads + kvh) * page_size + off) * D;
-                    for (int c = threadIdx.x; c < 2 * CHUNKS; c += THREADS) {
+                    const size_t cache_at = ((size_t)page * kv_heads + kvh) * page_size + off;
+                    for (int c = threadIdx.x; c < CHUNKS + CHUNKS_V; c += THREADS) {
                         const bool is_v = c >= CHUNKS;
                         const int chunk = is_v ? c - CHUNKS : c;
-                        *reinterpret_cast<uint4*>((is_v ? fused.v_cache : fused.k_cache) + at + chunk * 8) =
+                        *reinterpret_cast<uint4*>((is_v ? fused.v_cache + cache_at * DV : fused.k_cache + cache_at * D) + chunk * 8) =
                             *reinterpret_cast<const uint4*>((is_v ? new_v : new_k) + chunk * 8);
                     }
                 }
@@ -544,6 +577,10 @@ decode_kernel(const bf16* __restrict__ q, long q_stride, bf16* __restrict__ out,
             row_pos[rr] = row < group ? pos : -1;
             row_lo[rr] = lo;
         }
+        mrun::ScoreRow form_row[2];
+#pragma unroll
+        for (int rr = 0; rr < 2; ++rr)
+            form_row[rr] = make_score_row(form, scale_log2, pos, kvh * group + min((lane >> 2) + rr * 8, group - 1));
         for (int block = first_block; block <= last_block; ++block) {
             const int it = block - first_block;
             cp_async_wait<STAGES - 2>();        // tile `it` has landed
@@ -551,7 +588,7 @@ decode_kernel(const bf16* __restrict__ q, long q_stride, bf16* __restrict__ out,
             const int ahead = block + STAGES - 1;
             if (ahead <= last_block) {
                 const int s = (it + STAGES - 1) % STAGES;
-                load_kv_tiles(k_tiles + s * BLOCK_N * LD, v_tiles + s * BLOCK_N * LD, k_cache, v_cache, pg,
+                load_kv_tiles(k_tiles + s * BLOCK_N * LD, v_tiles + s * BLOCK_N * LDV, k_cache, v_cache, pg,
                               ahead * BLOCK_N, lo, pos);
             }
             cp_async_commit();
@@ -560,18 +597,19 @@ decode_kernel(const bf16* __restrict__ q, long q_stride, bf16* __restrict__ out,
             if (owns_new_token && block == b1) {
                 // the page row of this step's token was not written when the tile was requested
                 const int row = pos - key_base;
-                for (int c = threadIdx.x; c < 2 * CHUNKS; c += THREADS) {
+                for (int c = threadIdx.x; c < CHUNKS + CHUNKS_V; c += THREADS) {
                     const bool is_v = c >= CHUNKS;
                     const int chunk = is_v ? c - CHUNKS : c;
-                    *reinterpret_cast<uint4*>((is_v ? v_tiles : k_tiles) + (stage * BLOCK_N + row) * LD + chunk * 8) =
+                    *reinterpret_cast<uint4*>((is_v ? v_tiles + (stage * BLOCK_N + row) * LDV : k_tiles + (stage * BLOCK_N + row) * LD) + chunk * 8) =
                         *reinterpret_cast<const uint4*>((is_v ? new_v : new_k) + chunk * 8);
                 }
                 __syncthreads();
             }
             // warp w takes keys 16w .. 16w+15 of the tile
             if (key_base + warp * 16 <= pos && key_base + warp * 16 + 15 >= lo)
-                attend_tile<16>(q_tile, k_tiles + stage * BLOCK_N * LD, v_tiles + stage * BLOCK_N * LD, warp * 16,
-                                key_base, scale_log2, true, row_pos, row_lo, m, l, o);
+                attend_tile<16>(q_tile, k_tiles + stage * BLOCK_N * LD, v_tiles + stage * BLOCK_N * LDV, warp * 16,
+                                key_base, scale_log2, true, row_pos, row_lo, form_row,
+                                SCORED && pos - (key_base + warp * 16 + 15) < form.bias_len - 1, m, l, o);
         }
         cp_async_wait<0>();
 #pragma unroll
@@ -580,42 +618,44 @@ decode_kernel(const bf16* __restrict__ q, long q_stride, bf16* __restrict__ out,
             l[rr] += __shfl_xor_sync(0xffffffffu, l[rr], 2);
         }
 
-        // merge the four warps: merge[warp][16 rows][D + 2]
+        // merge the four warps: merge[warp][16 rows][DV + 2]
         __syncthreads();
 #pragma unroll
         for (int rr = 0; rr < 2; ++rr) {
             const int row = (lane >> 2) + rr * 8;
             float* dst = merge + (warp * 16 + row) * MS;
 #pragma unroll
-            for (int dt = 0; dt < D / 8; ++dt) {
+            for (int dt = 0; dt < DV / 8; ++dt) {
                 dst[dt * 8 + (lane & 3) * 2] = o[dt][2 * rr];
                 dst[dt * 8 + (lane & 3) * 2 + 1] = o[dt][2 * rr + 1];
             }
             if ((lane & 3) == 0) {
-                dst[D] = m[rr];
-                dst[D + 1] = l[rr];
+                dst[DV] = m[rr];
+                dst[DV + 1] = l[rr];
             }
         }
         __syncthreads();
         const size_t my_slot = (size_t)block_id * 2 + (seg == 0 ? 0 : 1);
-        for (int i = threadIdx.x; i < group * D; i += THREADS) {
-            const int row = i / D, d = i - row * D;
+        for (int i = threadIdx.x; i < group * DV; i += THREADS) {
+            const int row = i / DV, d = i - row * DV;
             float mm = -INFINITY;
 #pragma unroll
-            for (int w = 0; w < 4; ++w) mm = fmaxf(mm, merge[(w * 16 + row) * MS + D]);
+            for (int w = 0; w < 4; ++w) mm = fmaxf(mm, merge[(w * 16 + row) * MS + DV]);
             float acc = 0.f, ll = 0.f;
 #pragma unroll
             for (int w = 0; w < 4; ++w) {
                 const float* src = merge + (w * 16 + row) * MS;
-                const float c = (src[D] == -INFINITY) ? 0.f : exp2f(src[D] - mm);
+                const float c = (src[DV] == -INFINITY) ? 0.f : exp2f(src[DV] - mm);
                 acc += src[d] * c;
-                ll += src[D + 1] * c;
+                ll += src[DV + 1] * c;
             }
             if (complete) {
                 ll = with_sink(ll, mm, sink_log2);
-                out[((size_t)tok * heads + kvh * group + row) * D + d] = __float2bfloat16_rn(ll > 0.f ? acc / ll : 0.f);
+                float v = ll > 0.f ? acc / ll : 0.f;
+                if constexpr (SCORED) v = mrun::gate_output(form, tok, (kvh * group + row) * DV + d, v);
+                out[(size_t)tok * out_stride + (kvh * group + row) * DV + d] = __float2bfloat16_rn(v);
             } else {
-                part_o[(my_slot * 16 + row) * D + d] = acc;
+                part_o[(my_slot * 16 + row) * DV + d] = acc;
                 if (d == 0) {
                     part_ml[(my_slot * 16 + row) * 2] = mm;
                     part_ml[(my_slot * 16 + row) * 2 + 1] = ll;
@@ -641,8 +681,8 @@ decode_kernel(const bf16* __restrict__ q, long q_stride, bf16* __restrict__ out,
                 __threadfence();
                 // A thread takes four values of a row; the pieces are read four at a time, all loads
                 // of a round requested before any is used.
-                for (int i = threadIdx.x; i < group * (D / 4); i += THREADS) {
-                    const int row = i / (D / 4), d = (i - row * (D / 4)) * 4;
+                for (int i = threadIdx.x; i < group * (DV / 4); i += THREADS) {
+                    const int row = i / (DV / 4), d = (i - row * (DV / 4)) * 4;
                     // block p's piece of this pair is its first segment iff its range starts inside the pair
                     auto slot_of = [&](int p) -> size_t {
                         return (size_t)p * 2 + ((splits > 0 || p * per >= pair_start) ? 0 : 1);
@@ -668,7 +708,7 @@ decode_kernel(const bf16* __restrict__ q, long q_stride, bf16* __restrict__ out,
                             if (p0 + k <= p_last) {
                                 const size_t at = slot_of(p0 + k) * 16 + row;
                                 ml[k] = __ldcg(reinterpret_cast<const float2*>(part_ml + at * 2));
-                                po[k] = __ldcg(reinterpret_cast<const float4*>(part_o + at * D + d));
+                                po[k] = __ldcg(reinterpret_cast<const float4*>(part_o + at * DV + d));
                             }
                         }
 #pragma unroll
@@ -680,12 +720,10 @@ decode_kernel(const bf16* __restrict__ q, long q_stride, bf16* __restrict__ out,
                     }
                     ll = with_sink(ll, mm, sink_log2);
                     const float inv = ll > 0.f ? 1.f / ll : 0.f;
-                    __nv_bfloat162 lo2 = __floats2bfloat162_rn(acc.x * inv, acc.y * inv);
-                    __nv_bfloat162 hi2 = __floats2bfloat162_rn(acc.z * inv, acc.w * inv);
-                    uint2 packed;
-                    packed.x = *reinterpret_cast<unsigned*>(&lo2);
-                    packed.y = *reinterpret_cast<unsigned*>(&hi2);
-                    *reinterpret_cast<uint2*>(out + ((size_t)tok * heads + kvh * group + row) * D + d) = packed;
+                    float v[4] = {acc.x * inv, acc.y * inv, acc.z * inv, acc.w * inv};
+                    finish_outputs<4>(form, tok, (kvh * group + row) * DV + d, v);
+                    *reinterpret_cast<uint2*>(out + (size_t)tok * out_stride + (kvh * group + row) * DV + d) =
+                        make_uint2(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]));
                 }
                 if (threadIdx.x == 0) counters[tok * kv_heads + kvh] = 0;
             }
@@ -695,14 +733,17 @@ decode_kernel(const bf16* __restrict__ q, long q_stride, bf16* __restrict__ out,
     }
 }
 
-constexpr size_t PREFILL_SMEM = (size_t)(64 + 4 * BLOCK_N) * LD * sizeof(bf16);
-constexpr size_t DECODE_SMEM = (size_t)(16 + 2 * STAGES * BLOCK_N) * LD * sizeof(bf16);
-static_assert((size_t)4 * 16 * (D + 2) * sizeof(float) <= (size_t)2 * STAGES * BLOCK_N * LD * sizeof(bf16),
+constexpr size_t PREFILL_SMEM = ((size_t)(64 + 2 * BLOCK_N) * LD + (size_t)2 * BLOCK_N * LDV) * sizeof(bf16);
+constexpr size_t DECODE_SMEM = ((size_t)(16 + STAGES * BLOCK_N) * LD + (size_t)STAGES * BLOCK_N * LDV) * sizeof(bf16);
+static_assert((size_t)64 * LDV * sizeof(bf16) <= PREFILL_SMEM, "the output rows must fit");
+static_assert((size_t)4 * 16 * (DV + 2) * sizeof(float) <= (size_t)STAGES * BLOCK_N * (LD + LDV) * sizeof(bf16),
               "the warp merge area must fit in the key/value tiles");
 
 }  // namespace
 
 MRUN_API int mrun_attn_head_dim() { return D; }
+MRUN_API int mrun_attn_value_dim() { return DV; }
+MRUN_API int mrun_attn_scored() { return SCORED; }
 
 // Tiles: tile i covers tokens tile_tok0[i] .. +tile_ntok[i]-1 (consecutive positions of one request,
 // at most 64 / (heads / kv_heads) of them).
@@ -710,8 +751,9 @@ MRUN_API int mrun_attn_prefill(const void* q, long q_stride, void* out, const vo
                                const int* block_tables, int max_blocks, const int* token_slot,
                                const int* positions, const int* tile_tok0, const int* tile_ntok, int n_tiles,
                                int heads, int kv_heads, int head_dim, int page_size, float scale, int window,
-                               float sink, cudaStream_t stream) {
+                               float sink, const mrun_score_form* form, cudaStream_t stream) {
     if (int rc = check_common("attn_prefill", heads, kv_heads, head_dim, page_size, max_blocks, window, 64)) return rc;
+    if (int rc = check_form("attn_prefill", form, heads)) return rc;
     MRUN_REQUIRE(n_tiles >= 0, "attn_prefill: n_tiles=%d", n_tiles);
     if (n_tiles == 0) return 0;
     static bool configured = false;
@@ -725,7 +767,7 @@ MRUN_API int mrun_attn_prefill(const void* q, long q_stride, void* out, const vo
         prefill_kernel<<<dim3(kv_heads, now), THREADS, PREFILL_SMEM, stream>>>(
             (const bf16*)q, q_stride, (bf16*)out, (const bf16*)k_cache, (const bf16*)v_cache, block_tables, max_blocks,
             token_slot, positions, tile_tok0 + done, tile_ntok + done, heads, kv_heads, page_size, page_shift_of(page_size),
-            scale * LOG2E, window, sink * LOG2E);
+            scale * LOG2E, window, sink * LOG2E, form_or_none(form));
         MRUN_CHECK_LAUNCH("attn_prefill");
     }
     return 0;
@@ -761,11 +803,11 @@ MRUN_API int mrun_attn_decode_plan(const int* positions, int tokens, int window,
 // Every token is a row of its own (positions[t] < 0 = padding, output zero).  tile_prefix and
 // assignment: the plan from mrun_attn_decode_plan for the same positions, window, kv_heads and
 // blocks.  blocks: how many blocks share the tiles (as many as the device holds at once is best).
-// part_o and part_ml are scratch of blocks * 2 * 16 * (D and 2) floats; counters holds
+// part_o and part_ml are scratch of blocks * 2 * 16 * (DV and 2) floats; counters holds
 // tokens * kv_heads ints that are zero before the call and zero again after it.  Calls that share
 // scratch must not overlap on the device.
 //
-// fused != 0: `q` is the projection's raw output, rows of [heads | kv_heads | kv_heads] x D (q, k, v);
+// fused != 0: `q` is the projection's raw output, rows of q [heads x D], k [kv_heads x D], v [kv_heads x DV];
 // the kernel norms q and k with q_weight / k_weight (null: no norm) and eps, rotates them with
 // rot[token] (null: no rotation), writes the token's k and v to cache slot slots[token] (null or
 // negative: no write) and attends over the cache plus that token.  fused == 0: q is ready and the
@@ -776,7 +818,8 @@ MRUN_API int mrun_attn_decode(const void* q, long q_stride, void* out, void* k_c
                               float* part_o, float* part_ml, int* counters, int blocks, int heads, int kv_heads,
                               int head_dim, int page_size, float scale, int window, float sink, int fused,
                               const float* q_weight, const float* k_weight, float eps, const float* rot,
-                              int rotary_dim, const int* slots, cudaStream_t stream) {
+                              int rotary_dim, const int* slots, const mrun_score_form* form, cudaStream_t stream) {
+    if (int rc = check_form("attn_decode", form, heads)) return rc;
     if (int rc = check_common("attn_decode", heads, kv_heads, head_dim, page_size, max_blocks, window, 16)) return rc;
     MRUN_REQUIRE(tokens >= 0 && blocks >= 1 && blocks <= 65535, "attn_decode: tokens=%d blocks=%d", tokens, blocks);
     MRUN_REQUIRE(tile_prefix && assignment && part_o && part_ml && counters,
@@ -785,7 +828,7 @@ MRUN_API int mrun_attn_decode(const void* q, long q_stride, void* out, void* k_c
                  "attn_decode: rotary_dim=%d must be even and at most head_dim=%d", rotary_dim, head_dim);
     MRUN_REQUIRE(!fused || (q_weight == nullptr) == (k_weight == nullptr),
                  "attn_decode: q and k norm weights come together");
-    MRUN_REQUIRE(!fused || q_stride >= (long)(heads + 2 * kv_heads) * head_dim,
+    MRUN_REQUIRE(!fused || q_stride >= (long)(heads + kv_heads) * head_dim + (long)kv_heads * DV,
                  "attn_decode: the raw rows must hold q, k and v (stride %ld)", q_stride);
     if (tokens == 0) return 0;
     static bool configured = false;
@@ -810,7 +853,8 @@ MRUN_API int mrun_attn_decode(const void* q, long q_stride, void* out, void* k_c
                                      (const bf16*)q, q_stride, (bf16*)out, (const bf16*)k_cache, (const bf16*)v_cache,
                                      block_tables, max_blocks, token_slot, positions, tile_prefix,
                                      (const int4*)assignment, tokens, part_o, part_ml, counters, heads, kv_heads,
-                                     page_size, page_shift_of(page_size), scale * LOG2E, window, sink * LOG2E, in),
+                                     page_size, page_shift_of(page_size), scale * LOG2E, window, sink * LOG2E, in,
+                                     form_or_none(form)),
                     "attn_decode");
     return 0;
 }
@@ -824,9 +868,11 @@ MRUN_API int mrun_attn_decode_occupancy() {
     return blocks;
 }
 
+#if !MRUN_SCORED
 // ------------------------------------------------------------------------------------------
 // The same decode kernel for callers that cannot allocate: its scratch is a fixed array in this
-// library (see attention_static.h for who needs that, the limits and the rules).
+// library (see attention_static.h for who needs that, the limits and the rules).  Not in libraries
+// with a score form.
 // ------------------------------------------------------------------------------------------
 #include "attention_static.h"
 
@@ -834,7 +880,7 @@ MRUN_API int mrun_attn_decode_occupancy() {
 
 namespace {
 
-constexpr size_t STATIC_PART_O = (size_t)MRUN_STATIC_MAX_BLOCKS * 2 * 16 * D;      // floats
+constexpr size_t STATIC_PART_O = (size_t)MRUN_STATIC_MAX_BLOCKS * 2 * 16 * DV;      // floats
 constexpr size_t STATIC_PART_ML = (size_t)MRUN_STATIC_MAX_BLOCKS * 2 * 16 * 2;     // floats
 constexpr size_t STATIC_COUNTERS = MRUN_STATIC_MAX_PAIRS;                          // ints, stored as 4-byte words
 constexpr size_t STATIC_ASSIGNMENT = (size_t)MRUN_STATIC_MAX_BLOCKS * 8;            // ints, 16-byte aligned
@@ -906,7 +952,8 @@ MRUN_API int mrun_attn_decode_static(const void* q, long q_stride, void* out, co
     decode_kernel<<<dim3(blocks), THREADS, DECODE_SMEM, stream>>>(
         (const bf16*)q, q_stride, (bf16*)out, (const bf16*)k_cache, (const bf16*)v_cache, block_tables, max_blocks,
         token_slot, positions, tile_prefix, (const int4*)assignment, tokens, part_o, part_ml, counters, heads, kv_heads,
-        page_size, page_shift_of(page_size), scale * LOG2E, window, -INFINITY, FusedInput{});
+        page_size, page_shift_of(page_size), scale * LOG2E, window, -INFINITY, FusedInput{}, mrun_score_form{});
     MRUN_CHECK_LAUNCH("attn_decode_static");
     return 0;
 }
+#endif  // !MRUN_SCORED

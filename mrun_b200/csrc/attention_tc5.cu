@@ -1,6 +1,7 @@
 // Paged grouped-query attention for prompt portions on the fifth-generation tensor cores
 // (tcgen05, accumulators in tensor memory), compiled for one head size that is a multiple of 64
-// and at most 128: -DMRUN_HEAD_DIM=<64 | 128>.
+// and at most 128: -DMRUN_HEAD_DIM=<64 | 128> (values of another of these sizes: -DMRUN_VALUE_DIM;
+// worked-on scores and gated outputs, attention_score.cuh: -DMRUN_SCORED=1).
 //
 // One thread block per (tile of query tokens, kv head).  The tile's 128 rows are (token, query
 // head of the kv head's group) pairs, so a key/value tile read once serves the whole group.  Keys
@@ -41,6 +42,7 @@
 #include <cstdio>
 
 #include "attention_paging.cuh"
+#include "attention_score.cuh"
 #include "common.cuh"
 #include "tcgen05.cuh"
 
@@ -48,7 +50,14 @@
 #error "compile with -DMRUN_HEAD_DIM=<head size>"
 #endif
 
-#if MRUN_HEAD_DIM % 64 == 0 && MRUN_HEAD_DIM <= 128
+#ifndef MRUN_VALUE_DIM
+#define MRUN_VALUE_DIM MRUN_HEAD_DIM
+#endif
+#ifndef MRUN_SCORED
+#define MRUN_SCORED 0
+#endif
+
+#if MRUN_HEAD_DIM % 64 == 0 && MRUN_HEAD_DIM <= 128 && MRUN_VALUE_DIM % 64 == 0 && MRUN_VALUE_DIM <= 128
 #define MRUN_ATTN_TC5 1
 #else
 #define MRUN_ATTN_TC5 0
@@ -61,20 +70,22 @@ namespace {
 using bf16 = __nv_bfloat16;
 using namespace tc5;
 
-constexpr int D = MRUN_HEAD_DIM;
+constexpr int D = MRUN_HEAD_DIM, DV = MRUN_VALUE_DIM;
+constexpr bool SCORED = MRUN_SCORED;
 constexpr int ROWS = 128;                    // query rows per block = MMA M
 constexpr int KEYS = 128;                    // keys per tile = N of the first product, K of the second
-constexpr int SPANS_D = D / 64;              // 64-wide spans of the head dimension
+constexpr int SPANS_D = D / 64, SPANS_V = DV / 64;      // 64-wide spans of the head dimensions
 constexpr int SPAN_BYTES = 128 * 128;        // one swizzled tile of 128 rows x 64 bf16
-constexpr int KV_BYTES = SPANS_D * SPAN_BYTES;          // one stage of K (or V): 128 keys x D
+constexpr int K_BYTES = SPANS_D * SPAN_BYTES;           // one stage of K: 128 keys x D
+constexpr int V_BYTES = SPANS_V * SPAN_BYTES;           // one stage of V: 128 keys x DV
 constexpr int Q_BYTES = SPANS_D * SPAN_BYTES;
-constexpr int SMEM_BYTES = Q_BYTES + 4 * KV_BYTES + 1024;                // Q, two stages of K and of V
+constexpr int SMEM_BYTES = Q_BYTES + 2 * K_BYTES + 2 * V_BYTES + 1024;                // Q, two stages of K and of V
 constexpr int SOFTMAX_WARPS = 8, SOFTMAX_THREADS = SOFTMAX_WARPS * 32;
 constexpr int MMA_WARP = 8, K_WARP = 9, V_WARP = 10;
 constexpr int THREADS = SOFTMAX_THREADS + 3 * 32;                        // 352
-constexpr unsigned TMEM_COLS = 512;          // S0 [0,128) S1 [128,256) P0 [256,320) P1 [320,384) O [384, 384 + D)
+constexpr unsigned TMEM_COLS = 512;          // S0 [0,128) S1 [128,256) P0 [256,320) P1 [320,384) O [384, 384 + DV)
 constexpr unsigned P_COL = 256, O_COL = 384;
-constexpr int O_HALF = D / 2;                // columns of O a thread of a pair looks after
+constexpr int O_HALF = DV / 2;                // columns of O a thread of a pair looks after
 constexpr float LOG2E = 1.4426950408889634f;
 constexpr float RESCALE_STEP = 8.f;          // log2 of the growth of a row maximum that forces a rescale
 constexpr long long WAIT_CYCLES = 3000000000LL;         // about 1.5 s at 2 GHz
@@ -117,12 +128,12 @@ prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_const
                    const int* __restrict__ block_tables, int max_blocks, const int* __restrict__ token_slot,
                    const int* __restrict__ positions, const int* __restrict__ tile_tok0,
                    const int* __restrict__ tile_ntok, int heads, int kv_heads, int page_size, int page_shift,
-                   float scale_log2, int window, float sink_log2, int* __restrict__ status) {
+                   float scale_log2, int window, float sink_log2, const mrun_score_form form, int* __restrict__ status) {
     extern __shared__ __align__(1024) unsigned char smem_raw[];
     unsigned char* base = reinterpret_cast<unsigned char*>(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
     unsigned char* q_tile = base;
     unsigned char* k_stages = q_tile + Q_BYTES;
-    unsigned char* v_stages = k_stages + 2 * KV_BYTES;
+    unsigned char* v_stages = k_stages + 2 * K_BYTES;
     __shared__ Barriers bars;
     __shared__ unsigned tmem_base_slot;
     __shared__ int aborted;
@@ -158,7 +169,7 @@ prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_const
         mbar_init_fence();
     }
     // rows of a V stage that no copy ever fills must not hold NaN patterns: 0 * NaN is NaN
-    for (int i = threadIdx.x; i < 2 * KV_BYTES / 16; i += THREADS)
+    for (int i = threadIdx.x; i < 2 * V_BYTES / 16; i += THREADS)
         reinterpret_cast<uint4*>(v_stages)[i] = make_uint4(0, 0, 0, 0);
     fence_async_smem();
     __syncwarp();
@@ -192,6 +203,8 @@ prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_const
         const int row_lo = mrun::first_visible(row_pos, window);
         // the tile's last row sees the most recent keys, its first row the oldest
         const int lo_last = mrun::first_visible(pos_last, window);
+        mrun::ScoreRow form_row = {};
+        if constexpr (SCORED) form_row = mrun::score_row(form, scale_log2 / LOG2E, row_pos, kvh * group + min(row, n_rows - 1) % group);
         float m_used = -INFINITY, l = 0.f;                           // l: this half's share of the row's sum
         bool alive = true;
         // A warp that gave up on a wait still walks through the remaining tiles, doing nothing but
@@ -225,6 +238,32 @@ prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_const
                     pin(raw[i]);
                     sc[i] = __uint_as_float(raw[i]);
                 }
+                if constexpr (SCORED) {
+                    // scores in base-2 units from here on: two a step where the polynomial serves (every
+                    // row of the warp alike), then the bias, an entry a distance only near the query
+                    if (__all_sync(0xffffffffu, form_row.small)) {
+                        const float2 factor2 = make_float2(form_row.factor, form_row.factor);
+                        const float2 cap2 = make_float2(form_row.cap2, form_row.cap2);
+                        const float2 far2 = make_float2(form_row.far_bias, form_row.far_bias);
+#pragma unroll
+                        for (int i = 0; i < 64; i += 2) {
+                            const float2 th = mrun::tanh_small2(__fmul2_rn(make_float2(sc[i], sc[i + 1]), factor2));
+                            const float2 v = __ffma2_rn(th, cap2, far2);
+                            sc[i] = v.x; sc[i + 1] = v.y;
+                        }
+                    } else {
+#pragma unroll
+                        for (int i = 0; i < 64; ++i) sc[i] = mrun::capped_score(form_row, sc[i]) + form_row.far_bias;
+                    }
+                    if (form.bias != nullptr && pos_first - (key_base + 63) < form.bias_len - 1) {
+                        // every entry as its difference from the far one, which the scores hold already
+                        const float* table = form_row.bias;
+                        const int distance = row_pos - key_base;
+#pragma unroll
+                        for (int i = 0; i < 64; ++i)
+                            sc[i] += fmaf(__ldg(table + min(max(distance - i, 0), form_row.bias_last)), LOG2E, -form_row.far_bias);
+                    }
+                }
                 // the largest raw score first (the scale is positive, so it scales the maximum
                 // alike); masked scores become -inf and later give p = 0
                 if (need_mask) {
@@ -248,7 +287,8 @@ prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_const
             pair_max[buf][half][row] = mx;
             pair_sync(quarter);
             if (!alive) continue;
-            mx = fmaxf(mx, pair_max[buf][half ^ 1][row]) * scale_log2;
+            mx = fmaxf(mx, pair_max[buf][half ^ 1][row]);
+            if constexpr (!SCORED) mx *= scale_log2;
             // the maximum the probabilities are taken against moves only by large steps; both
             // halves of a row decide alike, from the same numbers
             float m_new = m_used;
@@ -279,7 +319,8 @@ prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_const
             const float m_sub = m_used == -INFINITY ? 0.f : -m_used;
             // Two scores an instruction where the hardware has one (fma.f32x2, add.f32x2): these
             // warps are bound by the instructions they issue.
-            const float2 scale2 = make_float2(scale_log2, scale_log2), m_sub2 = make_float2(m_sub, m_sub);
+            const float unit = SCORED ? 1.f : scale_log2;
+            const float2 scale2 = make_float2(unit, unit), m_sub2 = make_float2(m_sub, m_sub);
             float2 sums = make_float2(0.f, 0.f);
             float packed[32];                                         // two bf16 a word, even key low
 #pragma unroll
@@ -313,19 +354,21 @@ prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_const
             tc_fence_after();
             const float total = with_sink(l + pair_sum[half ^ 1][row], m_used, sink_log2);
             const float inv = total > 0.f ? 1.f / total : 0.f;
-            bf16* dst = out + ((size_t)(tok0 + row / group) * heads + kvh * group + row % group) * D + half * O_HALF;
+            const int col = (kvh * group + row % group) * DV + half * O_HALF;
+            bf16* dst = out + (size_t)(tok0 + row / group) * (SCORED ? form.out_stride : (long)heads * DV) + col;
 #pragma unroll 1
             for (int c = 0; c < O_HALF; c += 32) {
                 float v[32];
                 tmem_load32(lane_base + O_COL + half * O_HALF + c, v);       // every lane of the warp takes part
                 if (row < n_rows) {
 #pragma unroll
+                    for (int i = 0; i < 32; ++i) v[i] *= inv;
+                    if constexpr (SCORED) mrun::gate_outputs<32>(form, tok0 + row / group, col + c, v);
+#pragma unroll
                     for (int k = 0; k < 4; ++k)
                         *reinterpret_cast<uint4*>(dst + c + 8 * k) =
-                            make_uint4(pack_bf16(v[8 * k] * inv, v[8 * k + 1] * inv),
-                                       pack_bf16(v[8 * k + 2] * inv, v[8 * k + 3] * inv),
-                                       pack_bf16(v[8 * k + 4] * inv, v[8 * k + 5] * inv),
-                                       pack_bf16(v[8 * k + 6] * inv, v[8 * k + 7] * inv));
+                            make_uint4(pack_bf16(v[8 * k], v[8 * k + 1]), pack_bf16(v[8 * k + 2], v[8 * k + 3]),
+                                       pack_bf16(v[8 * k + 4], v[8 * k + 5]), pack_bf16(v[8 * k + 6], v[8 * k + 7]));
                 }
             }
         }
@@ -333,10 +376,10 @@ prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_const
         // ---------------------------------------------------------------------------- MMA issuer
         if (lane == 0) {
             constexpr unsigned idesc_qk = instruction_descriptor(ROWS, KEYS);
-            constexpr unsigned idesc_pv = instruction_descriptor(ROWS, D, true);
+            constexpr unsigned idesc_pv = instruction_descriptor(ROWS, DV, true);
             // The operand descriptors of stage 0, made once: this warp shares its scheduler with
             // two softmax warps, so every instruction it spends between two products delays them.
-            // Stage 1 lies KV_BYTES further (the address field counts 16-byte units).
+            // Stage 1 lies K_BYTES (V_BYTES) further (the address field counts 16-byte units).
             unsigned long long q_desc[D / 16], k_desc[D / 16], v_desc[KEYS / 16];
 #pragma unroll
             for (int kk = 0; kk < D / 16; ++kk) {
@@ -347,14 +390,14 @@ prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_const
 #pragma unroll
             for (int kk = 0; kk < KEYS / 16; ++kk)                            // sixteen rows (two groups) further per step
                 v_desc[kk] = smem_descriptor(v_stages + kk * 2048, SPAN_BYTES, 1024);
-            constexpr unsigned long long STAGE_STEP = KV_BYTES >> 4;
+            constexpr unsigned long long K_STEP = K_BYTES >> 4, V_STEP = V_BYTES >> 4;
             bool alive = mbar_wait(&bars.q_full, 0, WAIT_CYCLES, &aborted);
             auto issue_qk = [&](int j) -> bool {
                 const int s = j & 1;
                 if (!mbar_wait(&bars.k_full[s], (j >> 1) & 1, WAIT_CYCLES, &aborted)) return false;
                 if (j >= 2 && !mbar_wait(&bars.s_empty[s], ((j >> 1) - 1) & 1, WAIT_CYCLES, &aborted)) return false;
                 tc_fence_after();
-                const unsigned long long step = s * STAGE_STEP;
+                const unsigned long long step = s * K_STEP;
 #pragma unroll
                 for (int kk = 0; kk < D / 16; ++kk)
                     umma_bf16(tmem_base + s * KEYS, q_desc[kk], k_desc[kk] + step, idesc_qk, kk > 0 ? 1u : 0u);
@@ -370,7 +413,7 @@ prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_const
                 if (!mbar_wait(&bars.v_full[s], (j >> 1) & 1, WAIT_CYCLES, &aborted)) { alive = false; break; }
                 if (!mbar_wait(&bars.p_full[s], (j >> 1) & 1, WAIT_CYCLES, &aborted)) { alive = false; break; }
                 tc_fence_after();
-                const unsigned long long step = s * STAGE_STEP;
+                const unsigned long long step = s * V_STEP;
 #pragma unroll
                 for (int kk = 0; kk < KEYS / 16; ++kk)                        // P: eight columns (16 keys) further per step
                     umma_bf16_a_tmem(tmem_base + O_COL, tmem_base + P_COL + s * 64 + kk * 8, v_desc[kk] + step, idesc_pv,
@@ -401,13 +444,13 @@ prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_const
             const bool free_now = j < 2 || mbar_wait(&empty[s], ((j >> 1) - 1) & 1, WAIT_CYCLES, &aborted);
             if (!__all_sync(0xffffffffu, free_now)) { alive = false; break; }
             const int key0 = (first_block + j) * KEYS;
-            unsigned char* stage = stages + s * KV_BYTES;
+            unsigned char* stage = stages + s * (keys_role ? K_BYTES : V_BYTES);
             // a lane's boxes: lane, lane + 32, ...  It announces their bytes, then copies them.
             unsigned bytes = 0;
             for (int b = lane; b < boxes; b += 32) {
                 const int first_key = key0 + b * box_rows;
                 if (first_key <= pos_last && first_key + box_rows - 1 >= lo_tile && table[first_key >> page_shift] >= 0)
-                    bytes += (unsigned)(box_rows * D * 2);
+                    bytes += (unsigned)(box_rows * (keys_role ? D : DV) * 2);
             }
             if (bytes) mbar_expect_tx(&full[s], bytes);
             else mbar_arrive(&full[s]);
@@ -417,8 +460,9 @@ prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_const
                 const int page = table[first_key >> page_shift];
                 if (page < 0) continue;
 #pragma unroll
-                for (int h = 0; h < SPANS_D; ++h)
-                    tma_load_4d(stage + h * SPAN_BYTES + b * box_rows * 128, map, h * 64,
+                for (int h = 0; h < (SPANS_D > SPANS_V ? SPANS_D : SPANS_V); ++h)
+                    if (h < (keys_role ? SPANS_D : SPANS_V))
+                        tma_load_4d(stage + h * SPAN_BYTES + b * box_rows * 128, map, h * 64,
                                 first_key & (page_size - 1), kvh, page, &full[s]);
             }
         }
@@ -457,8 +501,8 @@ MRUN_API int mrun_attn_prefill_tc5(const void* q, long q_stride, void* out, cons
                                    const void* v_cache, const int* block_tables, int max_blocks,
                                    const int* token_slot, const int* positions, const int* tile_tok0,
                                    const int* tile_ntok, int n_tiles, int heads, int kv_heads, int head_dim,
-                                   int page_size, float scale, int window, float sink, long pages, int* status,
-                                   cudaStream_t stream) {
+                                   int page_size, float scale, int window, float sink, long pages,
+                                   const mrun_score_form* form, int* status, cudaStream_t stream) {
 #if MRUN_ATTN_TC5
     MRUN_REQUIRE(head_dim == D, "attn_prefill_tc5: this library was built for head_dim=%d, got %d", D, head_dim);
     MRUN_REQUIRE(heads > 0 && kv_heads > 0 && heads % kv_heads == 0,
@@ -470,6 +514,13 @@ MRUN_API int mrun_attn_prefill_tc5(const void* q, long q_stride, void* out, cons
     MRUN_REQUIRE(q_stride % 8 == 0 && ((uintptr_t)q & 15) == 0 && ((uintptr_t)out & 15) == 0 &&
                  ((uintptr_t)k_cache & 15) == 0 && ((uintptr_t)v_cache & 15) == 0,
                  "attn_prefill_tc5: q, out and the caches must be 16-byte aligned, q_stride a multiple of 8");
+    MRUN_REQUIRE(SCORED == (form != nullptr), "attn_prefill_tc5: this library was built %s a score form",
+                 SCORED ? "for" : "without");
+    if (form)
+        MRUN_REQUIRE(form->out_stride >= (long)heads * DV && form->out_stride % 8 == 0 &&
+                     (form->gate == nullptr || (form->gate_stride >= (long)heads * DV && form->gate_stride % 8 == 0 &&
+                                                ((uintptr_t)form->gate & 15) == 0)),
+                     "attn_prefill_tc5: the output's and the gate's rows must start on 16 bytes and hold %d features", heads * DV);
     MRUN_REQUIRE(status != nullptr, "attn_prefill_tc5: the status word is missing");
     MRUN_REQUIRE(page_shift_of(page_size) >= 0, "attn_prefill_tc5: page_size=%d is not a power of two", page_size);
     MRUN_REQUIRE(pages > 0 && pages < (1L << 31), "attn_prefill_tc5: pages=%ld", pages);
@@ -477,7 +528,7 @@ MRUN_API int mrun_attn_prefill_tc5(const void* q, long q_stride, void* out, cons
     CUtensorMap map_k, map_v;
     const int box_rows = page_size < KEYS ? page_size : KEYS;
     if (int rc = paged_cache_map(&map_k, k_cache, pages, kv_heads, page_size, D, box_rows, "attn_prefill_tc5")) return rc;
-    if (int rc = paged_cache_map(&map_v, v_cache, pages, kv_heads, page_size, D, box_rows, "attn_prefill_tc5")) return rc;
+    if (int rc = paged_cache_map(&map_v, v_cache, pages, kv_heads, page_size, DV, box_rows, "attn_prefill_tc5")) return rc;
     static bool configured = false;
     if (!configured) {
         MRUN_CHECK_CUDA(cudaFuncSetAttribute(prefill_tc5_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize,
@@ -489,7 +540,7 @@ MRUN_API int mrun_attn_prefill_tc5(const void* q, long q_stride, void* out, cons
         prefill_tc5_kernel<<<dim3(kv_heads, now), THREADS, SMEM_BYTES, stream>>>(
             map_k, map_v, (const bf16*)q, q_stride, (bf16*)out, block_tables, max_blocks,
             token_slot, positions, tile_tok0 + done, tile_ntok + done, heads, kv_heads, page_size, page_shift_of(page_size),
-            scale * LOG2E, window, sink * LOG2E, status);
+            scale * LOG2E, window, sink * LOG2E, form ? *form : mrun_score_form{}, status);
         MRUN_CHECK_LAUNCH("attn_prefill_tc5");
     }
     return 0;

@@ -15,6 +15,8 @@
 enum : int { MRUN_F32 = 0, MRUN_BF16 = 1 };
 // gate functions of a gated feed-forward (0 = the product has no gated epilogue)
 enum : int { MRUN_GATE_NONE = 0, MRUN_GATE_SILU = 1, MRUN_GATE_GELU_TANH = 2 };
+// functions of one argument (0 = none)
+enum : int { MRUN_ACT_NONE = 0, MRUN_ACT_RELU2 = 1, MRUN_ACT_TANH = 2 };
 #define MRUN_REQUIRE_GATE(act, name) \
     MRUN_REQUIRE((act) == MRUN_GATE_SILU || (act) == MRUN_GATE_GELU_TANH, "%s: unknown gate function code %d", name, act)
 
@@ -192,6 +194,15 @@ __device__ __forceinline__ float gated_mul(int act, float gate, float up) {
     }
     if constexpr (EXACT) return gate / (1.f + expf(-gate)) * up;
     else return __fdividef(gate, 1.f + __expf(-gate)) * up;
+}
+
+// A function of one argument, named by a code of the C ABI, in 32-bit.
+__device__ __forceinline__ float plain_act(int act, float v) {
+    if (act == MRUN_ACT_RELU2) {
+        v = fmaxf(v, 0.f);
+        return v * v;
+    }
+    return act == MRUN_ACT_TANH ? tanhf(v) : v;
 }
 
 }  // namespace mrun

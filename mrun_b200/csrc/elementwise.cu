@@ -973,3 +973,32 @@ MRUN_API int mrun_head_norm_rope_cache(void* x, long ld, long q_off, long k_off,
     MRUN_CHECK_LAUNCH("head_norm_rope_cache");
     return 0;
 }
+
+// ------------------------------------------------------------------------------------------
+// out[i] = act(x[i]) in 32-bit, a function of one argument (MRUN_ACT_*); x and out may differ in type.
+// ------------------------------------------------------------------------------------------
+template <typename TX, typename TA>
+__global__ void __launch_bounds__(256)
+plain_act_kernel(const TX* __restrict__ x, TA* __restrict__ out, long n, int act) {
+    const long i = (long)blockIdx.x * 256 + threadIdx.x;
+    if (i < n) out[i] = from_float<TA>(plain_act(act, to_float(x[i])));
+}
+
+MRUN_API int mrun_plain_act(const void* x, int x_dtype, void* out, int out_dtype, long n, int act, cudaStream_t stream) {
+    MRUN_REQUIRE(n >= 0 && (act == MRUN_ACT_RELU2 || act == MRUN_ACT_TANH), "plain_act: n=%ld, activation code %d", n, act);
+    MRUN_REQUIRE(x_dtype == MRUN_F32 || x_dtype == MRUN_BF16, "plain_act: unknown dtype code %d", x_dtype);
+    MRUN_REQUIRE(out_dtype == MRUN_F32 || out_dtype == MRUN_BF16, "plain_act: unknown dtype code %d", out_dtype);
+    if (n == 0) return 0;
+    const unsigned blocks = (unsigned)((n + 255) / 256);
+    if (x_dtype == MRUN_F32 && out_dtype == MRUN_F32)
+        plain_act_kernel<float, float><<<blocks, 256, 0, stream>>>((const float*)x, (float*)out, n, act);
+    else if (x_dtype == MRUN_F32)
+        plain_act_kernel<float, __nv_bfloat16><<<blocks, 256, 0, stream>>>((const float*)x, (__nv_bfloat16*)out, n, act);
+    else if (out_dtype == MRUN_F32)
+        plain_act_kernel<__nv_bfloat16, float><<<blocks, 256, 0, stream>>>((const __nv_bfloat16*)x, (float*)out, n, act);
+    else
+        plain_act_kernel<__nv_bfloat16, __nv_bfloat16><<<blocks, 256, 0, stream>>>((const __nv_bfloat16*)x,
+                                                                                   (__nv_bfloat16*)out, n, act);
+    MRUN_CHECK_LAUNCH("plain_act");
+    return 0;
+}

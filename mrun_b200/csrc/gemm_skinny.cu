@@ -45,7 +45,9 @@ constexpr float SUMS_SCALE = 1073741824.f, SUMS_UNIT = 1.f / 1073741824.f;
 
 // What a launch does beside the product itself.
 struct Fusion {
-    int act;                     // EPI_GATED: the gate's function (MRUN_GATE_*)
+    int act;                     // EPI_GATED: the gate's function (MRUN_GATE_*); EPI_PLAIN: MRUN_ACT_* or 0
+    // a batch of products in one launch (blockIdx.y): W matrices one after the other, x and y this far apart
+    long batch_x, batch_y;
     // x is the xw of a product before: the row's scale is rsqrt(in_sums[row] * 2^-30 / width + eps)
     const unsigned long long* in_sums;   // [16] totals of squares, or null: x is taken as it is
     float in_eps, in_inv_width;
@@ -94,6 +96,11 @@ skinny_kernel(const bf16* __restrict__ x, const bf16* __restrict__ w, TOut* __re
     const int rows = CUT ? rows_cut : MT * 16;
     const int n0 = blockIdx.x * rows;
     const int chunks = K >> 5;          // whole 32-wide chunks; K % 32 == 0 is checked by the host
+    if (EPI == EPI_PLAIN) {
+        w += (size_t)blockIdx.y * N * K;
+        x += blockIdx.y * f.batch_x;
+        y += blockIdx.y * f.batch_y;
+    }
 
     const bf16* w_rows[MT][2];
 #pragma unroll
@@ -229,7 +236,10 @@ skinny_kernel(const bf16* __restrict__ x, const bf16* __restrict__ w, TOut* __re
                 float s = 0.f;
 #pragma unroll
                 for (int wi = 0; wi < WARPS; ++wi) s += red[wi][row][token];
-                store_out<TOut>(y + (size_t)token * ldy + n0 + row, s * row_scale[token]);
+                s *= row_scale[token];
+                // an activation sees the sum as the layer would have stored it
+                if (f.act) s = mrun::plain_act(f.act, __bfloat162float(__float2bfloat16_rn(s)));
+                store_out<TOut>(y + (size_t)token * ldy + n0 + row, s);
             }
         }
     } else if constexpr (EPI == EPI_GATED) {
@@ -301,16 +311,16 @@ int rows_a_block(int N, int places, int forced) {
 
 template <int NT, int MT, int UNROLL, typename TOut, int EPI>
 void launch(const bf16* x, const bf16* w, TOut* y, int M, int N, int K, long ldx, long ldy, const Fusion& f,
-            int forced_rows, cudaStream_t stream) {
+            int forced_rows, int batch, cudaStream_t stream) {
     if constexpr (MT == 1 && EPI != EPI_GATED) {     // the gated epilogue pairs rows inside whole runs of 16
-        const int rows = rows_a_block(N, sm_count() * resident_blocks(NT, MT, UNROLL), forced_rows);
+        const int rows = rows_a_block(N * batch, sm_count() * resident_blocks(NT, MT, UNROLL), forced_rows);
         if (rows < 16) {
-            mrun::launch_kernel_overlapped(skinny_kernel<NT, MT, UNROLL, TOut, EPI, true>, dim3((N + rows - 1) / rows),
+            mrun::launch_kernel_overlapped(skinny_kernel<NT, MT, UNROLL, TOut, EPI, true>, dim3((N + rows - 1) / rows, batch),
                                            dim3(THREADS), 0, stream, x, w, y, M, N, K, ldx, ldy, f, rows);
             return;
         }
     }
-    mrun::launch_kernel_overlapped(skinny_kernel<NT, MT, UNROLL, TOut, EPI, false>, dim3((N + MT * 16 - 1) / (MT * 16)),
+    mrun::launch_kernel_overlapped(skinny_kernel<NT, MT, UNROLL, TOut, EPI, false>, dim3((N + MT * 16 - 1) / (MT * 16), batch),
                                    dim3(THREADS), 0, stream, x, w, y, M, N, K, ldx, ldy, f, MT * 16);
 }
 
@@ -327,24 +337,24 @@ int sm_count() {
 
 template <typename TOut, int EPI>
 void dispatch(const bf16* x, const bf16* w, TOut* y, int M, int N, int K, long ldx, long ldy, const Fusion& f,
-              int rows, cudaStream_t stream) {
+              int rows, int batch, cudaStream_t stream) {
     const int sms = sm_count();
-    const bool two_rounds = (N + 15) / 16 > 2 * sms;      // more 16-row blocks than two a multiprocessor
+    const bool two_rounds = (long)batch * ((N + 15) / 16) > 2 * sms;      // more 16-row blocks than two a multiprocessor
     if (M <= 8) {
         // With the deep batches two blocks fit on a multiprocessor (registers), with the shallow
         // ones three.  Plenty of blocks: two row tiles a block halve the reads of x.  More than
         // two rounds' worth of 16-row blocks run in one round with the shallow kind; fewer blocks
         // are faster with the deep kind.
         if constexpr (EPI != EPI_RESIDUAL) {
-            if (N >= 32 * sms * 4) return launch<1, 2, UNROLL_SHALLOW, TOut, EPI>(x, w, y, M, N, K, ldx, ldy, f, rows, stream);
+            if ((long)N * batch >= 32 * sms * 4) return launch<1, 2, UNROLL_SHALLOW, TOut, EPI>(x, w, y, M, N, K, ldx, ldy, f, rows, batch, stream);
         }
-        if (two_rounds) launch<1, 1, UNROLL_SHALLOW, TOut, EPI>(x, w, y, M, N, K, ldx, ldy, f, rows, stream);
-        else launch<1, 1, UNROLL_DEEP, TOut, EPI>(x, w, y, M, N, K, ldx, ldy, f, rows, stream);
+        if (two_rounds) launch<1, 1, UNROLL_SHALLOW, TOut, EPI>(x, w, y, M, N, K, ldx, ldy, f, rows, batch, stream);
+        else launch<1, 1, UNROLL_DEEP, TOut, EPI>(x, w, y, M, N, K, ldx, ldy, f, rows, batch, stream);
     } else {
         // 9 to 16 rows of x: every chunk carries twice the x, so one row tile a block, and with
         // more than two rounds' worth of blocks one chunk per batch
-        if (two_rounds) launch<2, 1, 1, TOut, EPI>(x, w, y, M, N, K, ldx, ldy, f, rows, stream);
-        else launch<2, 1, UNROLL_SHALLOW, TOut, EPI>(x, w, y, M, N, K, ldx, ldy, f, rows, stream);
+        if (two_rounds) launch<2, 1, 1, TOut, EPI>(x, w, y, M, N, K, ldx, ldy, f, rows, batch, stream);
+        else launch<2, 1, UNROLL_SHALLOW, TOut, EPI>(x, w, y, M, N, K, ldx, ldy, f, rows, batch, stream);
     }
 }
 
@@ -386,7 +396,7 @@ MRUN_API int mrun_gemm_skinny(const void* x, const void* w, void* y, int out_dty
         f.norm_w = norm_w;
         f.xw_out = (bf16*)xw_out;
         f.out_sums = out_sums;
-        dispatch<bf16, EPI_RESIDUAL>(xp, wp, (bf16*)nullptr, M, N, K, ldx, ldy, f, rows, stream);
+        dispatch<bf16, EPI_RESIDUAL>(xp, wp, (bf16*)nullptr, M, N, K, ldx, ldy, f, rows, 1, stream);
         MRUN_CHECK_LAUNCH("gemm_skinny");
         return 0;
     }
@@ -395,15 +405,44 @@ MRUN_API int mrun_gemm_skinny(const void* x, const void* w, void* y, int out_dty
     MRUN_REQUIRE(ldy >= (gate ? N / 2 : N), "gemm_skinny: ldy=%ld is below the output width", ldy);
     if (M == 0) return 0;
     if (out_dtype == MRUN_BF16) {
-        if (gate) dispatch<bf16, EPI_GATED>(xp, wp, (bf16*)y, M, N, K, ldx, ldy, f, rows, stream);
-        else dispatch<bf16, EPI_PLAIN>(xp, wp, (bf16*)y, M, N, K, ldx, ldy, f, rows, stream);
+        if (gate) dispatch<bf16, EPI_GATED>(xp, wp, (bf16*)y, M, N, K, ldx, ldy, f, rows, 1, stream);
+        else dispatch<bf16, EPI_PLAIN>(xp, wp, (bf16*)y, M, N, K, ldx, ldy, f, rows, 1, stream);
     } else if (out_dtype == MRUN_F32) {
         MRUN_REQUIRE(!gate, "gemm_skinny: the gated epilogue writes bfloat16");
-        dispatch<float, EPI_PLAIN>(xp, wp, (float*)y, M, N, K, ldx, ldy, f, rows, stream);
+        dispatch<float, EPI_PLAIN>(xp, wp, (float*)y, M, N, K, ldx, ldy, f, rows, 1, stream);
     } else {
         return mrun_set_error("gemm_skinny: unknown output dtype code %d", out_dtype);
     }
     MRUN_CHECK_LAUNCH("gemm_skinny");
+    return 0;
+}
+
+// y[b] = act(x[b] · w[b]^T) for `batch` products of one shape in one launch: w dense [batch, N, K], x and y
+// with the given strides between products.  act: MRUN_ACT_* or 0.
+MRUN_API int mrun_gemm_skinny_batched(const void* x, const void* w, void* y, int out_dtype, int act, int batch, int M,
+                                      int N, int K, long ldx, long ldy, long batch_x, long batch_y, cudaStream_t stream) {
+    MRUN_REQUIRE(M >= 0 && N > 0 && K > 0 && batch > 0 && batch <= 65535, "gemm_skinny_batched: bad sizes batch=%d M=%d N=%d K=%d",
+                 batch, M, N, K);
+    MRUN_REQUIRE(M <= 16, "gemm_skinny_batched: M=%d exceeds the 16 rows this kernel takes", M);
+    MRUN_REQUIRE(K % 32 == 0, "gemm_skinny_batched: K=%d is not a multiple of 32", K);
+    MRUN_REQUIRE(ldx >= K && ldx % 8 == 0 && batch_x % 8 == 0 && ldy >= N,
+                 "gemm_skinny_batched: ldx=%ld and the step between products (%ld) must be multiples of 8, ldy=%ld at least N",
+                 ldx, batch_x, ldy);
+    MRUN_REQUIRE(((uintptr_t)x & 15) == 0 && ((uintptr_t)w & 15) == 0, "gemm_skinny_batched: x and W must be 16-byte aligned");
+    MRUN_REQUIRE(act == 0 || act == MRUN_ACT_RELU2 || act == MRUN_ACT_TANH, "gemm_skinny_batched: unknown activation code %d", act);
+    if (M == 0) return 0;
+    Fusion f = {};
+    f.act = act;
+    f.in_inv_width = 1.f / (float)K;
+    f.batch_x = batch_x;
+    f.batch_y = batch_y;
+    if (out_dtype == MRUN_BF16)
+        dispatch<bf16, EPI_PLAIN>((const bf16*)x, (const bf16*)w, (bf16*)y, M, N, K, ldx, ldy, f, 0, batch, stream);
+    else if (out_dtype == MRUN_F32)
+        dispatch<float, EPI_PLAIN>((const bf16*)x, (const bf16*)w, (float*)y, M, N, K, ldx, ldy, f, 0, batch, stream);
+    else
+        return mrun_set_error("gemm_skinny_batched: unknown output dtype code %d", out_dtype);
+    MRUN_CHECK_LAUNCH("gemm_skinny_batched");
     return 0;
 }
 

@@ -18,8 +18,14 @@
 //                   S <- g * S (rows); u = beta (v - S^T k); S <- S + k u^T; o = S^T q
 //   gated_scan      per head, with a decay per key channel g = sigmoid(a + bias)^(1/tau) and q
 //                   times dim^-1/2: S <- g * S (rows) + k v^T; o = S^T q (gated linear attention)
+//   bonus_scan      per head, with a decay per key channel g = exp(-exp(a + bias)) and a bonus u for the
+//                   current token: o = S^T r + (r . (u * k)) v; S <- g * S (rows) + k v^T
+//   ssm_scan        per head, with a step dt = softplus(dt + bias) and a scalar decay exp(-exp(A_h) dt):
+//                   S <- decay S + (dt B) x^T; y = S^T C (B and C shared by the heads of a group)
+//   token_blend     rows h + (h' - h) * mu_s for several mu at once, h' the row of the token before
 //   gated_norm      per group of n outputs: o / sqrt(mean(o^2) + eps) * w * f(gate), f the sigmoid
 //                   or SiLU
+//   skip_gate_norm  per group of n outputs: y = (o + D_h x) * SiLU(z), then y / sqrt(mean(y^2) + eps) * w
 #include "common.cuh"
 
 using namespace mrun;
@@ -39,7 +45,8 @@ template <bool EXACT> __device__ __forceinline__ float silu_f(float z) {
 // block also leaves the new state once it has read the old one.
 template <typename TA>
 __global__ void __launch_bounds__(128)
-causal_conv_kernel(const TA* __restrict__ x, long ldx, const float* __restrict__ w, TA* __restrict__ state,
+causal_conv_kernel(const TA* __restrict__ x, long ldx, const float* __restrict__ w, const float* __restrict__ bias,
+                   TA* __restrict__ state,
                    TA* __restrict__ out, long ldo, const int* __restrict__ seg_q_start,
                    const int* __restrict__ seg_slot, int C, int taps, int residual, int silu) {
     const int c = blockIdx.x * blockDim.x + threadIdx.x;
@@ -59,6 +66,7 @@ causal_conv_kernel(const TA* __restrict__ x, long ldx, const float* __restrict__
             hist[j - 1] = l >= 0 ? to_float(x[(size_t)(q0 + l) * ldx + c]) : to_float(st[(size_t)(l + taps - 1) * C]);
         }
     }
+    const float shift = bias ? bias[c] : 0.f;
     const int end = min(n, l0 + CONV_TILE);
     for (int l = l0; l < end; ++l) {
         const float cur = to_float(x[(size_t)(q0 + l) * ldx + c]);
@@ -66,7 +74,7 @@ causal_conv_kernel(const TA* __restrict__ x, long ldx, const float* __restrict__
 #pragma unroll
         for (int j = MAX_TAPS - 1; j >= 1; --j)          // oldest input first
             if (j < taps) acc = fmaf(wv[j], hist[j - 1], acc);
-        acc = fmaf(wv[0], cur, acc);
+        acc = fmaf(wv[0], cur, acc) + shift;
         float y = residual ? cur + acc : acc;
         if (silu) y = silu_f<true>(y);
         out[(size_t)(q0 + l) * ldo + c] = from_float<TA>(y);
@@ -94,7 +102,8 @@ causal_conv_kernel(const TA* __restrict__ x, long ldx, const float* __restrict__
 // 16-byte loads and stores, four tokens' loads in flight.
 template <typename TA>
 __global__ void __launch_bounds__(128)
-causal_conv_vec_kernel(const TA* __restrict__ x, long ldx, const float* __restrict__ w, TA* __restrict__ state,
+causal_conv_vec_kernel(const TA* __restrict__ x, long ldx, const float* __restrict__ w, const float* __restrict__ bias,
+                       TA* __restrict__ state,
                        TA* __restrict__ out, long ldo, const int* __restrict__ seg_q_start,
                        const int* __restrict__ seg_slot, int C, int taps, int residual, int silu) {
     const int c = (blockIdx.x * blockDim.x + threadIdx.x) * 8;
@@ -119,6 +128,9 @@ causal_conv_vec_kernel(const TA* __restrict__ x, long ldx, const float* __restri
             for (int ch = 0; ch < 8; ++ch) hist[j - 1][ch] = 0.f;
         }
     }
+    float shift[8];
+#pragma unroll
+    for (int ch = 0; ch < 8; ++ch) shift[ch] = bias ? bias[c + ch] : 0.f;
     const int end = min(n, l0 + CONV_TILE);
     for (int lb = l0; lb < end; lb += 4) {
         float cur[4][8];
@@ -135,7 +147,7 @@ causal_conv_vec_kernel(const TA* __restrict__ x, long ldx, const float* __restri
 #pragma unroll
                 for (int j = MAX_TAPS - 1; j >= 1; --j)          // oldest input first
                     if (j < taps) acc = fmaf(wv[ch][j], hist[j - 1][ch], acc);
-                acc = fmaf(wv[ch][0], cur[k][ch], acc);
+                acc = fmaf(wv[ch][0], cur[k][ch], acc) + shift[ch];
                 float v = residual ? cur[k][ch] + acc : acc;
                 if (silu) v = silu_f<true>(v);
                 y[ch] = v;
@@ -170,8 +182,8 @@ causal_conv_vec_kernel(const TA* __restrict__ x, long ldx, const float* __restri
 //
 // scan_prepare (a block a token, nothing sequential): everything a token brings to the recurrence
 // as 32-bit rows: q and k per q/k head (through SiLU, or made unit vectors with q times D^-1/2),
-// v (through SiLU or as it is), and for the delta rule the decays g per head and key channel and
-// the write strengths beta.
+// v (through SiLU or as it is; times the step for the state-space scan), the decays g per head and
+// key channel, and one number a head (the delta rule's write strength beta, the state-space decay).
 //
 // scan (grid: value-column groups x heads x segments, SCAN_WARPS warps a block): a warp's lanes
 // are R row slices x C = 32 / R columns; lane (r, c) owns up to 16 key rows of column c of the
@@ -181,7 +193,12 @@ causal_conv_vec_kernel(const TA* __restrict__ x, long ldx, const float* __restri
 // of the next tokens run under the walk over the present ones); a slice's rows start on a
 // 16-byte boundary, one bank group after the slice before, and are read four at a time.
 // ------------------------------------------------------------------------------------------
-constexpr int SCAN_HEAD_DECAY = 0, SCAN_DELTA = 1, SCAN_GATED = 2;      // which recurrence a scan runs
+// which recurrence a scan runs
+constexpr int SCAN_HEAD_DECAY = 0, SCAN_DELTA = 1, SCAN_GATED = 2, SCAN_BONUS = 3, SCAN_SSM = 4;
+// whether every key row has a decay of its own (else one number a head), and whether a token brings
+// one number a head (the delta rule's write strength, the state-space decay)
+__host__ __device__ constexpr bool row_decays(int mode) { return mode == SCAN_DELTA || mode == SCAN_GATED || mode == SCAN_BONUS; }
+__host__ __device__ constexpr bool head_number(int mode) { return mode == SCAN_DELTA || mode == SCAN_SSM; }
 constexpr int SCAN_WARPS = 4;
 constexpr int SCAN_ROWS = 16;       // key rows a lane holds at most
 
@@ -225,6 +242,7 @@ scan_prepare_kernel(const TA* __restrict__ q, const TA* __restrict__ k, const TA
     for (int e = tid; e < H * V; e += 256) {
         float vv = to_float(v[t * ld + e]);
         if (silu_inputs) vv = silu_f<true>(vv);
+        if (mode == SCAN_SSM) vv *= softplus_f(to_float(b[t * ldb + e / V]) + dt_bias[e / V]);
         vf[t * H * V + e] = vv;
     }
     if (delta) {
@@ -236,6 +254,11 @@ scan_prepare_kernel(const TA* __restrict__ q, const TA* __restrict__ k, const TA
     } else if (mode == SCAN_GATED) {    // sigmoid(z)^(1/tau) = exp(-softplus(-z) / tau)
         for (int e = tid; e < H * D; e += 256)
             gf[t * H * D + e] = expf(-softplus_f(-(a[t * H * D + e] + dt_bias[e])) / tau);
+    } else if (mode == SCAN_BONUS) {
+        for (int e = tid; e < H * D; e += 256) gf[t * H * D + e] = expf(-expf(a[t * H * D + e] + dt_bias[e]));
+    } else if (mode == SCAN_SSM) {
+        for (int e = tid; e < H; e += 256)
+            bf[t * H + e] = expf(-expf(a_log[e]) * softplus_f(to_float(b[t * ldb + e]) + dt_bias[e]));
     }
 }
 
@@ -259,10 +282,10 @@ template <int R, int MODE, bool FULL>
 __global__ void __launch_bounds__(SCAN_WARPS * 32)
 scan_kernel(const float* __restrict__ qf, const float* __restrict__ kf, const float* __restrict__ gf,
             const float* __restrict__ vf, const float* __restrict__ bf, const float* __restrict__ decay,
-            float* __restrict__ state, float* __restrict__ out, const int* __restrict__ seg_q_start,
+            const float* __restrict__ bonus, float* __restrict__ state, float* __restrict__ out, const int* __restrict__ seg_q_start,
             const int* __restrict__ seg_slot, int group, int G, int H, int D, int V, int stage) {
     extern __shared__ __align__(16) float smem[];
-    constexpr bool DELTA = MODE == SCAN_DELTA, DECAYS = MODE != SCAN_HEAD_DECAY;     // DECAYS: a decay per key row
+    constexpr bool DELTA = MODE == SCAN_DELTA, DECAYS = row_decays(MODE);
     constexpr int C = 32 / R, COLS = SCAN_WARPS * C, THREADS = SCAN_WARPS * 32;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int h = blockIdx.y, seg = blockIdx.z;
@@ -283,7 +306,12 @@ scan_kernel(const float* __restrict__ qf, const float* __restrict__ kf, const fl
     float* st = state + (((size_t)seg_slot[seg] * H + h) * D) * V + col;
 #pragma unroll
     for (int i = 0; i < SCAN_ROWS; ++i) S[i] = (live && i < mine) ? st[(size_t)(row0 + i) * V] : 0.f;
-    const float head_decay = DECAYS ? 0.f : decay[h];
+    const float head_decay = MODE == SCAN_HEAD_DECAY ? decay[h] : 0.f;
+    float ur[SCAN_ROWS];
+    if constexpr (MODE == SCAN_BONUS) {
+#pragma unroll
+        for (int i = 0; i < SCAN_ROWS; ++i) ur[i] = i < mine ? bonus[(size_t)h * D + row0 + i] : 0.f;
+    }
 
     auto fetch = [&](int which, int t0) {             // tokens t0 .. of the segment into buffer `which`
         const int m = min(stage, n - t0);
@@ -316,7 +344,7 @@ scan_kernel(const float* __restrict__ qf, const float* __restrict__ kf, const fl
             const int tt = e / COLS, j = e - tt * COLS;
             if (col0 + j < V) copy_async_4(vs + e, vf + ((size_t)(q0 + t0 + tt) * H + h) * V + col0 + j);
         }
-        if constexpr (DELTA)
+        if constexpr (head_number(MODE))
             if (tid < m) copy_async_4(bs + tid, bf + (size_t)(q0 + t0 + tid) * H + h);
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
@@ -368,6 +396,19 @@ scan_kernel(const float* __restrict__ qf, const float* __restrict__ kf, const fl
 #pragma unroll
                 for (int i = 0; i < SCAN_ROWS; ++i)
                     if (FULL || i < mine) { S[i] = fmaf(gr[i], S[i], kr[i] * vv); o[i & 3] = fmaf(S[i], qr[i], o[i & 3]); }
+            } else if constexpr (MODE == SCAN_BONUS) {
+#pragma unroll
+                for (int i = 0; i < SCAN_ROWS; ++i)
+                    if (FULL || i < mine) {
+                        const float write = kr[i] * vv;
+                        o[i & 3] = fmaf(fmaf(ur[i], write, S[i]), qr[i], o[i & 3]);      // the state before this token's write
+                        S[i] = fmaf(gr[i], S[i], write);
+                    }
+            } else if constexpr (MODE == SCAN_SSM) {
+                const float dec = bs[tt];
+#pragma unroll
+                for (int i = 0; i < SCAN_ROWS; ++i)
+                    if (FULL || i < mine) { S[i] = fmaf(dec, S[i], kr[i] * vv); o[i & 3] = fmaf(S[i], qr[i], o[i & 3]); }
             } else {
 #pragma unroll
                 for (int i = 0; i < SCAN_ROWS; ++i)
@@ -386,7 +427,8 @@ scan_kernel(const float* __restrict__ qf, const float* __restrict__ kf, const fl
 template <typename TA>
 __global__ void __launch_bounds__(128)
 gated_norm_kernel(const float* __restrict__ o, const float* __restrict__ w, int w_len, const TA* __restrict__ gate,
-                  long ldg, float eps, TA* __restrict__ out, long pairs, int groups, int n, int gate_silu) {
+                  long ldg, float eps, TA* __restrict__ out, long ldo, float scale, long pairs, int groups, int n,
+                  int gate_silu) {
     const long pair = (long)blockIdx.x * 4 + (threadIdx.x >> 5);
     const int lane = threadIdx.x & 31;
     if (pair >= pairs) return;
@@ -396,21 +438,21 @@ gated_norm_kernel(const float* __restrict__ o, const float* __restrict__ w, int 
     float ss = 0.f;
     for (int i = lane; i < n; i += 32) ss = fmaf(row[i], row[i], ss);
     ss = warp_sum(ss);
-    const float inv = 1.f / sqrtf(ss / (float)n + eps);
+    const float inv = scale / sqrtf(ss / (float)n + eps);
     for (int i = lane; i < n; i += 32) {
         const int c = g * n + i;
         const float gv = to_float(gate[t * ldg + c]);
-        out[(t * groups + g) * n + i] = from_float<TA>(row[i] * inv * w[c % w_len] * ((gate_silu ? gv : 1.f) / (1.f + expf(-gv))));
+        out[t * ldo + c] = from_float<TA>(row[i] * inv * w[c % w_len] * ((gate_silu ? gv : 1.f) / (1.f + expf(-gv))));
     }
 }
 
-// scratch: float32, scan_scratch_floats() of them.
 // A block a (token, group), for groups of many features.  The sums differ from the warp kernel's in
 // their order; which of the two runs depends on the group's size only.
 template <typename TA>
 __global__ void __launch_bounds__(256)
 gated_norm_block_kernel(const float* __restrict__ o, const float* __restrict__ w, int w_len, const TA* __restrict__ gate,
-                        long ldg, float eps, TA* __restrict__ out, int groups, int n, int gate_silu) {
+                        long ldg, float eps, TA* __restrict__ out, long ldo, float scale, int groups, int n,
+                        int gate_silu) {
     __shared__ float scratch[33];
     const long pair = blockIdx.x;
     const long t = pair / groups;
@@ -419,20 +461,151 @@ gated_norm_block_kernel(const float* __restrict__ o, const float* __restrict__ w
     float ss = 0.f;
     for (int i = threadIdx.x; i < n; i += 256) ss = fmaf(row[i], row[i], ss);
     ss = block_sum(ss, scratch);
-    const float inv = 1.f / sqrtf(ss / (float)n + eps);
+    const float inv = scale / sqrtf(ss / (float)n + eps);
     for (int i = threadIdx.x; i < n; i += 256) {
         const int c = g * n + i;
         const float gv = to_float(gate[t * ldg + c]);
-        out[(t * groups + g) * n + i] = from_float<TA>(row[i] * inv * w[c % w_len] * ((gate_silu ? gv : 1.f) / (1.f + expf(-gv))));
+        out[t * ldo + c] = from_float<TA>(row[i] * inv * w[c % w_len] * ((gate_silu ? gv : 1.f) / (1.f + expf(-gv))));
     }
+}
+
+// ------------------------------------------------------------------------------------------
+// out[t, s] = h_t + (h_(t-1) - h_t) * mu_s for S vectors mu: the rows that several projections of a
+// time mixing read.  The row before a segment's first token is the request's state (zeros at the
+// start), and the segment's last row becomes it.  Grid as the convolution's; W channels a thread.
+// ------------------------------------------------------------------------------------------
+template <typename TA, int W>
+__global__ void __launch_bounds__(128)
+token_blend_kernel(const TA* __restrict__ x, long ldx, const float* __restrict__ mu, TA* __restrict__ state,
+                   TA* __restrict__ out, const int* __restrict__ seg_q_start, const int* __restrict__ seg_slot, int C,
+                   int S) {
+    const int c = (blockIdx.x * blockDim.x + threadIdx.x) * W;
+    const int seg = blockIdx.z;
+    const int q0 = seg_q_start[seg], n = seg_q_start[seg + 1] - q0;
+    const int l0 = blockIdx.y * CONV_TILE;
+    if (c >= C || l0 >= n) return;
+    TA* st = state + (size_t)seg_slot[seg] * C + c;
+    auto load = [](const TA* p, float (&v)[W]) {
+        if constexpr (W == 8) Vec8<TA>::load(p, v);
+        else v[0] = to_float(*p);
+    };
+    float before[W], last[W];
+    load(l0 > 0 ? x + (size_t)(q0 + l0 - 1) * ldx + c : st, before);
+    if (blockIdx.y == 0) load(x + (size_t)(q0 + n - 1) * ldx + c, last);
+    const int end = min(n, l0 + CONV_TILE);
+    for (int l = l0; l < end; ++l) {
+        float cur[W];
+        load(x + (size_t)(q0 + l) * ldx + c, cur);
+        for (int s = 0; s < S; ++s) {
+            float m[W], y[W];
+            if constexpr (W == 8) Vec8<float>::load(mu + (size_t)s * C + c, m);
+            else m[0] = mu[(size_t)s * C + c];
+#pragma unroll
+            for (int i = 0; i < W; ++i) y[i] = fmaf(before[i] - cur[i], m[i], cur[i]);
+            TA* dst = out + ((size_t)(q0 + l) * S + s) * C + c;
+            if constexpr (W == 8) Vec8<TA>::store(dst, y);
+            else *dst = from_float<TA>(y[0]);
+        }
+#pragma unroll
+        for (int i = 0; i < W; ++i) before[i] = cur[i];
+    }
+    if (blockIdx.y == 0) {           // the only block of these channels that has read the state
+        if constexpr (W == 8) Vec8<TA>::store(st, last);
+        else *st = from_float<TA>(last[0]);
+    }
+}
+
+// ------------------------------------------------------------------------------------------
+// y = (o + skip_h x) * SiLU(z), then per group of n features y / sqrt(mean(y^2) + eps) * w.
+// LANES threads a (token, group): a warp for groups of up to 1,024 features, a block of 256 beyond.
+// VEC: eight features at a time in 16-byte pieces, kept in registers between the two passes (n at
+// most 32 * LANES); otherwise element by element, y formed anew in the second pass.
+// ------------------------------------------------------------------------------------------
+template <typename TA, int LANES, bool VEC>
+__global__ void __launch_bounds__(LANES == 32 ? 128 : LANES)
+skip_gate_norm_kernel(const float* __restrict__ o, const TA* __restrict__ x, long ldx, const float* __restrict__ skip,
+                      int vdim, const TA* __restrict__ z, long ldz, const float* __restrict__ w, float eps,
+                      TA* __restrict__ out, long pairs, int groups, int n) {
+    __shared__ float scratch[33];
+    const long pair = LANES == 32 ? (long)blockIdx.x * 4 + (threadIdx.x >> 5) : (long)blockIdx.x;
+    const int lane = LANES == 32 ? (threadIdx.x & 31) : threadIdx.x;
+    if (pair >= pairs) return;
+    const long t = pair / groups;
+    const int c0 = (int)(pair - t * groups) * n;
+    const float* orow = o + pair * n;
+    const TA* xrow = x + t * ldx + c0;
+    const TA* zrow = z + t * ldz + c0;
+    TA* dst = out + pair * n;
+    float ss = 0.f;
+    if constexpr (VEC) {
+        float y[4][8];
+        const int chunks = n >> 3;
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const int c = lane + i * LANES;
+            if (c < chunks) {
+                float xv[8], zv[8];
+                Vec8<float>::load(orow + c * 8, y[i]);
+                Vec8<TA>::load(xrow + c * 8, xv);
+                Vec8<TA>::load(zrow + c * 8, zv);
+#pragma unroll
+                for (int e = 0; e < 8; ++e) {
+                    y[i][e] = fmaf(skip[(c0 + c * 8 + e) / vdim], xv[e], y[i][e]) * silu_f<true>(zv[e]);
+                    ss = fmaf(y[i][e], y[i][e], ss);
+                }
+            }
+        }
+        ss = LANES == 32 ? warp_sum(ss) : block_sum(ss, scratch);
+        const float inv = 1.f / sqrtf(ss / (float)n + eps);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const int c = lane + i * LANES;
+            if (c < chunks) {
+                float wv[8];
+                Vec8<float>::load(w + c0 + c * 8, wv);
+#pragma unroll
+                for (int e = 0; e < 8; ++e) wv[e] *= y[i][e] * inv;
+                Vec8<TA>::store(dst + c * 8, wv);
+            }
+        }
+    } else {
+        auto value = [&](int i) {
+            return fmaf(skip[(c0 + i) / vdim], to_float(xrow[i]), orow[i]) * silu_f<true>(to_float(zrow[i]));
+        };
+        for (int i = lane; i < n; i += LANES) {
+            const float y = value(i);
+            ss = fmaf(y, y, ss);
+        }
+        ss = LANES == 32 ? warp_sum(ss) : block_sum(ss, scratch);
+        const float inv = 1.f / sqrtf(ss / (float)n + eps);
+        for (int i = lane; i < n; i += LANES) dst[i] = from_float<TA>(value(i) * inv * w[c0 + i]);
+    }
+}
+
+template <typename TA>
+void launch_skip_gate_norm(const float* o, const void* x, long ldx, const float* skip, int vdim, const void* z, long ldz,
+                           const float* w, float eps, void* out, int tokens, int groups, int n, cudaStream_t stream) {
+    const long pairs = (long)tokens * groups;
+    const bool narrow = n <= 1024;
+    const bool vec = n % 8 == 0 && n <= 8192 && (ldx * sizeof(TA)) % 16 == 0 && (ldz * sizeof(TA)) % 16 == 0 &&
+                     (((uintptr_t)o | (uintptr_t)x | (uintptr_t)z | (uintptr_t)w | (uintptr_t)out) & 15) == 0;
+    const dim3 grid((unsigned)(narrow ? (pairs + 3) / 4 : pairs));
+#define MRUN_SKIP_GATE_NORM(LANES, VEC)                                                                                \
+    skip_gate_norm_kernel<TA, LANES, VEC><<<grid, LANES == 32 ? 128 : LANES, 0, stream>>>(                             \
+        o, (const TA*)x, ldx, skip, vdim, (const TA*)z, ldz, w, eps, (TA*)out, pairs, groups, n)
+    if (narrow && vec) MRUN_SKIP_GATE_NORM(32, true);
+    else if (narrow) MRUN_SKIP_GATE_NORM(32, false);
+    else if (vec) MRUN_SKIP_GATE_NORM(256, true);
+    else MRUN_SKIP_GATE_NORM(256, false);
+#undef MRUN_SKIP_GATE_NORM
 }
 
 template <typename TA, int MODE>
 int launch_scan(const void* q, const void* k, const void* v, long ld, int group, const float* a, const void* b,
-                long ldb, const float* a_log, const float* dt_bias, const float* decay, float* state, float* out,
+                long ldb, const float* a_log, const float* dt_bias, const float* decay, const float* bonus, float* state, float* out,
                 float* scratch, const int* seg_q_start, const int* seg_slot, int segments, int tokens, int H, int D,
                 int V, int silu_inputs, float tau, cudaStream_t stream) {
-    constexpr bool DECAYS = MODE != SCAN_HEAD_DECAY;
+    constexpr bool DECAYS = row_decays(MODE);
     const int G = H / group;
     float* qf = scratch;
     float* kf = qf + (size_t)tokens * G * D;
@@ -454,7 +627,7 @@ int launch_scan(const void* q, const void* k, const void* v, long ld, int group,
             cudaFuncSetAttribute(scan_kernel<SLICES, MODE, WHOLE>, cudaFuncAttributeMaxDynamicSharedMemorySize,    \
                                  (int)smem);                                                                       \
         scan_kernel<SLICES, MODE, WHOLE><<<grid, SCAN_WARPS * 32, smem, stream>>>(                                 \
-            qf, kf, gf, vf, bf, decay, state, out, seg_q_start, seg_slot, group, G, H, D, V, stage);               \
+            qf, kf, gf, vf, bf, decay, bonus, state, out, seg_q_start, seg_slot, group, G, H, D, V, stage);               \
     } while (0)
 #define MRUN_SCAN(SLICES)                                                                                          \
     do {                                                                                                           \
@@ -473,9 +646,9 @@ int launch_scan(const void* q, const void* k, const void* v, long ld, int group,
 
 }  // namespace
 
-// x: row t at x + t * ldx, C channels; w: float32 [C, taps]; state: [slots, taps - 1, C] in the
+// x: row t at x + t * ldx, C channels; w: float32 [C, taps]; bias: float32 [C] or null; state: [slots, taps - 1, C] in the
 // activation dtype; out: row t at out + t * ldo.  seg_q_start: int32 [segments + 1].
-MRUN_API int mrun_causal_conv(const void* x, long ldx, const float* w, void* state, void* out, long ldo, int act_dtype,
+MRUN_API int mrun_causal_conv(const void* x, long ldx, const float* w, const float* bias, void* state, void* out, long ldo, int act_dtype,
                               const int* seg_q_start, const int* seg_slot, int segments, int max_q_len, int C,
                               int taps, int residual, int silu, cudaStream_t stream) {
     MRUN_REQUIRE(C > 0 && segments >= 0 && max_q_len >= 0, "causal_conv: bad sizes");
@@ -491,11 +664,11 @@ MRUN_API int mrun_causal_conv(const void* x, long ldx, const float* w, void* sta
     if (vec) {
         const dim3 vec_grid((C / 8 + 127) / 128, tiles, segments);
         if (act_dtype == MRUN_F32)
-            causal_conv_vec_kernel<float><<<vec_grid, 128, 0, stream>>>((const float*)x, ldx, w, (float*)state, (float*)out,
+            causal_conv_vec_kernel<float><<<vec_grid, 128, 0, stream>>>((const float*)x, ldx, w, bias, (float*)state, (float*)out,
                                                                          ldo, seg_q_start, seg_slot, C, taps, residual, silu);
         else if (act_dtype == MRUN_BF16)
             causal_conv_vec_kernel<__nv_bfloat16><<<vec_grid, 128, 0, stream>>>(
-                (const __nv_bfloat16*)x, ldx, w, (__nv_bfloat16*)state, (__nv_bfloat16*)out, ldo, seg_q_start, seg_slot, C,
+                (const __nv_bfloat16*)x, ldx, w, bias, (__nv_bfloat16*)state, (__nv_bfloat16*)out, ldo, seg_q_start, seg_slot, C,
                 taps, residual, silu);
         else
             return mrun_set_error("causal_conv: unknown dtype code %d", act_dtype);
@@ -504,11 +677,11 @@ MRUN_API int mrun_causal_conv(const void* x, long ldx, const float* w, void* sta
     }
     const dim3 grid((C + 127) / 128, tiles, segments);
     if (act_dtype == MRUN_F32)
-        causal_conv_kernel<float><<<grid, 128, 0, stream>>>((const float*)x, ldx, w, (float*)state, (float*)out, ldo,
+        causal_conv_kernel<float><<<grid, 128, 0, stream>>>((const float*)x, ldx, w, bias, (float*)state, (float*)out, ldo,
                                                              seg_q_start, seg_slot, C, taps, residual, silu);
     else if (act_dtype == MRUN_BF16)
         causal_conv_kernel<__nv_bfloat16><<<grid, 128, 0, stream>>>(
-            (const __nv_bfloat16*)x, ldx, w, (__nv_bfloat16*)state, (__nv_bfloat16*)out, ldo, seg_q_start, seg_slot, C,
+            (const __nv_bfloat16*)x, ldx, w, bias, (__nv_bfloat16*)state, (__nv_bfloat16*)out, ldo, seg_q_start, seg_slot, C,
             taps, residual, silu);
     else
         return mrun_set_error("causal_conv: unknown dtype code %d", act_dtype);
@@ -531,10 +704,10 @@ MRUN_API int mrun_decay_scan(const void* q, const void* k, const void* v, long l
     MRUN_REQUIRE(H <= 65535 && segments <= 65535, "decay_scan: %d heads or %d segments exceed 65535", H, segments);
     if (segments == 0 || tokens == 0) return 0;
     if (act_dtype == MRUN_F32)
-        launch_scan<float, SCAN_HEAD_DECAY>(q, k, v, ld, 1, nullptr, nullptr, 0, nullptr, nullptr, decay, state, out, scratch,
+        launch_scan<float, SCAN_HEAD_DECAY>(q, k, v, ld, 1, nullptr, nullptr, 0, nullptr, nullptr, decay, nullptr, state, out, scratch,
                                             seg_q_start, seg_slot, segments, tokens, H, D, V, silu_inputs, 1.f, stream);
     else if (act_dtype == MRUN_BF16)
-        launch_scan<__nv_bfloat16, SCAN_HEAD_DECAY>(q, k, v, ld, 1, nullptr, nullptr, 0, nullptr, nullptr, decay, state, out,
+        launch_scan<__nv_bfloat16, SCAN_HEAD_DECAY>(q, k, v, ld, 1, nullptr, nullptr, 0, nullptr, nullptr, decay, nullptr, state, out,
                                                     scratch, seg_q_start, seg_slot, segments, tokens, H, D, V, silu_inputs,
                                                     1.f, stream);
     else
@@ -554,10 +727,10 @@ MRUN_API int mrun_delta_scan(const void* q, const void* k, const void* v, long l
     MRUN_REQUIRE(H <= 65535 && segments <= 65535, "delta_scan: %d heads or %d segments exceed 65535", H, segments);
     if (segments == 0 || tokens == 0) return 0;
     if (act_dtype == MRUN_F32)
-        launch_scan<float, SCAN_DELTA>(q, k, v, ld, group, a, b, ldb, a_log, dt_bias, nullptr, state, out, scratch,
+        launch_scan<float, SCAN_DELTA>(q, k, v, ld, group, a, b, ldb, a_log, dt_bias, nullptr, nullptr, state, out, scratch,
                                        seg_q_start, seg_slot, segments, tokens, H, D, V, 0, 1.f, stream);
     else if (act_dtype == MRUN_BF16)
-        launch_scan<__nv_bfloat16, SCAN_DELTA>(q, k, v, ld, group, a, b, ldb, a_log, dt_bias, nullptr, state, out, scratch,
+        launch_scan<__nv_bfloat16, SCAN_DELTA>(q, k, v, ld, group, a, b, ldb, a_log, dt_bias, nullptr, nullptr, state, out, scratch,
                                                seg_q_start, seg_slot, segments, tokens, H, D, V, 0, 1.f, stream);
     else
         return mrun_set_error("delta_scan: unknown dtype code %d", act_dtype);
@@ -576,10 +749,10 @@ MRUN_API int mrun_gated_scan(const void* q, const void* k, const void* v, long l
     MRUN_REQUIRE(H <= 65535 && segments <= 65535, "gated_scan: %d heads or %d segments exceed 65535", H, segments);
     if (segments == 0 || tokens == 0) return 0;
     if (act_dtype == MRUN_F32)
-        launch_scan<float, SCAN_GATED>(q, k, v, ld, 1, a, nullptr, 0, nullptr, bias, nullptr, state, out, scratch,
+        launch_scan<float, SCAN_GATED>(q, k, v, ld, 1, a, nullptr, 0, nullptr, bias, nullptr, nullptr, state, out, scratch,
                                        seg_q_start, seg_slot, segments, tokens, H, D, V, 0, tau, stream);
     else if (act_dtype == MRUN_BF16)
-        launch_scan<__nv_bfloat16, SCAN_GATED>(q, k, v, ld, 1, a, nullptr, 0, nullptr, bias, nullptr, state, out, scratch,
+        launch_scan<__nv_bfloat16, SCAN_GATED>(q, k, v, ld, 1, a, nullptr, 0, nullptr, bias, nullptr, nullptr, state, out, scratch,
                                                seg_q_start, seg_slot, segments, tokens, H, D, V, 0, tau, stream);
     else
         return mrun_set_error("gated_scan: unknown dtype code %d", act_dtype);
@@ -587,23 +760,120 @@ MRUN_API int mrun_gated_scan(const void* q, const void* k, const void* v, long l
     return 0;
 }
 
+// q (the read vector), k, v: [H, D] a row (stride ld); a: float32 [tokens, H * D], bias: float32 [H * D],
+// the decay is exp(-exp(a + bias)); bonus: float32 [H * D].
+MRUN_API int mrun_bonus_scan(const void* q, const void* k, const void* v, long ld, int act_dtype, const float* a,
+                             const float* bias, const float* bonus, float* state, float* out, float* scratch,
+                             const int* seg_q_start, const int* seg_slot, int segments, int tokens, int H, int D, int V,
+                             cudaStream_t stream) {
+    MRUN_REQUIRE(H > 0 && D > 0 && V > 0 && segments >= 0, "bonus_scan: bad sizes");
+    MRUN_REQUIRE(D <= 256, "bonus_scan: key size %d exceeds the supported 256", D);
+    MRUN_REQUIRE(H <= 65535 && segments <= 65535, "bonus_scan: %d heads or %d segments exceed 65535", H, segments);
+    if (segments == 0 || tokens == 0) return 0;
+    if (act_dtype == MRUN_F32)
+        launch_scan<float, SCAN_BONUS>(q, k, v, ld, 1, a, nullptr, 0, nullptr, bias, nullptr, bonus, state, out, scratch,
+                                       seg_q_start, seg_slot, segments, tokens, H, D, V, 0, 1.f, stream);
+    else if (act_dtype == MRUN_BF16)
+        launch_scan<__nv_bfloat16, SCAN_BONUS>(q, k, v, ld, 1, a, nullptr, 0, nullptr, bias, nullptr, bonus, state, out,
+                                               scratch, seg_q_start, seg_slot, segments, tokens, H, D, V, 0, 1.f, stream);
+    else
+        return mrun_set_error("bonus_scan: unknown dtype code %d", act_dtype);
+    MRUN_CHECK_LAUNCH("bonus_scan");
+    return 0;
+}
+
+// c, b: [H / group, N] a row, x: [H, V] a row (stride ld); dt: row t at dt + t * lddt, [H]; dt_bias, a_log:
+// float32 [H].  state: float32 [slots, H, N, V]; out: float32 [tokens, H * V].
+MRUN_API int mrun_ssm_scan(const void* c, const void* b, const void* x, long ld, int act_dtype, int group, const void* dt,
+                           long lddt, const float* dt_bias, const float* a_log, float* state, float* out, float* scratch,
+                           const int* seg_q_start, const int* seg_slot, int segments, int tokens, int H, int N, int V,
+                           cudaStream_t stream) {
+    MRUN_REQUIRE(H > 0 && N > 0 && V > 0 && segments >= 0 && group > 0 && H % group == 0, "ssm_scan: bad sizes");
+    MRUN_REQUIRE(N <= 256, "ssm_scan: state size %d exceeds the supported 256", N);
+    MRUN_REQUIRE(H <= 65535 && segments <= 65535, "ssm_scan: %d heads or %d segments exceed 65535", H, segments);
+    if (segments == 0 || tokens == 0) return 0;
+    if (act_dtype == MRUN_F32)
+        launch_scan<float, SCAN_SSM>(c, b, x, ld, group, nullptr, dt, lddt, a_log, dt_bias, nullptr, nullptr, state, out,
+                                     scratch, seg_q_start, seg_slot, segments, tokens, H, N, V, 0, 1.f, stream);
+    else if (act_dtype == MRUN_BF16)
+        launch_scan<__nv_bfloat16, SCAN_SSM>(c, b, x, ld, group, nullptr, dt, lddt, a_log, dt_bias, nullptr, nullptr,
+                                             state, out, scratch, seg_q_start, seg_slot, segments, tokens, H, N, V, 0, 1.f,
+                                             stream);
+    else
+        return mrun_set_error("ssm_scan: unknown dtype code %d", act_dtype);
+    MRUN_CHECK_LAUNCH("ssm_scan");
+    return 0;
+}
+
+// x: row t at x + t * ldx, C channels; mu: float32 [S, C]; state: [slots, C] in the activation type;
+// out: dense [tokens, S, C].
+MRUN_API int mrun_token_blend(const void* x, long ldx, const float* mu, void* state, void* out, int act_dtype,
+                              const int* seg_q_start, const int* seg_slot, int segments, int max_q_len, int C, int S,
+                              cudaStream_t stream) {
+    MRUN_REQUIRE(C > 0 && S > 0 && segments >= 0 && max_q_len >= 0, "token_blend: bad sizes");
+    MRUN_REQUIRE(ldx >= C, "token_blend: a row stride below the %d channels", C);
+    MRUN_REQUIRE(segments <= 65535, "token_blend: %d segments exceed 65535", segments);
+    MRUN_REQUIRE(act_dtype == MRUN_F32 || act_dtype == MRUN_BF16, "token_blend: unknown dtype code %d", act_dtype);
+    if (segments == 0 || max_q_len == 0) return 0;
+    const int tiles = (max_q_len + CONV_TILE - 1) / CONV_TILE;
+    MRUN_REQUIRE(tiles <= 65535, "token_blend: a segment of %d tokens is too long", max_q_len);
+    const size_t unit = act_dtype == MRUN_F32 ? 4 : 2;
+    const bool vec = C % 8 == 0 && (ldx * unit) % 16 == 0 &&
+                     (((uintptr_t)x | (uintptr_t)out | (uintptr_t)state | (uintptr_t)mu) & 15) == 0;
+    const dim3 grid(((vec ? C / 8 : C) + 127) / 128, tiles, segments);
+#define MRUN_TOKEN_BLEND(TA, W)                                                                                        \
+    token_blend_kernel<TA, W><<<grid, 128, 0, stream>>>((const TA*)x, ldx, mu, (TA*)state, (TA*)out, seg_q_start,      \
+                                                        seg_slot, C, S)
+    if (act_dtype == MRUN_F32) {
+        if (vec) MRUN_TOKEN_BLEND(float, 8);
+        else MRUN_TOKEN_BLEND(float, 1);
+    } else {
+        if (vec) MRUN_TOKEN_BLEND(__nv_bfloat16, 8);
+        else MRUN_TOKEN_BLEND(__nv_bfloat16, 1);
+    }
+#undef MRUN_TOKEN_BLEND
+    MRUN_CHECK_LAUNCH("token_blend");
+    return 0;
+}
+
+// o: float32 [tokens, groups * n]; x, z: rows of groups * n features (strides ldx, ldz); skip: float32, one
+// entry a head of vdim features; w: float32 [groups * n]; out: dense [tokens, groups * n].
+MRUN_API int mrun_skip_gate_norm(const float* o, const void* x, long ldx, const float* skip, int vdim, const void* z,
+                                 long ldz, const float* w, int act_dtype, float eps, void* out, int tokens, int groups,
+                                 int n, cudaStream_t stream) {
+    MRUN_REQUIRE(tokens >= 0 && groups > 0 && n > 0 && vdim > 0 && ((long)groups * n) % vdim == 0,
+                 "skip_gate_norm: bad sizes groups=%d n=%d vdim=%d", groups, n, vdim);
+    MRUN_REQUIRE(ldx >= (long)groups * n && ldz >= (long)groups * n, "skip_gate_norm: a row stride is below the row");
+    if (tokens == 0) return 0;
+    if (act_dtype == MRUN_F32)
+        launch_skip_gate_norm<float>(o, x, ldx, skip, vdim, z, ldz, w, eps, out, tokens, groups, n, stream);
+    else if (act_dtype == MRUN_BF16)
+        launch_skip_gate_norm<__nv_bfloat16>(o, x, ldx, skip, vdim, z, ldz, w, eps, out, tokens, groups, n, stream);
+    else
+        return mrun_set_error("skip_gate_norm: unknown dtype code %d", act_dtype);
+    MRUN_CHECK_LAUNCH("skip_gate_norm");
+    return 0;
+}
+
 // o: float32 [tokens, groups * n]; w: float32 [w_len], element c of a row takes w[c % w_len];
-// gate: row t at gate + t * ldg; out: dense [tokens, groups * n].  gate_silu: the gate passes SiLU
-// instead of the sigmoid.
+// gate: row t at gate + t * ldg; out: row t at out + t * ldo.  gate_silu: the gate passes SiLU
+// instead of the sigmoid.  scale: multiplies every output.
 MRUN_API int mrun_gated_norm(const float* o, const float* w, int w_len, const void* gate, long ldg, int act_dtype,
-                             float eps, void* out, int tokens, int groups, int n, int gate_silu, cudaStream_t stream) {
+                             float eps, void* out, long ldo, float scale, int tokens, int groups, int n, int gate_silu,
+                             cudaStream_t stream) {
     MRUN_REQUIRE(tokens >= 0 && groups > 0 && n > 0 && w_len > 0, "gated_norm: bad sizes");
-    MRUN_REQUIRE(ldg >= (long)groups * n, "gated_norm: the gate's row stride %ld is below the row", ldg);
+    MRUN_REQUIRE(ldg >= (long)groups * n && ldo >= (long)groups * n,
+                 "gated_norm: a row stride (gate %ld, output %ld) is below the row", ldg, ldo);
     if (tokens == 0) return 0;
     const long pairs = (long)tokens * groups;
     const unsigned blocks = (unsigned)((pairs + 3) / 4);
     if (n >= 1024) {            // a block a pair
         if (act_dtype == MRUN_F32)
             gated_norm_block_kernel<float><<<(unsigned)pairs, 256, 0, stream>>>(o, w, w_len, (const float*)gate, ldg, eps,
-                                                                                 (float*)out, groups, n, gate_silu);
+                                                                                 (float*)out, ldo, scale, groups, n, gate_silu);
         else if (act_dtype == MRUN_BF16)
             gated_norm_block_kernel<__nv_bfloat16><<<(unsigned)pairs, 256, 0, stream>>>(
-                o, w, w_len, (const __nv_bfloat16*)gate, ldg, eps, (__nv_bfloat16*)out, groups, n, gate_silu);
+                o, w, w_len, (const __nv_bfloat16*)gate, ldg, eps, (__nv_bfloat16*)out, ldo, scale, groups, n, gate_silu);
         else
             return mrun_set_error("gated_norm: unknown dtype code %d", act_dtype);
         MRUN_CHECK_LAUNCH("gated_norm");
@@ -611,10 +881,10 @@ MRUN_API int mrun_gated_norm(const float* o, const float* w, int w_len, const vo
     }
     if (act_dtype == MRUN_F32)
         gated_norm_kernel<float><<<blocks, 128, 0, stream>>>(o, w, w_len, (const float*)gate, ldg, eps, (float*)out,
-                                                              pairs, groups, n, gate_silu);
+                                                              ldo, scale, pairs, groups, n, gate_silu);
     else if (act_dtype == MRUN_BF16)
         gated_norm_kernel<__nv_bfloat16><<<blocks, 128, 0, stream>>>(o, w, w_len, (const __nv_bfloat16*)gate, ldg, eps,
-                                                                      (__nv_bfloat16*)out, pairs, groups, n, gate_silu);
+                                                                      (__nv_bfloat16*)out, ldo, scale, pairs, groups, n, gate_silu);
     else
         return mrun_set_error("gated_norm: unknown dtype code %d", act_dtype);
     MRUN_CHECK_LAUNCH("gated_norm");

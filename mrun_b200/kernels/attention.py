@@ -22,6 +22,7 @@ from __future__ import annotations
 
 import ctypes
 import math
+from typing import Optional
 
 import numpy as np
 import torch
@@ -33,13 +34,13 @@ from .ops import _c_float, _c_int, _c_long, _ptr, _stream
 COUNTER_CAPACITY = 1 << 16     # (token, kv head) pairs of one decode launch that may be split
 
 _counters = {}                 # device -> int32 zeros, handed to every split launch
-_slots = {}                    # head size -> blocks of the decode kernel resident on the device
+_slots = {}                    # library -> blocks of the decode kernel resident on the device
 
 
-def _decode_slots(head_dim: int, library, tma_group: int = 0) -> int:
+def _decode_slots(library, tma_group: int = 0) -> int:
     """Blocks of the decode kernel that the device holds at once: the cp.async kernel's, or, with
     ``tma_group`` query heads per kv head, the TMA kernel's."""
-    slots = _slots.get((head_dim, tma_group))
+    slots = _slots.get((library.path, tma_group))
     if slots is None:
         if tma_group:
             per_sm = max(1, int(library._dll.mrun_attn_decode_tma_occupancy(_c_int(tma_group))))
@@ -48,7 +49,7 @@ def _decode_slots(head_dim: int, library, tma_group: int = 0) -> int:
             query.restype = ctypes.c_int
             per_sm = max(1, query())
         sms = torch.cuda.get_device_properties(torch.cuda.current_device()).multi_processor_count
-        slots = _slots[(head_dim, tma_group)] = per_sm * sms
+        slots = _slots[(library.path, tma_group)] = per_sm * sms
     return slots
 
 
@@ -56,19 +57,18 @@ TMA_DECODE = True        # False: the cp.async kernel for every decode step (tes
 _tma_decode = {}
 
 
-def decode_uses_tma(library, head_dim: int, ratio: int, page_size: int) -> bool:
+def decode_uses_tma(library, ratio: int, page_size: int) -> bool:
     """Head sizes 64 and 128, pages of a power-of-two size (the kernel copies whole pages by TMA)."""
     if not TMA_DECODE or ratio > 16 or page_size & (page_size - 1):
         return False
-    have = _tma_decode.get(head_dim)
+    have = _tma_decode.get(library.path)
     if have is None:
-        have = _tma_decode[head_dim] = bool(library._dll.mrun_attn_decode_tma_available())
+        have = _tma_decode[library.path] = bool(library._dll.mrun_attn_decode_tma_available())
     return have
 
 
-def decode_slots(head_dim: int, ratio: int, page_size: int) -> int:
-    library = _lib.attention(head_dim)
-    return _decode_slots(head_dim, library, ratio if decode_uses_tma(library, head_dim, ratio, page_size) else 0)
+def decode_slots(library, ratio: int, page_size: int) -> int:
+    return _decode_slots(library, ratio if decode_uses_tma(library, ratio, page_size) else 0)
 
 
 def _split_counters(device: torch.device) -> torch.Tensor:
@@ -84,18 +84,17 @@ CLUSTER_DECODE = True    # False: the planned kernel for every decode step (test
 MAX_CLUSTER = 16
 
 
-def decode_cluster(library, head_dim: int, ratio: int, page_size: int, tokens: int, kv_heads: int,
-                   max_kv_len: int) -> int:
+def decode_cluster(library, ratio: int, page_size: int, tokens: int, kv_heads: int, max_kv_len: int) -> int:
     """Blocks of a thread-block cluster that takes one (token, kv head) pair of a decode step, or
     0 where the planned kernel runs instead.  The cluster kernel takes steps whose pairs fill at
     most half the device (each pair is then cut into as many pieces as fit), groups of up to 8,
     and contexts short enough for its pieces: a cluster has at most 16 blocks, so beyond 32 tiles
     a block (8 where the clusters leave a fifth of the device or more empty) the planned kernel,
     which cuts a pair into up to 32 pieces, spreads a long context further."""
-    if not CLUSTER_DECODE or ratio > 8 or not decode_uses_tma(library, head_dim, ratio, page_size):
+    if not CLUSTER_DECODE or ratio > 8 or not decode_uses_tma(library, ratio, page_size):
         return 0
     pairs = tokens * kv_heads
-    slots = _decode_slots(head_dim, library, ratio)
+    slots = _decode_slots(library, ratio)
     if pairs < 1 or 2 * pairs > slots:
         return 0
     cluster = 1
@@ -111,8 +110,10 @@ def decode_cluster(library, head_dim: int, ratio: int, page_size: int, tokens: i
     return cluster
 
 
-def supports_tensor_cores(dtype: torch.dtype, head_dim: int, group: int) -> bool:
-    return dtype == torch.bfloat16 and head_dim % 16 == 0 and 16 <= head_dim <= 256 and group <= 64
+def supports_tensor_cores(dtype: torch.dtype, head_dim: int, group: int, value_dim: Optional[int] = None) -> bool:
+    """``value_dim``: where it differs from ``head_dim``; only kernels with a score form take that."""
+    sizes = (head_dim,) if value_dim is None else (head_dim, value_dim)
+    return dtype == torch.bfloat16 and group <= 64 and all(n % 16 == 0 and 16 <= n <= 256 for n in sizes)
 
 
 MIN_TILES = 2      # the fewest 64-key tiles a block of the decode kernel takes
@@ -211,6 +212,36 @@ def decode_fuses_input(ctx, dtype: torch.dtype, heads: int, kv_heads: int, head_
     return ctx.all_decode and ratio <= 16 and supports_tensor_cores(dtype, head_dim, ratio)
 
 
+class ScoreForm(ctypes.Structure):
+    """What is done to a score between the product and the softmax and to the output behind it (see
+    ``csrc/attention_score.cuh``, whose ``mrun_score_form`` this mirrors)."""
+
+    _fields_ = [("cap", ctypes.c_float), ("temp_coef", ctypes.c_float), ("temp_every", ctypes.c_float),
+                ("dot_bound", ctypes.c_float), ("bias", ctypes.c_void_p), ("gate", ctypes.c_void_p),
+                ("gate_stride", ctypes.c_long), ("out_stride", ctypes.c_long), ("out_scale", ctypes.c_float),
+                ("bias_len", ctypes.c_int)]
+
+
+def score_form(out: torch.Tensor, soft_cap: Optional[float] = None, temperature=None, bias: Optional[torch.Tensor] = None,
+               gate: Optional[torch.Tensor] = None, out_scale: float = 1.0, dot_bound: float = math.inf) -> ScoreForm:
+    """``out``: the output's rows (may be a column slice of wider ones); ``bias``: float32 [heads,
+    distances], the last entry for every longer distance; ``gate``: rows of ``out``'s width whose
+    sigmoid multiplies it; ``dot_bound``: a bound of |q . k| where one is known (heads of unit
+    root mean square: their size), which lets a kernel choose a cheaper tanh."""
+    coef, every = temperature if temperature is not None else (0.0, 1.0)
+    if bias is not None:
+        ops._check(bias, "bias", torch.float32)
+    gate_stride = 0
+    if gate is not None:
+        gate_stride = ops._strided_rows(gate, "gate")
+        if gate.shape != out.shape or gate.dtype != out.dtype:
+            raise ops.KernelError(f"attention: gate {tuple(gate.shape)} {gate.dtype} vs out {tuple(out.shape)} {out.dtype}")
+    return ScoreForm(cap=soft_cap or 0.0, temp_coef=coef, temp_every=every, dot_bound=dot_bound,
+                     bias=None if bias is None else bias.data_ptr(), gate=None if gate is None else gate.data_ptr(),
+                     gate_stride=gate_stride, out_stride=ops._strided_rows(out, "out"), out_scale=out_scale,
+                     bias_len=0 if bias is None else bias.shape[1])
+
+
 LATENT_WIDE_MAX_SPLITS = 32     # the most blocks one token's keys are dealt to by the kernel for wide latent rows
 
 
@@ -222,7 +253,7 @@ def latent_wide_ok(dtype: torch.dtype, width: int, value_dim: int) -> bool:
 
 def paged_attention(q: torch.Tensor, q_stride: int, out: torch.Tensor, cache, group, ctx,
                     heads: int, scale: float, window: int, raw=None, value_dim: int = 0,
-                    sink: bool = False) -> torch.Tensor:
+                    sink: bool = False, form: Optional[ScoreForm] = None) -> torch.Tensor:
     """``q``: the step's queries (row t at ``q_stride * t``, heads contiguous); ``cache``: the
     schedule entry's pages; ``group``: the step's view of the cache's group.  ``raw``, only where
     :func:`decode_fuses_input` holds: ``(q_weight, k_weight, eps, rot, rotary_dim, slots)`` for a
@@ -231,10 +262,13 @@ def paged_attention(q: torch.Tensor, q_stride: int, out: torch.Tensor, cache, gr
     features the caller reads of the output; rows too wide for the per-head-size kernels then go
     to the kernel for wide latent rows.  ``sink``: one more term of score 0 without a value in
     every softmax's denominator (it enters where a kernel normalises a finished row, after the
-    pieces of split keys have been merged)."""
+    pieces of split keys have been merged).  ``form``: a score form, whose output rows may be a
+    column slice; with it the values may have another size than the keys."""
     pages, kv_heads, page_size, head_dim = cache.k.shape
+    v_dim = cache.v.shape[3] if form is not None else head_dim
+    formed = ctypes.byref(form) if form is not None else _ptr(None)
     ratio = heads // kv_heads
-    if (value_dim and cache.v is cache.k and kv_heads == 1 and window == 0 and raw is None and not sink
+    if (value_dim and cache.v is cache.k and kv_heads == 1 and window == 0 and raw is None and not sink and form is None
             and not supports_tensor_cores(q.dtype, head_dim, ratio) and latent_wide_ok(q.dtype, head_dim, value_dim)):
         ops._check(q, "q", torch.bfloat16, dense=False); ops._check(out, "out", torch.bfloat16)
         # few tokens and long contexts: every token's keys are dealt to several blocks, so that the
@@ -253,10 +287,10 @@ def paged_attention(q: torch.Tensor, q_stride: int, out: torch.Tensor, cache, gr
                          _c_long(pages * page_size), _c_float(scale), _c_int(splits), _ptr(part_o), _ptr(part_ml),
                          _stream())
         return out
-    if not supports_tensor_cores(q.dtype, head_dim, ratio):
+    if not supports_tensor_cores(q.dtype, head_dim, ratio, v_dim):
         return ops.paged_attention_generic(q, q_stride, out, cache.k, cache.v, group.block_tables,
-                                           ctx.token_slot, ctx.positions, heads, scale, window, sink=sink)
-    library = _lib.attention(head_dim)
+                                           ctx.token_slot, ctx.positions, heads, scale, window, sink=sink, form=form)
+    library = _lib.attention(head_dim, v_dim, form is not None)
     tokens = ctx.num_tokens
     common = (_ptr(cache.k), _ptr(cache.v), _ptr(group.block_tables), _c_int(group.max_blocks),
               _ptr(ctx.token_slot), _ptr(ctx.positions))
@@ -270,21 +304,21 @@ def paged_attention(q: torch.Tensor, q_stride: int, out: torch.Tensor, cache, gr
             q_weight, k_weight, eps, rot, rotary_dim, slots = raw
             fused = (_c_int(1), _ptr(q_weight), _ptr(k_weight), _c_float(eps), _ptr(rot), _c_int(rotary_dim),
                      _ptr(slots))
-        cluster = decode_cluster(library, head_dim, ratio, page_size, tokens, kv_heads, ctx.max_kv_len)
+        cluster = decode_cluster(library, ratio, page_size, tokens, kv_heads, ctx.max_kv_len)
         if cluster:
             status = ops.status_word(q.device, "attn_decode_tma", {1: "the TMA producer", 2: "the consumer warps"})
             library.call("mrun_attn_decode_cluster", _ptr(q), _c_long(q_stride), _ptr(out), *common, _c_int(tokens),
-                         _c_int(cluster), *tail[:-1], *fused, _ptr(None), _c_long(pages), _ptr(status), tail[-1])
+                         _c_int(cluster), *tail[:-1], *fused, _ptr(None), _c_long(pages), formed, _ptr(status), tail[-1])
             return out
-        tma = decode_uses_tma(library, head_dim, ratio, page_size)
-        blocks, splits = decode_launch(tokens, kv_heads, decode_slots(head_dim, ratio, page_size))
-        part_o = torch.empty((blocks, 2, 16, head_dim), dtype=torch.float32, device=q.device)
+        tma = decode_uses_tma(library, ratio, page_size)
+        blocks, splits = decode_launch(tokens, kv_heads, decode_slots(library, ratio, page_size))
+        part_o = torch.empty((blocks, 2, 16, v_dim), dtype=torch.float32, device=q.device)
         part_ml = torch.empty((blocks, 2, 16, 2), dtype=torch.float32, device=q.device)
         prefix, assignment = decode_plan(ctx, library, window, kv_heads, blocks, splits)
-        extra = ()
+        extra = (formed,)
         if tma:
             status = ops.status_word(q.device, "attn_decode_tma", {1: "the TMA producer", 2: "the consumer warps"})
-            extra = (_ptr(None), _c_long(pages), _ptr(status))
+            extra = (_ptr(None), _c_long(pages), formed, _ptr(status))
         library.call("mrun_attn_decode_tma" if tma else "mrun_attn_decode", _ptr(q), _c_long(q_stride), _ptr(out),
                      *common, _ptr(prefix), _ptr(assignment), _c_int(tokens), _ptr(part_o), _ptr(part_ml),
                      _ptr(_split_counters(q.device)), _c_int(blocks), *tail[:-1], *fused, *extra, tail[-1])
@@ -296,20 +330,20 @@ def paged_attention(q: torch.Tensor, q_stride: int, out: torch.Tensor, cache, gr
     # The single tokens of a step that also carries prompt portions: the decode kernel over that
     # selection of rows (split keys, every block busy), not one 64-row tile a token and kv head.
     shortest = 0
-    if ratio <= 16 and decode_uses_tma(library, head_dim, ratio, page_size):
+    if ratio <= 16 and decode_uses_tma(library, ratio, page_size):
         rows, row_positions, row_slots, n_single = single_tokens(ctx)
-        cluster = decode_cluster(library, head_dim, ratio, page_size, n_single, kv_heads, ctx.max_kv_len) if n_single else 0
+        cluster = decode_cluster(library, ratio, page_size, n_single, kv_heads, ctx.max_kv_len) if n_single else 0
         if cluster:
             status = ops.status_word(q.device, "attn_decode_tma", {1: "the TMA producer", 2: "the consumer warps"})
             library.call("mrun_attn_decode_cluster", _ptr(q), _c_long(q_stride), _ptr(out), _ptr(cache.k), _ptr(cache.v),
                          _ptr(group.block_tables), _c_int(group.max_blocks), _ptr(row_slots), _ptr(row_positions),
                          _c_int(n_single), _c_int(cluster), *tail[:-1],
                          _c_int(0), _ptr(None), _ptr(None), _c_float(0.0), _ptr(None), _c_int(0), _ptr(None),
-                         _ptr(rows), _c_long(pages), _ptr(status), tail[-1])
+                         _ptr(rows), _c_long(pages), formed, _ptr(status), tail[-1])
             shortest = 1
         elif n_single and n_single * kv_heads <= COUNTER_CAPACITY:
-            blocks, splits = decode_launch(n_single, kv_heads, decode_slots(head_dim, ratio, page_size))
-            part_o = torch.empty((blocks, 2, 16, head_dim), dtype=torch.float32, device=q.device)
+            blocks, splits = decode_launch(n_single, kv_heads, decode_slots(library, ratio, page_size))
+            part_o = torch.empty((blocks, 2, 16, v_dim), dtype=torch.float32, device=q.device)
             part_ml = torch.empty((blocks, 2, 16, 2), dtype=torch.float32, device=q.device)
             prefix, assignment = decode_plan(ctx, library, window, kv_heads, blocks, splits, positions=row_positions)
             status = ops.status_word(q.device, "attn_decode_tma", {1: "the TMA producer", 2: "the consumer warps"})
@@ -318,10 +352,10 @@ def paged_attention(q: torch.Tensor, q_stride: int, out: torch.Tensor, cache, gr
                          _ptr(prefix), _ptr(assignment), _c_int(n_single), _ptr(part_o), _ptr(part_ml),
                          _ptr(_split_counters(q.device)), _c_int(blocks), *tail[:-1],
                          _c_int(0), _ptr(None), _ptr(None), _c_float(0.0), _ptr(None), _c_int(0), _ptr(None),
-                         _ptr(rows), _c_long(pages), _ptr(status), tail[-1])
+                         _ptr(rows), _c_long(pages), formed, _ptr(status), tail[-1])
             shortest = 1
     short_up_to = 1 << 30
-    if prefill_uses_tcgen05(library, head_dim, ratio, page_size):
+    if prefill_uses_tcgen05(library, ratio, page_size):
         # segments with more rows than a 64-row tile go to the 128-row tcgen05 kernel
         short_up_to = (64 // ratio) if ratio <= 64 else 0
         first, count, n_tiles = prefill_tiles(ctx, 128 // ratio, longer_than=max(short_up_to, shortest))
@@ -329,12 +363,12 @@ def paged_attention(q: torch.Tensor, q_stride: int, out: torch.Tensor, cache, gr
             status = ops.status_word(q.device, "attn_prefill_tc5",
                                      {1: "a key/value loader", 2: "the MMA issuer", 3: "the softmax warps"})
             library.call("mrun_attn_prefill_tc5", _ptr(q), _c_long(q_stride), _ptr(out), *common, _ptr(first),
-                         _ptr(count), _c_int(n_tiles), *tail[:-1], _c_long(pages), _ptr(status), tail[-1])
+                         _ptr(count), _c_int(n_tiles), *tail[:-1], _c_long(pages), formed, _ptr(status), tail[-1])
     if short_up_to > shortest:
         first, count, n_tiles = prefill_tiles(ctx, 64 // ratio, longer_than=shortest, up_to=short_up_to)
         if n_tiles:
             library.call("mrun_attn_prefill", _ptr(q), _c_long(q_stride), _ptr(out), *common, _ptr(first),
-                         _ptr(count), _c_int(n_tiles), *tail)
+                         _ptr(count), _c_int(n_tiles), *tail[:-1], formed, tail[-1])
     return out
 
 
@@ -342,11 +376,11 @@ TC5_PREFILL = True       # False: the mma.sync kernel for every prompt portion (
 _tc5_prefill = {}
 
 
-def prefill_uses_tcgen05(library, head_dim: int, ratio: int, page_size: int) -> bool:
+def prefill_uses_tcgen05(library, ratio: int, page_size: int) -> bool:
     """Head sizes 64 and 128, pages of a power-of-two size (the kernel copies whole pages by TMA)."""
     if not TC5_PREFILL or ratio > 128 or page_size & (page_size - 1):
         return False
-    have = _tc5_prefill.get(head_dim)
+    have = _tc5_prefill.get(library.path)
     if have is None:
-        have = _tc5_prefill[head_dim] = bool(library._dll.mrun_attn_prefill_tc5_available())
+        have = _tc5_prefill[library.path] = bool(library._dll.mrun_attn_prefill_tc5_available())
     return have

@@ -194,18 +194,30 @@ def build_core() -> str:
 ATTENTION_SOURCES = ("common.cu", "attention_mma.cu", "attention_decode_tma.cu", "attention_tc5.cu")
 
 
-def build_attention(head_dim: int) -> str:
-    """The tensor-core attention kernels specialised for one head size."""
-    if head_dim % 16 or not 16 <= head_dim <= 256:
-        raise BuildError(f"the tensor-core attention takes head sizes 16, 32, ... 256, not {head_dim}")
-    return build_library(f"mrun_attn_d{head_dim}", ATTENTION_SOURCES, {"MRUN_HEAD_DIM": head_dim})
+def build_attention(head_dim: int, value_dim: Optional[int] = None, scored: bool = False) -> str:
+    """The tensor-core attention kernels specialised for one head size (and, where the values have
+    another, for a value size); ``scored``: with scores worked on before the softmax and a gated
+    output (``csrc/attention_score.cuh``)."""
+    value_dim = head_dim if value_dim is None else value_dim
+    for size in (head_dim, value_dim):
+        if size % 16 or not 16 <= size <= 256:
+            raise BuildError(f"the tensor-core attention takes head sizes 16, 32, ... 256, not {size}")
+    name, defines = f"mrun_attn_d{head_dim}", {"MRUN_HEAD_DIM": head_dim}
+    if value_dim != head_dim:
+        name, defines["MRUN_VALUE_DIM"] = f"{name}v{value_dim}", value_dim
+    if scored:
+        name, defines["MRUN_SCORED"] = f"{name}s", 1
+    return build_library(name, ATTENTION_SOURCES, defines)
 
 
 # head sizes of the configurations this repository measures and tests
 COMMON_HEAD_DIMS = (16, 32, 48, 64, 80, 96, 128, 144, 256)      # the head sizes the tests and the measured shapes use
+# (key size, value size) of the attentions with a score form among them
+COMMON_SCORED_DIMS = ((128, 128), (64, 64), (128, 64), (64, 128), (48, 16), (32, 80), (16, 16))
 
 
 def build_all() -> list[str]:
     """Every library the package loads for the configurations it measures and tests; other head
     sizes are built when a model with them is first run."""
-    return [build_host(), build_core()] + [build_attention(d) for d in COMMON_HEAD_DIMS]
+    return ([build_host(), build_core()] + [build_attention(d) for d in COMMON_HEAD_DIMS]
+            + [build_attention(d, v, scored=True) for d, v in COMMON_SCORED_DIMS])

@@ -56,7 +56,7 @@ def call_count() -> int:
 
 
 _core: Library | None = None
-_attention: Dict[int, Library] = {}
+_attention: Dict[tuple, Library] = {}
 
 
 def core() -> Library:
@@ -71,14 +71,16 @@ def core() -> Library:
     return _core
 
 
-def attention(head_dim: int) -> Library:
-    """The tensor-core attention library for ``head_dim`` (built at first use)."""
-    lib = _attention.get(head_dim)
+def attention(head_dim: int, value_dim: int | None = None, scored: bool = False) -> Library:
+    """The tensor-core attention library for ``head_dim`` (and another ``value_dim``, and with a score
+    form), built at first use."""
+    value_dim = head_dim if value_dim is None else value_dim
+    key = (head_dim, value_dim, bool(scored))
+    lib = _attention.get(key)
     if lib is None:
-        lib = Library(build.build_attention(head_dim))
-        query = lib._dll.mrun_attn_head_dim
-        query.restype = ctypes.c_int
-        if query() != head_dim:
-            raise KernelError(f"{lib.path} was built for head_dim={query()}, not {head_dim}")
-        _attention[head_dim] = lib
+        lib = Library(build.build_attention(head_dim, value_dim, scored))
+        found = tuple(int(getattr(lib._dll, f"mrun_attn_{what}")()) for what in ("head_dim", "value_dim", "scored"))
+        if found != (head_dim, value_dim, int(scored)):
+            raise KernelError(f"{lib.path} was built for {found}, not {(head_dim, value_dim, int(scored))}")
+        _attention[key] = lib
     return lib

@@ -75,9 +75,10 @@ def add_rmsnorm(resid: torch.Tensor, delta: Optional[torch.Tensor], weight: torc
 
 
 def add_layernorm(resid: torch.Tensor, delta: Optional[torch.Tensor], weight: torch.Tensor, eps: float,
-                  out: torch.Tensor, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """resid (+= delta) then out = (resid - mean) * rsqrt(variance + eps) * weight, the variance the
-    mean of the squared deviations; with ``rows`` only those rows are normed and resid is left as
+                  out: torch.Tensor, rows: Optional[torch.Tensor] = None,
+                  bias: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """resid (+= delta) then out = (resid - mean) * rsqrt(variance + eps) * weight (+ bias), the
+    variance the mean of the squared deviations; with ``rows`` only those rows are normed and resid is left as
     it is.  ``delta`` is 32-bit or of ``out``'s dtype."""
     _check(resid, "resid", torch.float32); _check(weight, "weight", torch.float32); _check(out, "out")
     hidden = resid.shape[-1]
@@ -87,14 +88,54 @@ def add_layernorm(resid: torch.Tensor, delta: Optional[torch.Tensor], weight: to
         if delta.shape != resid.shape or delta.dtype not in (torch.float32, out.dtype):
             raise KernelError(f"add_layernorm: delta {tuple(delta.shape)} {delta.dtype} vs resid {tuple(resid.shape)}, "
                               f"out {out.dtype}")
+    if bias is not None:
+        _check(bias, "bias", torch.float32)
+        if bias.numel() != hidden:
+            raise KernelError(f"add_layernorm: bias has {bias.numel()} entries, the width is {hidden}")
     if rows is not None:
         _check(rows, "rows", torch.int32)
     if weight.numel() != hidden or out.shape != (n_rows, hidden):
         raise KernelError(f"add_layernorm: weight {tuple(weight.shape)}, out {tuple(out.shape)}, "
                           f"expected hidden {hidden}, rows {n_rows}")
     _lib.core().call("mrun_add_layernorm", _ptr(resid), _ptr(delta), dtype_code(delta.dtype if delta is not None else out.dtype),
-                     _ptr(weight), _c_float(eps), _ptr(out), dtype_code(out.dtype), _ptr(rows), _c_int(n_rows),
+                     _ptr(weight), _ptr(bias), _c_float(eps), _ptr(out), dtype_code(out.dtype), _ptr(rows), _c_int(n_rows),
                      _c_int(hidden), _stream())
+    return out
+
+
+def post_layernorm_add(stream: torch.Tensor, pending, next_weight: Optional[torch.Tensor] = None,
+                       next_bias: Optional[torch.Tensor] = None, next_eps: float = 0.0,
+                       out: Optional[torch.Tensor] = None, rows: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
+    """stream += layer norm of a :class:`PendingPostLayerNorm`'s branch (None: nothing is added), in
+    place and in 32-bit; then ``out`` gets the new rows in its dtype or, with ``next_weight``, their
+    layer norm (``out`` None: nothing).  With ``rows`` only those rows are computed and the stream
+    is left as it is."""
+    _check(stream, "stream", torch.float32)
+    hidden = stream.shape[1]
+    n_rows = stream.shape[0] if rows is None else rows.numel()
+    branch = weight = bias = None
+    eps = 0.0
+    if pending is not None:
+        branch, weight, bias, eps = pending.branch, pending.weight, pending.bias, pending.eps
+        _check(branch, "branch", torch.float32)
+        if branch.shape != stream.shape:
+            raise KernelError(f"post_layernorm_add: stream {tuple(stream.shape)}, branch {tuple(branch.shape)}")
+    for name, v in (("weight", weight), ("bias", bias), ("next_weight", next_weight), ("next_bias", next_bias)):
+        if v is not None:
+            _check(v, name, torch.float32)
+            if v.numel() != hidden:
+                raise KernelError(f"post_layernorm_add: {name} has {v.numel()} entries, the width is {hidden}")
+    code = F32
+    if out is not None:
+        _check(out, "out")
+        code = dtype_code(out.dtype)
+        if out.shape != (n_rows, hidden):
+            raise KernelError(f"post_layernorm_add: out {tuple(out.shape)}, expected {(n_rows, hidden)}")
+    if rows is not None:
+        _check(rows, "rows", torch.int32)
+    _lib.core().call("mrun_post_layernorm_add", _ptr(stream), _ptr(branch), _ptr(weight), _ptr(bias), _c_float(eps),
+                     _ptr(next_weight), _ptr(next_bias), _c_float(next_eps), _ptr(out), _c_int(code), _ptr(rows),
+                     _c_int(n_rows), _c_int(hidden), _stream())
     return out
 
 
@@ -262,16 +303,17 @@ def head_norm_rope_cache(x: torch.Tensor, q_off: int, k_off: int, v_off: int, he
 def paged_attention_generic(q: torch.Tensor, q_stride: int, out: torch.Tensor, k_cache: torch.Tensor,
                             v_cache: torch.Tensor, block_tables: torch.Tensor, token_slot: torch.Tensor,
                             positions: torch.Tensor, heads: int, scale: float, window: int = 0, sink: bool = False,
-                            gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+                            gate: Optional[torch.Tensor] = None, form=None) -> torch.Tensor:
     """Attention of every token over its request's pages, 32-bit arithmetic on CUDA cores.
 
     ``q`` may be a view into a wider buffer: row t starts ``q_stride`` elements after row t-1.
     ``block_tables`` has one row per state slot; ``token_slot[t]`` names the row of token t.
     The value pages may have another feature size than the key pages.  ``sink``: one more term of
     score 0 without a value in the softmax's denominator.  ``gate``: [tokens, heads] in q's dtype
-    (rows may be strided), whose sigmoid multiplies each head's output.
+    (rows may be strided), whose sigmoid multiplies each head's output.  ``form``: a score form
+    (:class:`mrun_b200.kernels.attention.ScoreForm`), whose output rows may be strided.
     """
-    _check(q, "q", dense=False); _check(out, "out", q.dtype)
+    _check(q, "q", dense=False); _check(out, "out", q.dtype, dense=form is None)
     _check(k_cache, "k_cache", q.dtype); _check(v_cache, "v_cache", q.dtype)
     _check(block_tables, "block_tables", torch.int32); _check(token_slot, "token_slot", torch.int32)
     _check(positions, "positions", torch.int32)
@@ -294,7 +336,8 @@ def paged_attention_generic(q: torch.Tensor, q_stride: int, out: torch.Tensor, k
                      _ptr(v_cache), dtype_code(q.dtype), _ptr(block_tables), _c_int(block_tables.shape[1]),
                      _ptr(token_slot), _ptr(positions), _c_int(tokens), _c_int(heads), _c_int(kv_heads),
                      _c_int(head_dim), _c_int(value_dim), _c_int(page_size), _c_long(pages * kv_heads * page_size),
-                     _c_float(scale), _c_int(window), _c_int(1 if sink else 0), _ptr(gate), _c_long(gate_stride), _stream())
+                     _c_float(scale), _c_int(window), _c_int(1 if sink else 0), _ptr(gate), _c_long(gate_stride),
+                     ctypes.byref(form) if form is not None else _ptr(None), _stream())
     return out
 
 
@@ -457,7 +500,25 @@ class PendingPairNorm:
         return pair_norm_mean(self.a, self.b, self.weight_a, self.weight_b, self.eps, self.share)
 
 
-PENDING = (PendingLinear, PendingPostNorm, PendingPairNorm)      # what a block may hand to the norm after it unadded
+class PendingPostLayerNorm:
+    """A branch output (float32 rows) that joins the stream as its layer norm with ``weight`` and
+    ``bias`` and has not been added yet (:func:`post_layernorm_add`).  :meth:`compute` makes the
+    addend itself (float32)."""
+
+    def __init__(self, branch: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor], eps: float):
+        self.branch, self.weight, self.bias, self.eps = branch, weight, bias, float(eps)
+
+    @property
+    def shape(self):
+        return self.branch.shape
+
+    def compute(self) -> torch.Tensor:
+        addend = torch.zeros_like(self.branch)
+        post_layernorm_add(addend, self)
+        return addend
+
+
+PENDING = (PendingLinear, PendingPostNorm, PendingPairNorm, PendingPostLayerNorm)      # what a block may hand to the norm after it unadded
 
 
 def _normed(x):
@@ -644,6 +705,51 @@ def linear(x, w: torch.Tensor, out_dtype: Optional[torch.dtype] = None,
         else:
             y = torch.mm(x, w.t(), out_dtype=out_dtype)
     return y if bias is None else add_bias(y, bias)
+
+
+ACTIVATIONS = {"relu2": 1, "tanh": 2}      # codes of the C ABI (MRUN_ACT_*): functions of one argument
+
+
+def plain_act(x: torch.Tensor, activation: str, out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
+    """act(x) element by element in 32-bit."""
+    _check(x, "x")
+    out = torch.empty(x.shape, dtype=out_dtype or x.dtype, device=x.device)
+    _lib.core().call("mrun_plain_act", _ptr(x), _c_int(dtype_code(x.dtype)), _ptr(out), _c_int(dtype_code(out.dtype)),
+                     _c_long(x.numel()), _c_int(ACTIVATIONS[activation]), _stream())
+    return out
+
+
+def linear_act(x: torch.Tensor, w: torch.Tensor, activation: str) -> torch.Tensor:
+    """act(x @ w.T) in x's dtype; up to 16 bfloat16 rows the activation rides in the decode GEMM's
+    epilogue (which sees the sums as they would have been stored)."""
+    if skinny_ok(x, w):
+        return linears_batched(x.unsqueeze(1), w.unsqueeze(0), activation=activation)[:, 0]
+    y = linear(x, w)
+    if activation == "relu2":
+        return relu2_scaled(y, None, 0, 1)
+    return plain_act(y, activation)
+
+
+def linears_batched(x: torch.Tensor, w: torch.Tensor, activation: Optional[str] = None) -> torch.Tensor:
+    """y[:, b] = act(x[:, b] @ w[b].T): ``x`` [rows, batch, K] (may be strided along the first two
+    axes), ``w`` dense [batch, N, K]; returns dense [rows, batch, N].  One launch: up to 16
+    bfloat16 rows this library's decode GEMM, else as :func:`linear_per_head` (without an activation)."""
+    rows, batch, k = x.shape
+    n = w.shape[1]
+    out = torch.empty((rows, batch, n), dtype=x.dtype, device=x.device)
+    if not (x.dtype == torch.bfloat16 and rows <= SKINNY_ROWS and k % 32 == 0 and x.stride(0) % 8 == 0
+            and x.stride(1) % 8 == 0 and x.data_ptr() % 16 == 0):
+        if activation is not None:
+            raise KernelError("linears_batched: an activation comes with the decode GEMM only")
+        return linear_per_head(x, w, out)
+    _check(x, "x", torch.bfloat16, dense=False); _check(w, "w", torch.bfloat16)
+    if w.shape != (batch, n, k) or x.stride(2) != 1:
+        raise KernelError(f"linears_batched: x {tuple(x.shape)} (strides {x.stride()}) vs w {tuple(w.shape)}")
+    _lib.core().call("mrun_gemm_skinny_batched", _ptr(x), _ptr(w), _ptr(out), dtype_code(out.dtype),
+                     _c_int(ACTIVATIONS[activation] if activation else 0), _c_int(batch), _c_int(rows), _c_int(n), _c_int(k),
+                     _c_long(x.stride(0) if rows > 1 else max(k, x.stride(0))), _c_long(batch * n),
+                     _c_long(x.stride(1) if batch > 1 else 0), _c_long(n), _stream())
+    return out
 
 
 def linear_or_pending(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None):
@@ -1079,9 +1185,10 @@ def streams_step(streams: torch.Tensor, pending: Optional[PendingStreams], in_c:
 
 # ------------------------------------------------------------------ recurrent mixers
 
-def causal_conv(x: torch.Tensor, weight: torch.Tensor, state: torch.Tensor, ctx, residual: bool, silu: bool) -> torch.Tensor:
+def causal_conv(x: torch.Tensor, weight: torch.Tensor, state: torch.Tensor, ctx, residual: bool, silu: bool,
+                bias: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Causal convolution per channel over each request's tokens (the last tap meets the token
-    itself), added to x (``residual``) and/or passed through SiLU.  ``x``: [tokens, channels],
+    itself) plus ``bias`` (float32 [channels]), added to x (``residual``) and/or passed through SiLU.  ``x``: [tokens, channels],
     rows may be strided; ``weight``: float32 [channels, taps]; ``state``: [slots, taps - 1,
     channels] in x's dtype, the request's last inputs, read and left up to date (empty with one
     tap, which sees the token itself only)."""
@@ -1090,8 +1197,12 @@ def causal_conv(x: torch.Tensor, weight: torch.Tensor, state: torch.Tensor, ctx,
     taps = weight.shape[1]
     if x.stride(1) != 1 or weight.shape[0] != channels or state.shape[1:] != (taps - 1, channels):
         raise KernelError(f"causal_conv: x {tuple(x.shape)}, weight {tuple(weight.shape)}, state {tuple(state.shape)}")
+    if bias is not None:
+        _check(bias, "bias", torch.float32)
+        if bias.numel() != channels:
+            raise KernelError(f"causal_conv: bias has {bias.numel()} entries for {channels} channels")
     out = torch.empty((tokens, channels), dtype=x.dtype, device=x.device)
-    _lib.core().call("mrun_causal_conv", _ptr(x), _c_long(x.stride(0)), _ptr(weight), _ptr(state), _ptr(out),
+    _lib.core().call("mrun_causal_conv", _ptr(x), _c_long(x.stride(0)), _ptr(weight), _ptr(bias), _ptr(state), _ptr(out),
                      _c_long(channels), dtype_code(x.dtype), _ptr(ctx.seg_q_start), _ptr(ctx.seg_slot),
                      _c_int(ctx.num_segments), _c_int(ctx.max_q_len), _c_int(channels), _c_int(taps),
                      _c_int(1 if residual else 0), _c_int(1 if silu else 0), _stream())
@@ -1181,20 +1292,113 @@ GATE_SHAPES = {"sigmoid": 0, "silu": 1}        # what a gated norm passes its ga
 
 
 def gated_norm(o: torch.Tensor, weight: torch.Tensor, gate: torch.Tensor, eps: float, groups: int,
-               out_dtype: torch.dtype, gate_function: str = "sigmoid") -> torch.Tensor:
+               out_dtype: torch.dtype, gate_function: str = "sigmoid", out: Optional[torch.Tensor] = None,
+               scale: float = 1.0) -> torch.Tensor:
     """Per group of ``o.shape[1] // groups`` features: o / sqrt(mean(o^2) + eps) * weight *
     f(gate), f the sigmoid or SiLU (``gate_function``).  ``o``: float32 [tokens, features]; ``weight``: float32, one entry per feature
-    of a row or of a group; ``gate``: [tokens, features] in ``out_dtype``, rows may be strided."""
+    of a row or of a group; ``gate``: [tokens, features] in ``out_dtype``, rows may be strided.
+    ``out``: where the result goes, times ``scale`` (rows may be strided)."""
     _check(o, "o", torch.float32); _check(weight, "weight", torch.float32)
     ldg = _strided_rows(gate, "gate")
     tokens, features = o.shape
     n = features // groups
     if gate.shape != o.shape or gate.dtype != out_dtype or weight.numel() not in (n, features) or n * groups != features:
         raise KernelError("gated_norm: sizes do not match")
-    out = torch.empty((tokens, features), dtype=out_dtype, device=o.device)
+    if out is None:
+        out = torch.empty((tokens, features), dtype=out_dtype, device=o.device)
+    ldo = _strided_rows(out, "out")
+    if out.shape != o.shape or out.dtype != out_dtype:
+        raise KernelError(f"gated_norm: out is {tuple(out.shape)} {out.dtype}")
     _lib.core().call("mrun_gated_norm", _ptr(o), _ptr(weight), _c_int(weight.numel()), _ptr(gate), _c_long(ldg),
-                     dtype_code(out_dtype), _c_float(eps), _ptr(out), _c_int(tokens), _c_int(groups), _c_int(n),
+                     dtype_code(out_dtype), _c_float(eps), _ptr(out), _c_long(ldo), _c_float(scale), _c_int(tokens), _c_int(groups), _c_int(n),
                      _c_int(GATE_SHAPES[gate_function]), _stream())
+    return out
+
+
+def skip_gate_norm(o: torch.Tensor, x: torch.Tensor, skip: torch.Tensor, z: torch.Tensor, weight: torch.Tensor, eps: float,
+                   groups: int) -> torch.Tensor:
+    """y = (o + skip_h * x) * SiLU(z), then per group of ``o.shape[1] // groups`` features y /
+    sqrt(mean(y^2) + eps) * weight.  ``o``: float32 [tokens, features]; ``x``, ``z``: [tokens,
+    features] of the activation type, rows may be strided; ``skip``: float32, one entry a head;
+    ``weight``: float32 [features].  Returns rows of the activation type."""
+    _check(o, "o", torch.float32); _check(weight, "weight", torch.float32); _check(skip, "skip", torch.float32)
+    ldx, ldz = _strided_rows(x, "x"), _strided_rows(z, "z")
+    tokens, features = o.shape
+    if x.shape != o.shape or z.shape != o.shape or x.dtype != z.dtype or weight.numel() != features or features % groups \
+            or features % skip.numel():
+        raise KernelError(f"skip_gate_norm: o {tuple(o.shape)}, x {tuple(x.shape)}, z {tuple(z.shape)}, {groups} groups")
+    out = torch.empty((tokens, features), dtype=x.dtype, device=o.device)
+    _lib.core().call("mrun_skip_gate_norm", _ptr(o), _ptr(x), _c_long(ldx), _ptr(skip), _c_int(features // skip.numel()),
+                     _ptr(z), _c_long(ldz), _ptr(weight), _c_int(dtype_code(x.dtype)), _c_float(eps), _ptr(out),
+                     _c_int(tokens), _c_int(groups), _c_int(features // groups), _stream())
+    return out
+
+
+def token_blend(x: torch.Tensor, mu: torch.Tensor, state: torch.Tensor, ctx) -> torch.Tensor:
+    """[tokens, S, channels]: x_t + (x_(t-1) - x_t) * mu[s] over each request's tokens, the row before
+    a portion's first token from ``state`` ([slots, 1, channels] in x's dtype, zeros at the start),
+    which is left holding the portion's last row.  ``mu``: float32 [S, channels]."""
+    ldx = _strided_rows(x, "x")
+    _check(mu, "mu", torch.float32); _check(state, "state", x.dtype)
+    tokens, channels = x.shape
+    if mu.dim() != 2 or mu.shape[1] != channels or state.shape[1:] != (1, channels):
+        raise KernelError(f"token_blend: x {tuple(x.shape)}, mu {tuple(mu.shape)}, state {tuple(state.shape)}")
+    out = torch.empty((tokens, mu.shape[0], channels), dtype=x.dtype, device=x.device)
+    _lib.core().call("mrun_token_blend", _ptr(x), _c_long(ldx), _ptr(mu), _ptr(state), _ptr(out), _c_int(dtype_code(x.dtype)),
+                     _ptr(ctx.seg_q_start), _ptr(ctx.seg_slot), _c_int(ctx.num_segments), _c_int(ctx.max_q_len),
+                     _c_int(channels), _c_int(mu.shape[0]), _stream())
+    return out
+
+
+def bonus_scan(r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, a: torch.Tensor, bias: torch.Tensor, bonus: torch.Tensor,
+               state: torch.Tensor, ctx, heads: int, dim: int, vdim: int) -> torch.Tensor:
+    """Linear attention with a decay per head and key channel and a bonus for the current token, over
+    each request's tokens: g = exp(-exp(a + bias)), o = S^T r + (r . (bonus * k)) v, S <- g * S
+    (rows) + k v^T, from and into ``state`` (float32 [slots, heads, dim, vdim]).  r, k ([tokens,
+    heads * dim]) and v ([tokens, heads * vdim]): column slices of one matrix; ``a``: float32 [tokens,
+    heads * dim]; ``bias`` and ``bonus``: float32 [heads * dim].  Returns float32 [tokens, heads *
+    vdim]."""
+    ld = _strided_rows(r, "r")
+    if _strided_rows(k, "k") != ld or _strided_rows(v, "v") != ld or k.dtype != r.dtype or v.dtype != r.dtype:
+        raise KernelError("bonus_scan: r, k and v must be slices of one matrix")
+    for name, t in (("a", a), ("bias", bias), ("bonus", bonus), ("state", state)):
+        _check(t, name, torch.float32)
+    tokens = r.shape[0]
+    if r.shape[1] != heads * dim or k.shape[1] != heads * dim or v.shape[1] != heads * vdim \
+            or a.shape != (tokens, heads * dim) or bias.numel() != heads * dim or bonus.numel() != heads * dim \
+            or state.shape[1:] != (heads, dim, vdim):
+        raise KernelError("bonus_scan: sizes do not match")
+    out = torch.empty((tokens, heads * vdim), dtype=torch.float32, device=r.device)
+    scratch = torch.empty(tokens * heads * (3 * dim + vdim), dtype=torch.float32, device=r.device)
+    _lib.core().call("mrun_bonus_scan", _ptr(r), _ptr(k), _ptr(v), _c_long(ld), dtype_code(r.dtype), _ptr(a), _ptr(bias),
+                     _ptr(bonus), _ptr(state), _ptr(out), _ptr(scratch), _ptr(ctx.seg_q_start), _ptr(ctx.seg_slot),
+                     _c_int(ctx.num_segments), _c_int(tokens), _c_int(heads), _c_int(dim), _c_int(vdim), _stream())
+    return out
+
+
+def ssm_scan(c: torch.Tensor, b: torch.Tensor, x: torch.Tensor, dt: torch.Tensor, dt_bias: torch.Tensor,
+             a_log: torch.Tensor, state: torch.Tensor, ctx, heads: int, groups: int, size: int, vdim: int) -> torch.Tensor:
+    """A selective state-space recurrence over each request's tokens: step = softplus(dt + dt_bias) and
+    decay = exp(-exp(a_log) * step) per head; S <- decay * S + step * b x^T, y = S^T c, from and into
+    ``state`` (float32 [slots, heads, size, vdim]).  c, b ([tokens, groups * size]) and x ([tokens,
+    heads * vdim]): column slices of one matrix; ``dt``: [tokens, heads] in the same type, rows may be
+    strided; ``dt_bias``, ``a_log``: float32 [heads].  Returns float32 [tokens, heads * vdim]."""
+    ld, lddt = _strided_rows(c, "c"), _strided_rows(dt, "dt")
+    if _strided_rows(b, "b") != ld or _strided_rows(x, "x") != ld or len({t.dtype for t in (c, b, x, dt)}) != 1:
+        raise KernelError("ssm_scan: c, b and x must be slices of one matrix, dt of its type")
+    for name, t in (("dt_bias", dt_bias), ("a_log", a_log), ("state", state)):
+        _check(t, name, torch.float32)
+    tokens = c.shape[0]
+    if c.shape[1] != groups * size or b.shape[1] != groups * size or x.shape[1] != heads * vdim or heads % groups \
+            or dt.shape != (tokens, heads) or dt_bias.numel() != heads or a_log.numel() != heads \
+            or state.shape[1:] != (heads, size, vdim):
+        raise KernelError("ssm_scan: sizes do not match")
+    out = torch.empty((tokens, heads * vdim), dtype=torch.float32, device=c.device)
+    scratch = torch.empty(tokens * (2 * groups * size + heads * (vdim + 1)), dtype=torch.float32, device=c.device)
+    _lib.core().call("mrun_ssm_scan", _ptr(c), _ptr(b), _ptr(x), _c_long(ld), dtype_code(c.dtype), _c_int(heads // groups),
+                     _ptr(dt), _c_long(lddt), _ptr(dt_bias), _ptr(a_log), _ptr(state), _ptr(out), _ptr(scratch),
+                     _ptr(ctx.seg_q_start), _ptr(ctx.seg_slot), _c_int(ctx.num_segments), _c_int(tokens), _c_int(heads),
+                     _c_int(size), _c_int(vdim), _stream())
     return out
 
 

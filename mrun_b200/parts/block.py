@@ -150,6 +150,74 @@ class SandwichBlock:
         return self._branch(f, self.feed_forward_post_norm)
 
 
+@register_arrangement("post_norm")
+class PostNormBlock:
+    """``x += norm_1(mixer(x)); x += norm_2(ff(x))``: the sublayers read the stream itself (narrowed to the
+    activation type) and a branch passes a layer norm on its way into it.  A layer without a
+    feed-forward has the first half only.
+
+    The branch's last product writes 32-bit sums; their norm, the residual sum and the narrowed rows
+    that the next sublayer reads are one kernel (``ops.post_layernorm_add``), so the block hands its own
+    last branch output on unadded, as the other arrangements do."""
+
+    accepts_pending = True
+
+    tensor_specs = staticmethod(PreNormBlock.tensor_specs)
+
+    def __init__(self, spec: LayerSpec, tensors, runtime: Runtime):
+        for norm in (spec.mixer_norm, spec.feed_forward_norm):
+            if norm is not None and norm.kind != "layernorm":
+                raise ValueError(f"the post_norm arrangement norms its branches by layer norms, not by {norm.kind!r}")
+        mine = local(tensors, spec.prefix)
+        self.act = runtime.precision.act
+        self.mixer_norm = NORMS.build(spec.mixer_norm, local(mine, spec.mixer_norm_prefix), runtime)
+        self.mixer = MIXERS.build(spec.mixer, local(mine, spec.mixer_prefix), runtime)
+        self.feed_forward_norm = self.feed_forward = None
+        if spec.feed_forward is not None:
+            self.feed_forward_norm = NORMS.build(spec.feed_forward_norm, local(mine, spec.feed_forward_norm_prefix), runtime)
+            self.feed_forward = FEED_FORWARDS.build(spec.feed_forward, local(mine, spec.feed_forward_prefix), runtime)
+        self._mixer_defers = bool(getattr(self.mixer, "can_defer_output", False))
+        self._feed_forward_defers = bool(getattr(self.feed_forward, "can_defer_output", False))
+
+    def _input(self, resid: torch.Tensor, delta) -> torch.Tensor:
+        """The stream with the pending branch in it, as the rows a sublayer reads (in 32-bit the stream
+        itself: it changes only after the sublayer has read it)."""
+        if delta is not None and not isinstance(delta, ops.PendingPostLayerNorm):
+            resid.add_(delta.compute() if isinstance(delta, ops.PENDING) else delta)     # from a layer of another arrangement
+            delta = None
+        wide = self.act == torch.float32
+        if wide and delta is None:
+            return resid
+        out = None if wide else torch.empty(resid.shape, dtype=self.act, device=resid.device)
+        ops.post_layernorm_add(resid, delta, out=out)
+        return resid if wide else out
+
+    @staticmethod
+    def _branch(y, norm) -> "ops.PendingPostLayerNorm":
+        """The branch output as 32-bit rows, with the norm that it still has to pass."""
+        if isinstance(y, ops.PendingLinear):
+            y = ops.linear(y.x, y.w, out_dtype=torch.float32)
+        elif isinstance(y, ops.PENDING):
+            y = y.compute()
+        return ops.PendingPostLayerNorm(y if y.dtype == torch.float32 else y.to(torch.float32), norm.weight, norm.bias, norm.eps)
+
+    def forward(self, resid: torch.Tensor, delta, ctx, cache):
+        h = self._input(resid, delta)
+        if self._mixer_defers:
+            a = self.mixer.forward(h, ctx, cache, defer_output=True)
+        else:
+            a = self.mixer.forward(h, ctx, cache)
+        a = self._branch(a, self.mixer_norm)
+        if self.feed_forward is None:
+            return a
+        h = self._input(resid, a)
+        if self._feed_forward_defers:
+            f = self.feed_forward.forward(h, ctx, defer_output=True)
+        else:
+            f = self.feed_forward.forward(h, ctx)
+        return self._branch(f, self.feed_forward_norm)
+
+
 @register_arrangement("streams")
 class StreamsBlock:
     """A pre-norm layer over several residual streams a token (hyper-connections).  The stream

@@ -8,7 +8,7 @@ from __future__ import annotations
 
 import torch
 
-from ..config.spec import ClampedGatedMLPSpec, GatedMLPSpec, TensorSpec
+from ..config.spec import ClampedGatedMLPSpec, DenseMLPSpec, GatedMLPSpec, TensorSpec
 from ..kernels import ops
 from .base import Runtime, register_feed_forward
 
@@ -78,6 +78,36 @@ class GatedMLP:
         if defer_output:
             return ops.linear_or_pending(act, self.w_down, self.b_down)
         return ops.linear(act, self.w_down, bias=self.b_down)
+
+
+@register_feed_forward("dense_mlp")
+class DenseMLP:
+    """Feed-forward without a gate: ``down(act(up(x)))``.  Up to 16 bfloat16 rows the activation rides in
+    the first product's epilogue."""
+
+    can_defer_output = True
+
+    @staticmethod
+    def tensor_specs(spec: DenseMLPSpec, prefix: str):
+        up, down = spec.tensor_names
+        return [TensorSpec(f"{prefix}.{up}", (spec.intermediate, spec.hidden)),
+                TensorSpec(f"{prefix}.{down}", (spec.hidden, spec.intermediate))]
+
+    def __init__(self, spec: DenseMLPSpec, tensors, runtime: Runtime):
+        if spec.activation not in ops.ACTIVATIONS:
+            raise ValueError(f"no kernel has the activation {spec.activation!r} (known: {', '.join(sorted(ops.ACTIVATIONS))})")
+        self.spec = spec
+        up, down = spec.tensor_names
+        self.w_up, self.w_down = runtime.matrix(tensors[up]), runtime.matrix(tensors[down])
+
+    def activation_elements(self) -> int:
+        return 2 * self.spec.intermediate
+
+    def forward(self, x, ctx, defer_output: bool = False):
+        act = ops.linear_act(x, self.w_up, self.spec.activation)
+        if defer_output:
+            return ops.linear_or_pending(act, self.w_down)
+        return ops.linear(act, self.w_down)
 
 
 @register_feed_forward("clamped_gated_mlp")

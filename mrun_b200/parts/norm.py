@@ -43,7 +43,7 @@ class RMSNorm:
             out = torch.empty(resid.shape, dtype=self.act, device=resid.device)
             return ops.post_norm_add(resid, delta.branch, delta.weight, delta.scale, delta.eps, self.weight,
                                      self.eps, out)
-        if isinstance(delta, ops.PendingPairNorm):
+        if isinstance(delta, (ops.PendingPairNorm, ops.PendingPostLayerNorm)):
             delta = delta.compute().to(self.act)        # no fused form with this norm: the addend, in the activation type
         if isinstance(delta, ops.PendingLinear):
             if ops.norm_fusable(delta, resid, self.weight):
@@ -61,7 +61,7 @@ class RMSNorm:
             out = torch.empty((rows.numel(), self.size), dtype=self.act, device=resid.device)
             return ops.post_norm_add(resid, delta.branch, delta.weight, delta.scale, delta.eps, self.weight,
                                      self.eps, out, rows=rows)
-        if isinstance(delta, ops.PendingPairNorm):
+        if isinstance(delta, (ops.PendingPairNorm, ops.PendingPostLayerNorm)):
             delta = delta.compute().to(self.act)
         if isinstance(delta, ops.PendingLinear):
             delta = delta.compute()
@@ -74,13 +74,16 @@ class RMSNorm:
 
 @register_norm("layernorm")
 class LayerNorm:
-    """Layer norm with a weight and no bias, in 32-bit: ``y = (x - mean) * rsqrt(var + eps) * w``,
+    """Layer norm with a weight (and a bias), in 32-bit: ``y = (x - mean) * rsqrt(var + eps) * w (+ b)``,
     the variance taken from the deviations.  The residual sum rides in the same kernel; a branch
     output may come in 32-bit or in the activation type."""
 
     @staticmethod
     def tensor_specs(spec: LayerNormSpec, prefix: str):
-        return [TensorSpec(prefix if spec.bare else f"{prefix}.weight", (spec.size,), "norm")]
+        out = [TensorSpec(prefix if spec.bare else f"{prefix}.weight", (spec.size,), "norm")]
+        if spec.bias:
+            out.append(TensorSpec(f"{prefix}.b" if spec.bare else f"{prefix}.bias", (spec.size,), "norm_zero"))
+        return out
 
     # ``delta`` may be a product that has not run yet: above 16 bfloat16 rows the vendor GEMM adds
     # it into the 32-bit stream itself, otherwise it is computed first
@@ -90,6 +93,7 @@ class LayerNorm:
     def __init__(self, spec: LayerNormSpec, tensors, runtime: Runtime):
         self.size, self.eps = spec.size, float(spec.eps)
         self.weight = runtime.vector_f32(tensors["" if spec.bare else "weight"])
+        self.bias = runtime.vector_f32(tensors["b" if spec.bare else "bias"]) if spec.bias else None
         self.act = runtime.precision.act
 
     def _settle(self, resid: torch.Tensor, delta, in_place: bool):
@@ -104,17 +108,21 @@ class LayerNorm:
 
     def add_forward(self, resid: torch.Tensor, delta):
         out = torch.empty(resid.shape, dtype=self.act, device=resid.device)
-        if isinstance(delta, ops.PendingPairNorm):      # two branches still to be normed and averaged: one kernel
+        if isinstance(delta, ops.PendingPostLayerNorm):     # a branch still to be normed itself: one kernel
+            return ops.post_layernorm_add(resid, delta, self.weight, self.bias, self.eps, out)
+        if isinstance(delta, ops.PendingPairNorm) and self.bias is None:    # two branches still to be normed and averaged: one kernel
             return ops.pair_norm_add_layernorm(resid, delta, self.weight, self.eps, out)
         delta = self._settle(resid, delta, True)
-        return ops.add_layernorm(resid, delta, self.weight, self.eps, out)
+        return ops.add_layernorm(resid, delta, self.weight, self.eps, out, bias=self.bias)
 
     def rows_forward(self, resid: torch.Tensor, delta, rows: torch.Tensor) -> torch.Tensor:
         out = torch.empty((rows.numel(), self.size), dtype=self.act, device=resid.device)
-        if isinstance(delta, ops.PendingPairNorm):
+        if isinstance(delta, ops.PendingPostLayerNorm):
+            return ops.post_layernorm_add(resid, delta, self.weight, self.bias, self.eps, out, rows=rows)
+        if isinstance(delta, ops.PendingPairNorm) and self.bias is None:
             return ops.pair_norm_add_layernorm(resid, delta, self.weight, self.eps, out, rows=rows)
         delta = self._settle(resid, delta, False)
-        return ops.add_layernorm(resid, delta, self.weight, self.eps, out, rows=rows)
+        return ops.add_layernorm(resid, delta, self.weight, self.eps, out, rows=rows, bias=self.bias)
 
     def forward(self, x: torch.Tensor) -> torch.Tensor:
         return self.add_forward(x.to(torch.float32), None)

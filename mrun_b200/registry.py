@@ -68,11 +68,13 @@ def _register_builtin() -> None:
     from .config.balivik import BalivikConfig
     from .config.fikudra import FikudraConfig
     from .config.nisotar import NisotarConfig
+    from .config.katadra import KatadraConfig
     register_architecture(Qwen3Config)
     register_architecture(ZasesunConfig)
     register_architecture(BalivikConfig)
     register_architecture(FikudraConfig)
     register_architecture(NisotarConfig)
+    register_architecture(KatadraConfig)
 
 
 _register_builtin()

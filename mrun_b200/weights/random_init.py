@@ -4,7 +4,7 @@ and a seed.
 Each tensor has a generator of its own, seeded from (seed, tensor name), so a tensor's values do
 not depend on which other tensors exist or on their order.  Matrices and tables are N(0, std);
 scale vectors of norms are 1, or 1 + N(0, norm_noise); the few other kinds (an integer table of
-distinct entries per row, weights between residual streams, logarithms of decay rates) are named
+distinct entries per row, weights between residual streams, shares, convolution taps, logarithms of decay rates) are named
 by ``TensorSpec.init``.  The reference's test helper fills its tiny
 model the same way with its own generator (crates/mrun-engine/src/testing.rs:42-51, 91-149).
 """
@@ -51,6 +51,11 @@ def random_tensor(t: TensorSpec, seed: int, std: float, norm_noise: float, dtype
     if t.init == "streams_mix":         # stream-to-stream weights: near the identity
         noise = torch.randn(t.shape, generator=gen, dtype=torch.float32, device=device)
         return (torch.eye(t.shape[0], dtype=torch.float32, device=device) + 0.15 * noise).to(dtype)
+    if t.init == "share":               # blending weights: between 0 and 1
+        return torch.rand(t.shape, generator=gen, dtype=torch.float32, device=device).to(dtype)
+    if t.init == "taps":                # a short convolution: an even share a tap, about
+        noise = torch.randn(t.shape, generator=gen, dtype=torch.float32, device=device)
+        return ((1.0 + 0.5 * noise) / t.shape[-1]).to(dtype)
     if t.init == "log_rate":            # logarithms of decay rates between e^-3 and 1
         return (torch.rand(t.shape, generator=gen, dtype=torch.float32, device=device) * 3.0 - 3.0).to(dtype)
     if t.init != "normal":

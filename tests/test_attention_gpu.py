@@ -179,7 +179,7 @@ def test_decode_tiles_dealt_to_any_number_of_blocks(blocks, min_tiles, splits, e
     part_ml = torch.full((blocks, 2, 16, 2), float("nan"), device=DEV)
     counters = torch.zeros(n * kv_heads, dtype=torch.int32, device=DEV)
     status = torch.zeros(1, dtype=torch.int32, device=DEV)
-    extra = (_ptr(None), _c_long(case.kd.shape[0]), _ptr(status)) if entry.endswith("tma") else ()
+    extra = (_ptr(None), _c_long(case.kd.shape[0]), _ptr(None), _ptr(status)) if entry.endswith("tma") else (_ptr(None),)
     for _ in range(2):
         out = torch.full((n, heads * head_dim), 3.0, dtype=torch.bfloat16, device=DEV)
         library.call(
@@ -252,7 +252,7 @@ def test_decode_contexts_of_unequal_length_and_raw_input(contexts, blocks, min_t
     part_ml = torch.full((blocks, 2, 16, 2), float("nan"), device=DEV)
     counters = torch.zeros(n * kv_heads, dtype=torch.int32, device=DEV)
     status = torch.zeros(1, dtype=torch.int32, device=DEV)
-    extra = (_ptr(None), _c_long(case.kd.shape[0]), _ptr(status)) if entry.endswith("tma") else ()
+    extra = (_ptr(None), _c_long(case.kd.shape[0]), _ptr(None), _ptr(status)) if entry.endswith("tma") else (_ptr(None),)
     for _ in range(2):
         k_got, v_got = case.kd.clone(), case.vd.clone()
         q_in = qkv if raw else case.qd
@@ -325,7 +325,7 @@ def test_cluster_decode_with_every_cluster_size(cluster, heads, kv_heads, head_d
             "mrun_attn_decode_cluster", _ptr(q_in), _c_long(q_in.stride(0)), _ptr(out), _ptr(k_got), _ptr(v_got),
             _ptr(case.table), _c_int(case.group.max_blocks), _ptr(case.ctx.token_slot), _ptr(case.ctx.positions),
             _c_int(n), _c_int(cluster), _c_int(heads), _c_int(kv_heads), _c_int(head_dim), _c_int(page_size),
-            _c_float(scale), _c_int(window), _c_float(float("-inf")), *fused, _ptr(None), _c_long(case.kd.shape[0]), _ptr(status), _stream())
+            _c_float(scale), _c_int(window), _c_float(float("-inf")), *fused, _ptr(None), _c_long(case.kd.shape[0]), _ptr(None), _ptr(status), _stream())
         got = out.float().cpu()
         assert int(status.item()) == 0
         assert (got - want).abs().max() <= 2e-2 * want.abs().max()
@@ -349,7 +349,7 @@ def test_cluster_decode_refuses_what_it_cannot_take():
             _ptr(case.table), _c_int(case.group.max_blocks), _ptr(case.ctx.token_slot), _ptr(case.ctx.positions),
             _c_int(1), _c_int(cluster), _c_int(heads), _c_int(2), _c_int(64), _c_int(16), _c_float(0.125), _c_int(0),
             _c_float(float("-inf")), _c_int(0), _ptr(None), _ptr(None), _c_float(0.0), _ptr(None), _c_int(0), _ptr(None), _ptr(None),
-            _c_long(case.kd.shape[0]), _ptr(status), _stream())
+            _c_long(case.kd.shape[0]), _ptr(None), _ptr(status), _stream())
     with pytest.raises(KernelError, match="query heads per kv head exceed"):
         call(4, 32)
     with pytest.raises(KernelError, match="cluster of 3 blocks"):
@@ -366,7 +366,7 @@ def test_the_router_gives_small_decode_steps_to_clusters_and_large_ones_to_the_p
     case = Case(segments, heads, kv_heads, head_dim, page_size, torch.bfloat16, seed=3, pad=1)
     want = case.reference(scale)
     library = attention._lib.attention(head_dim)
-    pick = lambda group, tokens, reach=1024: attention.decode_cluster(library, head_dim, group, page_size, tokens, kv_heads, reach)
+    pick = lambda group, tokens, reach=1024: attention.decode_cluster(library, group, page_size, tokens, kv_heads, reach)
     assert pick(4, 8) == 4 and pick(4, 1) == 16 and pick(4, 16) == 2
     assert pick(4, 2) == 8                        # sixteen would crowd
     assert pick(4, 19) == 0                       # 152 pairs: more than half the device

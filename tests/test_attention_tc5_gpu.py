@@ -37,7 +37,7 @@ def reference(case: Case, scale: float) -> torch.Tensor:
 def uses_tcgen05(head_dim: int, ratio: int, page_size: int) -> bool:
     from mrun_b200.kernels import lib
     from mrun_b200.kernels.attention import prefill_uses_tcgen05
-    return prefill_uses_tcgen05(lib.attention(head_dim), head_dim, ratio, page_size)
+    return prefill_uses_tcgen05(lib.attention(head_dim), ratio, page_size)
 
 
 def check_status():
