@@ -3,7 +3,7 @@
 random weights and seeded synthetic token ids.
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--layers L] [--impl ours|reference]
-                    [--shape 8b|4b|32b] [--serve] [--design zasesun|balivik|fikudra|nisotar]
+                    [--shape 8b|4b|32b] [--serve] [--design zasesun|balivik|fikudra|nisotar|katadra]
 
 A *step* is one decode step of a batch of 8 requests that each hold 1,024 tokens of context.
 ``value`` is decoded tokens per second over exactly K steps, timed on the device with CUDA events
@@ -26,6 +26,9 @@ widths, depths, head counts and expert sizes.
 beside a gated delta rule, attention and latent attention under sliding windows, all under layer
 norms; a clamped dense and logit-routed feed-forwards) beside the Fikudra decoder at equal widths,
 depths, head counts and expert sizes.
+``--design katadra`` measures the Katadra decoder (an attention with a soft cap, a distance bias and a
+gate per feature beside a time mixing, state-space mixers, dense feed-forwards, layer norms on branch
+outputs) beside the Nisotar decoder at equal widths, depths and head counts.
 """
 from __future__ import annotations
 
@@ -489,15 +492,64 @@ def nisotar_counts(cfg: dict, tokens: int, context: int):
     return flops + 2.0 * cfg["vocab"] * h, row_bytes, state_bytes
 
 
+# Layer sizes for --design katadra: (Katadra sizes, the Nisotar sizes of equal width, depth and head counts,
+# from the table above).  Eight layers: parallel (the attention beside a time mixing with heads of the
+# delta rule's size) with a dense feed-forward, two state-space mixers of twice the width without one,
+# and again; keys and values of one size (the tcgen05 and TMA attention kernels).
+def _katadra_sizes(width, heads, kv_heads, att_dim, dim, dense_ff, rank, layers, vocab):
+    left = {"heads": heads, "kv_heads": kv_heads, "dim": att_dim, "vdim": att_dim, "scale": att_dim ** -0.5, "softcap": 50.0,
+            "bias_max": 256, "bias_rows": 64, "q_temp": {"coef": 0.1, "every": 1024}}
+    par = {"left": left, "right": {"heads": heads, "dim": dim, "rank": rank}, "left_scale": 0.7, "right_scale": 0.7}
+    ssm = {"heads": width // 32, "vdim": 64, "state": 128, "groups": 8, "conv": 4, "norm_groups": 8}
+    return {"architecture": "Katadra", "vocab": vocab, "width": width, "norm": {"eps": 1e-6},
+            "layers": [{"type": "mamba2", "mixer": ssm, "mlp": None} if i % 3 else
+                       {"type": "parallel", "mixer": par, "mlp": {"kind": "dense", "ff": dense_ff}} for i in range(layers)]}
+
+
+KATADRA_SIZES = {
+    "w2048": (_katadra_sizes(2048, 16, 4, 128, 128, 8192, 64, 8, 32768), NISOTAR_SIZES["w2048"][0]),
+    "w4096": (_katadra_sizes(4096, 32, 8, 128, 128, 16384, 128, 8, 32768), NISOTAR_SIZES["w4096"][0]),
+}
+
+
+def katadra_counts(cfg: dict, tokens: int):
+    """(FLOPs of a prompt of ``tokens`` tokens as the design states them, cache bytes a token, bytes of one
+    request's recurrent states) of a Katadra configuration over all layers: products count two FLOPs a
+    weight and token, the attention the scores and weighted sums of every visible key, a recurrence the
+    decay, the update and the read-out of its state for every token."""
+    h, flops, kv_bytes, state_bytes = cfg["width"], 0.0, 0, 0
+    for layer in cfg["layers"]:
+        m = layer["mixer"]
+        if layer["type"] == "parallel":
+            a, r = m["left"], m["right"]
+            params = h * (a["heads"] * (a["dim"] + 2 * a["vdim"]) + a["kv_heads"] * (a["dim"] + a["vdim"]))
+            flops += 2.0 * tokens * (tokens + 1) / 2.0 * a["heads"] * (a["dim"] + a["vdim"])
+            kv_bytes += 2 * a["kv_heads"] * (a["dim"] + a["vdim"])
+            inner = r["heads"] * r["dim"]
+            params += h * (5 * inner + r["rank"]) + r["rank"] * inner
+            flops += 2.0 * tokens * 3 * r["heads"] * r["dim"] ** 2
+            state_bytes += 4 * r["heads"] * r["dim"] ** 2
+        else:
+            inner = m["heads"] * m["vdim"]
+            params = h * (3 * inner + 2 * m["groups"] * m["state"] + m["heads"])
+            flops += 2.0 * tokens * 3 * inner * m["state"]
+            state_bytes += 4 * inner * m["state"]
+        if layer["mlp"]:
+            params += 2 * h * layer["mlp"]["ff"]
+        flops += 2.0 * tokens * params
+    return flops + 2.0 * cfg["vocab"] * h, kv_bytes, state_bytes
+
+
 def compare_designs(args, peaks: dict) -> int:
     """Prefill of 2,048 tokens and decode at batch 8 with 1,024-token contexts, the named design
-    beside Qwen3 (Fikudra: beside Balivik; Nisotar: beside Fikudra) at equal sizes, each through
+    beside Qwen3 (Fikudra: beside Balivik; Nisotar: beside Fikudra; Katadra: beside Nisotar) at equal sizes, each through
     the same ``Executor.step`` and captured decode step."""
     import torch
     from mrun_b200 import Engine
     from mrun_b200.config import Qwen3Config, ZasesunConfig
     from mrun_b200.config.balivik import BalivikConfig
     from mrun_b200.config.fikudra import FikudraConfig
+    from mrun_b200.config.katadra import KatadraConfig
     from mrun_b200.config.nisotar import NisotarConfig
     from mrun_b200.engine import StepEntry
     context, batch = 1024, 8
@@ -505,17 +557,22 @@ def compare_designs(args, peaks: dict) -> int:
     sampler = ClockSampler()
     sampler.start()
     size_sets = {"zasesun": DESIGN_SIZES, "balivik": BALIVIK_SIZES, "fikudra": FIKUDRA_SIZES,
-                 "nisotar": NISOTAR_SIZES}[args.design]
-    beside = {"fikudra": "balivik", "nisotar": "fikudra"}.get(args.design, "qwen3")
+                 "nisotar": NISOTAR_SIZES, "katadra": KATADRA_SIZES}[args.design]
+    beside = {"fikudra": "balivik", "nisotar": "fikudra", "katadra": "nisotar"}.get(args.design, "qwen3")
     for name in (args.sizes.split(",") if args.sizes else sorted(size_sets)):
         z_sizes, q_sizes = size_sets[name]
         row = {}
         for design in (args.design, beside):
             state_bytes = 0
-            if design == "nisotar":
-                config = NisotarConfig.from_dict(z_sizes)
+            if design == "katadra":
+                config = KatadraConfig.from_dict(z_sizes)
                 vocab, h = z_sizes["vocab"], z_sizes["width"]
-                flops, kv_bytes, state_bytes = nisotar_counts(z_sizes, PREFILL_TOKENS, context)
+                flops, kv_bytes, state_bytes = katadra_counts(z_sizes, PREFILL_TOKENS)
+            elif design == "nisotar":
+                sizes = q_sizes if args.design == "katadra" else z_sizes
+                config = NisotarConfig.from_dict(sizes)
+                vocab, h = sizes["vocab"], sizes["width"]
+                flops, kv_bytes, state_bytes = nisotar_counts(sizes, PREFILL_TOKENS, context)
             elif design == "fikudra" and args.design == "nisotar":
                 config = FikudraConfig.from_dict(q_sizes)
                 vocab, h = q_sizes["vocab"], q_sizes["width"]
@@ -619,8 +676,8 @@ def main() -> int:
     parser.add_argument("--profiler-range", nargs="?", const="decode", default=None, choices=["decode", "prefill"],
                         help="bracket the timed decode steps (or the last timed prefill) with "
                              "cudaProfilerStart/Stop, for a profiler started with --profile-from-start off")
-    parser.add_argument("--design", choices=["zasesun", "balivik", "fikudra", "nisotar"], default=None,
-                        help="instead of the default workload: the named design beside Qwen3 (fikudra: beside Balivik; nisotar: beside Fikudra) at equal sizes "
+    parser.add_argument("--design", choices=["zasesun", "balivik", "fikudra", "nisotar", "katadra"], default=None,
+                        help="instead of the default workload: the named design beside Qwen3 (fikudra: beside Balivik; nisotar: beside Fikudra; katadra: beside Nisotar) at equal sizes "
                              "(prefill of 2,048 tokens, decode at batch 8)")
     parser.add_argument("--sizes", default=None, help="with --design: which of its size sets to run, comma separated")
     args = parser.parse_args()

@@ -27,6 +27,7 @@
 //                   or SiLU
 //   skip_gate_norm  per group of n outputs: y = (o + D_h x) * SiLU(z), then y / sqrt(mean(y^2) + eps) * w
 #include "common.cuh"
+#include "recurrent_walk.h"
 
 using namespace mrun;
 
@@ -99,26 +100,39 @@ causal_conv_kernel(const TA* __restrict__ x, long ldx, const float* __restrict__
 }
 
 // The same with eight channels a thread (channels a multiple of 8, rows on 16-byte boundaries):
-// 16-byte loads and stores, four tokens' loads in flight.
-template <typename TA>
+// 16-byte loads and stores, four tokens' loads in flight.  TAPS: the taps where they are known when the
+// kernel is compiled, else 0 (up to MAX_TAPS, registers for all of them).
+template <typename TA, int TAPS>
 __global__ void __launch_bounds__(128)
 causal_conv_vec_kernel(const TA* __restrict__ x, long ldx, const float* __restrict__ w, const float* __restrict__ bias,
-                       TA* __restrict__ state,
-                       TA* __restrict__ out, long ldo, const int* __restrict__ seg_q_start,
-                       const int* __restrict__ seg_slot, int C, int taps, int residual, int silu) {
+                       TA* __restrict__ state, TA* __restrict__ out, long ldo, const int* __restrict__ seg_q_start,
+                       const int* __restrict__ seg_slot, int C, int taps_given, int residual, int silu) {
+    constexpr int HELD = TAPS ? TAPS : MAX_TAPS;
+    const int taps = TAPS ? TAPS : taps_given;
     const int c = (blockIdx.x * blockDim.x + threadIdx.x) * 8;
     const int seg = blockIdx.z;
     const int q0 = seg_q_start[seg], n = seg_q_start[seg + 1] - q0;
     const int l0 = blockIdx.y * CONV_TILE;
     if (c >= C || l0 >= n) return;
     TA* st = state + (size_t)seg_slot[seg] * (taps - 1) * C + c;
-    float wv[8][MAX_TAPS], hist[MAX_TAPS - 1][8];      // hist[j - 1]: the inputs j tokens back
+    float wv[HELD][8], hist[HELD > 1 ? HELD - 1 : 1][8];      // wv[j], hist[j - 1]: of the input j tokens back
+    if constexpr (TAPS != 0) {          // a thread's 8 * TAPS weights lie side by side
+        float flat[8 * HELD];
 #pragma unroll
-    for (int ch = 0; ch < 8; ++ch)
+        for (int i = 0; i < HELD; ++i)
+            Vec8<float>::load(w + (size_t)c * TAPS + i * 8, *reinterpret_cast<float (*)[8]>(flat + i * 8));
 #pragma unroll
-        for (int j = 0; j < MAX_TAPS; ++j) wv[ch][j] = j < taps ? w[(size_t)(c + ch) * taps + (taps - 1 - j)] : 0.f;
+        for (int j = 0; j < HELD; ++j)
 #pragma unroll
-    for (int j = 1; j < MAX_TAPS; ++j) {
+            for (int ch = 0; ch < 8; ++ch) wv[j][ch] = flat[ch * HELD + (HELD - 1 - j)];
+    } else {
+#pragma unroll
+        for (int j = 0; j < HELD; ++j)
+#pragma unroll
+            for (int ch = 0; ch < 8; ++ch) wv[j][ch] = j < taps ? w[(size_t)(c + ch) * taps + (taps - 1 - j)] : 0.f;
+    }
+#pragma unroll
+    for (int j = 1; j < HELD; ++j) {
         if (j < taps) {
             const int l = l0 - j;
             if (l >= 0) Vec8<TA>::load(x + (size_t)(q0 + l) * ldx + c, hist[j - 1]);
@@ -130,7 +144,8 @@ causal_conv_vec_kernel(const TA* __restrict__ x, long ldx, const float* __restri
     }
     float shift[8];
 #pragma unroll
-    for (int ch = 0; ch < 8; ++ch) shift[ch] = bias ? bias[c + ch] : 0.f;
+    for (int ch = 0; ch < 8; ++ch) shift[ch] = 0.f;
+    if (bias) Vec8<float>::load(bias + c, shift);
     const int end = min(n, l0 + CONV_TILE);
     for (int lb = l0; lb < end; lb += 4) {
         float cur[4][8];
@@ -145,26 +160,28 @@ causal_conv_vec_kernel(const TA* __restrict__ x, long ldx, const float* __restri
             for (int ch = 0; ch < 8; ++ch) {
                 float acc = 0.f;
 #pragma unroll
-                for (int j = MAX_TAPS - 1; j >= 1; --j)          // oldest input first
-                    if (j < taps) acc = fmaf(wv[ch][j], hist[j - 1][ch], acc);
-                acc = fmaf(wv[ch][0], cur[k][ch], acc) + shift[ch];
+                for (int j = HELD - 1; j >= 1; --j)          // oldest input first
+                    if (j < taps) acc = fmaf(wv[j][ch], hist[j - 1][ch], acc);
+                acc = fmaf(wv[0][ch], cur[k][ch], acc) + shift[ch];
                 float v = residual ? cur[k][ch] + acc : acc;
-                if (silu) v = silu_f<true>(v);
+                if (silu) v = silu_f<sizeof(TA) == 4>(v);
                 y[ch] = v;
             }
             Vec8<TA>::store(out + (size_t)(q0 + lb + k) * ldo + c, y);
+            if constexpr (HELD > 1) {
 #pragma unroll
-            for (int j = MAX_TAPS - 1; j >= 2; --j)
+                for (int j = HELD - 1; j >= 2; --j)
 #pragma unroll
-                for (int ch = 0; ch < 8; ++ch) hist[j - 1][ch] = hist[j - 2][ch];
+                    for (int ch = 0; ch < 8; ++ch) hist[j - 1][ch] = hist[j - 2][ch];
 #pragma unroll
-            for (int ch = 0; ch < 8; ++ch) hist[0][ch] = cur[k][ch];
+                for (int ch = 0; ch < 8; ++ch) hist[0][ch] = cur[k][ch];
+            }
         }
     }
-    if (blockIdx.y == 0) {
-        float fresh[MAX_TAPS - 1][8];
+    if (HELD > 1 && blockIdx.y == 0) {
+        float fresh[HELD][8];
 #pragma unroll
-        for (int i = 0; i < MAX_TAPS - 1; ++i) {
+        for (int i = 0; i < HELD - 1; ++i) {
             if (i < taps - 1) {
                 const int l = n - (taps - 1) + i;
                 if (l >= 0) Vec8<TA>::load(x + (size_t)(q0 + l) * ldx + c, fresh[i]);
@@ -172,9 +189,22 @@ causal_conv_vec_kernel(const TA* __restrict__ x, long ldx, const float* __restri
             }
         }
 #pragma unroll
-        for (int i = 0; i < MAX_TAPS - 1; ++i)
+        for (int i = 0; i < HELD - 1; ++i)
             if (i < taps - 1) Vec8<TA>::store(st + (size_t)i * C, fresh[i]);
     }
+}
+
+template <typename TA>
+void launch_conv_vec(dim3 grid, const void* x, long ldx, const float* w, const float* bias, void* state, void* out, long ldo,
+                     const int* seg_q_start, const int* seg_slot, int C, int taps, int residual, int silu, cudaStream_t stream) {
+#define MRUN_CONV(TAPS)                                                                                                 \
+    causal_conv_vec_kernel<TA, TAPS><<<grid, 128, 0, stream>>>((const TA*)x, ldx, w, bias, (TA*)state, (TA*)out, ldo,    \
+                                                               seg_q_start, seg_slot, C, taps, residual, silu)
+    if (taps == 2) MRUN_CONV(2);
+    else if (taps == 3) MRUN_CONV(3);
+    else if (taps == 4) MRUN_CONV(4);
+    else MRUN_CONV(0);
+#undef MRUN_CONV
 }
 
 // ------------------------------------------------------------------------------------------
@@ -660,16 +690,14 @@ MRUN_API int mrun_causal_conv(const void* x, long ldx, const float* w, const flo
     MRUN_REQUIRE(tiles <= 65535, "causal_conv: a segment of %d tokens is too long", max_q_len);
     const size_t unit = act_dtype == MRUN_F32 ? 4 : 2;
     const bool vec = C % 8 == 0 && (ldx * unit) % 16 == 0 && (ldo * unit) % 16 == 0 &&
-                     ((((uintptr_t)x) | ((uintptr_t)out) | ((uintptr_t)state)) & 15) == 0 && (C * unit) % 16 == 0;
+                     ((((uintptr_t)x) | ((uintptr_t)out) | ((uintptr_t)state) | ((uintptr_t)w) | ((uintptr_t)bias)) & 15) == 0 && (C * unit) % 16 == 0;
     if (vec) {
         const dim3 vec_grid((C / 8 + 127) / 128, tiles, segments);
         if (act_dtype == MRUN_F32)
-            causal_conv_vec_kernel<float><<<vec_grid, 128, 0, stream>>>((const float*)x, ldx, w, bias, (float*)state, (float*)out,
-                                                                         ldo, seg_q_start, seg_slot, C, taps, residual, silu);
+            launch_conv_vec<float>(vec_grid, x, ldx, w, bias, state, out, ldo, seg_q_start, seg_slot, C, taps, residual, silu, stream);
         else if (act_dtype == MRUN_BF16)
-            causal_conv_vec_kernel<__nv_bfloat16><<<vec_grid, 128, 0, stream>>>(
-                (const __nv_bfloat16*)x, ldx, w, bias, (__nv_bfloat16*)state, (__nv_bfloat16*)out, ldo, seg_q_start, seg_slot, C,
-                taps, residual, silu);
+            launch_conv_vec<__nv_bfloat16>(vec_grid, x, ldx, w, bias, state, out, ldo, seg_q_start, seg_slot, C, taps, residual, silu,
+                                           stream);
         else
             return mrun_set_error("causal_conv: unknown dtype code %d", act_dtype);
         MRUN_CHECK_LAUNCH("causal_conv");
@@ -760,6 +788,17 @@ MRUN_API int mrun_gated_scan(const void* q, const void* k, const void* v, long l
     return 0;
 }
 
+// 1 where the register-tiled walk (recurrent_walk.cu) runs a bonus (ssm = 0) or a state-space scan (ssm = 1)
+// with these rows: the scan then needs no scratch.
+MRUN_API int mrun_scan_walks(int ssm, const void* q, const void* k, const void* v, long ld, int act_dtype, const float* a,
+                             const float* bias, const float* bonus, const float* state, int D, int V) {
+    WalkArgs w = {};
+    w.mode = ssm ? WALK_SSM : WALK_BONUS;
+    w.q = q; w.k = k; w.v = v; w.ld = ld; w.a = a; w.bias = bias; w.bonus = bonus; w.state = (float*)state; w.D = D; w.V = V;
+    return walk_takes(w, act_dtype) ? 1 : 0;
+}
+
+// scratch: may be null where mrun_scan_walks() says so.
 // q (the read vector), k, v: [H, D] a row (stride ld); a: float32 [tokens, H * D], bias: float32 [H * D],
 // the decay is exp(-exp(a + bias)); bonus: float32 [H * D].
 MRUN_API int mrun_bonus_scan(const void* q, const void* k, const void* v, long ld, int act_dtype, const float* a,
@@ -770,6 +809,9 @@ MRUN_API int mrun_bonus_scan(const void* q, const void* k, const void* v, long l
     MRUN_REQUIRE(D <= 256, "bonus_scan: key size %d exceeds the supported 256", D);
     MRUN_REQUIRE(H <= 65535 && segments <= 65535, "bonus_scan: %d heads or %d segments exceed 65535", H, segments);
     if (segments == 0 || tokens == 0) return 0;
+    const WalkArgs w = {WALK_BONUS, q, k, v, ld, a, nullptr, 0, bias, nullptr, bonus, state, out, seg_q_start, seg_slot, 1, H, D, V, 0};
+    if (walk_takes(w, act_dtype)) return launch_walk(w, act_dtype, segments, stream);
+    MRUN_REQUIRE(scratch != nullptr, "bonus_scan: these sizes need scratch");
     if (act_dtype == MRUN_F32)
         launch_scan<float, SCAN_BONUS>(q, k, v, ld, 1, a, nullptr, 0, nullptr, bias, nullptr, bonus, state, out, scratch,
                                        seg_q_start, seg_slot, segments, tokens, H, D, V, 0, 1.f, stream);
@@ -792,6 +834,10 @@ MRUN_API int mrun_ssm_scan(const void* c, const void* b, const void* x, long ld,
     MRUN_REQUIRE(N <= 256, "ssm_scan: state size %d exceeds the supported 256", N);
     MRUN_REQUIRE(H <= 65535 && segments <= 65535, "ssm_scan: %d heads or %d segments exceed 65535", H, segments);
     if (segments == 0 || tokens == 0) return 0;
+    const WalkArgs w = {WALK_SSM, c, b, x, ld, nullptr, dt, lddt, dt_bias, a_log, nullptr, state, out, seg_q_start, seg_slot,
+                        group, H, N, V, 0};
+    if (walk_takes(w, act_dtype)) return launch_walk(w, act_dtype, segments, stream);
+    MRUN_REQUIRE(scratch != nullptr, "ssm_scan: these sizes need scratch");
     if (act_dtype == MRUN_F32)
         launch_scan<float, SCAN_SSM>(c, b, x, ld, group, nullptr, dt, lddt, a_log, dt_bias, nullptr, nullptr, state, out,
                                      scratch, seg_q_start, seg_slot, segments, tokens, H, N, V, 0, 1.f, stream);

@@ -1,0 +1,690 @@
+"""Katadra on the GPU against the plain implementation (``plain_katadra``): every new kernel and every
+part alone (whole requests, token by token, portions down to one and two tokens, unequal requests
+side by side, state slots and pages given back and used again), inputs made so that one far key, one
+bucket of the distance table, the cap, the temperature or a kept state decides the result, then whole
+models replayed through ``bin/trace_run`` cut in every way, then greedy generation through
+``Engine.generate`` and the command line."""
+from __future__ import annotations
+
+import numpy as np
+import pytest
+import torch
+
+import plain_katadra as plain
+from test_fikudra_gpu import LENGTHS, SIZES, TRACE_LENGTHS, Steps, check_rows, close, named, random_tensors, runtime
+from test_nisotar_gpu import edge_cuts, run_cut
+from tiny_katadra import KTINY, load_folder, make_folder, tokens_of
+from trace_tools import TraceBuilder, TraceRunner, cut_decode_tail, cut_mixed, cut_portions, cut_whole
+
+pytestmark = pytest.mark.gpu
+DEV = "cuda:0"
+F64 = torch.float64
+
+
+# ------------------------------------------------------------------ kernels alone
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("hidden", [8, 100, 1027, 4096, 13000])
+def test_post_layernorm_add_kernel(dtype, hidden):
+    """A branch's layer norm on its way into the stream; what comes out are the new rows, their layer
+    norm, or nothing; in place and at chosen rows; a large common offset of the branch must not cost
+    its variance the digits."""
+    from mrun_b200.kernels import ops
+    act = getattr(torch, dtype)
+    gen = torch.Generator().manual_seed(hidden)
+    rand = lambda *s: torch.randn(*s, generator=gen)
+    resid, branch = rand(9, hidden) * 2 - 5.0, rand(9, hidden) * 3 + 40.0
+    w, b, w2, b2 = 1 + 0.3 * rand(hidden), 0.4 * rand(hidden), 1 + 0.3 * rand(hidden), 0.4 * rand(hidden)
+    bound = 2e-5 if dtype == "float32" else 1e-2
+    rows = torch.tensor([8, 0, 3], dtype=torch.int32)
+    for bias in (True, False):
+        zero = torch.zeros(hidden)
+        addend = plain.layer_norm(branch.double(), w.double(), (b if bias else zero).double(), 1e-5)
+        pending = ops.PendingPostLayerNorm(branch.to(DEV), w.to(DEV), b.to(DEV) if bias else None, 1e-5)
+        close(pending.compute(), addend, "float32", "the addend alone", bound=2e-5)
+        total = resid.double() + addend
+        for next_norm in (False, True):
+            want = plain.layer_norm(total, w2.double(), (b2 if bias else zero).double(), 1e-4) if next_norm else total
+            args = (w2.to(DEV), b2.to(DEV) if bias else None, 1e-4) if next_norm else (None, None, 0.0)
+            stream = resid.to(DEV)
+            out = torch.empty((9, hidden), dtype=act, device=DEV)
+            ops.post_layernorm_add(stream, pending, *args, out=out)
+            close(out, want, dtype, "all rows", bound=bound)
+            close(stream, total, "float32", "the stream", bound=2e-5)
+            stream = resid.to(DEV)
+            out = torch.empty((3, hidden), dtype=act, device=DEV)
+            ops.post_layernorm_add(stream, pending, *args, out=out, rows=rows.to(DEV))
+            close(out, want[rows.long()], dtype, "chosen rows", bound=bound)
+            assert torch.equal(stream.cpu(), resid)
+    stream = resid.to(DEV)
+    ops.post_layernorm_add(stream, pending)                                    # nothing comes out
+    close(stream, total, "float32", "the stream alone", bound=2e-5)
+    out = torch.empty((9, hidden), dtype=act, device=DEV)
+    ops.post_layernorm_add(stream, None, out=out)                              # no branch: the rows, narrowed
+    assert torch.equal(out, stream.to(act))
+    # the layer norm of the framework's other arrangements, with a bias
+    out = torch.empty((9, hidden), dtype=act, device=DEV)
+    ops.add_layernorm(resid.to(DEV), None, w.to(DEV), 1e-5, out, bias=b.to(DEV))
+    close(out, plain.layer_norm(resid.double(), w.double(), b.double(), 1e-5), dtype, "with a bias", bound=bound)
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("heads, vdim, groups", [(3, 7, 1), (3, 7, 3), (16, 64, 8), (20, 64, 1), (64, 64, 2), (96, 128, 1), (24, 40, 12)])
+def test_skip_gate_norm_kernel(dtype, heads, vdim, groups):
+    from mrun_b200.kernels import ops
+    act = getattr(torch, dtype)
+    gen = torch.Generator().manual_seed(heads * vdim + groups)
+    inner, tokens = heads * vdim, 11
+    o = torch.randn(tokens, inner, generator=gen)
+    pad = 8 if inner % 8 == 0 else 5
+    x = torch.randn(tokens, inner + pad, generator=gen).to(act)
+    z = torch.randn(tokens, inner + pad, generator=gen).to(act)
+    skip, w = torch.randn(heads, generator=gen), 1 + 0.3 * torch.randn(inner, generator=gen)
+    got = ops.skip_gate_norm(o.to(DEV), x.to(DEV)[:, :inner], skip.to(DEV), z.to(DEV)[:, :inner], w.to(DEV), 1e-3, groups)
+    y = (o.double() + skip.double().repeat_interleave(vdim) * x[:, :inner].double()) * plain.silu(z[:, :inner].double())
+    want = plain.unit_rms(y.view(tokens, groups, -1), 1e-3).reshape(tokens, inner) * w.double()
+    close(got, want, dtype, "rows", bound=1e-5 if dtype == "float32" else 1e-2)
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("rows, batch, n, k", [(1, 4, 64, 64), (8, 3, 40, 96), (13, 4, 200, 2048), (16, 1, 7, 32), (5, 2, 24, 37),
+                                               (40, 4, 64, 96), (3, 5, 4096, 128)])
+def test_batched_products_and_products_with_an_activation(dtype, rows, batch, n, k):
+    """One launch for several products of different inputs; relu^2 and tanh behind a product, in the
+    decode GEMM's epilogue and behind the other products."""
+    from mrun_b200.kernels import ops
+    act = getattr(torch, dtype)
+    gen = torch.Generator().manual_seed(rows * n + k)
+    wide = torch.randn(rows, batch + 1, k, generator=gen).to(act)
+    w = (torch.randn(batch, n, k, generator=gen) * k ** -0.5).to(act)
+    x = wide.to(DEV)[:, :batch]
+    got = ops.linears_batched(x, w.to(DEV))
+    want = torch.einsum("tbk,bnk->tbn", wide[:, :batch].double(), w.double())
+    close(got, want, dtype, "products", bound=1e-5 if dtype == "float32" else 1e-2)
+    for name, fn in (("relu2", lambda v: torch.relu(v) ** 2), ("tanh", torch.tanh)):
+        got = ops.linear_act(x[:, 0], w[0].to(DEV), name)
+        close(got, fn(want[:, 0]), dtype, name, bound=1e-5 if dtype == "float32" else 2e-2)
+
+
+# ------------------------------------------------------------------ attention
+
+def attention_spec(hidden, m):
+    from mrun_b200.config.spec import GatedAttentionSpec
+    return GatedAttentionSpec(hidden=hidden, heads=m["heads"], kv_heads=m["kv_heads"], dim=m["dim"], vdim=m["vdim"],
+                              softmax_scale=m["scale"], eps=1e-5, qk_norm="unit", sink=False, head_gate=False,
+                              temperature=(m["q_temp"]["coef"], m["q_temp"]["every"]), soft_cap=m["softcap"],
+                              distance_bias=(m["bias_rows"], m["bias_max"]), element_gate=True)
+
+
+def entry(heads, kv_heads, dim, vdim, scale=0.3, cap=4.0, rows=8, reach=60, coef=0.5, every=9):
+    return {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale, "softcap": cap, "bias_rows": rows,
+            "bias_max": reach, "q_temp": {"coef": coef, "every": every}}
+
+
+def attention_weights(spec, seed, bias=1.0):
+    from mrun_b200.parts import MIXERS
+    w = random_tensors(MIXERS.tensor_specs(spec, "m"), "m", torch.Generator().manual_seed(seed))
+    w["rel"] = (w["rel"] / 0.3 * bias).to(torch.bfloat16).float()
+    return w
+
+
+ATTENTION_SHAPES = [
+    (entry(6, 3, 24, 40, cap=2.0, rows=6, reach=33.5), 16),
+    (entry(5, 5, 11, 7, cap=30.0, rows=2, reach=9), 4),
+    (entry(4, 2, 64, 64, scale=0.125, cap=30.0, rows=32, reach=128), 16),      # bfloat16: tcgen05 and TMA, every tanh small
+    (entry(4, 2, 64, 64, scale=0.4, cap=5.0, rows=16, reach=100), 16),         # the same, no tanh small
+    (entry(3, 1, 128, 64, scale=0.09, cap=9.0, rows=8, reach=40, coef=2.0, every=3), 8),      # small for the first positions only
+    (entry(2, 2, 64, 128, scale=0.2, cap=8.0), 16),
+    (entry(4, 1, 128, 128, scale=0.1, cap=40.0, rows=64, reach=1000), 16),     # a table longer than every request
+    (entry(6, 3, 48, 16), 8),
+    (entry(4, 4, 32, 80, coef=0.0), 16),
+    (entry(34, 2, 16, 16, cap=50.0), 16),                                      # seventeen query heads a kv head
+    (entry(2, 1, 96, 32, rows=10, reach=10), 16),
+]
+
+
+@pytest.mark.parametrize("dtype, tensor_cores", [("float32", False), ("bfloat16", False), ("bfloat16", True)])
+@pytest.mark.parametrize("m, page", ATTENTION_SHAPES)
+def test_attention_alone(dtype, tensor_cores, m, page, monkeypatch):
+    from mrun_b200.parts import MIXERS, gated_attention
+    monkeypatch.setattr(gated_attention, "TENSOR_CORES", tensor_cores)
+    rt = runtime(dtype, page)
+    spec = attention_spec(40, m)
+    w = attention_weights(spec, m["dim"] + m["vdim"])
+    part = MIXERS.build(spec, w, rt)
+    if tensor_cores and not part.tensor_cores:
+        pytest.skip("the tensor-core kernels do not take this shape")
+    W = named(w, "m.")
+    check_rows(lambda rows, ctx, caches: part.forward(rows, ctx, caches[0]), 40, dtype, LENGTHS,
+               lambda h, _: plain.biased_attention(m, W, "m.", h, 1e-5), [part.cache_need()], rt)
+
+
+@pytest.mark.parametrize("tma, tc5, cluster", [(True, True, True), (True, True, False), (False, False, False)])
+@pytest.mark.parametrize("m", [entry(4, 2, 128, 128, scale=0.1, cap=25.0, rows=32, reach=200), entry(8, 1, 64, 128, scale=0.3, cap=6.0, rows=8, reach=30),
+                               entry(2, 2, 128, 64, scale=0.1, cap=20.0, rows=64, reach=2000), entry(3, 3, 48, 16, rows=16, reach=300)])
+def test_long_context_on_every_tensor_core_kernel(m, tma, tc5, cluster, monkeypatch):
+    """Prompt tiles and decode splits that lie wholly beyond the table's reach, wholly within and across
+    its end, on the tcgen05 / TMA kernels and on the older ones, in one piece and cut."""
+    from mrun_b200.kernels import attention
+    from mrun_b200.parts import MIXERS
+    for name, value in (("TMA_DECODE", tma), ("TC5_PREFILL", tc5), ("CLUSTER_DECODE", cluster)):
+        monkeypatch.setattr(attention, name, value)
+    rt = runtime("bfloat16", 16)
+    spec = attention_spec(40, m)
+    w = attention_weights(spec, 3, bias=2.0)
+    part = MIXERS.build(spec, w, rt)
+    assert part.tensor_cores
+    W = named(w, "m.")
+    total = 1100
+    x = torch.randn(total, 40, generator=torch.Generator().manual_seed(9)).to(torch.bfloat16).float()
+    want = plain.biased_attention(m, W, "m.", x.double(), 1e-5)
+    for portions in ([total], [1060] + [1] * 40, [500, 1, 300, 2, 257] + [1] * 40, [70] * 15 + [50]):
+        got = run_cut(part, rt, x, portions, pages=-(-total // 16) + 2)
+        close(got, want, "bfloat16", f"portions {portions[:6]}")
+
+
+@pytest.mark.parametrize("dtype, tensor_cores", [("float32", False), ("bfloat16", False), ("bfloat16", True)])
+@pytest.mark.parametrize("dim, vdim, rows, reach, page", [(64, 64, 8, 40, 16), (20, 12, 6, 21, 8), (48, 16, 8, 64, 16), (128, 64, 16, 90, 4)])
+def test_one_bucket_of_the_distance_table(dtype, tensor_cores, dim, vdim, rows, reach, page, monkeypatch):
+    """One row of the table stands far above the others, so that a query sees the keys of that bucket
+    only: the first, each side of where distances begin to share a row, one in the middle, the last one
+    before the end and the one that takes everything beyond.  The plain run is asserted to change at
+    every later position when the bucket next to it stands out instead."""
+    from mrun_b200.parts import MIXERS, gated_attention
+    monkeypatch.setattr(gated_attention, "TENSOR_CORES", tensor_cores)
+    rt = runtime(dtype, page)
+    m = entry(2, 1, dim, vdim, scale=0.2, cap=20.0, rows=rows, reach=reach, coef=0.0)
+    spec = attention_spec(32, m)
+    total = 2 * reach + 60
+    gen = torch.Generator().manual_seed(dim)
+    x = torch.randn(total, 32, generator=gen).to(rt.precision.act).float()
+    for bucket in sorted({0, 1, rows // 2 - 1, rows // 2, (3 * rows) // 4, rows - 2, rows - 1}):
+        w = attention_weights(spec, 5, bias=0.3)
+        w["rel"][bucket] += 25.0
+        part = MIXERS.build(spec, w, rt)
+        if tensor_cores and not part.tensor_cores:
+            pytest.skip("the tensor-core kernels do not take this shape")
+        W = named(w, "m.")
+        want = plain.biased_attention(m, W, "m.", x.double(), 1e-5)
+        other = W["m.rel"].clone()
+        other[[bucket, (bucket + 1) % rows]] = other[[(bucket + 1) % rows, bucket]]
+        change = plain.biased_attention(m, dict(W, **{"m.rel": other}), "m.", x.double(), 1e-5) - want
+        assert float(change[reach + 5:].abs().max(1).values.min() / want.abs().max()) > 0.01
+        for portions in edge_cuts(total, total // 2):
+            got = run_cut(part, rt, x, portions, pages=-(-total // page) + 2)
+            close(got, want, dtype, f"bucket {bucket}, portions {portions[:8]}")
+
+
+@pytest.mark.parametrize("dtype, tensor_cores", [("float32", False), ("bfloat16", False), ("bfloat16", True)])
+@pytest.mark.parametrize("dim, vdim, page", [(16, 48, 8), (64, 64, 16), (128, 128, 16), (20, 33, 4)])
+def test_one_far_key_finds_its_queries(dtype, tensor_cores, dim, vdim, page, monkeypatch):
+    """One key and the queries that look for it are made so that their score dominates a head: at the
+    first token, on both sides of a page border and hundreds of tokens back, asked for from inside a
+    prompt portion, by tokens decoded alone and from portions of two and three tokens."""
+    from mrun_b200.parts import MIXERS, gated_attention
+    monkeypatch.setattr(gated_attention, "TENSOR_CORES", tensor_cores)
+    rt = runtime(dtype, page)
+    hidden, heads = 32, 2
+    m = entry(heads, 1, dim, vdim, scale=0.9, cap=60.0, rows=8, reach=30, coef=0.3, every=50)
+    spec = attention_spec(hidden, m)
+    w = attention_weights(spec, 17 + dim, bias=0.5)
+    w = {k: (v * 0.3 if k in ("q", "k") else v) for k, v in w.items()}
+    w["q"][:, :2] = 0; w["k"][:, :2] = 0; w["g"][:, :2] = 0; w["v"][:, 1] = 0
+    for row in (dim - 1, 2 * dim - 1):                  # the last feature of both heads' queries reads input column 1 alone
+        w["q"][row] = 0; w["q"][row, 1] = 1
+    w["k"][dim - 1] = 0; w["k"][dim - 1, 0] = 1         # and the key's column 0
+    part = MIXERS.build(spec, w, rt)
+    if tensor_cores and not part.tensor_cores:
+        pytest.skip("the tensor-core kernels do not take this shape")
+    W = named(w, "m.")
+    total = 360
+    gen = torch.Generator().manual_seed(4)
+    for far in (0, page - 1, page, 130):
+        x = torch.randn(total, hidden, generator=gen) * 0.5
+        x[:, :2] = 0
+        x[far, 0] = 30.0
+        asking = sorted({far + 1, far + 31, 200, 345, 359})
+        x[asking, 1] = 30.0
+        x = x.to(rt.precision.act).float()
+        want = plain.biased_attention(m, W, "m.", x.double(), 1e-5)
+        lost = x.clone(); lost[far, 0] = 0
+        change = (want - plain.biased_attention(m, W, "m.", lost.double(), 1e-5)).abs().max(1).values / want.abs().max()
+        assert float(change[asking].min()) > 0.1
+        for portions in edge_cuts(total, 346):
+            got = run_cut(part, rt, x, portions, pages=-(-total // page) + 2)
+            close(got[asking], want[asking], dtype, f"key at {far}, portions {portions[:8]}: the queries that look for it")
+            close(got, want, dtype, f"key at {far}, portions {portions[:8]}: all tokens")
+
+
+def test_cap_and_temperature_change_the_plain_result():
+    """The shapes above would notice a cap or a temperature left out."""
+    m = entry(4, 2, 64, 64, scale=0.4, cap=5.0, rows=16, reach=100)
+    spec = attention_spec(40, m)
+    W = named(attention_weights(spec, 128), "m.")
+    h = torch.randn(60, 40, generator=torch.Generator().manual_seed(1), dtype=F64)
+    want = plain.biased_attention(m, W, "m.", h, 1e-5)
+    for other in (dict(m, softcap=1e6), dict(m, q_temp={"coef": 0.0, "every": 9}), dict(m, q_temp={"coef": 0.5, "every": 10}),
+                  dict(m, bias_max=101)):
+        got = plain.biased_attention(other, W, "m.", h, 1e-5)
+        assert float((got - want).abs().max() / want.abs().max()) > 1e-3
+
+
+# ------------------------------------------------------------------ recurrent mixers
+
+def time_spec(hidden, heads, dim, rank):
+    from mrun_b200.config.spec import TimeMixingSpec
+    return TimeMixingSpec(hidden=hidden, heads=heads, dim=dim, rank=rank, eps=1e-5)
+
+
+def time_weights(spec, seed):
+    from mrun_b200.parts import MIXERS
+    gen = torch.Generator().manual_seed(seed)
+    w = random_tensors(MIXERS.tensor_specs(spec, "m"), "m", gen)
+    w["w0"] = (torch.rand(w["w0"].shape, generator=gen) * 7 - 6).to(torch.bfloat16).float()       # decays from near 1 to near 0
+    w["u"] = (w["u"] * 4).to(torch.bfloat16).float()
+    return w
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("hidden, heads, dim, rank", [(48, 4, 16, 8), (37, 1, 13, 3), (64, 3, 32, 32), (40, 2, 64, 5), (64, 2, 128, 16), (24, 16, 72, 8),
+                                                      (32, 5, 8, 2),
+                                                      (96, 1, 200, 7)])
+def test_time_mixing_alone(dtype, hidden, heads, dim, rank):
+    from mrun_b200.parts import MIXERS
+    rt = runtime(dtype)
+    spec = time_spec(hidden, heads, dim, rank)
+    w = time_weights(spec, heads + dim)
+    part = MIXERS.build(spec, w, rt)
+    W = named(w, "m.")
+    m = {"heads": heads, "dim": dim}
+    # sixteen heads of 72: a step of one request and one of three take different register tiles of the walk;
+    # a head whose first read-outs are all but zero before their norm is ill-conditioned in bfloat16
+    check_rows(lambda rows, ctx, caches: part.forward(rows, ctx, caches[0]), hidden, dtype, LENGTHS,
+               lambda h, _: plain.time_mixing(m, W, "m.", h, 1e-5), [part.cache_need()], rt,
+               bound=None if dtype == "float32" else 6e-2)
+
+
+def ssm_spec(hidden, heads, vdim, state, groups, conv, parts):
+    from mrun_b200.config.spec import StateSpaceSpec
+    return StateSpaceSpec(hidden=hidden, heads=heads, vdim=vdim, state=state, groups=groups, conv=conv, norm_groups=parts, eps=1e-5)
+
+
+def ssm_weights(spec, seed):
+    from mrun_b200.parts import MIXERS
+    gen = torch.Generator().manual_seed(seed)
+    w = random_tensors(MIXERS.tensor_specs(spec, "m"), "m", gen)
+    w["A_log"] = (torch.rand(w["A_log"].shape, generator=gen) * 6 - 5).to(torch.bfloat16).float()
+    w["dt_bias"] = (w["dt_bias"] * 6).to(torch.bfloat16).float()
+    w["D"] = torch.randn(w["D"].shape, generator=gen).to(torch.bfloat16).float()
+    return w
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("hidden, heads, vdim, state, groups, conv, parts", [
+    (48, 4, 24, 16, 2, 4, 2), (37, 3, 7, 9, 1, 1, 3), (64, 8, 16, 64, 8, 2, 1), (40, 2, 33, 130, 1, 8, 6), (64, 16, 64, 128, 4, 3, 1),
+    (32, 6, 10, 200, 3, 5, 12), (32, 3, 12, 200, 1, 4, 1), (32, 5, 8, 8, 5, 2, 1), (24, 48, 32, 128, 4, 2, 1), (24, 4, 20, 40, 2, 3, 4)])
+def test_state_space_alone(dtype, hidden, heads, vdim, state, groups, conv, parts):
+    from mrun_b200.parts import MIXERS
+    rt = runtime(dtype)
+    spec = ssm_spec(hidden, heads, vdim, state, groups, conv, parts)
+    w = ssm_weights(spec, heads + state)
+    part = MIXERS.build(spec, w, rt)
+    W = named(w, "m.")
+    m = {"heads": heads, "vdim": vdim, "state": state, "groups": groups, "conv": conv, "norm_groups": parts}
+    check_rows(lambda rows, ctx, caches: part.forward(rows, ctx, caches[0]), hidden, dtype, LENGTHS,
+               lambda h, _: plain.mamba2(m, W, "m.", h, 1e-5), [part.cache_need()], rt,
+               bound=None if dtype == "float32" else 6e-2)
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_time_mixing_keeps_a_far_key_by_channel(dtype):
+    """Key channel 0 never decays, channel 1 forgets at once.  A key written into both answers a query
+    on channel 0 hundreds of tokens later (in the prompt, in a later portion, decoded alone) and one
+    on channel 1 only as the current token's bonus."""
+    from mrun_b200.parts import MIXERS
+    rt = runtime(dtype)
+    hidden, heads, dim = 32, 1, 16
+    spec = time_spec(hidden, heads, dim, 2)
+    w = time_weights(spec, 3)
+    w = {k: (v * 0.1 if k in ("r", "k", "v") else v) for k, v in w.items()}
+    for name in "rkvgw":
+        w["mu." + name].zero_()                         # no shift: every row reads itself
+    w["w1"].zero_()
+    w["w0"][:] = -1.0
+    w["w0"][0], w["w0"][1] = -60.0, 5.0                 # exp(-e^-60) = 1; exp(-e^5) = 0
+    for row, column in ((0, 1), (1, 2)):
+        w["k"][row] = 0; w["k"][row, 0] = 1             # both channels' keys read column 0; the queries columns 1 and 2
+        w["r"][row] = 0; w["r"][row, column] = 1
+    w["r"][2:, :3] = 0; w["k"][2:, :3] = 0; w["v"][:, 1:3] = 0; w["g"][:, :3] = 0
+    part = MIXERS.build(spec, w, rt)
+    W = named(w, "m.")
+    m = {"heads": heads, "dim": dim}
+    total = 420
+    x = torch.randn(total, hidden, generator=torch.Generator().manual_seed(8)) * 0.3
+    x[:, :3] = 0
+    x[5, 0] = 8.0
+    keepers, forgetters = [6, 130, 300, 401, 419], [131, 402]
+    x[keepers, 1] = 8.0
+    x[forgetters, 2] = 8.0
+    x = x.to(rt.precision.act).float()
+    want = plain.time_mixing(m, W, "m.", x.double(), 1e-5)
+    lost = x.clone(); lost[5, 0] = 0
+    change = (want - plain.time_mixing(m, W, "m.", lost.double(), 1e-5)).abs().max(1).values / want.abs().max()
+    assert float(change[keepers].min()) > 0.1 and float(change[forgetters].max()) < 1e-3
+    for portions in ([400] + [1] * 20, [3, 2, 2, 100, 193, 100] + [1] * 20):
+        got = run_cut(part, rt, x, portions, pages=8)
+        close(got[keepers], want[keepers], dtype, "queries on the kept channel")
+        close(got, want, dtype, "all tokens", bound=None if dtype == "float32" else 6e-2)
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_state_space_keeps_a_far_input_by_head(dtype):
+    """Head 0 never decays, head 1 forgets at once: an input written once is read from head 0 hundreds
+    of tokens later by the tokens whose C points at it."""
+    from mrun_b200.parts import MIXERS
+    rt = runtime(dtype)
+    hidden, heads, vdim, state = 32, 2, 8, 16
+    spec = ssm_spec(hidden, heads, vdim, state, 1, 2, 2)
+    w = ssm_weights(spec, 5)
+    inner = heads * vdim
+    w["in"] = w["in"] * 0.1
+    w["in"][:, :3] = 0
+    w["in"][2 * inner, 0] = 1                           # B_0 reads column 0
+    w["in"][2 * inner + state, 1] = 1                   # C_0 reads column 1
+    w["in"][inner:2 * inner, 0] = 0.5                   # and the input itself
+    w["in"][-heads:] = 0
+    w["dt_bias"][:] = 1.0
+    w["A_log"][0], w["A_log"][1] = -60.0, 6.0
+    w["conv"][:, 0] = 0; w["conv"][:, 1] = 1; w["conv.b"][:] = 0
+    part = MIXERS.build(spec, w, rt)
+    W = named(w, "m.")
+    m = {"heads": heads, "vdim": vdim, "state": state, "groups": 1, "conv": 2, "norm_groups": 2}
+    total = 420
+    x = torch.randn(total, hidden, generator=torch.Generator().manual_seed(8)) * 0.3
+    x[:, :3] = 0
+    x[5, 0] = 6.0
+    asking = [6, 130, 300, 401, 419]
+    x[asking, 1] = 8.0
+    x = x.to(rt.precision.act).float()
+    want = plain.mamba2(m, W, "m.", x.double(), 1e-5)
+    lost = x.clone(); lost[5, 0] = 0
+    change = (want - plain.mamba2(m, W, "m.", lost.double(), 1e-5)).abs().max(1).values / want.abs().max()
+    assert float(change[asking].min()) > 0.1
+    for portions in ([400] + [1] * 20, [3, 2, 2, 100, 193, 100] + [1] * 20):
+        got = run_cut(part, rt, x, portions, pages=8)
+        close(got[asking], want[asking], dtype, "the tokens that ask")
+        close(got, want, dtype, "all tokens", bound=None if dtype == "float32" else 6e-2)
+
+
+@pytest.mark.parametrize("dtype, tensor_cores", [("float32", False), ("bfloat16", False), ("bfloat16", True)])
+@pytest.mark.parametrize("a, r, scales, page", [(entry(4, 2, 32, 80), (3, 24, 5), (0.7, 1.2), 8), (entry(3, 1, 11, 5), (1, 13, 2), (-0.5, 1.0), 16),
+                                                (entry(2, 1, 128, 64, scale=0.1), (2, 64, 16), (1.0, 0.3), 16),
+                                                (entry(4, 4, 64, 64, scale=0.2), (4, 16, 8), (0.0, 1.0), 4)])
+def test_scaled_sum_of_two_mixers_alone(dtype, tensor_cores, a, r, scales, page, monkeypatch):
+    from mrun_b200.config.spec import ParallelMixerSpec
+    from mrun_b200.parts import MIXERS, gated_attention
+    monkeypatch.setattr(gated_attention, "TENSOR_CORES", tensor_cores)
+    rt = runtime(dtype, page)
+    spec = ParallelMixerSpec(hidden=48, left=attention_spec(48, a), right=time_spec(48, *r), eps=1e-5, combine="sum", scales=scales)
+    w = {f"left.{k}": v for k, v in attention_weights(spec.left, 2).items()}
+    w.update({f"right.{k}": v for k, v in time_weights(spec.right, 7).items()})
+    part = MIXERS.build(spec, w, rt)
+    W = named(w, "m.")
+    m = {"left": a, "right": {"heads": r[0], "dim": r[1]}, "left_scale": scales[0], "right_scale": scales[1]}
+    check_rows(lambda rows, ctx, caches: part.forward(rows, ctx, caches[0]), 48, dtype, LENGTHS,
+               lambda h, _: plain.parallel_mixer(m, W, "m.", h, 1e-5), [part.cache_need()], rt,
+               bound=None if dtype == "float32" else 6e-2)
+
+
+def test_two_mixers_with_states_of_one_name_are_refused():
+    from mrun_b200.config.spec import ParallelMixerSpec
+    from mrun_b200.parts import MIXERS
+    left, right = ssm_spec(48, 4, 8, 16, 1, 3, 1), time_spec(48, 2, 16, 4)
+    spec = ParallelMixerSpec(hidden=48, left=left, right=right, eps=1e-5, combine="sum", scales=(0.4, -1.5))
+    w = {f"left.{k}": v for k, v in ssm_weights(left, 2).items()}
+    w.update({f"right.{k}": v for k, v in time_weights(right, 7).items()})
+    with pytest.raises(TypeError, match="different names"):
+        MIXERS.build(spec, w, runtime("float32"))
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_scaled_sum_of_mixers_that_keep_their_products(dtype):
+    """A side that does not offer its rows in front of its output projection (the state space): the two
+    outputs are scaled and added as they are."""
+    from mrun_b200.config.spec import ParallelMixerSpec
+    from mrun_b200.parts import MIXERS
+    rt = runtime(dtype)
+    a = entry(4, 2, 32, 16)
+    left, right = attention_spec(48, a), ssm_spec(48, 4, 8, 16, 1, 3, 1)
+    spec = ParallelMixerSpec(hidden=48, left=left, right=right, eps=1e-5, combine="sum", scales=(0.4, -1.5))
+    w = {f"left.{k}": v for k, v in attention_weights(left, 2).items()}
+    w.update({f"right.{k}": v for k, v in ssm_weights(right, 7).items()})
+    part = MIXERS.build(spec, w, rt)
+    assert part.w_o is None
+    W = named(w, "m.")
+    m = {"heads": 4, "vdim": 8, "state": 16, "groups": 1, "conv": 3, "norm_groups": 1}
+    check_rows(lambda rows, ctx, caches: part.forward(rows, ctx, caches[0]), 48, dtype, LENGTHS,
+               lambda h, _: 0.4 * plain.biased_attention(a, W, "m.left.", h, 1e-5) - 1.5 * plain.mamba2(m, W, "m.right.", h, 1e-5),
+               [part.cache_need()], rt)
+
+
+# ------------------------------------------------------------------ whole models
+
+@pytest.fixture(scope="module", params=sorted(KTINY))
+def ktiny(request, tmp_path_factory):
+    name = request.param
+    return name, make_folder(name, str(tmp_path_factory.mktemp(f"katadra_{name}"))), KTINY[name]
+
+
+def rounding_alone(cfg, weights, tokens, want, scale):
+    """[T]: how far the plain logits move, at most, when every weight moves by up to a bfloat16 rounding
+    (two draws).  A head whose read-out is all but zero before its norm takes the size away makes a few
+    positions ill-conditioned; the bounds below follow them."""
+    worst = torch.zeros(len(tokens), dtype=F64)
+    for seed in (1, 2):
+        gen = torch.Generator().manual_seed(seed)
+        moved = {n: t.double() * (1 + 2 ** -9 * (2 * torch.rand(t.shape, generator=gen, dtype=F64) - 1)) for n, t in weights.items()}
+        worst = torch.maximum(worst, (plain.forward(cfg, moved, tokens) - want).abs().max(1).values / scale)
+    return worst.numpy()
+
+
+def test_layers_of_the_plain_run_and_the_engine_agree(ktiny):
+    """The engine's 32-bit residual stream after every layer run is the plain run's."""
+    from mrun_b200.engine import StepEntry
+    from mrun_b200.engine.loading import executor_from_folder
+    name, folder, settings = ktiny
+    cfg, weights = load_folder(folder)
+    tokens = tokens_of(cfg["vocab"], 41, seed=4)
+    logits, layers = plain.forward(cfg, weights, tokens, want_layers=True)
+    assert layers.shape == (len(cfg["layers"]), 41, cfg["width"])
+    ex = executor_from_folder(folder, dtype="float32", page_size=settings["page_size"], num_pages=32, max_requests=1)
+    assert len(ex.model.blocks) < len(ex.model.order) or not any("weights_of" in l for l in cfg["layers"])
+    seen = []
+    for block in ex.model.blocks:
+        def forward(resid, delta, ctx, cache, inner=block.forward):
+            out = inner(resid, delta, ctx, cache)
+            seen.append((resid + out.compute()).cpu().double())
+            return out
+        block.forward = forward
+    got = ex.step([StepEntry(ex.admit("r"), tokens, list(range(41)))]).cpu().double()
+    assert len(seen) == len(layers)
+    for i, layer in enumerate(seen):
+        error = float((layer - layers[i]).abs().max() / layers[i].abs().max())
+        assert error < 2e-5, f"{name}: after layer {i} ({cfg['layers'][i]['type']}): {error:.3e}"
+    assert float((got - logits).abs().max() / logits.abs().max()) < 2e-5
+
+
+@pytest.mark.parametrize("dtype, tensor_cores", [("float32", False), ("bfloat16", False), ("bfloat16", True)])
+def test_every_cutting_matches_plain(ktiny, dtype, tensor_cores, tmp_path, monkeypatch):
+    """Whole prompts, a prefix and then token by token, portions of changing size down to one and two
+    tokens, and up to four requests side by side in a pool so small that pages and state slots are
+    used again."""
+    name, folder, settings = ktiny
+    cfg, weights = load_folder(folder)
+    vocab = cfg["vocab"]
+    requests = {f"r{i}": tokens_of(vocab, n, seed=200 + i) for i, n in enumerate(TRACE_LENGTHS)}
+    exact = {rid: plain.forward(cfg, weights, tokens) for rid, tokens in requests.items()}
+    scale = max(float(w.abs().max()) for w in exact.values())
+    moves = {rid: rounding_alone(cfg, weights, requests[rid], w, scale) for rid, w in exact.items()}
+    want = {rid: w.to(torch.float32).numpy() for rid, w in exact.items()}
+    b = TraceBuilder()
+    cuts = {}
+
+    def section(label):
+        cuts[label] = len(b.where)
+    section("whole")
+    for rid in ("r0", "r1", "r3", "r5"):
+        cut_whole(b, rid, requests[rid])
+    section("decode_tail")
+    cut_decode_tail(b, "r0", requests["r0"])
+    cut_decode_tail(b, "r7", requests["r7"], tail=2)
+    cut_decode_tail(b, "r5", requests["r5"], tail=200 if name == "tensor" else 40)          # long decoding
+    section("portions")
+    for k, rid in enumerate(("r2", "r4", "r5", "r3")):
+        cut_portions(b, rid, requests[rid], SIZES[k:] + SIZES[:k])
+    section("mixed")
+    cut_mixed(b, requests, SIZES, live=4, seed=6)
+    rounded = sorted((-(-n // 64) * 64 for n in TRACE_LENGTHS), reverse=True)
+    monkeypatch.setenv("MRUN_GATED_ATTENTION_TENSOR_CORES", "1" if tensor_cores else "0")
+    runner = TraceRunner(folder, dtype, str(tmp_path / "out"), sum(rounded[:4]), settings["page_size"], max_requests=4)
+    try:
+        runner.run(b.steps)
+    finally:
+        assert runner.close() == 0
+    # (a 32-bit rounding is 2^-15 of a bfloat16 one; sums of many terms collect some)
+    limit = {rid: np.maximum(2e-5, 8 * 2.0 ** -14 * m) if dtype == "float32" else np.maximum(4e-2, 8 * m) for rid, m in moves.items()}
+    files, first_seen, errors = {}, {}, {}
+    for index, (step, row, rid, position) in enumerate(b.where):
+        if step not in files:
+            files[step] = runner.logits(step, vocab)
+        got = files[step][row]
+        if dtype == "float32":
+            seen = first_seen.setdefault((rid, position), (got, step))
+            assert np.array_equal(seen[0], got), (f"{name}: request {rid}, position {position}: steps {seen[1]} and "
+                                                  f"{step} differ in bits")
+        label = [l for l in cuts if cuts[l] <= index][-1]
+        error = float(np.max(np.abs(got - want[rid][position]))) / scale
+        errors.setdefault(label, []).append((error / limit[rid][position], error, step, rid, position))
+    tight = 2e-5 if dtype == "float32" else 4e-2
+    for label, found in errors.items():
+        worst = max(found)
+        over = sum(e[1] > tight for e in found)
+        print(name, dtype, label, f"{worst[0]:.2f} of its limit, {max(e[1] for e in found):.2e}", over, len(found))
+        assert worst[0] <= 1.0, f"{name}/{dtype}/{label}: {worst}"
+        # and nearly every position stays within the bound that asks nothing of the conditioning
+        assert over <= max(2, len(found) // 12), f"{name}/{dtype}/{label}: {over} of {len(found)} over {tight}"
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_greedy_generation_matches_plain(ktiny, dtype):
+    """Greedy generation through ``Engine.generate``: the scheduler cuts prompts into portions of seven
+    tokens beside decoded tokens of other requests, with four state slots for five requests."""
+    from mrun_b200 import Engine
+    name, folder, settings = ktiny
+    cfg, weights = load_folder(folder)
+    prompts = [tokens_of(cfg["vocab"], n, seed=300 + n) for n in (1, 9, 40, 71, 5)]
+    engine = Engine.from_folder(folder, dtype=dtype, page_size=settings["page_size"], context=512, max_batch_tokens=7, max_requests=4)
+    results = engine.generate(prompts, max_tokens=10, ignore_eos=True)
+    assert bool(engine.executor._graphs) == engine.executor.model.graph_safe
+    for prompt, result in zip(prompts, results):
+        assert result.finish_reason == "length" and len(result.tokens) == 10
+        tokens = list(prompt)
+        for n, token in enumerate(result.tokens):
+            logits = plain.forward(cfg, weights, tokens)[-1]
+            best = int(torch.argmax(logits))
+            top = float(logits.abs().max())
+            margin = 1e-3 if dtype == "float32" else 8e-2 * top
+            if dtype == "bfloat16" and token != best:
+                margin = max(margin, 12 * top * float(rounding_alone(cfg, weights, tokens, plain.forward(cfg, weights, tokens), top)[-1]))
+            assert token == best or float(logits[best] - logits[token]) < margin, \
+                f"{name}: output token {n}: engine {token}, plain {best}, behind by {float(logits[best] - logits[token]):.4f}"
+            tokens.append(token)
+    engine.executor.cache.check_invariants()
+    assert not engine.executor.cache.live
+
+
+def test_captured_decode_steps_are_used():
+    """Every tiny model whose attention takes at most sixteen query heads a kv head decodes captured."""
+    from mrun_b200.parts import MIXERS
+    from tiny_katadra import kconfig
+    safe = {}
+    for name in KTINY:
+        for i, layer in enumerate(kconfig(name).to_spec().layers):
+            w = {t.name[2:]: torch.zeros(t.shape) for t in MIXERS.tensor_specs(layer.mixer, "m")}
+            safe[name, i] = MIXERS.build(layer.mixer, w, runtime("bfloat16")).graph_safe
+    assert [key for key, value in safe.items() if not value] == [("groups", 1)]
+
+
+def test_command_line_random_then_run(tmp_path):
+    """``mrun random`` writes a Katadra folder from its config.json (the sizes that only tensors give from
+    the keys), ``mrun run`` reads them back from the checkpoint and generates."""
+    import json
+    import os
+    import subprocess
+    import sys
+    root = os.path.normpath(os.path.join(os.path.dirname(os.path.abspath(__file__)), os.pardir))
+    mrun = os.path.join(root, "bin", "mrun")
+    run = lambda *args: subprocess.run([sys.executable, mrun, *args], capture_output=True, text=True, timeout=600)
+    (tmp_path / "cfg.json").write_text(json.dumps(KTINY["mixed"]["config"]))
+    folder = str(tmp_path / "model")
+    made = run("random", folder, "--config", str(tmp_path / "cfg.json"), "--seed", "21", "--std", "0.1")
+    assert made.returncode == 0, made.stderr
+    cfg, weights = load_folder(folder)
+    for layer in cfg["layers"]:
+        if layer["type"] == "parallel":
+            layer["mixer"]["left"].pop("bias_rows"); layer["mixer"]["right"].pop("rank")
+    with open(os.path.join(folder, "config.json"), "w") as f:
+        json.dump(cfg, f)
+    prompt = tokens_of(cfg["vocab"], 19, seed=8)
+    result = run("run", folder, "--prompt", ",".join(map(str, prompt)), "--max-tokens", "6", "--dtype", "float32",
+                 "--ignore-eos", "--context", "1K")
+    assert result.returncode == 0, result.stderr
+    tokens = list(prompt)
+    for token in (int(t) for t in result.stdout.strip().split(",")):
+        logits = plain.forward(cfg, weights, tokens)[-1]
+        best = int(torch.argmax(logits))
+        assert token == best or float(logits[best] - logits[token]) < 1e-3
+        tokens.append(token)
+    assert len(tokens) == 19 + 6 and "Katadra" in result.stderr
+
+
+# ------------------------------------------------------------------ layer sizes of a real model
+
+def real_sizes(vdim):
+    a = {"heads": 8, "kv_heads": 2, "dim": 128, "vdim": vdim, "scale": 128 ** -0.5, "softcap": 50.0, "bias_max": 100, "bias_rows": 48,
+         "q_temp": {"coef": 0.1, "every": 64}}
+    par = {"type": "parallel", "mixer": {"left": a, "right": {"heads": 16, "dim": 64, "rank": 32}, "left_scale": 0.7, "right_scale": 0.9},
+           "mlp": {"kind": "dense", "ff": 2816}}
+    ssm = {"type": "mamba2", "mixer": {"heads": 32, "vdim": 64, "state": 128, "groups": 4, "conv": 4, "norm_groups": 4}, "mlp": None}
+    return {"architecture": "Katadra", "vocab": 4096, "width": 1024, "norm": {"eps": 1e-6},
+            "layers": [ssm, par, dict(ssm, weights_of=0), dict(par, weights_of=1)]}
+
+
+@pytest.mark.parametrize("dtype, vdim", [("float32", 64), ("bfloat16", 64), ("bfloat16", 128)])
+def test_real_layer_sizes(dtype, vdim, tmp_path):
+    """A width of 1,024, heads of 128 (in bfloat16 the tcgen05 and TMA attention kernels), sixteen heads of
+    64 in the time mixing, a state of 128 x 64 a head: a prompt whole and in portions, then decoded token
+    by token, against the plain model."""
+    from mrun_b200.config.katadra import KatadraConfig
+    from mrun_b200.engine import StepEntry
+    from mrun_b200.engine.loading import executor_from_folder
+    from mrun_b200.weights import write_random_model
+    folder = write_random_model(KatadraConfig.from_dict(real_sizes(vdim)), str(tmp_path / "real"), seed=7, std=0.03, norm_noise=0.1)
+    cfg, weights = load_folder(folder)
+    tokens = tokens_of(cfg["vocab"], 330, seed=77)
+    want = plain.forward(cfg, weights, tokens).to(torch.float32)
+    ex = executor_from_folder(folder, dtype=dtype, page_size=16, num_pages=64, max_requests=2)
+    seen = {}
+    for label, portions in (("whole", [330]), ("portions", [200, 3, 65, 30] + [1] * 32)):
+        request, at, got = ex.admit(label), 0, []
+        for n in portions:
+            got.append(ex.step([StepEntry(request, tokens[at:at + n], list(range(n)))]).cpu())
+            at += n
+        ex.release(request)
+        got = torch.cat(got)
+        errors = (got - want).abs().max(1).values / want.abs().max()
+        print(dtype, vdim, label, f"{float(errors.max()):.2e}")
+        assert float(errors.max()) <= (2e-5 if dtype == "float32" else 4e-2), f"{label}: {float(errors.max()):.3e}"
+        if dtype == "float32":
+            assert torch.equal(seen.setdefault("logits", got), got), "the cuttings differ in bits"
+    ex.check()
