@@ -78,10 +78,10 @@ def test_constants_reach_the_parts():
     spec = kconfig("odd").to_spec()
     mix = spec.layers[1].mixer
     a, r = mix.left, mix.right
-    assert mix.combine == "sum" and mix.scales == (0.6, 1.3)
+    assert mix.combine == "sum" and mix.scales == (0.9, 0.4)
     assert a.temperature == (0.8, 3.5) and a.soft_cap == 3.0 and a.distance_bias == (8, 30.0) and a.softmax_scale == 0.4
     assert a.qk_norm == "unit" and a.element_gate and not a.sink and not a.head_gate and a.position is None and a.window is None
-    assert (a.heads, a.kv_heads, a.dim, a.vdim) == (3, 1, 11, 5) and (r.heads, r.dim, r.rank) == (1, 13, 3)
+    assert (a.heads, a.kv_heads, a.dim, a.vdim) == (3, 1, 11, 5) and (r.heads, r.dim, r.rank) == (3, 13, 3)
     s = spec.layers[0].mixer
     assert (s.heads, s.vdim, s.state, s.groups, s.conv, s.norm_groups) == (3, 7, 9, 1, 1, 3)
     assert kconfig("groups").to_spec().layers[0].mixer.left.kv_heads == 5      # left out: one a query head
@@ -195,6 +195,6 @@ def test_two_mixers_side_by_side_need_names_of_their_own():
     part = MIXERS.build(spec, w, rt)
     paged, states = split_need(part.cache_need())
     assert paged == PagedKV(1, 11, None, value_dim=5)
-    assert {s.name: s for s in states} == {"state": FixedState((1, 13, 13), "float32", "state"),
+    assert {s.name: s for s in states} == {"state": FixedState((3, 13, 13), "float32", "state"),
                                            "shift": FixedState((1, 37), "float32", "shift")}
-    assert part.w_o.shape == (37, 3 * 5 + 13) and part.graph_safe
+    assert part.w_o.shape == (37, 3 * 5 + 3 * 13) and part.graph_safe

@@ -46,9 +46,9 @@ def again(layers, *owners):
 
 KTINY = {
     # every kernel's element-by-element form: sizes that fit no vector width, one tap, one-row parts
-    "odd": {"page_size": 8, "seed": 31, "std": 0.2, "norm_noise": 0.2, "config": {
+    "odd": {"page_size": 8, "seed": 37, "std": 0.15, "norm_noise": 0.2, "config": {
         "architecture": "Katadra", "vocab": 83, "width": 37, "norm": {"eps": 1e-5},
-        "layers": again([mamba2(3, 7, 9, 1, 1, 3, 19), parallel(left(3, 1, 11, 5, 0.4, 3.0, 8, 30, 0.8, 3.5), right(1, 13, 3), (0.6, 1.3))],
+        "layers": again([mamba2(3, 7, 9, 1, 1, 3, 19), parallel(left(3, 1, 11, 5, 0.4, 3.0, 8, 30, 0.8, 3.5), right(3, 13, 3), (0.9, 0.4))],
                         1, 0, 0)}},
     # heads the mma.sync kernels take, keys wider than values and the other way round; a chain of owners
     "wide": {"page_size": 4, "seed": 32, "std": 0.12, "norm_noise": 0.15, "config": {
