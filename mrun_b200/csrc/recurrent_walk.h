@@ -6,8 +6,6 @@
 
 enum : int { WALK_BONUS = 0, WALK_SSM = 1 };
 
-template <int N> struct Count { static constexpr int value = N; };
-
 struct WalkArgs {
     int mode;
     const void *q, *k, *v;          // rows of one matrix, `ld` elements apart: q, k [H / group, D], v [H, V]
