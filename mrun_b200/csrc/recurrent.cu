@@ -798,18 +798,19 @@ MRUN_API int mrun_scan_walks(int ssm, const void* q, const void* k, const void* 
     return walk_takes(w, act_dtype) ? 1 : 0;
 }
 
-// scratch: may be null where mrun_scan_walks() says so.
+// scratch: may be null where mrun_scan_walks() says so.  max_q_len: the longest segment.
 // q (the read vector), k, v: [H, D] a row (stride ld); a: float32 [tokens, H * D], bias: float32 [H * D],
 // the decay is exp(-exp(a + bias)); bonus: float32 [H * D].
 MRUN_API int mrun_bonus_scan(const void* q, const void* k, const void* v, long ld, int act_dtype, const float* a,
                              const float* bias, const float* bonus, float* state, float* out, float* scratch,
-                             const int* seg_q_start, const int* seg_slot, int segments, int tokens, int H, int D, int V,
-                             cudaStream_t stream) {
+                             const int* seg_q_start, const int* seg_slot, int segments, int max_q_len, int tokens, int H,
+                             int D, int V, cudaStream_t stream) {
     MRUN_REQUIRE(H > 0 && D > 0 && V > 0 && segments >= 0, "bonus_scan: bad sizes");
     MRUN_REQUIRE(D <= 256, "bonus_scan: key size %d exceeds the supported 256", D);
     MRUN_REQUIRE(H <= 65535 && segments <= 65535, "bonus_scan: %d heads or %d segments exceed 65535", H, segments);
     if (segments == 0 || tokens == 0) return 0;
-    const WalkArgs w = {WALK_BONUS, q, k, v, ld, a, nullptr, 0, bias, nullptr, bonus, state, out, seg_q_start, seg_slot, 1, H, D, V, 0};
+    const WalkArgs w = {WALK_BONUS, q, k, v, ld, a, nullptr, 0, bias, nullptr, bonus, state, out, seg_q_start, seg_slot, 1, H, D, V,
+                        max_q_len, 0};
     if (walk_takes(w, act_dtype)) return launch_walk(w, act_dtype, segments, stream);
     MRUN_REQUIRE(scratch != nullptr, "bonus_scan: these sizes need scratch");
     if (act_dtype == MRUN_F32)
@@ -828,14 +829,14 @@ MRUN_API int mrun_bonus_scan(const void* q, const void* k, const void* v, long l
 // float32 [H].  state: float32 [slots, H, N, V]; out: float32 [tokens, H * V].
 MRUN_API int mrun_ssm_scan(const void* c, const void* b, const void* x, long ld, int act_dtype, int group, const void* dt,
                            long lddt, const float* dt_bias, const float* a_log, float* state, float* out, float* scratch,
-                           const int* seg_q_start, const int* seg_slot, int segments, int tokens, int H, int N, int V,
-                           cudaStream_t stream) {
+                           const int* seg_q_start, const int* seg_slot, int segments, int max_q_len, int tokens, int H,
+                           int N, int V, cudaStream_t stream) {
     MRUN_REQUIRE(H > 0 && N > 0 && V > 0 && segments >= 0 && group > 0 && H % group == 0, "ssm_scan: bad sizes");
     MRUN_REQUIRE(N <= 256, "ssm_scan: state size %d exceeds the supported 256", N);
     MRUN_REQUIRE(H <= 65535 && segments <= 65535, "ssm_scan: %d heads or %d segments exceed 65535", H, segments);
     if (segments == 0 || tokens == 0) return 0;
     const WalkArgs w = {WALK_SSM, c, b, x, ld, nullptr, dt, lddt, dt_bias, a_log, nullptr, state, out, seg_q_start, seg_slot,
-                        group, H, N, V, 0};
+                        group, H, N, V, max_q_len, 0};
     if (walk_takes(w, act_dtype)) return launch_walk(w, act_dtype, segments, stream);
     MRUN_REQUIRE(scratch != nullptr, "ssm_scan: these sizes need scratch");
     if (act_dtype == MRUN_F32)

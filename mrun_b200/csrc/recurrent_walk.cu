@@ -15,7 +15,8 @@
 // slice order.  The three meet at one barrier a stage.
 // There is no kernel in front and no scratch memory.  Nothing in a token's arithmetic depends on the
 // tile, on the stage or on how a request was cut into steps.
-// grid: value-column groups x heads x segments; a segment of zero rows is padding.
+// grid: value-column groups x heads x segments; a segment of zero rows is padding.  A step of single
+// tokens has a smaller kernel of its own, below.
 #include "recurrent_walk.h"
 
 #include "common.cuh"
@@ -75,6 +76,95 @@ template <> struct Raw4<__nv_bfloat16> {
     }
 };
 
+// ------------------------------------------------------------------------------------------
+// What both kernels do with a lane's tile: rows of pair p, and columns col .. col + CL - 1.
+// ------------------------------------------------------------------------------------------
+template <int R> __device__ __forceinline__ int pair_row(int r, int p) { return (p >> 1) * 4 * R + 4 * r + (p & 1) * 2; }
+
+template <int CL> __device__ __forceinline__ void load_columns(const float* p, float (&x)[CL]) {
+    if constexpr (CL == 4) {
+        const float4 t = *reinterpret_cast<const float4*>(p);
+        x[0] = t.x; x[1] = t.y; x[2] = t.z; x[3] = t.w;
+    } else if constexpr (CL == 2) {
+        const float2 t = *reinterpret_cast<const float2*>(p);
+        x[0] = t.x; x[1] = t.y;
+    } else {
+        x[0] = p[0];
+    }
+}
+template <int CL> __device__ __forceinline__ void store_columns(float* p, const float (&x)[CL]) {
+    if constexpr (CL == 4) *reinterpret_cast<float4*>(p) = make_float4(x[0], x[1], x[2], x[3]);
+    else if constexpr (CL == 2) *reinterpret_cast<float2*>(p) = make_float2(x[0], x[1]);
+    else p[0] = x[0];
+}
+
+template <int R, int CL>
+__device__ __forceinline__ void load_tile(const float* st, int r, bool live, int D, int V, float2 (&S)[4][CL]) {
+#pragma unroll
+    for (int p = 0; p < 4; ++p) {
+        const int row = pair_row<R>(r, p);
+#pragma unroll
+        for (int j = 0; j < CL; ++j) S[p][j] = make_float2(0.f, 0.f);
+        if (live && row < D) {
+            float x[CL], y[CL];
+            load_columns<CL>(st + (size_t)row * V, x);
+            load_columns<CL>(st + (size_t)(row + 1) * V, y);
+#pragma unroll
+            for (int j = 0; j < CL; ++j) S[p][j] = make_float2(x[j], y[j]);
+        }
+    }
+}
+template <int R, int CL>
+__device__ __forceinline__ void store_tile(float* st, int r, bool live, int D, int V, const float2 (&S)[4][CL]) {
+#pragma unroll
+    for (int p = 0; p < 4; ++p) {
+        const int row = pair_row<R>(r, p);
+        if (live && row < D) {
+            float x[CL], y[CL];
+#pragma unroll
+            for (int j = 0; j < CL; ++j) { x[j] = S[p][j].x; y[j] = S[p][j].y; }
+            store_columns<CL>(st + (size_t)row * V, x);
+            store_columns<CL>(st + (size_t)(row + 1) * V, y);
+        }
+    }
+}
+
+// One token: the state advances, o gets the tile's share of the read-out.  gg: the decays of the pairs
+// (bonus), or the head's in gg[0] (state space).
+template <int MODE, int CL>
+__device__ __forceinline__ void advance(float2 (&S)[4][CL], const float2 (&qq)[4], const float2 (&kk)[4],
+                                        const float2 (&gg)[4], const float2 (&u)[4], const float (&vv)[CL], float (&o)[CL]) {
+    // neighbouring columns' steps stand side by side: none waits for the one before
+    float2 v2[CL], acc[CL];
+#pragma unroll
+    for (int j = 0; j < CL; ++j) {
+        v2[j] = both(vv[j]);
+        acc[j] = make_float2(0.f, 0.f);
+    }
+#pragma unroll
+    for (int p = 0; p < 4; ++p) {
+        float2 write[CL];
+#pragma unroll
+        for (int j = 0; j < CL; ++j) write[j] = __fmul2_rn(kk[p], v2[j]);
+        if constexpr (MODE == WALK_BONUS) {             // the state before this token's write, the write weighed by u
+            float2 seen[CL];
+#pragma unroll
+            for (int j = 0; j < CL; ++j) seen[j] = __ffma2_rn(u[p], write[j], S[p][j]);
+#pragma unroll
+            for (int j = 0; j < CL; ++j) S[p][j] = __ffma2_rn(gg[p], S[p][j], write[j]);
+#pragma unroll
+            for (int j = 0; j < CL; ++j) acc[j] = __ffma2_rn(seen[j], qq[p], acc[j]);
+        } else {
+#pragma unroll
+            for (int j = 0; j < CL; ++j) S[p][j] = __ffma2_rn(gg[0], S[p][j], write[j]);
+#pragma unroll
+            for (int j = 0; j < CL; ++j) acc[j] = __ffma2_rn(S[p][j], qq[p], acc[j]);
+        }
+    }
+#pragma unroll
+    for (int j = 0; j < CL; ++j) o[j] = acc[j].x + acc[j].y;
+}
+
 // Floats of the shared-memory areas: a stage's input rows, and the slices' shares of its read-outs (a
 // walking warp's start C * CL banks after the one's before, so that a row of columns is read without conflicts).
 template <int MODE, int R, int CL> __host__ __device__ constexpr int input_floats(int stage) {
@@ -109,29 +199,12 @@ walk_kernel(const WalkArgs w) {
         const int r = lane / C, c = lane % C;
         const int my_col = (warp * C + c) * CL, col = block_col + my_col;
         const bool live = col < V;                      // V is a multiple of CL
-        auto row_of = [&](int p) { return (p >> 1) * 4 * R + 4 * r + (p & 1) * 2; };      // first row of pair p
         float2 S[4][CL], u[4];
         float* st = w.state + (((size_t)w.seg_slot[seg] * H + h) * D) * V + col;
+        load_tile<R, CL>(st, r, live, D, V, S);
 #pragma unroll
         for (int p = 0; p < 4; ++p) {
-            const int row = row_of(p);
-#pragma unroll
-            for (int j = 0; j < CL; ++j) S[p][j] = make_float2(0.f, 0.f);
-            if (live && row < D) {
-                float x[CL], y[CL];
-                if constexpr (CL == 4) {
-                    *reinterpret_cast<float4*>(x) = load4(st + (size_t)row * V);
-                    *reinterpret_cast<float4*>(y) = load4(st + (size_t)(row + 1) * V);
-                } else if constexpr (CL == 2) {
-                    *reinterpret_cast<float2*>(x) = *reinterpret_cast<const float2*>(st + (size_t)row * V);
-                    *reinterpret_cast<float2*>(y) = *reinterpret_cast<const float2*>(st + (size_t)(row + 1) * V);
-                } else {
-                    x[0] = st[(size_t)row * V];
-                    y[0] = st[(size_t)(row + 1) * V];
-                }
-#pragma unroll
-                for (int j = 0; j < CL; ++j) S[p][j] = make_float2(x[j], y[j]);
-            }
+            const int row = pair_row<R>(r, p);
             u[p] = make_float2(0.f, 0.f);
             if (BONUS && row < D) u[p] = *reinterpret_cast<const float2*>(w.bonus + (size_t)h * D + row);
         }
@@ -147,9 +220,7 @@ walk_kernel(const WalkArgs w) {
                 [[maybe_unused]] const float4* g4 = reinterpret_cast<const float4*>(base + (2 * stage + t) * ROWS);
                 float vv[CL];
                 const float* vs = base + VECTORS * stage * ROWS + t * COLS + my_col;
-                if constexpr (CL == 4) *reinterpret_cast<float4*>(vv) = *reinterpret_cast<const float4*>(vs);
-                else if constexpr (CL == 2) *reinterpret_cast<float2*>(vv) = *reinterpret_cast<const float2*>(vs);
-                else vv[0] = vs[0];
+                load_columns<CL>(vs, vv);
                 const float4 qa = q4[r], qb = q4[R + r], ka = k4[r], kb = k4[R + r];
                 const float2 qq[4] = {{qa.x, qa.y}, {qa.z, qa.w}, {qb.x, qb.y}, {qb.z, qb.w}};
                 const float2 kk[4] = {{ka.x, ka.y}, {ka.z, ka.w}, {kb.x, kb.y}, {kb.z, kb.w}};
@@ -160,62 +231,13 @@ walk_kernel(const WalkArgs w) {
                 } else {
                     gg[0] = both(base[VECTORS * stage * ROWS + stage * COLS + t]);
                 }
-                // neighbouring columns' steps stand side by side: none waits for the one before
-                float2 v2[CL], acc[CL];
-#pragma unroll
-                for (int j = 0; j < CL; ++j) {
-                    v2[j] = both(vv[j]);
-                    acc[j] = make_float2(0.f, 0.f);
-                }
-#pragma unroll
-                for (int p = 0; p < 4; ++p) {
-                    float2 write[CL];
-#pragma unroll
-                    for (int j = 0; j < CL; ++j) write[j] = __fmul2_rn(kk[p], v2[j]);
-                    if constexpr (BONUS) {              // the state before this token's write, the write weighed by u
-                        float2 seen[CL];
-#pragma unroll
-                        for (int j = 0; j < CL; ++j) seen[j] = __ffma2_rn(u[p], write[j], S[p][j]);
-#pragma unroll
-                        for (int j = 0; j < CL; ++j) S[p][j] = __ffma2_rn(gg[p], S[p][j], write[j]);
-#pragma unroll
-                        for (int j = 0; j < CL; ++j) acc[j] = __ffma2_rn(seen[j], qq[p], acc[j]);
-                    } else {
-#pragma unroll
-                        for (int j = 0; j < CL; ++j) S[p][j] = __ffma2_rn(gg[0], S[p][j], write[j]);
-#pragma unroll
-                        for (int j = 0; j < CL; ++j) acc[j] = __ffma2_rn(S[p][j], qq[p], acc[j]);
-                    }
-                }
                 float o[CL];
-#pragma unroll
-                for (int j = 0; j < CL; ++j) o[j] = acc[j].x + acc[j].y;
-                float* dst = share + t * (WARPS * SHARE_WARP<R, CL>);
-                if constexpr (CL == 4) *reinterpret_cast<float4*>(dst) = *reinterpret_cast<float4*>(o);
-                else if constexpr (CL == 2) *reinterpret_cast<float2*>(dst) = *reinterpret_cast<float2*>(o);
-                else dst[0] = o[0];
+                advance<MODE, CL>(S, qq, kk, gg, u, vv, o);
+                store_columns<CL>(share + t * (WARPS * SHARE_WARP<R, CL>), o);
             }
             stage_barrier();
         }
-#pragma unroll
-        for (int p = 0; p < 4; ++p) {
-            const int row = row_of(p);
-            if (live && row < D) {
-                float x[CL], y[CL];
-#pragma unroll
-                for (int j = 0; j < CL; ++j) { x[j] = S[p][j].x; y[j] = S[p][j].y; }
-                if constexpr (CL == 4) {
-                    *reinterpret_cast<float4*>(st + (size_t)row * V) = *reinterpret_cast<float4*>(x);
-                    *reinterpret_cast<float4*>(st + (size_t)(row + 1) * V) = *reinterpret_cast<float4*>(y);
-                } else if constexpr (CL == 2) {
-                    *reinterpret_cast<float2*>(st + (size_t)row * V) = *reinterpret_cast<float2*>(x);
-                    *reinterpret_cast<float2*>(st + (size_t)(row + 1) * V) = *reinterpret_cast<float2*>(y);
-                } else {
-                    st[(size_t)row * V] = x[0];
-                    st[(size_t)(row + 1) * V] = y[0];
-                }
-            }
-        }
+        store_tile<R, CL>(st, r, live, D, V, S);
     } else if (tid < 2 * ROLE) {
         // ------------------------------------------------------------------------- bringing input
         const int me = tid - ROLE;
@@ -342,9 +364,84 @@ walk_kernel(const WalkArgs w) {
     }
 }
 
+// ------------------------------------------------------------------------------------------
+// The same for a step in which every segment is a single token (or none): the state's tile is asked for
+// first, a lane makes its own rows of q, k and the decays, the slices' shares meet in shared memory
+// once.  Nothing is staged and a block is four warps, so that many tiles are in flight; the arithmetic
+// and the order of the sums are the walk's.
+// ------------------------------------------------------------------------------------------
+template <typename TA, int MODE, int R, int CL>
+__global__ void __launch_bounds__(ROLE)
+single_kernel(const WalkArgs w) {
+    constexpr bool BONUS = MODE == WALK_BONUS;
+    constexpr int C = 32 / R, COLS = WARPS * C * CL;
+    __shared__ __align__(16) float shares[WARPS * SHARE_WARP<R, CL>];
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int h = blockIdx.y, seg = blockIdx.z;
+    const int q0 = w.seg_q_start[seg];
+    if (w.seg_q_start[seg + 1] <= q0) return;
+    const int D = w.D, V = w.V, H = w.H;
+    const int block_col = blockIdx.x * COLS;
+    const int r = lane / C, c = lane % C, col = block_col + (warp * C + c) * CL;
+    const bool live = col < V;
+    float2 S[4][CL];
+    float* st = w.state + (((size_t)w.seg_slot[seg] * H + h) * D) * V + col;
+    load_tile<R, CL>(st, r, live, D, V, S);
+    float2 qq[4], kk[4], gg[4], u[4];
+    const int kh = h / w.group;
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+        const int row = half * 4 * R + 4 * r;           // pairs 2 half and 2 half + 1
+        float4 x = make_float4(0.f, 0.f, 0.f, 0.f), y = x, g = x, b = x;
+        if (row < D) {
+            Raw4<TA> raw;
+            raw.load((const TA*)w.q + (size_t)q0 * w.ld + (size_t)kh * D + row);
+            x = raw.widen();
+            raw.load((const TA*)w.k + (size_t)q0 * w.ld + (size_t)kh * D + row);
+            y = raw.widen();
+            if constexpr (BONUS) {
+                const float4 z = load4(w.a + ((size_t)q0 * H + h) * D + row), bias = load4(w.bias + (size_t)h * D + row);
+                g = make_float4(expf(-expf(z.x + bias.x)), expf(-expf(z.y + bias.y)), expf(-expf(z.z + bias.z)), expf(-expf(z.w + bias.w)));
+                b = load4(w.bonus + (size_t)h * D + row);
+            }
+        }
+        qq[2 * half] = make_float2(x.x, x.y); qq[2 * half + 1] = make_float2(x.z, x.w);
+        kk[2 * half] = make_float2(y.x, y.y); kk[2 * half + 1] = make_float2(y.z, y.w);
+        gg[2 * half] = make_float2(g.x, g.y); gg[2 * half + 1] = make_float2(g.z, g.w);
+        u[2 * half] = make_float2(b.x, b.y); u[2 * half + 1] = make_float2(b.z, b.w);
+    }
+    float step = 1.f;
+    if constexpr (!BONUS) {
+        step = softplus_f(to_float(((const TA*)w.dt)[(size_t)q0 * w.lddt + h]) + w.bias[h]);
+        gg[0] = both(expf(-expf(w.a_log[h]) * step));
+    }
+    float vv[CL], o[CL];
+#pragma unroll
+    for (int j = 0; j < CL; ++j) vv[j] = live ? to_float(((const TA*)w.v)[(size_t)q0 * w.ld + (size_t)h * V + col + j]) * step : 0.f;
+    advance<MODE, CL>(S, qq, kk, gg, u, vv, o);
+    store_columns<CL>(shares + warp * SHARE_WARP<R, CL> + lane * CL, o);
+    store_tile<R, CL>(st, r, live, D, V, S);
+    __syncthreads();
+    for (int j = tid; j < COLS; j += ROLE) {
+        if (block_col + j >= V) continue;
+        const float* from = shares + (j / (C * CL)) * SHARE_WARP<R, CL> + j % (C * CL);
+        float x[R];
+#pragma unroll
+        for (int i = 0; i < R; ++i) x[i] = from[i * C * CL];
+#pragma unroll
+        for (int i = 1; i < R; ++i) x[0] += x[i];
+        w.out[(size_t)q0 * H * V + (size_t)h * V + block_col + j] = x[0];
+    }
+}
+
 template <typename TA, int MODE, int R, int CL>
 int launch(WalkArgs w, int segments, cudaStream_t stream) {
     constexpr int COLS = WARPS * (32 / R) * CL;
+    if (w.max_q_len == 1) {
+        single_kernel<TA, MODE, R, CL><<<dim3((w.V + COLS - 1) / COLS, w.H, segments), ROLE, 0, stream>>>(w);
+        MRUN_CHECK_LAUNCH("scan step");
+        return 0;
+    }
     const int carried = CHUNKS * ROLE * 8 / w.D;     // tokens whose chunks the bringing threads carry
     w.stage = carried > STAGE ? STAGE : carried / 4 * 4;
     const size_t smem = sizeof(float) * 2 * ((size_t)input_floats<MODE, R, CL>(w.stage) + (size_t)w.stage * WARPS * SHARE_WARP<R, CL>);

@@ -17,6 +17,7 @@ struct WalkArgs {
     float *state, *out;             // [slots, H, D, V]; [tokens, H * V]
     const int *seg_q_start, *seg_slot;
     int group, H, D, V;
+    int max_q_len;                  // the longest segment
     int stage;                      // tokens a stage (set at the launch)
 };
 

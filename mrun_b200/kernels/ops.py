@@ -1375,7 +1375,7 @@ def bonus_scan(r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, a: torch.Tenso
         scratch = torch.empty(tokens * heads * (3 * dim + vdim), dtype=torch.float32, device=r.device)
     _lib.core().call("mrun_bonus_scan", _ptr(r), _ptr(k), _ptr(v), _c_long(ld), dtype_code(r.dtype), _ptr(a), _ptr(bias),
                      _ptr(bonus), _ptr(state), _ptr(out), _ptr(scratch), _ptr(ctx.seg_q_start), _ptr(ctx.seg_slot),
-                     _c_int(ctx.num_segments), _c_int(tokens), _c_int(heads), _c_int(dim), _c_int(vdim), _stream())
+                     _c_int(ctx.num_segments), _c_int(ctx.max_q_len), _c_int(tokens), _c_int(heads), _c_int(dim), _c_int(vdim), _stream())
     return out
 
 
@@ -1403,7 +1403,7 @@ def ssm_scan(c: torch.Tensor, b: torch.Tensor, x: torch.Tensor, dt: torch.Tensor
         scratch = torch.empty(tokens * (2 * groups * size + heads * (vdim + 1)), dtype=torch.float32, device=c.device)
     _lib.core().call("mrun_ssm_scan", _ptr(c), _ptr(b), _ptr(x), _c_long(ld), dtype_code(c.dtype), _c_int(heads // groups),
                      _ptr(dt), _c_long(lddt), _ptr(dt_bias), _ptr(a_log), _ptr(state), _ptr(out), _ptr(scratch),
-                     _ptr(ctx.seg_q_start), _ptr(ctx.seg_slot), _c_int(ctx.num_segments), _c_int(tokens), _c_int(heads),
+                     _ptr(ctx.seg_q_start), _ptr(ctx.seg_slot), _c_int(ctx.num_segments), _c_int(ctx.max_q_len), _c_int(tokens), _c_int(heads),
                      _c_int(size), _c_int(vdim), _stream())
     return out
 
