@@ -213,7 +213,7 @@ def build_attention(head_dim: int, value_dim: Optional[int] = None, scored: bool
 # head sizes of the configurations this repository measures and tests
 COMMON_HEAD_DIMS = (16, 32, 48, 64, 80, 96, 128, 144, 256)      # the head sizes the tests and the measured shapes use
 # (key size, value size) of the attentions with a score form among them
-COMMON_SCORED_DIMS = ((128, 128), (64, 64), (128, 64), (64, 128), (48, 16), (32, 80), (16, 16))
+COMMON_SCORED_DIMS = ((128, 128), (64, 64), (128, 64), (64, 128), (48, 16), (32, 80), (16, 16), (96, 48), (16, 48), (32, 16))
 
 
 def build_all() -> list[str]:

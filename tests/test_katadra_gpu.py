@@ -139,7 +139,7 @@ ATTENTION_SHAPES = [
     (entry(6, 3, 48, 16), 8),
     (entry(4, 4, 32, 80, coef=0.0), 16),
     (entry(34, 2, 16, 16, cap=50.0), 16),                                      # seventeen query heads a kv head
-    (entry(2, 1, 96, 32, rows=10, reach=10), 16),
+    (entry(2, 1, 96, 48, rows=10, reach=10), 16),
 ]
 
 
