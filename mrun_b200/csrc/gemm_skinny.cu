@@ -38,15 +38,16 @@ constexpr int WARPS = 8;
 constexpr int THREADS = WARPS * 32;
 constexpr int UNROLL_DEEP = 4;      // chunks per batch with one row tile and one token tile per block
 constexpr int UNROLL_SHALLOW = 2;   // ... with two row tiles or two token tiles (more registers per chunk)
-enum : int { EPI_PLAIN = 0, EPI_GATED = 1, EPI_RESIDUAL = 2 };
+// EPI_BATCHED: several products of one shape in one launch, each with a function of one argument behind it
+enum : int { EPI_PLAIN = 0, EPI_GATED = 1, EPI_RESIDUAL = 2, EPI_BATCHED = 3 };
 // Sums of squares travel as unsigned 64-bit integers in units of 2^-30: room for 1.7e10, steps of
 // 1e-9 (a row of unit-scale values sums to its width; eps times the width is 1e-6 times that).
 constexpr float SUMS_SCALE = 1073741824.f, SUMS_UNIT = 1.f / 1073741824.f;
 
 // What a launch does beside the product itself.
 struct Fusion {
-    int act;                     // EPI_GATED: the gate's function (MRUN_GATE_*); EPI_PLAIN: MRUN_ACT_* or 0
-    // a batch of products in one launch (blockIdx.y): W matrices one after the other, x and y this far apart
+    int act;                     // EPI_GATED: the gate's function (MRUN_GATE_*); EPI_BATCHED: MRUN_ACT_* or 0
+    // EPI_BATCHED (the product is blockIdx.y): W matrices one after the other, x and y this far apart
     long batch_x, batch_y;
     // x is the xw of a product before: the row's scale is rsqrt(in_sums[row] * 2^-30 / width + eps)
     const unsigned long long* in_sums;   // [16] totals of squares, or null: x is taken as it is
@@ -96,7 +97,7 @@ skinny_kernel(const bf16* __restrict__ x, const bf16* __restrict__ w, TOut* __re
     const int rows = CUT ? rows_cut : MT * 16;
     const int n0 = blockIdx.x * rows;
     const int chunks = K >> 5;          // whole 32-wide chunks; K % 32 == 0 is checked by the host
-    if (EPI == EPI_PLAIN) {
+    if constexpr (EPI == EPI_BATCHED) {
         w += (size_t)blockIdx.y * N * K;
         x += blockIdx.y * f.batch_x;
         y += blockIdx.y * f.batch_y;
@@ -229,7 +230,7 @@ skinny_kernel(const bf16* __restrict__ x, const bf16* __restrict__ w, TOut* __re
             red[warp][mt * 16 + g + 8][nt * 8 + 2 * t + 1] = acc[mt][nt][3];
         }
     __syncthreads();
-    if constexpr (EPI == EPI_PLAIN) {
+    if constexpr (EPI == EPI_PLAIN || EPI == EPI_BATCHED) {
         for (int i = threadIdx.x; i < MT * 16 * NT * 8; i += THREADS) {
             const int row = i % (MT * 16), token = i / (MT * 16);
             if (token < M && row < rows && n0 + row < N) {
@@ -238,7 +239,7 @@ skinny_kernel(const bf16* __restrict__ x, const bf16* __restrict__ w, TOut* __re
                 for (int wi = 0; wi < WARPS; ++wi) s += red[wi][row][token];
                 s *= row_scale[token];
                 // an activation sees the sum as the layer would have stored it
-                if (f.act) s = mrun::plain_act(f.act, __bfloat162float(__float2bfloat16_rn(s)));
+                if (EPI == EPI_BATCHED && f.act) s = mrun::plain_act(f.act, __bfloat162float(__float2bfloat16_rn(s)));
                 store_out<TOut>(y + (size_t)token * ldy + n0 + row, s);
             }
         }
@@ -437,9 +438,9 @@ MRUN_API int mrun_gemm_skinny_batched(const void* x, const void* w, void* y, int
     f.batch_x = batch_x;
     f.batch_y = batch_y;
     if (out_dtype == MRUN_BF16)
-        dispatch<bf16, EPI_PLAIN>((const bf16*)x, (const bf16*)w, (bf16*)y, M, N, K, ldx, ldy, f, 0, batch, stream);
+        dispatch<bf16, EPI_BATCHED>((const bf16*)x, (const bf16*)w, (bf16*)y, M, N, K, ldx, ldy, f, 0, batch, stream);
     else if (out_dtype == MRUN_F32)
-        dispatch<float, EPI_PLAIN>((const bf16*)x, (const bf16*)w, (float*)y, M, N, K, ldx, ldy, f, 0, batch, stream);
+        dispatch<float, EPI_BATCHED>((const bf16*)x, (const bf16*)w, (float*)y, M, N, K, ldx, ldy, f, 0, batch, stream);
     else
         return mrun_set_error("gemm_skinny_batched: unknown output dtype code %d", out_dtype);
     MRUN_CHECK_LAUNCH("gemm_skinny_batched");

@@ -42,6 +42,8 @@ rows fold the residual sum and the norm into the products around them:
 last product unrun, ``kernels.ops.PendingLinear``); ``accepts_pending`` on a norm or arrangement
 (``delta`` may be such a product; a norm may answer with ``kernels.ops.NormedRows``);
 ``accepts_normed_rows`` on a mixer or feed-forward (``x`` may be ``NormedRows``).
+``heads_forward(x, ctx, cache, out, scale)`` and ``w_o`` on a mixer (everything in front of its output
+projection, times ``scale``, into the rows ``out``) let two mixers side by side share one output product.
 """
 from __future__ import annotations
 
