@@ -128,7 +128,9 @@ class LatentAttentionSpec:
     the key/value latent of ``kv_rank`` features (RMS-normed) and ``rot_dim`` more that are the
     rotated key part all heads share.  A head's plain key is an up-projection of the latent, its
     value (``vdim`` features) another; the score is (plain . plain + rotated . rotated) *
-    ``softmax_scale``.  The cache holds the latent and the shared rotated part only.  ``window``
+    ``softmax_scale``.  The cache holds the latent and the shared rotated part only (``rot_dim`` = 0: the
+    latent alone, an attention without positions).  ``head_gate``: head h's output is multiplied by
+    sigmoid(g x)_h, one projection row a head that reads the mixer's input.  ``window``
     = W: a token sees the last W keys, itself included."""
 
     kind: ClassVar[str] = "latent_attention"
@@ -143,6 +145,7 @@ class LatentAttentionSpec:
     eps: float
     position: Optional[Any] = None
     window: Optional[int] = None
+    head_gate: bool = False
 
 
 @dataclass(frozen=True)
@@ -193,7 +196,13 @@ class GatedAttentionSpec:
     ``rel`` of ``rows`` rows; bucket(n) = n for n < rows / 2, else min(rows - 1, rows / 2 +
     floor(ln(n / (rows / 2)) / ln(reach / (rows / 2)) * (rows - rows / 2))).  ``element_gate``: the
     heads' outputs together are multiplied element by element by sigmoid(g x), ``g`` with a row a
-    feature (in place of ``head_gate``)."""
+    feature (in place of ``head_gate``).
+
+    ``biases``: the q, k and v projections have biases ``q.b``, ``k.b``, ``v.b``.  ``learned_sink`` (with
+    ``sink``): the softmax's extra term has the score sink[head] instead of 0.  ``value_mix``: the values of a
+    token are shared between layers of the step.  ``"first"``: this layer's values, as projected, are
+    what later layers read; ``"blend"``: v <- (1 - vmix) v + vmix v_first with one number ``vmix`` a layer,
+    v_first the values of the layer marked ``"first"``; the blended v is what is cached."""
 
     kind: ClassVar[str] = "gated_attention"
     hidden: int
@@ -215,6 +224,9 @@ class GatedAttentionSpec:
     soft_cap: Optional[float] = None
     distance_bias: Optional[Tuple[int, float]] = None
     element_gate: bool = False
+    biases: bool = False
+    learned_sink: bool = False
+    value_mix: Optional[str] = None
 
 
 @dataclass(frozen=True)
@@ -318,6 +330,23 @@ class StateSpaceSpec:
 
 
 @dataclass(frozen=True)
+class SelectiveScanSpec:
+    """A selective state-space mixer with a decay per channel and state (Mamba-1).  One projection makes
+    [x: ``inner`` | z: ``inner``]; x passes a causal convolution of ``conv`` taps per channel with a bias, and
+    SiLU.  A product of x makes [r: ``dt_rank`` | B: ``state`` | C: ``state``]; step = softplus(dt r + bias), one
+    a channel.  S_t[c, n] = exp(-exp(A_log[c, n]) step_c) S_(t-1)[c, n] + step_c x_c B_n, y_c = sum over n
+    of S_t[c, n] C_n + D_c x_c; y * SiLU(z) is projected out.  The convolution's last inputs are part of
+    the state."""
+
+    kind: ClassVar[str] = "selective_scan"
+    hidden: int
+    inner: int
+    state: int
+    dt_rank: int
+    conv: int
+
+
+@dataclass(frozen=True)
 class ParallelMixerSpec:
     """Two mixers side by side that read the same input.  ``combine`` = ``"norm_mean"``: the result
     is ``share`` times the sum of their outputs, each first divided by its root mean square over
@@ -401,11 +430,14 @@ class RoutedMLPSpec:
 @dataclass(frozen=True)
 class GroupedRoutedMLPSpec:
     """A mixture of ``experts`` gated feed-forwards ``down(act(gate x) * up x)`` without biases,
-    chosen by a router whose scores are sigmoid(router x) in 32-bit.  The experts form ``groups``
-    equal groups of neighbours; a group's score is the sum of its ``group_top`` largest scores and
-    only experts of the ``keep_groups`` best groups can be chosen (``groups`` = 1: no limit).
-    Each token takes the ``top`` allowed experts with the largest scores; their weights are the
-    scores divided by their sum (+ 1e-20) times ``route_scale``.  ``shared_ff`` > 0: one more
+    chosen by a router whose scores are sigmoid(router x) or, with ``score`` = ``"softmax"``, the softmax over
+    all of router x, in 32-bit.  ``correction``: experts are ranked by score + correction[expert] (they weigh
+    the score alone).  ``identity``: the router's last ``identity`` rows stand for experts without tensors
+    whose output is the input.  The experts (these included) form ``groups`` equal groups of neighbours; a
+    group's rank is the sum of its ``group_top`` largest ranks and only experts of the ``keep_groups`` best
+    groups can be chosen (``groups`` = 1: no limit).  Each token takes the ``top`` allowed experts with the
+    largest ranks; their weights are the scores times ``route_scale``, divided by their sum (+ 1e-20) when
+    ``renormalize``.  ``shared_ff`` > 0: one more
     expert of that size runs for every token, weighed by sigmoid(sg x) (one number a token) when
     ``shared_gate``, else by 1.  ``score`` = ``"logit"`` (without groups): the router's logits
     themselves are ranked, and the chosen experts weigh the softmax over the chosen logits only.
@@ -425,6 +457,9 @@ class GroupedRoutedMLPSpec:
     activation: str = "silu"
     score: str = "sigmoid"
     router_bias: bool = False
+    correction: bool = False
+    identity: int = 0
+    renormalize: bool = True
 
 
 @dataclass(frozen=True)

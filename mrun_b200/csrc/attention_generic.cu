@@ -13,8 +13,8 @@
 // crates/mrun-engine/src/tensor/nuvec.rs:866-872).
 //
 // Options: values of another size than the keys (value pages [pages, kv_heads, page_size,
-// value_dim]); a sink, one more term of score 0 without a value in the softmax's denominator (the
-// running maximum starts at 0 and the running sum at 1); a gate per (token, head), whose sigmoid
+// value_dim]); a sink, one more term without a value in the softmax's denominator, of a score per
+// query head (the running maximum starts there and the running sum at 1); a gate per (token, head), whose sigmoid
 // multiplies the head's output; a score form (attention_score.cuh).
 #include "attention_score.cuh"
 #include "common.cuh"
@@ -32,7 +32,7 @@ paged_attention_generic_kernel(const TA* __restrict__ q, long q_stride, TA* __re
                                const int* __restrict__ block_tables, int max_blocks,
                                const int* __restrict__ token_slot, const int* __restrict__ positions,
                                int heads, int kv_heads, int head_dim, int value_dim, int page_size, float scale,
-                               int window, int sink, const TA* __restrict__ gate, long gate_stride,
+                               int window, const float* __restrict__ sinks, const TA* __restrict__ gate, long gate_stride,
                                const mrun_score_form form, int formed) {
     extern __shared__ float smem[];
     float* qs = smem;                 // head_dim
@@ -55,7 +55,7 @@ paged_attention_generic_kernel(const TA* __restrict__ q, long q_stride, TA* __re
 
     if (formed) scale *= query_temperature(form, pos);
     const int lo = first_visible(pos, window);
-    float m = sink ? 0.f : -INFINITY, l = sink ? 1.f : 0.f;
+    float m = sinks ? sinks[h] : -INFINITY, l = sinks ? 1.f : 0.f;
     float acc[8];  // value_dim <= 8 * THREADS = 1024
 #pragma unroll
     for (int i = 0; i < 8; ++i) acc[i] = 0.f;
@@ -125,7 +125,7 @@ MRUN_API int mrun_paged_attention_generic(const void* q, long q_stride, void* ou
                                           const void* v_cache, int act_dtype, const int* block_tables,
                                           int max_blocks, const int* token_slot, const int* positions,
                                           int tokens, int heads, int kv_heads, int head_dim, int value_dim,
-                                          int page_size, long cache_rows, float scale, int window, int sink,
+                                          int page_size, long cache_rows, float scale, int window, const float* sinks,
                                           const void* gate, long gate_stride, const mrun_score_form* form,
                                           cudaStream_t stream) {
     MRUN_REQUIRE(tokens >= 0 && heads > 0 && kv_heads > 0 && head_dim > 0 && page_size > 0 && max_blocks > 0,
@@ -153,12 +153,12 @@ MRUN_API int mrun_paged_attention_generic(const void* q, long q_stride, void* ou
         paged_attention_generic_kernel<float><<<grid, THREADS, smem, stream>>>(
             (const float*)q, q_stride, (float*)out, (const float*)k_cache, (const float*)v_cache,
             block_tables, max_blocks, token_slot, positions, heads, kv_heads, head_dim, value_dim, page_size, scale,
-            window, sink, (const float*)gate, gate_stride, f, formed);
+            window, sinks, (const float*)gate, gate_stride, f, formed);
     else if (act_dtype == MRUN_BF16)
         paged_attention_generic_kernel<__nv_bfloat16><<<grid, THREADS, smem, stream>>>(
             (const __nv_bfloat16*)q, q_stride, (__nv_bfloat16*)out, (const __nv_bfloat16*)k_cache,
             (const __nv_bfloat16*)v_cache, block_tables, max_blocks, token_slot, positions, heads, kv_heads,
-            head_dim, value_dim, page_size, scale, window, sink, (const __nv_bfloat16*)gate, gate_stride, f, formed);
+            head_dim, value_dim, page_size, scale, window, sinks, (const __nv_bfloat16*)gate, gate_stride, f, formed);
     else
         return mrun_set_error("paged_attention_generic: unknown dtype code %d", act_dtype);
     MRUN_CHECK_LAUNCH("paged_attention_generic");

@@ -176,7 +176,7 @@ prefill_kernel(const bf16* __restrict__ q, long q_stride, bf16* __restrict__ out
                const int* __restrict__ block_tables, int max_blocks, const int* __restrict__ token_slot,
                const int* __restrict__ positions, const int* __restrict__ tile_tok0,
                const int* __restrict__ tile_ntok, int heads, int kv_heads, int page_size, int page_shift,
-               float scale_log2, int window, float sink_log2, const mrun_score_form form) {
+               float scale_log2, int window, const float* __restrict__ sinks, const mrun_score_form form) {
     extern __shared__ __align__(16) unsigned char smem_raw[];
     bf16* q_tile = reinterpret_cast<bf16*>(smem_raw);           // [64][LD]
     bf16* k_tiles = q_tile + 64 * LD;                           // [2][64][LD]
@@ -263,8 +263,9 @@ prefill_kernel(const bf16* __restrict__ q, long q_stride, bf16* __restrict__ out
         l[r] += __shfl_xor_sync(0xffffffffu, l[r], 1);
         l[r] += __shfl_xor_sync(0xffffffffu, l[r], 2);
     }
-    l[0] = with_sink(l[0], m[0], sink_log2);
-    l[1] = with_sink(l[1], m[1], sink_log2);
+#pragma unroll
+    for (int r = 0; r < 2; ++r)
+        l[r] = with_sink(l[r], m[r], sinks, kvh * group + (w_row0 + (lane >> 2) + r * 8) % group);
     bf16* stage_rows = q_tile + w_row0 * LDV;
 #pragma unroll
     for (int r = 0; r < 2; ++r) {
@@ -455,7 +456,7 @@ decode_kernel(const bf16* __restrict__ q, long q_stride, bf16* __restrict__ out,
               const int* __restrict__ positions, const int* __restrict__ tile_prefix,
               const int4* __restrict__ assignment, int tokens, float* __restrict__ part_o,
               float* __restrict__ part_ml, int* __restrict__ counters, int heads, int kv_heads, int page_size,
-              int page_shift, float scale_log2, int window, float sink_log2, const FusedInput fused,
+              int page_shift, float scale_log2, int window, const float* __restrict__ sinks, const FusedInput fused,
               const mrun_score_form form) {
     extern __shared__ __align__(16) unsigned char smem_raw[];
     bf16* q_tile = reinterpret_cast<bf16*>(smem_raw);           // [16][LD]
@@ -650,7 +651,7 @@ decode_kernel(const bf16* __restrict__ q, long q_stride, bf16* __restrict__ out,
                 ll += src[DV + 1] * c;
             }
             if (complete) {
-                ll = with_sink(ll, mm, sink_log2);
+                ll = with_sink(ll, mm, sinks, kvh * group + row);
                 float v = ll > 0.f ? acc / ll : 0.f;
                 if constexpr (SCORED) v = mrun::gate_output(form, tok, (kvh * group + row) * DV + d, v);
                 out[(size_t)tok * out_stride + (kvh * group + row) * DV + d] = __float2bfloat16_rn(v);
@@ -718,7 +719,7 @@ decode_kernel(const bf16* __restrict__ q, long q_stride, bf16* __restrict__ out,
                             ll += ml[k].y * c;
                         }
                     }
-                    ll = with_sink(ll, mm, sink_log2);
+                    ll = with_sink(ll, mm, sinks, kvh * group + row);
                     const float inv = ll > 0.f ? 1.f / ll : 0.f;
                     float v[4] = {acc.x * inv, acc.y * inv, acc.z * inv, acc.w * inv};
                     finish_outputs<4>(form, tok, (kvh * group + row) * DV + d, v);
@@ -751,7 +752,7 @@ MRUN_API int mrun_attn_prefill(const void* q, long q_stride, void* out, const vo
                                const int* block_tables, int max_blocks, const int* token_slot,
                                const int* positions, const int* tile_tok0, const int* tile_ntok, int n_tiles,
                                int heads, int kv_heads, int head_dim, int page_size, float scale, int window,
-                               float sink, const mrun_score_form* form, cudaStream_t stream) {
+                               const float* sinks, const mrun_score_form* form, cudaStream_t stream) {
     if (int rc = check_common("attn_prefill", heads, kv_heads, head_dim, page_size, max_blocks, window, 64)) return rc;
     if (int rc = check_form("attn_prefill", form, heads)) return rc;
     MRUN_REQUIRE(n_tiles >= 0, "attn_prefill: n_tiles=%d", n_tiles);
@@ -767,7 +768,7 @@ MRUN_API int mrun_attn_prefill(const void* q, long q_stride, void* out, const vo
         prefill_kernel<<<dim3(kv_heads, now), THREADS, PREFILL_SMEM, stream>>>(
             (const bf16*)q, q_stride, (bf16*)out, (const bf16*)k_cache, (const bf16*)v_cache, block_tables, max_blocks,
             token_slot, positions, tile_tok0 + done, tile_ntok + done, heads, kv_heads, page_size, page_shift_of(page_size),
-            scale * LOG2E, window, sink * LOG2E, form_or_none(form));
+            scale * LOG2E, window, sinks, form_or_none(form));
         MRUN_CHECK_LAUNCH("attn_prefill");
     }
     return 0;
@@ -816,7 +817,7 @@ MRUN_API int mrun_attn_decode(const void* q, long q_stride, void* out, void* k_c
                               const int* block_tables, int max_blocks, const int* token_slot,
                               const int* positions, const int* tile_prefix, const int* assignment, int tokens,
                               float* part_o, float* part_ml, int* counters, int blocks, int heads, int kv_heads,
-                              int head_dim, int page_size, float scale, int window, float sink, int fused,
+                              int head_dim, int page_size, float scale, int window, const float* sinks, int fused,
                               const float* q_weight, const float* k_weight, float eps, const float* rot,
                               int rotary_dim, const int* slots, const mrun_score_form* form, cudaStream_t stream) {
     if (int rc = check_form("attn_decode", form, heads)) return rc;
@@ -853,7 +854,7 @@ MRUN_API int mrun_attn_decode(const void* q, long q_stride, void* out, void* k_c
                                      (const bf16*)q, q_stride, (bf16*)out, (const bf16*)k_cache, (const bf16*)v_cache,
                                      block_tables, max_blocks, token_slot, positions, tile_prefix,
                                      (const int4*)assignment, tokens, part_o, part_ml, counters, heads, kv_heads,
-                                     page_size, page_shift_of(page_size), scale * LOG2E, window, sink * LOG2E, in,
+                                     page_size, page_shift_of(page_size), scale * LOG2E, window, sinks, in,
                                      form_or_none(form)),
                     "attn_decode");
     return 0;
@@ -952,7 +953,7 @@ MRUN_API int mrun_attn_decode_static(const void* q, long q_stride, void* out, co
     decode_kernel<<<dim3(blocks), THREADS, DECODE_SMEM, stream>>>(
         (const bf16*)q, q_stride, (bf16*)out, (const bf16*)k_cache, (const bf16*)v_cache, block_tables, max_blocks,
         token_slot, positions, tile_prefix, (const int4*)assignment, tokens, part_o, part_ml, counters, heads, kv_heads,
-        page_size, page_shift_of(page_size), scale * LOG2E, window, -INFINITY, FusedInput{}, mrun_score_form{});
+        page_size, page_shift_of(page_size), scale * LOG2E, window, nullptr, FusedInput{}, mrun_score_form{});
     MRUN_CHECK_LAUNCH("attn_decode_static");
     return 0;
 }

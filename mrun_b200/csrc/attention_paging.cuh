@@ -32,8 +32,9 @@ inline int page_shift_of(int page_size) {
     return -1;
 }
 
-// A softmax sink: one more term of score `sink_log2` (in the kernels' base-2 units; -infinity:
-// none) that has no value, added to the denominator `l` of a row whose running maximum is `m`.
-__device__ __forceinline__ float with_sink(float l, float m, float sink_log2) {
-    return sink_log2 > -INFINITY ? l + exp2f(sink_log2 - m) : l;
+// A softmax sink: one more term that has no value, with the score sinks[head] (one number per query
+// head, not scaled; null: no such term), added to the denominator `l` of a row of that head whose
+// running maximum is `m` (in the kernels' base-2 units).
+__device__ __forceinline__ float with_sink(float l, float m, const float* __restrict__ sinks, int head) {
+    return sinks ? l + exp2f(sinks[head] * 1.4426950408889634f - m) : l;
 }

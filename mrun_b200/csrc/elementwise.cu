@@ -41,7 +41,8 @@ MRUN_API int mrun_embed(const void* table, int table_dtype, const int* ids, floa
 
 // ------------------------------------------------------------------------------------------
 // Residual add + RMSNorm.
-//   v = resid[src] + delta[src]   (delta may be null)
+//   v = resid[src] + delta[src]   (delta may be null; 32-bit or of out's type)
+//                  + share[src] * extra[src]   (a second branch with one factor a row, or null)
 //   if rows == null: resid[src] = v            (the stream advances)
 //   out[r] = v * rsqrt(mean(v^2) + eps) * weight
 // With `rows` the kernel reads row rows[r] and leaves the stream untouched (final norm at the
@@ -49,18 +50,23 @@ MRUN_API int mrun_embed(const void* table, int table_dtype, const int* ids, floa
 // (crates/mrun-engine/src/models/gated_delta.rs:11-13 states the form).
 // One block of 256 threads per row whatever the batch, so the order of additions is fixed.
 // ------------------------------------------------------------------------------------------
-template <typename TA>
-__global__ void add_rmsnorm_kernel(float* __restrict__ resid, const TA* __restrict__ delta,
+template <typename TA, typename TD>
+__global__ void add_rmsnorm_kernel(float* __restrict__ resid, const TD* __restrict__ delta,
                                    const float* __restrict__ weight, float eps, TA* __restrict__ out,
-                                   const int* __restrict__ rows, int hidden) {
+                                   const int* __restrict__ rows, int hidden, const TA* __restrict__ extra,
+                                   const float* __restrict__ share) {
     extern __shared__ float row_buf[];
     __shared__ float scratch[33];
     const int r = blockIdx.x;
-    const size_t src = (size_t)(rows ? rows[r] : r) * hidden;
+    const int row = rows ? rows[r] : r;
+    const size_t src = (size_t)row * hidden;
+    const float part = extra ? share[row] : 0.f;
+    const bool moved = delta || part != 0.f;
     float ss = 0.f;
     for (int h = threadIdx.x; h < hidden; h += blockDim.x) {
         float v = resid[src + h];
         if (delta) v += to_float(delta[src + h]);
+        if (part != 0.f) v = fmaf(part, to_float(extra[src + h]), v);
         row_buf[h] = v;
         ss += v * v;
     }
@@ -69,7 +75,7 @@ __global__ void add_rmsnorm_kernel(float* __restrict__ resid, const TA* __restri
     TA* dst = out + (size_t)r * hidden;
     for (int h = threadIdx.x; h < hidden; h += blockDim.x) {
         const float v = row_buf[h];
-        if (!rows && delta) resid[src + h] = v;
+        if (!rows && moved) resid[src + h] = v;
         dst[h] = from_float<TA>(v * inv * weight[h]);
     }
 }
@@ -78,14 +84,18 @@ __global__ void add_rmsnorm_kernel(float* __restrict__ resid, const TA* __restri
 // to four 8-element chunks in registers and moves them with 16-byte loads and stores, so a row
 // takes one pass and the latency of a few independent loads.  One block of 256 threads per row
 // whatever the batch: the order of additions depends on the width only.
-template <typename TA>
+template <typename TA, typename TD>
 __global__ void __launch_bounds__(256)
-add_rmsnorm_vec_kernel(float* __restrict__ resid, const TA* __restrict__ delta,
+add_rmsnorm_vec_kernel(float* __restrict__ resid, const TD* __restrict__ delta,
                        const float* __restrict__ weight, float eps, TA* __restrict__ out,
-                       const int* __restrict__ rows, int hidden) {
+                       const int* __restrict__ rows, int hidden, const TA* __restrict__ extra,
+                       const float* __restrict__ share) {
     __shared__ float scratch[33];
     const int r = blockIdx.x;
-    const size_t src = (size_t)(rows ? rows[r] : r) * hidden;
+    const int row = rows ? rows[r] : r;
+    const size_t src = (size_t)row * hidden;
+    const float part = extra ? share[row] : 0.f;
+    const bool moved = delta || part != 0.f;
     const int chunks = hidden >> 3;
     float v[4][8];
     float ss = 0.f;
@@ -96,9 +106,15 @@ add_rmsnorm_vec_kernel(float* __restrict__ resid, const TA* __restrict__ delta,
             Vec8<float>::load(resid + src + c * 8, v[i]);
             if (delta) {
                 float d[8];
-                Vec8<TA>::load(delta + src + c * 8, d);
+                Vec8<TD>::load(delta + src + c * 8, d);
 #pragma unroll
                 for (int e = 0; e < 8; ++e) v[i][e] += d[e];
+            }
+            if (part != 0.f) {
+                float d[8];
+                Vec8<TA>::load(extra + src + c * 8, d);
+#pragma unroll
+                for (int e = 0; e < 8; ++e) v[i][e] = fmaf(part, d[e], v[i][e]);
             }
 #pragma unroll
             for (int e = 0; e < 8; ++e) ss += v[i][e] * v[i][e];
@@ -110,7 +126,7 @@ add_rmsnorm_vec_kernel(float* __restrict__ resid, const TA* __restrict__ delta,
     for (int i = 0; i < 4; ++i) {
         const int c = threadIdx.x + i * 256;
         if (c < chunks) {
-            if (!rows && delta) Vec8<float>::store(resid + src + c * 8, v[i]);
+            if (!rows && moved) Vec8<float>::store(resid + src + c * 8, v[i]);
             float w[8], y[8];
             Vec8<float>::load(weight + c * 8, w);
 #pragma unroll
@@ -120,40 +136,77 @@ add_rmsnorm_vec_kernel(float* __restrict__ resid, const TA* __restrict__ delta,
     }
 }
 
-template <typename TA>
+template <typename TA, typename TD>
 static int launch_add_rmsnorm(float* resid, const void* delta, const float* weight, float eps, void* out,
-                              const int* rows, int n_rows, int hidden, cudaStream_t stream) {
-    const bool aligned = (((uintptr_t)resid | (uintptr_t)delta | (uintptr_t)weight | (uintptr_t)out) & 15) == 0;
+                              const int* rows, int n_rows, int hidden, const void* extra, const float* share,
+                              cudaStream_t stream) {
+    const bool aligned = (((uintptr_t)resid | (uintptr_t)delta | (uintptr_t)weight | (uintptr_t)out | (uintptr_t)extra) & 15) == 0;
     if (hidden % 8 == 0 && hidden <= 8192 && aligned) {
-        MRUN_CHECK_CUDA(launch_kernel(add_rmsnorm_vec_kernel<TA>, dim3(n_rows), dim3(256), 0, stream, resid,
-                                   (const TA*)delta, weight, eps, (TA*)out, rows, hidden), "add_rmsnorm");
+        MRUN_CHECK_CUDA(launch_kernel(add_rmsnorm_vec_kernel<TA, TD>, dim3(n_rows), dim3(256), 0, stream, resid,
+                                   (const TD*)delta, weight, eps, (TA*)out, rows, hidden, (const TA*)extra, share), "add_rmsnorm");
         return 0;
     }
     const size_t smem = (size_t)hidden * sizeof(float);
     if (smem > 48 * 1024)
-        MRUN_CHECK_CUDA(cudaFuncSetAttribute(add_rmsnorm_kernel<TA>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+        MRUN_CHECK_CUDA(cudaFuncSetAttribute(add_rmsnorm_kernel<TA, TD>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                              (int)smem), "add_rmsnorm");
-    add_rmsnorm_kernel<TA><<<n_rows, 256, smem, stream>>>(resid, (const TA*)delta, weight, eps, (TA*)out, rows,
-                                                          hidden);
+    add_rmsnorm_kernel<TA, TD><<<n_rows, 256, smem, stream>>>(resid, (const TD*)delta, weight, eps, (TA*)out, rows,
+                                                              hidden, (const TA*)extra, share);
     return 0;
 }
 
-MRUN_API int mrun_add_rmsnorm(float* resid, const void* delta, const float* weight, float eps, void* out,
-                              int act_dtype, const int* rows, int n_rows, int hidden,
-                              cudaStream_t stream) {
+// act_dtype: out's and extra's; delta_dtype: that or 32-bit.  extra and share (one factor a row) come together.
+MRUN_API int mrun_add_rmsnorm(float* resid, const void* delta, int delta_dtype, const float* weight, float eps, void* out,
+                              int act_dtype, const int* rows, int n_rows, int hidden, const void* extra,
+                              const float* share, cudaStream_t stream) {
     MRUN_REQUIRE(n_rows >= 0 && hidden > 0, "add_rmsnorm: bad sizes rows=%d hidden=%d", n_rows, hidden);
     MRUN_REQUIRE((size_t)hidden * sizeof(float) <= 200 * 1024, "add_rmsnorm: hidden=%d exceeds the supported 51200",
                  hidden);
+    MRUN_REQUIRE((extra == nullptr) == (share == nullptr), "add_rmsnorm: a second branch comes with its factors");
+    MRUN_REQUIRE(delta_dtype == MRUN_F32 || delta_dtype == act_dtype, "add_rmsnorm: the branch is 32-bit or of the output's type");
     if (n_rows == 0) return 0;
     int rc;
     if (act_dtype == MRUN_F32)
-        rc = launch_add_rmsnorm<float>(resid, delta, weight, eps, out, rows, n_rows, hidden, stream);
+        rc = launch_add_rmsnorm<float, float>(resid, delta, weight, eps, out, rows, n_rows, hidden, extra, share, stream);
+    else if (act_dtype == MRUN_BF16 && delta_dtype == MRUN_F32)
+        rc = launch_add_rmsnorm<__nv_bfloat16, float>(resid, delta, weight, eps, out, rows, n_rows, hidden, extra, share, stream);
     else if (act_dtype == MRUN_BF16)
-        rc = launch_add_rmsnorm<__nv_bfloat16>(resid, delta, weight, eps, out, rows, n_rows, hidden, stream);
+        rc = launch_add_rmsnorm<__nv_bfloat16, __nv_bfloat16>(resid, delta, weight, eps, out, rows, n_rows, hidden, extra, share,
+                                                              stream);
     else
         return mrun_set_error("add_rmsnorm: unknown dtype code %d", act_dtype);
     if (rc) return rc;
     MRUN_CHECK_LAUNCH("add_rmsnorm");
+    return 0;
+}
+
+// ------------------------------------------------------------------------------------------
+// y[t, :] += share[t] * x[t, :], the sum in 32-bit and rounded once to y's type: a branch that is a row
+// itself with a factor (an identity expert) where no other kernel adds it.
+// ------------------------------------------------------------------------------------------
+template <typename TY, typename TX>
+__global__ void add_scaled_rows_kernel(TY* __restrict__ y, const TX* __restrict__ x, const float* __restrict__ share,
+                                       int width) {
+    const float part = share[blockIdx.x];
+    if (part == 0.f) return;
+    const size_t row = (size_t)blockIdx.x * width;
+    for (int c = threadIdx.x; c < width; c += blockDim.x) y[row + c] = from_float<TY>(fmaf(part, to_float(x[row + c]), to_float(y[row + c])));
+}
+
+MRUN_API int mrun_add_scaled_rows(void* y, int y_dtype, const void* x, int x_dtype, const float* share, int rows, int width,
+                                  cudaStream_t stream) {
+    MRUN_REQUIRE(rows >= 0 && width > 0 && share != nullptr, "add_scaled_rows: bad sizes rows=%d width=%d", rows, width);
+    if (rows == 0) return 0;
+    using bf16 = __nv_bfloat16;
+    if (y_dtype == MRUN_F32 && x_dtype == MRUN_F32)
+        add_scaled_rows_kernel<float, float><<<rows, 256, 0, stream>>>((float*)y, (const float*)x, share, width);
+    else if (y_dtype == MRUN_F32 && x_dtype == MRUN_BF16)
+        add_scaled_rows_kernel<float, bf16><<<rows, 256, 0, stream>>>((float*)y, (const bf16*)x, share, width);
+    else if (y_dtype == MRUN_BF16 && x_dtype == MRUN_BF16)
+        add_scaled_rows_kernel<bf16, bf16><<<rows, 256, 0, stream>>>((bf16*)y, (const bf16*)x, share, width);
+    else
+        return mrun_set_error("add_scaled_rows: no kernel for the dtype codes %d and %d", y_dtype, x_dtype);
+    MRUN_CHECK_LAUNCH("add_scaled_rows");
     return 0;
 }
 
@@ -758,16 +811,42 @@ MRUN_API int mrun_head_gate(void* y, const void* gate, long ldg, int act_dtype, 
 // and whose keys (`dim` a head) and values (`vdim` a head) may differ in size.
 //   v_off < 0: the layer has no value projection and the values are the keys as they were
 //   projected, before the norm and the rotation (vdim = dim).
+//   HeadExtras: biases of the projections, added before anything else; values kept for a later layer
+//   of the step, and values blended with those an earlier layer kept.
 // q is worked on in place; a negative slot skips the page writes.  One warp per (token, q or k
 // or v head); the head's vector is staged in shared memory in 32-bit.
 // ------------------------------------------------------------------------------------------
+struct HeadExtras {
+    const float* bias;          // [q heads | k heads | v heads] or null
+    const void* first;          // row t's values of an earlier layer at first + t * ld_first (the activation type), or null
+    long ld_first;
+    float share;                // v <- (1 - share) * v + share * first
+    void* keep;                 // gets v (with its bias, before the blend), row t at keep + t * ld_keep; or null
+    long ld_keep;
+};
+
+// Eight (or fewer) features of a value head from feature e of the token's value row on.
+template <typename TA, int N>
+__device__ __forceinline__ void extend_values(const HeadExtras& x, const float* vbias, int t, int e, float (&v)[N]) {
+    if (vbias)
+#pragma unroll
+        for (int i = 0; i < N; ++i) v[i] += vbias[e + i];
+    if (x.keep)
+#pragma unroll
+        for (int i = 0; i < N; ++i) ((TA*)x.keep)[(size_t)t * x.ld_keep + e + i] = from_float<TA>(v[i]);
+    if (x.first)
+#pragma unroll
+        for (int i = 0; i < N; ++i)
+            v[i] = (1.f - x.share) * v[i] + x.share * to_float(((const TA*)x.first)[(size_t)t * x.ld_first + e + i]);
+}
+
 template <typename TA>
 __global__ void head_norm_rope_cache_kernel(TA* __restrict__ x, long ld, long q_off, long k_off, long v_off,
                                             const float* __restrict__ q_weight, const float* __restrict__ k_weight,
                                             float eps, const float2* __restrict__ rot, int rotary_dim, int interleaved,
                                             const int* __restrict__ slots, TA* __restrict__ k_cache,
                                             TA* __restrict__ v_cache, int tokens, int heads, int kv_heads, int dim,
-                                            int vdim, int page_size) {
+                                            int vdim, int page_size, const HeadExtras extras) {
     extern __shared__ float vec_buf[];
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int per_token = heads + (v_off >= 0 ? 2 : 1) * kv_heads;
@@ -777,29 +856,35 @@ __global__ void head_norm_rope_cache_kernel(TA* __restrict__ x, long ld, long q_
     const bool is_q = slot_head < heads;
     const bool is_k = !is_q && slot_head < heads + kv_heads;
     const int slot = slots ? slots[t] : -1;
-    if (!is_q && slot < 0) return;
+    if (!is_q && slot < 0 && (is_k || !extras.keep)) return;
     const int page = slot >= 0 ? slot / page_size : 0, off = slot >= 0 ? slot - page * page_size : 0;
     TA* row = x + (size_t)t * ld;
-    if (!is_q && !is_k) {       // a value head of a projection of its own: plain copy
+    if (!is_q && !is_k) {       // a value head of a projection of its own
         const int g = slot_head - heads - kv_heads;
         const TA* src = row + v_off + (size_t)g * vdim;
-        TA* dst = v_cache + (((size_t)page * kv_heads + g) * page_size + off) * vdim;
-        for (int e = lane; e < vdim; e += 32) dst[e] = src[e];
+        TA* dst = slot < 0 ? nullptr : v_cache + (((size_t)page * kv_heads + g) * page_size + off) * vdim;
+        const float* vbias = extras.bias ? extras.bias + (size_t)(heads + kv_heads) * dim : nullptr;
+        for (int e = lane; e < vdim; e += 32) {
+            float v[1] = {to_float(src[e])};
+            extend_values<TA, 1>(extras, vbias, t, g * vdim + e, v);
+            if (dst) dst[e] = from_float<TA>(v[0]);
+        }
         return;
     }
     const int g = is_q ? slot_head : slot_head - heads;
     TA* src = row + (is_q ? q_off : k_off) + (size_t)g * dim;
     TA* dst = is_q ? src : k_cache + (((size_t)page * kv_heads + g) * page_size + off) * dim;
     float* vec = vec_buf + warp * dim;
+    const float* bias = extras.bias ? extras.bias + (size_t)slot_head * dim : nullptr;
     float ss = 0.f;
     for (int e = lane; e < dim; e += 32) {
-        const float v = to_float(src[e]);
+        const float v = to_float(src[e]) + (bias ? bias[e] : 0.f);
         vec[e] = v;
         ss += v * v;
     }
     if (is_k && v_off < 0) {    // the values are the keys as projected
         TA* vdst = v_cache + (((size_t)page * kv_heads + g) * page_size + off) * vdim;
-        for (int e = lane; e < dim; e += 32) vdst[e] = src[e];
+        for (int e = lane; e < dim; e += 32) vdst[e] = from_float<TA>(vec[e]);
     }
     const float* weight = is_q ? q_weight : k_weight;
     if (weight) {
@@ -825,7 +910,7 @@ __global__ void head_norm_rope_cache_kernel(TA* __restrict__ x, long ld, long q_
     }
 }
 
-// The same for bfloat16 heads of 16, 32, 64, 128 or 256 features with keys and values of one size,
+// The same for bfloat16 heads of 16, 32, 64, 128 or 256 features with values of a multiple of 8,
 // half-split pairs and a rotating part that is a multiple of 16 features (or none): LANES = dim / 8
 // lanes share a head, eight values (16 bytes) a lane, so a row is read and written in whole 16-byte
 // pieces; the sum of squares and the rotation's partner values (the lane rotary_dim / 16 further
@@ -837,7 +922,7 @@ head_norm_rope_cache_vec_kernel(__nv_bfloat16* __restrict__ x, long ld, long q_o
                                 const float* __restrict__ q_weight, const float* __restrict__ k_weight, float eps,
                                 const float2* __restrict__ rot, int rotary_dim, const int* __restrict__ slots,
                                 __nv_bfloat16* __restrict__ k_cache, __nv_bfloat16* __restrict__ v_cache, int tokens,
-                                int heads, int kv_heads, int page_size) {
+                                int heads, int kv_heads, int vdim, int page_size, const HeadExtras extras) {
     constexpr int dim = LANES * 8;
     const int sub = threadIdx.x % LANES;                       // this lane's place in its head
     const int per_token = heads + (v_off >= 0 ? 2 : 1) * kv_heads;
@@ -850,22 +935,30 @@ head_norm_rope_cache_vec_kernel(__nv_bfloat16* __restrict__ x, long ld, long q_o
     const bool is_q = slot_head < heads;
     const bool is_k = !is_q && slot_head < heads + kv_heads;
     const int slot = slots ? slots[t] : -1;
-    if (!is_q && slot < 0) return;
+    if (!is_q && slot < 0 && (is_k || !extras.keep)) return;
     const int page = slot >= 0 ? slot / page_size : 0, off = slot >= 0 ? slot - page * page_size : 0;
     __nv_bfloat16* row = x + (size_t)t * ld;
-    if (!is_q && !is_k) {       // a value head of a projection of its own: plain copy
+    if (!is_q && !is_k) {       // a value head of a projection of its own
         const int g = slot_head - heads - kv_heads;
-        const uint4* src = reinterpret_cast<const uint4*>(row + v_off + (size_t)g * dim);
-        uint4* dst = reinterpret_cast<uint4*>(v_cache + (((size_t)page * kv_heads + g) * page_size + off) * dim);
-        dst[sub] = src[sub];
+        const __nv_bfloat16* src = row + v_off + (size_t)g * vdim;
+        __nv_bfloat16* dst = slot < 0 ? nullptr : v_cache + (((size_t)page * kv_heads + g) * page_size + off) * vdim;
+        const float* vbias = extras.bias ? extras.bias + (size_t)(heads + kv_heads) * dim : nullptr;
+        for (int c = sub; c < (vdim >> 3); c += LANES) {
+            if (vbias || extras.keep || extras.first) {
+                float v[8];
+                Vec8<__nv_bfloat16>::load(src + c * 8, v);
+                extend_values<__nv_bfloat16, 8>(extras, vbias, t, g * vdim + c * 8, v);
+                if (dst) Vec8<__nv_bfloat16>::store(dst + c * 8, v);
+            } else {
+                reinterpret_cast<uint4*>(dst)[c] = reinterpret_cast<const uint4*>(src)[c];
+            }
+        }
         return;
     }
     const int g = is_q ? slot_head : slot_head - heads;
     __nv_bfloat16* src = row + (is_q ? q_off : k_off) + (size_t)g * dim;
     __nv_bfloat16* dst = is_q ? src : k_cache + (((size_t)page * kv_heads + g) * page_size + off) * dim;
     const uint4 raw = reinterpret_cast<const uint4*>(src)[sub];
-    if (is_k && v_off < 0)      // the values are the keys as projected
-        reinterpret_cast<uint4*>(v_cache + (((size_t)page * kv_heads + g) * page_size + off) * dim)[sub] = raw;
     float v[8];
     {
         const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&raw);
@@ -875,6 +968,14 @@ head_norm_rope_cache_vec_kernel(__nv_bfloat16* __restrict__ x, long ld, long q_o
             v[2 * i] = f.x; v[2 * i + 1] = f.y;
         }
     }
+    if (extras.bias) {
+        float b[8];
+        Vec8<float>::load(extras.bias + (size_t)slot_head * dim + sub * 8, b);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) v[i] += b[i];
+    }
+    if (is_k && v_off < 0)      // the values are the keys as projected
+        Vec8<__nv_bfloat16>::store(v_cache + (((size_t)page * kv_heads + g) * page_size + off) * dim + sub * 8, v);
     const float* weight = is_q ? q_weight : k_weight;
     if (weight) {
         float ss = 0.f;
@@ -912,19 +1013,21 @@ template <int LANES>
 static void launch_head_norm_rope_cache_vec(void* x, long ld, long q_off, long k_off, long v_off, const float* q_weight,
                                             const float* k_weight, float eps, const float* rot, int rotary_dim,
                                             const int* slots, void* k_cache, void* v_cache, int tokens, int heads,
-                                            int kv_heads, int page_size, cudaStream_t stream) {
+                                            int kv_heads, int vdim, int page_size, const HeadExtras& extras,
+                                            cudaStream_t stream) {
     const long items = (long)tokens * (heads + (v_off >= 0 ? 2 : 1) * kv_heads);
     const long threads = items * LANES;
     head_norm_rope_cache_vec_kernel<LANES><<<(unsigned)((threads + 127) / 128), 128, 0, stream>>>(
         (__nv_bfloat16*)x, ld, q_off, k_off, v_off, q_weight, k_weight, eps, (const float2*)rot, rotary_dim, slots,
-        (__nv_bfloat16*)k_cache, (__nv_bfloat16*)v_cache, tokens, heads, kv_heads, page_size);
+        (__nv_bfloat16*)k_cache, (__nv_bfloat16*)v_cache, tokens, heads, kv_heads, vdim, page_size, extras);
 }
 
 MRUN_API int mrun_head_norm_rope_cache(void* x, long ld, long q_off, long k_off, long v_off, int act_dtype,
                                        const float* q_weight, const float* k_weight, float eps, const float* rot,
                                        int rotary_dim, int pairing, const int* slots, void* k_cache, void* v_cache,
                                        int tokens, int heads, int kv_heads, int dim, int vdim, int page_size,
-                                       cudaStream_t stream) {
+                                       const float* bias, const void* first, long ld_first, float share, void* keep,
+                                       long ld_keep, cudaStream_t stream) {
     MRUN_REQUIRE(tokens >= 0 && heads > 0 && kv_heads > 0 && dim > 0 && vdim > 0 && page_size > 0,
                  "head_norm_rope_cache: bad sizes tokens=%d heads=%d kv_heads=%d dim=%d vdim=%d page_size=%d", tokens,
                  heads, kv_heads, dim, vdim, page_size);
@@ -934,6 +1037,11 @@ MRUN_API int mrun_head_norm_rope_cache(void* x, long ld, long q_off, long k_off,
     MRUN_REQUIRE(v_off >= 0 || vdim == dim, "head_norm_rope_cache: values that are the keys have the keys' size (%d), not %d",
                  dim, vdim);
     MRUN_REQUIRE(q_off >= 0 && k_off >= 0, "head_norm_rope_cache: negative column of q or k");
+    MRUN_REQUIRE(v_off >= 0 || (first == nullptr && keep == nullptr),
+                 "head_norm_rope_cache: values that are the keys are neither kept nor blended");
+    MRUN_REQUIRE((first == nullptr || ld_first >= (long)kv_heads * vdim) && (keep == nullptr || ld_keep >= (long)kv_heads * vdim),
+                 "head_norm_rope_cache: the kept values' rows do not hold %d features", kv_heads * vdim);
+    const HeadExtras extras = {bias, first, ld_first, share, keep, ld_keep};
     MRUN_REQUIRE((size_t)dim * sizeof(float) * 4 <= 48 * 1024, "head_norm_rope_cache: dim=%d exceeds the supported 3072", dim);
     if (tokens == 0) return 0;
     const int warps = 4;
@@ -942,13 +1050,13 @@ MRUN_API int mrun_head_norm_rope_cache(void* x, long ld, long q_off, long k_off,
     const size_t smem = (size_t)warps * dim * sizeof(float);
     if (slots == nullptr) k_cache = v_cache = nullptr;
     const bool aligned = ((((uintptr_t)x) | ((uintptr_t)k_cache) | ((uintptr_t)v_cache) | ((uintptr_t)q_weight) |
-                           ((uintptr_t)k_weight)) & 15) == 0 &&
+                           ((uintptr_t)k_weight) | ((uintptr_t)bias)) & 15) == 0 &&
                          ld % 8 == 0 && q_off % 8 == 0 && k_off % 8 == 0 && (v_off < 0 || v_off % 8 == 0);
-    if (act_dtype == MRUN_BF16 && aligned && dim == vdim && pairing == 0 && rotary_dim % 16 == 0 &&
+    if (act_dtype == MRUN_BF16 && aligned && vdim % 8 == 0 && (v_off >= 0 || vdim == dim) && pairing == 0 && rotary_dim % 16 == 0 &&
         (dim == 16 || dim == 32 || dim == 64 || dim == 128 || dim == 256)) {
 #define MRUN_HEAD_VEC(L)                                                                                              \
     launch_head_norm_rope_cache_vec<L>(x, ld, q_off, k_off, v_off, q_weight, k_weight, eps, rot, rot ? rotary_dim : 0, \
-                                       slots, k_cache, v_cache, tokens, heads, kv_heads, page_size, stream)
+                                       slots, k_cache, v_cache, tokens, heads, kv_heads, vdim, page_size, extras, stream)
         switch (dim) {
             case 16: MRUN_HEAD_VEC(2); break;
             case 32: MRUN_HEAD_VEC(4); break;
@@ -963,11 +1071,11 @@ MRUN_API int mrun_head_norm_rope_cache(void* x, long ld, long q_off, long k_off,
     if (act_dtype == MRUN_F32)
         head_norm_rope_cache_kernel<float><<<blocks, warps * 32, smem, stream>>>(
             (float*)x, ld, q_off, k_off, v_off, q_weight, k_weight, eps, (const float2*)rot, rotary_dim, pairing, slots,
-            (float*)k_cache, (float*)v_cache, tokens, heads, kv_heads, dim, vdim, page_size);
+            (float*)k_cache, (float*)v_cache, tokens, heads, kv_heads, dim, vdim, page_size, extras);
     else if (act_dtype == MRUN_BF16)
         head_norm_rope_cache_kernel<__nv_bfloat16><<<blocks, warps * 32, smem, stream>>>(
             (__nv_bfloat16*)x, ld, q_off, k_off, v_off, q_weight, k_weight, eps, (const float2*)rot, rotary_dim, pairing,
-            slots, (__nv_bfloat16*)k_cache, (__nv_bfloat16*)v_cache, tokens, heads, kv_heads, dim, vdim, page_size);
+            slots, (__nv_bfloat16*)k_cache, (__nv_bfloat16*)v_cache, tokens, heads, kv_heads, dim, vdim, page_size, extras);
     else
         return mrun_set_error("head_norm_rope_cache: unknown dtype code %d", act_dtype);
     MRUN_CHECK_LAUNCH("head_norm_rope_cache");

@@ -49,12 +49,26 @@ struct Fusion {
     int act;                     // EPI_GATED: the gate's function (MRUN_GATE_*); EPI_BATCHED: MRUN_ACT_* or 0
     // EPI_BATCHED (the product is blockIdx.y): W matrices one after the other, x and y this far apart
     long batch_x, batch_y;
+    // EPI_BATCHED, in this order, in 32-bit: bias[N] is added; columns from blend_col on become
+    // (1 - blend_share) * y + blend_share * blend[row, column - blend_col]; the product is multiplied by
+    // sigmoid(gate[row, b]); act.  Null: left out.
+    const float* bias;
+    const bf16* blend;
+    long ld_blend;
+    int blend_col, blend_cols;
+    float blend_share;
+    const bf16* gate;
+    long ld_gate;
     // x is the xw of a product before: the row's scale is rsqrt(in_sums[row] * 2^-30 / width + eps)
     const unsigned long long* in_sums;   // [16] totals of squares, or null: x is taken as it is
     float in_eps, in_inv_width;
     // EPI_RESIDUAL: resid[M, ldr] += y; xw_out[M, N] = bf16(resid * norm_w); out_sums[16] += squares
+    // extra (or null): rows of x's type that join the stream too, with one factor a row
     float* resid;
     long ldr;
+    const bf16* extra;
+    long ld_extra;
+    const float* share;
     const float* norm_w;
     bf16* xw_out;
     unsigned long long* out_sums;
@@ -238,6 +252,13 @@ skinny_kernel(const bf16* __restrict__ x, const bf16* __restrict__ w, TOut* __re
 #pragma unroll
                 for (int wi = 0; wi < WARPS; ++wi) s += red[wi][row][token];
                 s *= row_scale[token];
+                if constexpr (EPI == EPI_BATCHED) {
+                    const int n = n0 + row, c = n - f.blend_col;
+                    if (f.bias) s += f.bias[n];
+                    if (f.blend && c >= 0 && c < f.blend_cols)
+                        s = (1.f - f.blend_share) * s + f.blend_share * __bfloat162float(f.blend[(size_t)token * f.ld_blend + c]);
+                    if (f.gate) s /= 1.f + expf(-__bfloat162float(f.gate[(size_t)token * f.ld_gate + blockIdx.y]));
+                }
                 // an activation sees the sum as the layer would have stored it
                 if (EPI == EPI_BATCHED && f.act) s = mrun::plain_act(f.act, __bfloat162float(__float2bfloat16_rn(s)));
                 store_out<TOut>(y + (size_t)token * ldy + n0 + row, s);
@@ -273,6 +294,10 @@ skinny_kernel(const bf16* __restrict__ x, const bf16* __restrict__ w, TOut* __re
 #pragma unroll
                 for (int wi = 0; wi < WARPS; ++wi) s += red[wi][row][token];
                 v = stream_tile[i] + s * row_scale[token];
+                if (f.extra) {
+                    const float part = f.share[token];
+                    if (part != 0.f) v = fmaf(part, __bfloat162float(f.extra[(size_t)token * f.ld_extra + n0 + row]), v);
+                }
                 f.resid[(size_t)token * f.ldr + n0 + row] = v;
                 f.xw_out[(size_t)token * N + n0 + row] = __float2bfloat16_rn(v * norm_tile[row]);
             }
@@ -368,18 +393,21 @@ void dispatch(const bf16* x, const bf16* w, TOut* y, int M, int N, int K, long l
 // multiplied by rsqrt(in_sums[row] * 2^-30 / K + in_eps).
 // resid != null: nothing is written to y; instead resid[M, N] (32-bit, dense) += the product,
 // xw_out[M, N] = bf16(resid * norm_w) and out_sums[row] (16 unsigned 64-bit integers, zero before
-// the call) gets the row's sum of squares of resid in units of 2^-30.
+// the call) gets the row's sum of squares of resid in units of 2^-30.  extra != null (with resid): rows
+// [M, N] of bfloat16, ld_extra elements apart, that are added to resid too, times share[row].
 // rows: the rows of W a block takes, 8..16, or 0 for the count that fills the device most evenly.
 MRUN_API int mrun_gemm_skinny(const void* x, const void* w, void* y, int out_dtype, int gate, int M, int N,
                               int K, long ldx, long ldy, const unsigned long long* in_sums, float in_eps,
                               float* resid, const float* norm_w, void* xw_out, unsigned long long* out_sums,
-                              int rows, cudaStream_t stream) {
+                              int rows, const void* extra, long ld_extra, const float* share, cudaStream_t stream) {
     MRUN_REQUIRE(M >= 0 && N > 0 && K > 0, "gemm_skinny: bad sizes M=%d N=%d K=%d", M, N, K);
     MRUN_REQUIRE(rows == 0 || (rows >= 8 && rows <= 16), "gemm_skinny: rows=%d a block must be 0 (chosen here) or 8..16", rows);
     MRUN_REQUIRE(M <= 16, "gemm_skinny: M=%d exceeds the 16 rows this kernel takes", M);
     MRUN_REQUIRE(K % 32 == 0, "gemm_skinny: K=%d is not a multiple of 32", K);
     MRUN_REQUIRE(ldx >= K && ldx % 8 == 0, "gemm_skinny: ldx=%ld must be a multiple of 8 and at least K=%d", ldx, K);
     MRUN_REQUIRE(((uintptr_t)x & 15) == 0 && ((uintptr_t)w & 15) == 0, "gemm_skinny: x and W must be 16-byte aligned");
+    MRUN_REQUIRE((extra == nullptr) == (share == nullptr) && (extra == nullptr || (resid != nullptr && ld_extra >= N)),
+                 "gemm_skinny: extra rows come with their factors and the residual epilogue");
     Fusion f = {};
     f.act = gate;
     f.in_sums = in_sums;
@@ -394,6 +422,9 @@ MRUN_API int mrun_gemm_skinny(const void* x, const void* w, void* y, int out_dty
         if (M == 0) return 0;
         f.resid = resid;
         f.ldr = N;
+        f.extra = (const bf16*)extra;
+        f.ld_extra = ld_extra;
+        f.share = share;
         f.norm_w = norm_w;
         f.xw_out = (bf16*)xw_out;
         f.out_sums = out_sums;
@@ -419,9 +450,15 @@ MRUN_API int mrun_gemm_skinny(const void* x, const void* w, void* y, int out_dty
 }
 
 // y[b] = act(x[b] · w[b]^T) for `batch` products of one shape in one launch: w dense [batch, N, K], x and y
-// with the given strides between products.  act: MRUN_ACT_* or 0.
+// with the given strides between products.  act: MRUN_ACT_* or 0.  bias (or null): float32 [N]; blend (or
+// null): rows of bfloat16, ld_blend apart, that columns blend_col .. blend_col + blend_cols - 1 are blended
+// with by blend_share; both for one product only.  gate (or null): rows of bfloat16, ld_gate apart, one entry
+// a product, whose sigmoid multiplies it.  What comes out of in_sums != null (one product only) is as for mrun_gemm_skinny.
 MRUN_API int mrun_gemm_skinny_batched(const void* x, const void* w, void* y, int out_dtype, int act, int batch, int M,
-                                      int N, int K, long ldx, long ldy, long batch_x, long batch_y, cudaStream_t stream) {
+                                      int N, int K, long ldx, long ldy, long batch_x, long batch_y, const float* bias,
+                                      const void* blend, long ld_blend, int blend_col, int blend_cols, float blend_share,
+                                      const void* gate, long ld_gate, const unsigned long long* in_sums, float in_eps,
+                                      cudaStream_t stream) {
     MRUN_REQUIRE(M >= 0 && N > 0 && K > 0 && batch > 0 && batch <= 65535, "gemm_skinny_batched: bad sizes batch=%d M=%d N=%d K=%d",
                  batch, M, N, K);
     MRUN_REQUIRE(M <= 16, "gemm_skinny_batched: M=%d exceeds the 16 rows this kernel takes", M);
@@ -437,6 +474,21 @@ MRUN_API int mrun_gemm_skinny_batched(const void* x, const void* w, void* y, int
     f.in_inv_width = 1.f / (float)K;
     f.batch_x = batch_x;
     f.batch_y = batch_y;
+    MRUN_REQUIRE(batch == 1 || (bias == nullptr && blend == nullptr && in_sums == nullptr),
+                 "gemm_skinny_batched: a bias, a blend and unfinished norms go with one product");
+    MRUN_REQUIRE(blend == nullptr || (blend_col >= 0 && blend_cols >= 0 && blend_col + blend_cols <= N && ld_blend >= blend_cols),
+                 "gemm_skinny_batched: the blended columns %d .. do not lie within %d", blend_col, N);
+    MRUN_REQUIRE(gate == nullptr || ld_gate >= batch, "gemm_skinny_batched: the gate's rows hold fewer than %d entries", batch);
+    f.bias = bias;
+    f.blend = (const bf16*)blend;
+    f.ld_blend = ld_blend;
+    f.blend_col = blend_col;
+    f.blend_cols = blend_cols;
+    f.blend_share = blend_share;
+    f.gate = (const bf16*)gate;
+    f.ld_gate = ld_gate;
+    f.in_sums = in_sums;
+    f.in_eps = in_eps;
     if (out_dtype == MRUN_BF16)
         dispatch<bf16, EPI_BATCHED>((const bf16*)x, (const bf16*)w, (bf16*)y, M, N, K, ldx, ldy, f, 0, batch, stream);
     else if (out_dtype == MRUN_F32)

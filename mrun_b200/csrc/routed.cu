@@ -16,13 +16,18 @@
 //                 u = clamp(up, -limit, limit), y = g * sigmoid(alpha * g) * (u + 1), times the
 //                 token's weight of the block's expert or the row's weight
 //
-// And the choice of a router with sigmoid scores and groups of experts:
+// And the choice of a router with groups of experts:
 //
-//   route_grouped the experts form equal groups of neighbours; a group's score is the sum of its
-//                 group_top largest scores; only experts of the keep best groups can be chosen;
-//                 the top allowed experts with the largest scores weigh score / (sum + 1e-20) *
-//                 scale; one more logit column, if there is one, becomes the sigmoid weight of a
-//                 shared expert
+//   route_grouped scores are the logits' sigmoids or their softmax; experts are ranked by score (+ a
+//                 correction per expert); they form equal groups of neighbours; a group's score is the
+//                 sum of its group_top largest ranks; only experts of the keep best groups can be
+//                 chosen; the top allowed experts with the largest ranks weigh score / (sum + 1e-20) *
+//                 scale, or score * scale; the last `identity` experts hand the token's row on
+//                 unchanged, so that one number a token, the sum of their weights, stands for them;
+//                 one more logit column, if there is one, becomes the sigmoid weight of a shared expert
+//
+// A pair that has no rows (an identity expert) is -1 in the chosen list: it is not counted, its dest is
+// -1, and combine_rows adds the token's row times its factor instead.
 //
 // Inside an expert's range the rows stand in the order in which the pairs arrived (an atomic
 // counter); a row's result does not depend on where in the range it stands, and the combine adds
@@ -65,6 +70,10 @@ __global__ void moe_place_kernel(const int* __restrict__ chosen, const float* __
     const int i = blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= pairs) return;
     const int e = chosen[i], t = i / top;
+    if (e < 0 || e >= experts) {
+        dest[i] = -1;
+        return;
+    }
     const int row = atomicAdd(cursor + e, 1);
     source[row] = t;
     row_weight[row] = weights[(size_t)t * experts + e];
@@ -110,10 +119,13 @@ __global__ void relu2_rows_kernel(const TA* __restrict__ u, TA* __restrict__ act
     }
 }
 
+// base may be null; extra: rows of TA with one factor a token each, or null.
 template <typename TA, typename TB, bool VEC>
 __global__ void combine_rows_kernel(const TB* __restrict__ base, const TA* __restrict__ rows,
-                                    const int* __restrict__ dest, float* __restrict__ out, int top, int width) {
+                                    const int* __restrict__ dest, float* __restrict__ out, int top, int width,
+                                    const TA* __restrict__ extra, const float* __restrict__ share) {
     const size_t t = blockIdx.x;
+    const float part = extra ? share[t] : 0.f;
     if constexpr (VEC) {
         for (int c = threadIdx.x * 8; c < width; c += blockDim.x * 8) {
             float s[8];
@@ -121,9 +133,17 @@ __global__ void combine_rows_kernel(const TB* __restrict__ base, const TA* __res
             else
 #pragma unroll
                 for (int i = 0; i < 8; ++i) s[i] = 0.f;
-            for (int k = 0; k < top; ++k) {
+            if (part != 0.f) {
                 float r[8];
-                Vec8<TA>::load(rows + (size_t)dest[t * top + k] * width + c, r);
+                Vec8<TA>::load(extra + t * width + c, r);
+#pragma unroll
+                for (int i = 0; i < 8; ++i) s[i] = fmaf(part, r[i], s[i]);
+            }
+            for (int k = 0; k < top; ++k) {
+                const int row = dest[t * top + k];
+                if (row < 0) continue;
+                float r[8];
+                Vec8<TA>::load(rows + (size_t)row * width + c, r);
 #pragma unroll
                 for (int i = 0; i < 8; ++i) s[i] += r[i];
             }
@@ -132,7 +152,11 @@ __global__ void combine_rows_kernel(const TB* __restrict__ base, const TA* __res
     } else {
         for (int c = threadIdx.x; c < width; c += blockDim.x) {
             float s = base ? to_float(base[t * width + c]) : 0.f;
-            for (int k = 0; k < top; ++k) s += to_float(rows[(size_t)dest[t * top + k] * width + c]);
+            if (part != 0.f) s = fmaf(part, to_float(extra[t * width + c]), s);
+            for (int k = 0; k < top; ++k) {
+                const int row = dest[t * top + k];
+                if (row >= 0) s += to_float(rows[(size_t)row * width + c]);
+            }
             out[t * width + c] = s;
         }
     }
@@ -155,38 +179,55 @@ __global__ void table_route_kernel(const int* __restrict__ ids, const int* __res
     }
 }
 
-// A warp a token.  logits: row t at logits + t * ldz, experts columns and then `extra` (0 or 1)
-// more.  weights: dense [tokens, experts]; shared_w: [tokens] or null; chosen: [tokens, top] or
-// null.  Ties go to the lower index.  Shared memory: experts + groups floats a warp.
+// A warp a token.  logits: row t at logits + t * ldz, `total` = experts + identity columns and then one
+// more where shared_w is not null.  softmax: the scores are the softmax over the `total` logits, else their
+// sigmoids.  correction: [total] or null.  weights: dense [tokens, experts]; identity_w, shared_w: [tokens]
+// or null; chosen: [tokens, top] or null.  Ties go to the lower index; a rank that is not a number is
+// never chosen (its pair is -1).  in_sums != null: the rows that the identity experts hand on still lack their
+// norm's factor rsqrt(in_sums[t] * 2^-30 / width + eps), which then goes into identity_w.  Shared memory:
+// total + groups floats a warp.
 __global__ void __launch_bounds__(128)
-route_grouped_kernel(const float* __restrict__ logits, long ldz, float* __restrict__ weights,
-                     float* __restrict__ shared_w, int* __restrict__ chosen, int tokens, int experts, int top,
-                     int groups, int keep, int group_top, float scale) {
+route_grouped_kernel(const float* __restrict__ logits, long ldz, int softmax, const float* __restrict__ correction,
+                     float* __restrict__ weights, float* __restrict__ identity_w, float* __restrict__ shared_w,
+                     int* __restrict__ chosen, int tokens, int experts, int total, int top, int groups, int keep,
+                     int group_top, int renormalize, float scale, const unsigned long long* __restrict__ in_sums,
+                     float in_inv_width, float in_eps) {
     extern __shared__ float route_smem[];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int t = blockIdx.x * 4 + warp;
     if (t >= tokens) return;
-    float* s = route_smem + (size_t)warp * (experts + groups);
-    float* gs = s + experts;
+    float* rank = route_smem + (size_t)warp * (total + groups);
+    float* gs = rank + total;
     const float* z = logits + (size_t)t * ldz;
-    for (int e = lane; e < experts; e += 32) {
-        s[e] = 1.f / (1.f + expf(-z[e]));
-        weights[(size_t)t * experts + e] = 0.f;
+    float largest = 0.f, inv_sum = 1.f;
+    if (softmax) {
+        largest = -INFINITY;
+        for (int e = lane; e < total; e += 32) largest = fmaxf(largest, z[e]);
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) largest = fmaxf(largest, __shfl_xor_sync(0xffffffffu, largest, o));
+        float sum = 0.f;
+        for (int e = lane; e < total; e += 32) sum += expf(z[e] - largest);
+        inv_sum = 1.f / warp_sum(sum);
     }
-    if (shared_w && lane == 0) shared_w[t] = 1.f / (1.f + expf(-z[experts]));
+    auto score = [&](int e) { return softmax ? expf(z[e] - largest) * inv_sum : 1.f / (1.f + expf(-z[e])); };
+    for (int e = lane; e < total; e += 32) {
+        rank[e] = score(e) + (correction ? correction[e] : 0.f);
+        if (e < experts) weights[(size_t)t * experts + e] = 0.f;
+    }
+    if (shared_w && lane == 0) shared_w[t] = 1.f / (1.f + expf(-z[total]));
     __syncwarp();
-    const int size = experts / groups;
+    const int size = total / groups;
     if (groups > 1) {
-        // a group's score: its group_top largest scores, found one after the other in the order
-        // (larger score, then lower index)
+        // a group's score: its group_top largest ranks, found one after the other in the order
+        // (larger rank, then lower index)
         for (int g = lane; g < groups; g += 32) {
             float sum = 0.f, last = INFINITY;
             int last_i = -1;
             for (int k = 0; k < group_top && k < size; ++k) {
-                float best = -1.f;
+                float best = -INFINITY;
                 int best_i = size;
                 for (int i = 0; i < size; ++i) {
-                    const float v = s[g * size + i];
+                    const float v = rank[g * size + i];
                     const bool after = v < last || (v == last && i > last_i);
                     if (after && (v > best || (v == best && i < best_i))) { best = v; best_i = i; }
                 }
@@ -195,12 +236,12 @@ route_grouped_kernel(const float* __restrict__ logits, long ldz, float* __restri
             gs[g] = sum;
         }
         __syncwarp();
-        // the keep best groups stay; the scores of the others leave the choice
+        // the keep best groups stay (+infinity marks them); the ranks of the others leave the choice
         for (int k = 0; k < keep; ++k) {
             float best = -INFINITY;
             int best_g = 0x7fffffff;
             for (int g = lane; g < groups; g += 32)
-                if (gs[g] > best || (gs[g] == best && g < best_g)) { best = gs[g]; best_g = g; }
+                if (gs[g] != INFINITY && (gs[g] > best || (gs[g] == best && g < best_g))) { best = gs[g]; best_g = g; }
 #pragma unroll
             for (int o = 16; o > 0; o >>= 1) {
                 const float ob = __shfl_xor_sync(0xffffffffu, best, o);
@@ -208,42 +249,46 @@ route_grouped_kernel(const float* __restrict__ logits, long ldz, float* __restri
                 if (ob > best || (ob == best && og < best_g)) { best = ob; best_g = og; }
             }
             __syncwarp();
-            if (lane == 0) gs[best_g] = -INFINITY;      // marks a group that stays
+            if (lane == 0 && best_g < groups) gs[best_g] = INFINITY;
             __syncwarp();
         }
-        for (int e = lane; e < experts; e += 32)
-            if (gs[e / size] != -INFINITY) s[e] = -1.f;
+        for (int e = lane; e < total; e += 32)
+            if (gs[e / size] != INFINITY) rank[e] = -INFINITY;
         __syncwarp();
     }
-    float total = 0.f, mine = 0.f;       // lane k keeps the score of the k-th choice
-    int mine_e = -1;
+    float sum = 0.f, unchanged = 0.f;
     for (int k = 0; k < top; ++k) {
-        float best = -1.f;
+        float best = -INFINITY;
         int best_e = 0x7fffffff;
-        for (int e = lane; e < experts; e += 32)
-            if (s[e] > best || (s[e] == best && e < best_e)) { best = s[e]; best_e = e; }
+        for (int e = lane; e < total; e += 32)
+            if (rank[e] > best) { best = rank[e]; best_e = e; }
 #pragma unroll
         for (int o = 16; o > 0; o >>= 1) {
             const float ob = __shfl_xor_sync(0xffffffffu, best, o);
             const int oe = __shfl_xor_sync(0xffffffffu, best_e, o);
             if (ob > best || (ob == best && oe < best_e)) { best = ob; best_e = oe; }
         }
+        const bool found = best_e < total;
         __syncwarp();
-        if (lane == 0) s[best_e] = -2.f;
+        if (lane == 0 && found) rank[best_e] = -INFINITY;
         __syncwarp();
-        total += best;
-        if (chosen && lane == 0) chosen[(size_t)t * top + k] = best_e;
-        if (k == lane) { mine = best; mine_e = best_e; }
+        const float s = found ? score(best_e) : 0.f;
+        sum += s;
+        if (found && best_e >= experts) unchanged += s;
+        if (chosen && lane == 0) chosen[(size_t)t * top + k] = found && best_e < experts ? best_e : -1;
+        if (lane == 0 && found && best_e < experts) weights[(size_t)t * experts + best_e] = s;
     }
-    // the weights need the total of all choices: lane k kept the k-th choice (chosen experts
-    // stand as -2 in s)
-    const float norm = scale / (total + 1e-20f);
-    if (top <= 32) {
-        if (lane < top) weights[(size_t)t * experts + mine_e] = mine * norm;
-    } else {
-        // more than 32 choices: recompute every chosen expert's score from its logit
-        for (int e = lane; e < experts; e += 32)
-            if (s[e] == -2.f) weights[(size_t)t * experts + e] = (1.f / (1.f + expf(-z[e]))) * norm;
+    const float norm = renormalize ? scale / (sum + 1e-20f) : scale;
+    if (identity_w && lane == 0) {
+        const float row = in_sums ? rsqrtf(__ull2float_rn(in_sums[t]) * (1.f / 1073741824.f) * in_inv_width + in_eps) : 1.f;
+        identity_w[t] = unchanged * norm * row;
+    }
+    if (norm != 1.f) {
+        __syncwarp();
+        for (int e = lane; e < experts; e += 32) {
+            const float w = weights[(size_t)t * experts + e];
+            if (w != 0.f) weights[(size_t)t * experts + e] = w * norm;
+        }
     }
 }
 
@@ -316,19 +361,27 @@ MRUN_API int mrun_table_route(const int* ids, const int* table, float* weights, 
     return 0;
 }
 
-MRUN_API int mrun_route_grouped(const float* logits, long ldz, float* weights, float* shared_w, int* chosen, int tokens,
-                                int experts, int top, int groups, int keep, int group_top, float scale,
-                                cudaStream_t stream) {
-    MRUN_REQUIRE(tokens >= 0 && experts > 0 && top > 0 && groups > 0 && keep > 0 && group_top > 0,
-                 "route_grouped: bad sizes tokens=%d experts=%d top=%d groups=%d", tokens, experts, top, groups);
-    MRUN_REQUIRE(experts % groups == 0 && keep <= groups && top <= keep * (experts / groups),
-                 "route_grouped: %d experts in %d groups of which %d stay cannot give %d choices", experts, groups, keep, top);
-    MRUN_REQUIRE(experts + groups <= 2048, "route_grouped: %d experts exceed the supported 2048", experts + groups);
-    MRUN_REQUIRE(ldz >= experts + (shared_w ? 1 : 0), "route_grouped: the logits' row stride is below the row");
+// score: 0 the softmax over all logits but the shared expert's, 1 the sigmoids.  The experts + identity
+// columns form the groups together.
+MRUN_API int mrun_route_grouped(const float* logits, long ldz, int score, const float* correction, float* weights,
+                                float* identity_w, float* shared_w, int* chosen, int tokens, int experts, int identity,
+                                int top, int groups, int keep, int group_top, int renormalize, float scale,
+                                const unsigned long long* in_sums, int in_width, float in_eps, cudaStream_t stream) {
+    MRUN_REQUIRE(tokens >= 0 && experts > 0 && identity >= 0 && top > 0 && groups > 0 && keep > 0 && group_top > 0,
+                 "route_grouped: bad sizes tokens=%d experts=%d identity=%d top=%d groups=%d", tokens, experts, identity, top, groups);
+    const int total = experts + identity;
+    MRUN_REQUIRE(score == 0 || score == 1, "route_grouped: unknown score code %d", score);
+    MRUN_REQUIRE(total % groups == 0 && keep <= groups && top <= keep * (total / groups),
+                 "route_grouped: %d experts in %d groups of which %d stay cannot give %d choices", total, groups, keep, top);
+    MRUN_REQUIRE(total + groups <= 2048, "route_grouped: %d experts exceed the supported 2048", total + groups);
+    MRUN_REQUIRE(ldz >= total + (shared_w ? 1 : 0), "route_grouped: the logits' row stride is below the row");
+    MRUN_REQUIRE(identity == 0 || identity_w != nullptr, "route_grouped: identity experts without a place for their weight");
     if (tokens == 0) return 0;
-    const size_t smem = 4 * (size_t)(experts + groups) * sizeof(float);
-    route_grouped_kernel<<<(tokens + 3) / 4, 128, smem, stream>>>(logits, ldz, weights, shared_w, chosen, tokens, experts,
-                                                                top, groups, keep, group_top, scale);
+    const size_t smem = 4 * (size_t)(total + groups) * sizeof(float);
+    route_grouped_kernel<<<(tokens + 3) / 4, 128, smem, stream>>>(logits, ldz, score == 0, correction, weights, identity_w, shared_w,
+                                                                chosen, tokens, experts, total, top, groups, keep, group_top,
+                                                                renormalize, scale, in_sums, 1.f / (float)(in_width > 0 ? in_width : 1),
+                                                                in_eps);
     MRUN_CHECK_LAUNCH("route_grouped");
     return 0;
 }
@@ -423,22 +476,26 @@ MRUN_API int mrun_relu2_rows(const void* u, void* act, int act_dtype, const floa
     return 0;
 }
 
-// base: [tokens, width] in the activation dtype (base_f32 = 0) or float32 (1), or null.
+// base: [tokens, width] in the activation dtype (base_f32 = 0) or float32 (1), or null; extra: rows of the
+// activation dtype that join with the factors share[t], or both null.
 MRUN_API int mrun_combine_rows(const void* base, int base_f32, const void* rows, int act_dtype, const int* dest,
-                               float* out, int tokens, int top, int width, cudaStream_t stream) {
+                               float* out, int tokens, int top, int width, const void* extra, const float* share,
+                               cudaStream_t stream) {
     MRUN_REQUIRE(tokens >= 0 && top > 0 && width > 0, "combine_rows: bad sizes tokens=%d top=%d width=%d", tokens, top, width);
     MRUN_REQUIRE(act_dtype == MRUN_BF16, "combine_rows: the sorted path runs in bfloat16");
+    MRUN_REQUIRE((extra == nullptr) == (share == nullptr), "combine_rows: extra rows come with their factors");
     if (tokens == 0) return 0;
-    const bool vec = width % 8 == 0 && ((((uintptr_t)base) | ((uintptr_t)rows) | ((uintptr_t)out)) & 15) == 0;
+    const bool vec = width % 8 == 0 && ((((uintptr_t)base) | ((uintptr_t)rows) | ((uintptr_t)out) | ((uintptr_t)extra)) & 15) == 0;
     using bf16 = __nv_bfloat16;
+    const bf16 *r = (const bf16*)rows, *x = (const bf16*)extra;
     if (base_f32 && vec)
-        combine_rows_kernel<bf16, float, true><<<tokens, 128, 0, stream>>>((const float*)base, (const bf16*)rows, dest, out, top, width);
+        combine_rows_kernel<bf16, float, true><<<tokens, 128, 0, stream>>>((const float*)base, r, dest, out, top, width, x, share);
     else if (base_f32)
-        combine_rows_kernel<bf16, float, false><<<tokens, 256, 0, stream>>>((const float*)base, (const bf16*)rows, dest, out, top, width);
+        combine_rows_kernel<bf16, float, false><<<tokens, 256, 0, stream>>>((const float*)base, r, dest, out, top, width, x, share);
     else if (vec)
-        combine_rows_kernel<bf16, bf16, true><<<tokens, 128, 0, stream>>>((const bf16*)base, (const bf16*)rows, dest, out, top, width);
+        combine_rows_kernel<bf16, bf16, true><<<tokens, 128, 0, stream>>>((const bf16*)base, r, dest, out, top, width, x, share);
     else
-        combine_rows_kernel<bf16, bf16, false><<<tokens, 256, 0, stream>>>((const bf16*)base, (const bf16*)rows, dest, out, top, width);
+        combine_rows_kernel<bf16, bf16, false><<<tokens, 256, 0, stream>>>((const bf16*)base, r, dest, out, top, width, x, share);
     MRUN_CHECK_LAUNCH("combine_rows");
     return 0;
 }

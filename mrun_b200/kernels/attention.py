@@ -111,7 +111,7 @@ def decode_cluster(library, ratio: int, page_size: int, tokens: int, kv_heads: i
 
 
 def supports_tensor_cores(dtype: torch.dtype, head_dim: int, group: int, value_dim: Optional[int] = None) -> bool:
-    """``value_dim``: where it differs from ``head_dim``; only kernels with a score form take that."""
+    """``value_dim``: where it differs from ``head_dim``."""
     sizes = (head_dim,) if value_dim is None else (head_dim, value_dim)
     return dtype == torch.bfloat16 and group <= 64 and all(n % 16 == 0 and 16 <= n <= 256 for n in sizes)
 
@@ -253,22 +253,23 @@ def latent_wide_ok(dtype: torch.dtype, width: int, value_dim: int) -> bool:
 
 def paged_attention(q: torch.Tensor, q_stride: int, out: torch.Tensor, cache, group, ctx,
                     heads: int, scale: float, window: int, raw=None, value_dim: int = 0,
-                    sink: bool = False, form: Optional[ScoreForm] = None) -> torch.Tensor:
+                    sink: Optional[torch.Tensor] = None, form: Optional[ScoreForm] = None) -> torch.Tensor:
     """``q``: the step's queries (row t at ``q_stride * t``, heads contiguous); ``cache``: the
     schedule entry's pages; ``group``: the step's view of the cache's group.  ``raw``, only where
     :func:`decode_fuses_input` holds: ``(q_weight, k_weight, eps, rot, rotary_dim, slots)`` for a
     ``q`` that is the projection's raw [q | k | v] rows.  ``value_dim``, for a cache whose rows
     are key and value at once (one tensor of pages, one kv head): how many of a row's first
     features the caller reads of the output; rows too wide for the per-head-size kernels then go
-    to the kernel for wide latent rows.  ``sink``: one more term of score 0 without a value in
-    every softmax's denominator (it enters where a kernel normalises a finished row, after the
+    to the kernel for wide latent rows.  ``sink`` (float32, a score a query head): one more term
+    without a value in every softmax's denominator (it enters where a kernel normalises a finished row, after the
     pieces of split keys have been merged).  ``form``: a score form, whose output rows may be a
-    column slice; with it the values may have another size than the keys."""
+    column slice.  The values may have another size than the keys."""
     pages, kv_heads, page_size, head_dim = cache.k.shape
-    v_dim = cache.v.shape[3] if form is not None else head_dim
+    v_dim = cache.v.shape[3]
+    ops.check_sink(sink, heads)
     formed = ctypes.byref(form) if form is not None else _ptr(None)
     ratio = heads // kv_heads
-    if (value_dim and cache.v is cache.k and kv_heads == 1 and window == 0 and raw is None and not sink and form is None
+    if (value_dim and cache.v is cache.k and kv_heads == 1 and window == 0 and raw is None and sink is None and form is None
             and not supports_tensor_cores(q.dtype, head_dim, ratio) and latent_wide_ok(q.dtype, head_dim, value_dim)):
         ops._check(q, "q", torch.bfloat16, dense=False); ops._check(out, "out", torch.bfloat16)
         # few tokens and long contexts: every token's keys are dealt to several blocks, so that the
@@ -295,7 +296,7 @@ def paged_attention(q: torch.Tensor, q_stride: int, out: torch.Tensor, cache, gr
     common = (_ptr(cache.k), _ptr(cache.v), _ptr(group.block_tables), _c_int(group.max_blocks),
               _ptr(ctx.token_slot), _ptr(ctx.positions))
     tail = (_c_int(heads), _c_int(kv_heads), _c_int(head_dim), _c_int(page_size), _c_float(scale),
-            _c_int(window), _c_float(0.0 if sink else -math.inf), _stream())
+            _c_int(window), _ptr(sink), _stream())
     if ctx.all_decode and ratio <= 16:
         if tokens * kv_heads > COUNTER_CAPACITY:
             raise ValueError(f"a decode step of {tokens} tokens x {kv_heads} kv heads exceeds {COUNTER_CAPACITY} pairs")

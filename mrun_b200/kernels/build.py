@@ -183,7 +183,7 @@ def build_host() -> str:
         return target
 
 
-CORE_SOURCES = ("common.cu", "elementwise.cu", "layernorm.cu", "latent.cu", "routed.cu", "streams.cu", "recurrent.cu", "recurrent_walk.cu", "attention_diff.cu", "gemm_f32.cu", "gemm_skinny.cu", "gemm_tc5.cu",
+CORE_SOURCES = ("common.cu", "elementwise.cu", "layernorm.cu", "latent.cu", "routed.cu", "streams.cu", "recurrent.cu", "recurrent_walk.cu", "selective_scan.cu", "attention_diff.cu", "gemm_f32.cu", "gemm_skinny.cu", "gemm_tc5.cu",
                 "attention_generic.cu", "attention_latent.cu", "sampling.cu")
 
 
@@ -214,10 +214,13 @@ def build_attention(head_dim: int, value_dim: Optional[int] = None, scored: bool
 COMMON_HEAD_DIMS = (16, 32, 48, 64, 80, 96, 128, 144, 256)      # the head sizes the tests and the measured shapes use
 # (key size, value size) of the attentions with a score form among them
 COMMON_SCORED_DIMS = ((128, 128), (64, 64), (128, 64), (64, 128), (48, 16), (32, 80), (16, 16), (96, 48), (16, 48), (32, 16))
+# and of those whose values have another size and no score form
+COMMON_VALUE_DIMS = ((32, 16), (64, 128), (128, 64), (80, 48))
 
 
 def build_all() -> list[str]:
     """Every library the package loads for the configurations it measures and tests; other head
     sizes are built when a model with them is first run."""
     return ([build_host(), build_core()] + [build_attention(d) for d in COMMON_HEAD_DIMS]
+            + [build_attention(d, v) for d, v in COMMON_VALUE_DIMS]
             + [build_attention(d, v, scored=True) for d, v in COMMON_SCORED_DIMS])

@@ -54,24 +54,42 @@ def embed(table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor) -> torch.Te
 
 
 def add_rmsnorm(resid: torch.Tensor, delta: Optional[torch.Tensor], weight: torch.Tensor, eps: float,
-                out: torch.Tensor, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """resid (+= delta) then out = rmsnorm(resid) * weight; with ``rows`` only those rows are
-    normed and resid is left as it is."""
+                out: torch.Tensor, rows: Optional[torch.Tensor] = None, scaled=None) -> torch.Tensor:
+    """resid (+= delta, += share * extra row by row for ``scaled`` = (extra, share)) then out =
+    rmsnorm(resid) * weight; with ``rows`` only those rows are normed and resid is left as it is.
+    ``delta`` is 32-bit or of ``out``'s dtype, ``extra`` of ``out``'s, ``share`` float32 [rows of resid]."""
     _check(resid, "resid", torch.float32); _check(weight, "weight", torch.float32); _check(out, "out")
     hidden = resid.shape[-1]
     n_rows = resid.shape[0] if rows is None else rows.numel()
     if delta is not None:
-        _check(delta, "delta", out.dtype)
-        if delta.shape != resid.shape:
-            raise KernelError(f"add_rmsnorm: delta {tuple(delta.shape)} vs resid {tuple(resid.shape)}")
+        _check(delta, "delta")
+        if delta.shape != resid.shape or delta.dtype not in (torch.float32, out.dtype):
+            raise KernelError(f"add_rmsnorm: delta {tuple(delta.shape)} {delta.dtype} vs resid {tuple(resid.shape)}, out {out.dtype}")
+    extra = share = None
+    if scaled is not None:
+        extra, share = scaled
+        _check(extra, "extra", out.dtype); _check(share, "share", torch.float32)
+        if extra.shape != resid.shape or share.numel() != resid.shape[0]:
+            raise KernelError(f"add_rmsnorm: extra {tuple(extra.shape)}, share {tuple(share.shape)} vs resid {tuple(resid.shape)}")
     if rows is not None:
         _check(rows, "rows", torch.int32)
     if weight.numel() != hidden or out.shape != (n_rows, hidden):
         raise KernelError(f"add_rmsnorm: weight {tuple(weight.shape)}, out {tuple(out.shape)}, "
                           f"expected hidden {hidden}, rows {n_rows}")
-    _lib.core().call("mrun_add_rmsnorm", _ptr(resid), _ptr(delta), _ptr(weight), _c_float(eps), _ptr(out),
-                     dtype_code(out.dtype), _ptr(rows), _c_int(n_rows), _c_int(hidden), _stream())
+    _lib.core().call("mrun_add_rmsnorm", _ptr(resid), _ptr(delta), dtype_code(delta.dtype if delta is not None else out.dtype),
+                     _ptr(weight), _c_float(eps), _ptr(out), dtype_code(out.dtype), _ptr(rows), _c_int(n_rows), _c_int(hidden),
+                     _ptr(extra), _ptr(share), _stream())
     return out
+
+
+def add_scaled_rows(y: torch.Tensor, x: torch.Tensor, share: torch.Tensor) -> torch.Tensor:
+    """y[t] += share[t] * x[t] in place, the sum in 32-bit; ``x`` of y's dtype, or bfloat16 with a 32-bit y."""
+    _check(y, "y"); _check(x, "x"); _check(share, "share", torch.float32)
+    if y.dim() != 2 or x.shape != y.shape or share.numel() != y.shape[0]:
+        raise KernelError(f"add_scaled_rows: y {tuple(y.shape)}, x {tuple(x.shape)}, share {tuple(share.shape)}")
+    _lib.core().call("mrun_add_scaled_rows", _ptr(y), dtype_code(y.dtype), _ptr(x), dtype_code(x.dtype), _ptr(share),
+                     _c_int(y.shape[0]), _c_int(y.shape[1]), _stream())
+    return y
 
 
 def add_layernorm(resid: torch.Tensor, delta: Optional[torch.Tensor], weight: torch.Tensor, eps: float,
@@ -265,13 +283,16 @@ def proj_norm_rope_cache(x: torch.Tensor, q_off: int, k_off: int, v_off: int, he
 def head_norm_rope_cache(x: torch.Tensor, q_off: int, k_off: int, v_off: int, heads: int, kv_heads: int, dim: int,
                          vdim: int, q_weight: Optional[torch.Tensor], k_weight: Optional[torch.Tensor], eps: float,
                          rot: Optional[torch.Tensor], rotary_dim: int, pairing: str, slots: Optional[torch.Tensor],
-                         k_cache: Optional[torch.Tensor], v_cache: Optional[torch.Tensor], page_size: int) -> None:
+                         k_cache: Optional[torch.Tensor], v_cache: Optional[torch.Tensor], page_size: int,
+                         bias: Optional[torch.Tensor] = None, keep: Optional[torch.Tensor] = None, blend=None) -> None:
     """RMS norm of every q and k head over its own ``dim`` features (weights of ``dim`` entries that
     the heads share; None: no norm), rotation of the first ``rotary_dim`` features of every head,
     k and v into the pages ``slots`` names (key pages [pages, kv_heads, page, dim], value pages
     [.., vdim]).  ``x``: rows whose q, k and v heads start at columns ``q_off``, ``k_off``,
     ``v_off``; q is worked on in place.  ``v_off`` < 0: the values are the keys as projected,
-    before norm and rotation."""
+    before norm and rotation.  ``bias`` (float32, [q | k | v] features) is added first.  ``keep`` (rows of
+    kv_heads * vdim features of x's dtype, may be strided) gets the values; ``blend`` = (rows, share): the
+    values then become (1 - share) * v + share * rows."""
     ld = _strided_rows(x, "x")
     tokens = x.shape[0]
     for name, w in (("q_weight", q_weight), ("k_weight", k_weight)):
@@ -290,6 +311,16 @@ def head_norm_rope_cache(x: torch.Tensor, q_off: int, k_off: int, v_off: int, he
             if c.dim() != 4 or c.shape[1:] != (kv_heads, page_size, n):
                 raise KernelError(f"head_norm_rope_cache: {name} is {tuple(c.shape)}, expected "
                                   f"[pages, {kv_heads}, {page_size}, {n}]")
+    if bias is not None:
+        _check(bias, "bias", torch.float32)
+        if bias.numel() != (heads + kv_heads) * dim + (kv_heads * vdim if v_off >= 0 else 0):
+            raise KernelError(f"head_norm_rope_cache: bias has {bias.numel()} entries")
+    first, share = blend if blend is not None else (None, 0.0)
+    strides = []
+    for name, t in (("keep", keep), ("blend", first)):
+        strides.append(_strided_rows(t, name) if t is not None else 0)
+        if t is not None and (t.shape != (tokens, kv_heads * vdim) or t.dtype != x.dtype):
+            raise KernelError(f"head_norm_rope_cache: {name} is {tuple(t.shape)} {t.dtype}, expected {(tokens, kv_heads * vdim)} {x.dtype}")
     width = x.shape[1]
     if q_off + heads * dim > width or k_off + kv_heads * dim > width or (v_off >= 0 and v_off + kv_heads * vdim > width):
         raise KernelError("head_norm_rope_cache: the heads do not fit the rows")
@@ -297,19 +328,27 @@ def head_norm_rope_cache(x: torch.Tensor, q_off: int, k_off: int, v_off: int, he
                      dtype_code(x.dtype), _ptr(q_weight), _ptr(k_weight), _c_float(eps), _ptr(rot),
                      _c_int(rotary_dim if rot is not None else 0), _c_int(PAIRINGS[pairing]), _ptr(slots), _ptr(k_cache),
                      _ptr(v_cache), _c_int(tokens), _c_int(heads), _c_int(kv_heads), _c_int(dim), _c_int(vdim),
-                     _c_int(page_size), _stream())
+                     _c_int(page_size), _ptr(bias), _ptr(first), _c_long(strides[1]), _c_float(share), _ptr(keep),
+                     _c_long(strides[0]), _stream())
+
+
+def check_sink(sink: Optional[torch.Tensor], heads: int) -> None:
+    if sink is not None:
+        _check(sink, "sink", torch.float32)
+        if sink.numel() != heads:
+            raise KernelError(f"attention: sink has {sink.numel()} scores for {heads} query heads")
 
 
 def paged_attention_generic(q: torch.Tensor, q_stride: int, out: torch.Tensor, k_cache: torch.Tensor,
                             v_cache: torch.Tensor, block_tables: torch.Tensor, token_slot: torch.Tensor,
-                            positions: torch.Tensor, heads: int, scale: float, window: int = 0, sink: bool = False,
+                            positions: torch.Tensor, heads: int, scale: float, window: int = 0, sink: Optional[torch.Tensor] = None,
                             gate: Optional[torch.Tensor] = None, form=None) -> torch.Tensor:
     """Attention of every token over its request's pages, 32-bit arithmetic on CUDA cores.
 
     ``q`` may be a view into a wider buffer: row t starts ``q_stride`` elements after row t-1.
     ``block_tables`` has one row per state slot; ``token_slot[t]`` names the row of token t.
-    The value pages may have another feature size than the key pages.  ``sink``: one more term of
-    score 0 without a value in the softmax's denominator.  ``gate``: [tokens, heads] in q's dtype
+    The value pages may have another feature size than the key pages.  ``sink`` (float32, a score a
+    query head): one more term without a value in the softmax's denominator.  ``gate``: [tokens, heads] in q's dtype
     (rows may be strided), whose sigmoid multiplies each head's output.  ``form``: a score form
     (:class:`mrun_b200.kernels.attention.ScoreForm`), whose output rows may be strided.
     """
@@ -327,6 +366,7 @@ def paged_attention_generic(q: torch.Tensor, q_stride: int, out: torch.Tensor, k
                           f"do not match {tokens} tokens of {heads}x{value_dim}")
     if block_tables.dim() != 2:
         raise KernelError("paged_attention: block_tables must be [slots, max_blocks]")
+    check_sink(sink, heads)
     gate_stride = 0
     if gate is not None:
         gate_stride = _strided_rows(gate, "gate")
@@ -336,7 +376,7 @@ def paged_attention_generic(q: torch.Tensor, q_stride: int, out: torch.Tensor, k
                      _ptr(v_cache), dtype_code(q.dtype), _ptr(block_tables), _c_int(block_tables.shape[1]),
                      _ptr(token_slot), _ptr(positions), _c_int(tokens), _c_int(heads), _c_int(kv_heads),
                      _c_int(head_dim), _c_int(value_dim), _c_int(page_size), _c_long(pages * kv_heads * page_size),
-                     _c_float(scale), _c_int(window), _c_int(1 if sink else 0), _ptr(gate), _c_long(gate_stride),
+                     _c_float(scale), _c_int(window), _ptr(sink), _ptr(gate), _c_long(gate_stride),
                      ctypes.byref(form) if form is not None else _ptr(None), _stream())
     return out
 
@@ -450,17 +490,19 @@ class RowSums:
 class PendingLinear:
     """A product ``x @ w.T`` that has not run yet: a part returns it as its output where the norm
     that follows can run it with the residual sum and the norm folded into its epilogue
-    (:func:`linear_into_norm`).  :meth:`compute` runs it as an ordinary product."""
+    (:func:`linear_into_norm`).  :meth:`compute` runs it as an ordinary product.  ``scaled`` = (rows,
+    share): rows of the output's shape that join it, row t times share[t] (float32)."""
 
-    def __init__(self, x: torch.Tensor, w: torch.Tensor):
-        self.x, self.w = x, w
+    def __init__(self, x: torch.Tensor, w: torch.Tensor, scaled=None):
+        self.x, self.w, self.scaled = x, w, scaled
 
     @property
     def shape(self):
         return (self.x.shape[0], self.w.shape[0])
 
-    def compute(self) -> torch.Tensor:
-        return linear(self.x, self.w)
+    def compute(self, out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
+        y = linear(self.x, self.w, out_dtype=out_dtype)
+        return y if self.scaled is None else add_scaled_rows(y, *self.scaled)
 
 
 class PendingPostNorm:
@@ -546,7 +588,8 @@ def gemm_skinny(x, w: torch.Tensor, out_dtype: torch.dtype = torch.bfloat16,
     _lib.core().call("mrun_gemm_skinny", _ptr(x), _ptr(w), _ptr(out), dtype_code(out_dtype),
                      _c_int(gate_code(activation) if swiglu_rows else 0), _c_int(m), _c_int(n), _c_int(k),
                      _c_long(x.stride(0) if m > 1 else max(k, x.stride(0))), _c_long(out.shape[1]),
-                     sums, eps, _ptr(None), _ptr(None), _ptr(None), _ptr(None), _c_int(rows), _stream())
+                     sums, eps, _ptr(None), _ptr(None), _ptr(None), _ptr(None), _c_int(rows), _ptr(None), _c_long(0), _ptr(None),
+                     _stream())
     return out
 
 
@@ -572,13 +615,22 @@ def linear_into_norm(pending: PendingLinear, resid: torch.Tensor, weight: torch.
     if w.shape[1] != k or resid.shape != (m, n) or weight.numel() != n:
         raise KernelError(f"linear_into_norm: x {tuple(x.shape)}, w {tuple(w.shape)}, resid {tuple(resid.shape)}, "
                           f"weight {tuple(weight.shape)}")
+    extra = share = None
+    ld_extra = 0
+    if pending.scaled is not None:
+        extra, share = pending.scaled
+        ld_extra = _strided_rows(extra, "extra"); _check(share, "share", torch.float32)
+        if extra.shape != (m, n) or extra.dtype != torch.bfloat16 or share.numel() != m:
+            raise KernelError(f"linear_into_norm: extra {tuple(extra.shape)} {extra.dtype}, share {tuple(share.shape)}")
+        if not skinny:          # the tcgen05 product's epilogue has no such rows
+            add_scaled_rows(resid, extra.contiguous(), share)
     xw = torch.empty((m, n), dtype=torch.bfloat16, device=x.device)
     out_sums = RowSums.take(x.device, m)
     head = (_ptr(x), _ptr(w), _ptr(None), dtype_code(torch.bfloat16), _c_int(0), _c_int(m), _c_int(n), _c_int(k),
             _c_long(x.stride(0) if m > 1 else max(k, x.stride(0))), _c_long(n), in_sums, in_eps, _ptr(resid),
             _ptr(weight), _ptr(xw), _ptr(out_sums))
     if skinny:
-        _lib.core().call("mrun_gemm_skinny", *head, _c_int(rows), _stream())
+        _lib.core().call("mrun_gemm_skinny", *head, _c_int(rows), _ptr(extra), _c_long(ld_extra), _ptr(share), _stream())
     else:
         _lib.core().call("mrun_gemm_tc5", *head, _c_int(0), _ptr(_tc5_status(x.device)), _stream())
     return NormedRows(xw, out_sums, eps)
@@ -719,47 +771,90 @@ def plain_act(x: torch.Tensor, activation: str, out_dtype: Optional[torch.dtype]
     return out
 
 
-def linear_act(x: torch.Tensor, w: torch.Tensor, activation: str) -> torch.Tensor:
+def linear_act(x, w: torch.Tensor, activation: str) -> torch.Tensor:
     """act(x @ w.T) in x's dtype; up to 16 bfloat16 rows the activation rides in the decode GEMM's
-    epilogue (which sees the sums as they would have been stored)."""
+    epilogue (which sees the sums as they would have been stored).  ``x`` may be :class:`NormedRows`."""
     if skinny_ok(x, w):
-        return linears_batched(x.unsqueeze(1), w.unsqueeze(0), activation=activation)[:, 0]
+        return linear_blended(x, w, activation=activation)
     y = linear(x, w)
     if activation == "relu2":
         return relu2_scaled(y, None, 0, 1)
     return plain_act(y, activation)
 
 
-def linears_batched(x: torch.Tensor, w: torch.Tensor, activation: Optional[str] = None) -> torch.Tensor:
-    """y[:, b] = act(x[:, b] @ w[b].T): ``x`` [rows, batch, K] (may be strided along the first two
-    axes), ``w`` dense [batch, N, K]; returns dense [rows, batch, N].  One launch: up to 16
-    bfloat16 rows this library's decode GEMM, else as :func:`linear_per_head` (without an activation)."""
+def linears_batched(x: torch.Tensor, w: torch.Tensor, activation: Optional[str] = None, gate: Optional[torch.Tensor] = None,
+                    out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """y[:, b] = act(x[:, b] @ w[b].T * sigmoid(gate[:, b])): ``x`` [rows, batch, K] and ``out`` [rows, batch, N]
+    (may be strided along the first two axes; None: a dense one is made), ``w`` dense [batch, N, K], ``gate``
+    [rows, batch] in x's dtype (rows may be strided) or None.  One launch up to 16 bfloat16 rows (this
+    library's decode GEMM), else as :func:`linear_per_head` and :func:`head_gate` (without an activation)."""
     rows, batch, k = x.shape
     n = w.shape[1]
-    out = torch.empty((rows, batch, n), dtype=x.dtype, device=x.device)
+    if out is None:
+        out = torch.empty((rows, batch, n), dtype=x.dtype, device=x.device)
     if not (x.dtype == torch.bfloat16 and rows <= SKINNY_ROWS and k % 32 == 0 and x.stride(0) % 8 == 0
             and x.stride(1) % 8 == 0 and x.data_ptr() % 16 == 0):
         if activation is not None:
             raise KernelError("linears_batched: an activation comes with the decode GEMM only")
-        return linear_per_head(x, w, out)
-    _check(x, "x", torch.bfloat16, dense=False); _check(w, "w", torch.bfloat16)
-    if w.shape != (batch, n, k) or x.stride(2) != 1:
-        raise KernelError(f"linears_batched: x {tuple(x.shape)} (strides {x.stride()}) vs w {tuple(w.shape)}")
+        linear_per_head(x, w, out)
+        if gate is not None:
+            head_gate(out.view(rows, batch * n), gate, batch)
+        return out
+    _check(x, "x", torch.bfloat16, dense=False); _check(w, "w", torch.bfloat16); _check(out, "out", torch.bfloat16, dense=False)
+    if w.shape != (batch, n, k) or x.stride(2) != 1 or out.shape != (rows, batch, n) or out.stride(2) != 1:
+        raise KernelError(f"linears_batched: x {tuple(x.shape)} (strides {x.stride()}) vs w {tuple(w.shape)}, out {tuple(out.shape)}")
+    ld_gate = 0
+    if gate is not None:
+        ld_gate = _strided_rows(gate, "gate")
+        if gate.shape != (rows, batch) or gate.dtype != x.dtype:
+            raise KernelError(f"linears_batched: gate {tuple(gate.shape)} {gate.dtype}")
     _lib.core().call("mrun_gemm_skinny_batched", _ptr(x), _ptr(w), _ptr(out), dtype_code(out.dtype),
                      _c_int(ACTIVATIONS[activation] if activation else 0), _c_int(batch), _c_int(rows), _c_int(n), _c_int(k),
-                     _c_long(x.stride(0) if rows > 1 else max(k, x.stride(0))), _c_long(batch * n),
-                     _c_long(x.stride(1) if batch > 1 else 0), _c_long(n), _stream())
+                     _c_long(x.stride(0) if rows > 1 else max(k, x.stride(0))), _c_long(out.stride(0) if rows > 1 else max(n, out.stride(0))),
+                     _c_long(x.stride(1) if batch > 1 else 0), _c_long(out.stride(1) if batch > 1 else n), _ptr(None), _ptr(None), _c_long(0),
+                     _c_int(0), _c_int(0), _c_float(0.0), _ptr(gate), _c_long(ld_gate), _ptr(None), _c_float(0.0), _stream())
     return out
 
 
-def linear_or_pending(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None):
+def linear_blended(x, w: torch.Tensor, bias: Optional[torch.Tensor] = None, blend=None,
+                   activation: Optional[str] = None) -> torch.Tensor:
+    """act(x @ w.T + bias) for at most 16 bfloat16 rows (:func:`skinny_ok`), the bias (float32 [N]) added to the 32-bit
+    sums.  ``blend`` = (rows, share, column): the columns from ``column`` on, as many as ``rows`` has, then
+    become (1 - share) * y + share * rows.  ``x`` may be :class:`NormedRows`."""
+    x, sums, eps = _normed(x)
+    _check(x, "x", torch.bfloat16, dense=False); _check(w, "w", torch.bfloat16)
+    m, k = x.shape
+    n = w.shape[0]
+    if w.shape[1] != k:
+        raise KernelError(f"linear_blended: x {tuple(x.shape)} vs w {tuple(w.shape)}")
+    if bias is not None:
+        _check(bias, "bias", torch.float32)
+        if bias.numel() != n:
+            raise KernelError(f"linear_blended: bias has {bias.numel()} entries for {n} columns")
+    rows, share, column = blend if blend is not None else (None, 0.0, 0)
+    ld_rows = columns = 0
+    if rows is not None:
+        ld_rows, columns = _strided_rows(rows, "blend"), rows.shape[1]
+        if rows.shape[0] != m or rows.dtype != torch.bfloat16:
+            raise KernelError(f"linear_blended: blend {tuple(rows.shape)} {rows.dtype}")
+    out = torch.empty((m, n), dtype=torch.bfloat16, device=x.device)
+    _lib.core().call("mrun_gemm_skinny_batched", _ptr(x), _ptr(w), _ptr(out), dtype_code(out.dtype),
+                     _c_int(ACTIVATIONS[activation] if activation else 0), _c_int(1),
+                     _c_int(m), _c_int(n), _c_int(k), _c_long(x.stride(0) if m > 1 else max(k, x.stride(0))), _c_long(n), _c_long(0),
+                     _c_long(n), _ptr(bias), _ptr(rows), _c_long(ld_rows), _c_int(column), _c_int(columns), _c_float(share), _ptr(None),
+                     _c_long(0), sums, eps, _stream())
+    return out
+
+
+def linear_or_pending(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None, scaled=None):
     """The last product of a part whose caller accepts a :class:`PendingLinear`: left pending in
     bfloat16 without a bias (the norm after it then runs it with the residual sum folded in: in
     the decode GEMM's epilogue up to 16 rows, as the vendor GEMM's accumulate-into-C above),
-    computed otherwise."""
+    computed otherwise.  ``scaled`` as for :class:`PendingLinear`."""
     if bias is None and x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16:
-        return PendingLinear(x, w)
-    return linear(x, w, bias=bias)
+        return PendingLinear(x, w, scaled)
+    y = linear(x, w, bias=bias)
+    return y if scaled is None else add_scaled_rows(y, *scaled)
 
 
 def accumulate_ok(pending, resid: torch.Tensor) -> bool:
@@ -773,7 +868,8 @@ def accumulate_ok(pending, resid: torch.Tensor) -> bool:
 def linear_add_into(resid: torch.Tensor, pending: PendingLinear) -> torch.Tensor:
     """resid += pending.x @ pending.w.T in place: the vendor GEMM with bfloat16 operands, 32-bit
     accumulation and the 32-bit stream as its C and D, so that the product is never rounded to
-    bfloat16, written and read again (prompt portions and decode batches above 16 rows)."""
+    bfloat16, written and read again (prompt portions and decode batches above 16 rows).  Its scaled
+    rows are the caller's to add."""
     return torch.addmm(resid, pending.x, pending.w.t(), out_dtype=torch.float32, out=resid)
 
 
@@ -1027,7 +1123,8 @@ def scale(x: torch.Tensor, factor: float) -> torch.Tensor:
 # ------------------------------------------------------------------ a routed feed-forward's rows sorted by expert
 
 def moe_sort(chosen: torch.Tensor, weights: torch.Tensor):
-    """Sorts the (token, chosen expert) pairs by expert.  ``chosen``: int32 [tokens, top];
+    """Sorts the (token, chosen expert) pairs by expert.  ``chosen``: int32 [tokens, top], a negative entry a
+    pair without a row (its ``dest`` is -1; rows that no pair takes stand at the end, with source 0);
     ``weights``: float32 [tokens, experts].  Returns ``ends`` (int32 [experts]: where each expert's
     rows end), ``source`` (int32 [pairs]: the token of every row), ``row_weight`` (float32
     [pairs]) and ``dest`` (int32 [tokens, top]: the row of every pair)."""
@@ -1038,8 +1135,8 @@ def moe_sort(chosen: torch.Tensor, weights: torch.Tensor):
         raise KernelError(f"moe_sort: chosen {tuple(chosen.shape)} vs weights {tuple(weights.shape)}")
     dev = chosen.device
     books = torch.zeros((3, experts), dtype=torch.int32, device=dev)          # counts, ends, cursor
-    source = torch.empty(tokens * top, dtype=torch.int32, device=dev)
-    row_weight = torch.empty(tokens * top, dtype=torch.float32, device=dev)
+    source = torch.zeros(tokens * top, dtype=torch.int32, device=dev)
+    row_weight = torch.zeros(tokens * top, dtype=torch.float32, device=dev)
     dest = torch.empty((tokens, top), dtype=torch.int32, device=dev)
     _lib.core().call("mrun_moe_sort", _ptr(chosen), _ptr(weights), _c_int(tokens), _c_int(experts), _c_int(top),
                      _ptr(books[0]), _ptr(books[1]), _ptr(books[2]), _ptr(source), _ptr(row_weight), _ptr(dest), _stream())
@@ -1066,8 +1163,9 @@ def relu2_rows(u: torch.Tensor, row_weight: torch.Tensor) -> torch.Tensor:
     return act
 
 
-def combine_rows(base: Optional[torch.Tensor], rows: torch.Tensor, dest: torch.Tensor) -> torch.Tensor:
-    """float32 out[t] = base[t] + sum over k of rows[dest[t, k]], added in the order of k."""
+def combine_rows(base: Optional[torch.Tensor], rows: torch.Tensor, dest: torch.Tensor, scaled=None) -> torch.Tensor:
+    """float32 out[t] = base[t] (+ share[t] * extra[t] for ``scaled`` = (extra, share)) + sum over k of
+    rows[dest[t, k]], added in the order of k; a negative dest has no row."""
     _check(rows, "rows", torch.bfloat16); _check(dest, "dest", torch.int32)
     tokens, top = dest.shape
     width = rows.shape[1]
@@ -1075,10 +1173,16 @@ def combine_rows(base: Optional[torch.Tensor], rows: torch.Tensor, dest: torch.T
         _check(base, "base")
         if base.shape != (tokens, width) or base.dtype not in (torch.float32, torch.bfloat16):
             raise KernelError(f"combine_rows: base {tuple(base.shape)} {base.dtype}")
+    extra = share = None
+    if scaled is not None:
+        extra, share = scaled
+        _check(extra, "extra", rows.dtype); _check(share, "share", torch.float32)
+        if extra.shape != (tokens, width) or share.numel() != tokens:
+            raise KernelError(f"combine_rows: extra {tuple(extra.shape)}, share {tuple(share.shape)}")
     out = torch.empty((tokens, width), dtype=torch.float32, device=rows.device)
     _lib.core().call("mrun_combine_rows", _ptr(base), _c_int(1 if base is not None and base.dtype == torch.float32 else 0),
                      _ptr(rows), dtype_code(rows.dtype), _ptr(dest), _ptr(out), _c_int(tokens), _c_int(top),
-                     _c_int(width), _stream())
+                     _c_int(width), _ptr(extra), _ptr(share), _stream())
     return out
 
 
@@ -1408,6 +1512,30 @@ def ssm_scan(c: torch.Tensor, b: torch.Tensor, x: torch.Tensor, dt: torch.Tensor
     return out
 
 
+def selective_scan(x: torch.Tensor, z: torch.Tensor, dt: torch.Tensor, dt_bias: torch.Tensor, a: torch.Tensor, b: torch.Tensor,
+                   c: torch.Tensor, skip: torch.Tensor, state: torch.Tensor, ctx) -> torch.Tensor:
+    """A state-space recurrence with a decay per channel and state over each request's tokens: step =
+    softplus(dt + dt_bias); S <- exp(step * a) * S + step * x * b; y = (S . c + skip * x) * SiLU(z), from and into
+    ``state`` (float32 [slots, inner, states]).  ``x``, ``z``: [tokens, inner]; ``b``, ``c``: [tokens, states] column
+    slices of one matrix; ``dt``: float32 [tokens, inner]; rows may be strided; ``a``: float32 [inner,
+    states] (negative rates).  Returns dense rows of x's dtype."""
+    ldx, ldz, ldb, lddt = _strided_rows(x, "x"), _strided_rows(z, "z"), _strided_rows(b, "b"), _strided_rows(dt, "dt")
+    for name, t in (("dt_bias", dt_bias), ("a", a), ("skip", skip), ("state", state)):
+        _check(t, name, torch.float32)
+    tokens, inner = x.shape
+    states = b.shape[1]
+    if z.shape != x.shape or dt.shape != x.shape or dt.dtype != torch.float32 or c.shape != b.shape or b.shape[0] != tokens \
+            or _strided_rows(c, "c") != ldb or a.shape != (inner, states) or dt_bias.numel() != inner or skip.numel() != inner \
+            or state.shape[1:] != (inner, states) or len({t.dtype for t in (x, z, b, c)}) != 1:
+        raise KernelError("selective_scan: sizes or types do not match")
+    out = torch.empty((tokens, inner), dtype=x.dtype, device=x.device)
+    _lib.core().call("mrun_selective_scan", _ptr(x), _c_long(ldx), _ptr(z), _c_long(ldz), _ptr(b), _ptr(c), _c_long(ldb),
+                     dtype_code(x.dtype), _ptr(dt), _c_long(lddt), _ptr(dt_bias), _ptr(a), _ptr(skip), _ptr(state), _ptr(out),
+                     _c_long(inner), _ptr(ctx.seg_q_start), _ptr(ctx.seg_slot), _c_int(ctx.num_segments), _c_int(ctx.max_q_len),
+                     _c_int(tokens), _c_int(inner), _c_int(states), _stream())
+    return out
+
+
 def head_gate(y: torch.Tensor, gate: torch.Tensor, heads: int) -> torch.Tensor:
     """In place: every head of ``y`` ([tokens, heads * n]) times the 32-bit sigmoid of its entry
     of ``gate`` ([tokens, heads] in the dtype of ``y``, rows may be strided)."""
@@ -1542,28 +1670,41 @@ def clamped_glu(u: torch.Tensor, weights: Optional[torch.Tensor], blocks: int, f
 
 
 def route_grouped(logits: torch.Tensor, experts: int, top: int, groups: int, keep: int, group_top: int, scale: float,
-                  chosen: Optional[torch.Tensor] = None):
-    """The choice of a router with sigmoid scores over groups of experts.  ``logits``: float32
-    [tokens, experts] or [tokens, experts + 1] (the last column the gate of a shared expert).
-    Returns (float32 [tokens, experts]: score / (sum of the chosen + 1e-20) * ``scale`` at the
-    chosen experts, zero elsewhere; float32 [tokens]: the sigmoid of the last column, or None).
-    The experts form ``groups`` equal groups of neighbours, a group's score is the sum of its
-    ``group_top`` largest scores, and only experts of the ``keep`` best groups can be chosen.
-    ``logits`` may be the first columns of wider rows (a product padded to a vendor-friendly
-    width): its row stride is passed on."""
+                  chosen: Optional[torch.Tensor] = None, score: str = "sigmoid", correction: Optional[torch.Tensor] = None,
+                  identity: int = 0, renormalize: bool = True, handed_on=None):
+    """The choice of a router over groups of experts.  ``logits``: float32 [tokens, experts + identity] or one
+    column more (the gate of a shared expert).  Scores are the logits' sigmoids or their softmax
+    (``score``); ``correction`` (float32, one entry an expert) is added where experts are ranked, not where
+    they weigh.  The experts form ``groups`` equal groups of neighbours, a group's rank is the sum of its
+    ``group_top`` largest ranks, and only experts of the ``keep`` best groups can be chosen.
+    Returns (float32 [tokens, experts]: score * ``scale``, divided by the sum of the chosen + 1e-20 with
+    ``renormalize``, at the chosen experts and zero elsewhere; float32 [tokens]: the sigmoid of the last
+    column, or None; float32 [tokens]: the sum of the weights of the chosen among the last ``identity``
+    experts, or None; for ``handed_on`` = :class:`NormedRows`, the rows those experts hand on, it contains
+    their norm's factor).  In ``chosen`` an identity expert is -1.  ``logits`` may be the first columns of wider
+    rows (a product padded to a vendor-friendly width): its row stride is passed on."""
     _check(logits, "logits", torch.float32, dense=False)
     tokens, columns = logits.shape
-    if columns not in (experts, experts + 1):
-        raise KernelError(f"route_grouped: logits is {tuple(logits.shape)}, expected {experts} or {experts + 1} columns")
+    total = experts + identity
+    if columns not in (total, total + 1):
+        raise KernelError(f"route_grouped: logits is {tuple(logits.shape)}, expected {total} or {total + 1} columns")
     if logits.stride(1) != 1 or logits.stride(0) < columns:
         raise KernelError(f"route_grouped: logits has strides {logits.stride()}, expected rows of unit stride")
+    if correction is not None:
+        _check(correction, "correction", torch.float32)
+        if correction.numel() != total:
+            raise KernelError(f"route_grouped: correction has {correction.numel()} entries for {total} experts")
     weights = torch.empty((tokens, experts), dtype=torch.float32, device=logits.device)
-    shared = torch.empty(tokens, dtype=torch.float32, device=logits.device) if columns > experts else None
+    shared = torch.empty(tokens, dtype=torch.float32, device=logits.device) if columns > total else None
+    unchanged = torch.empty(tokens, dtype=torch.float32, device=logits.device) if identity else None
     if chosen is not None:
         _check(chosen, "chosen", torch.int32)
         if chosen.shape != (tokens, top):
             raise KernelError(f"route_grouped: chosen is {tuple(chosen.shape)}, expected {(tokens, top)}")
-    _lib.core().call("mrun_route_grouped", _ptr(logits), _c_long(logits.stride(0)), _ptr(weights), _ptr(shared), _ptr(chosen),
-                     _c_int(tokens), _c_int(experts), _c_int(top), _c_int(groups), _c_int(keep), _c_int(group_top),
-                     _c_float(scale), _stream())
-    return weights, shared
+    _lib.core().call("mrun_route_grouped", _ptr(logits), _c_long(logits.stride(0)), _c_int(ROUTER_SCORES[score]), _ptr(correction),
+                     _ptr(weights), _ptr(unchanged), _ptr(shared), _ptr(chosen), _c_int(tokens), _c_int(experts),
+                     _c_int(identity), _c_int(top), _c_int(groups), _c_int(keep), _c_int(group_top),
+                     _c_int(1 if renormalize else 0), _c_float(scale),
+                     *((_ptr(handed_on.sums), _c_int(handed_on.shape[1]), _c_float(handed_on.eps)) if handed_on is not None
+                       else (_ptr(None), _c_int(0), _c_float(0.0))), _stream())
+    return weights, shared, unchanged

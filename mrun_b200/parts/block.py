@@ -126,7 +126,7 @@ class SandwichBlock:
     def _branch(self, y, post_norm) -> "ops.PendingPostNorm":
         """The branch output as 32-bit rows, with the post-norm that it still has to pass."""
         if isinstance(y, ops.PendingLinear):
-            y = ops.linear(y.x, y.w, out_dtype=torch.float32)
+            y = y.compute(torch.float32)
         elif isinstance(y, ops.PENDING):
             y = y.compute()
         if y.dtype != torch.float32:
@@ -196,7 +196,7 @@ class PostNormBlock:
     def _branch(y, norm) -> "ops.PendingPostLayerNorm":
         """The branch output as 32-bit rows, with the norm that it still has to pass."""
         if isinstance(y, ops.PendingLinear):
-            y = ops.linear(y.x, y.w, out_dtype=torch.float32)
+            y = y.compute(torch.float32)
         elif isinstance(y, ops.PENDING):
             y = y.compute()
         return ops.PendingPostLayerNorm(y if y.dtype == torch.float32 else y.to(torch.float32), norm.weight, norm.bias, norm.eps)
@@ -293,7 +293,7 @@ class StreamsBlock:
     def _rows(y) -> torch.Tensor:
         """A sublayer's output as 32-bit rows (its last product writes them where it was left unrun)."""
         if isinstance(y, ops.PendingLinear):
-            return ops.linear(y.x, y.w, out_dtype=torch.float32)
+            return y.compute(torch.float32)
         if isinstance(y, ops.PENDING):
             y = y.compute()
         return y if y.dtype == torch.float32 else y.to(torch.float32)

@@ -85,6 +85,7 @@ class DenseMLP:
     """Feed-forward without a gate: ``down(act(up(x)))``.  Up to 16 bfloat16 rows the activation rides in
     the first product's epilogue."""
 
+    accepts_normed_rows = True
     can_defer_output = True
 
     @staticmethod

@@ -1,8 +1,8 @@
 """Grouped-query attention with keys and values of different sizes, a norm of q and k (over the
 whole projection, or head by head, with or without a weight), a sink term in the softmax, scores
 with a query temperature, a soft cap and a learned bias over distances, an output gate per head or
-per feature, values that may be the unnormed keys, and a causal, sliding-window or chunked mask (the
-formulas are with :class:`GatedAttentionSpec`).
+per feature, values that may be the unnormed keys or a blend with an earlier layer's, projection
+biases, and a causal, sliding-window or chunked mask (the formulas are with :class:`GatedAttentionSpec`).
 
 One product makes [q | k | v | gate] (or [q | gate] for a layer that reads another layer's pages,
 [q | k] for one whose values are its keys); ``ops.proj_norm_rope_cache`` or
@@ -10,7 +10,9 @@ One product makes [q | k | v | gate] (or [q | gate] for a layer that reads anoth
 attention kernel applies the sink and the gate's sigmoid to every head's output; the output
 projection follows.  In a step of single tokens the tensor-core decode kernels take the rows of
 a layer with a norm per head raw and do the norm, the rotation and the page write themselves, as
-they do for :class:`Attention`.  Scores, softmax, the sink and the gate are 32-bit in both
+they do for :class:`Attention`.  Biases and blended values enter in ``ops.head_norm_rope_cache`` or, where a
+decode step has a handful of rows, in the product's epilogue; the first layer's values of a step travel
+to the later ones through ``ctx.shared`` (a token's values are always of the same step).  Scores, softmax, the sink and the gate are 32-bit in both
 precisions.  A chunked mask reaches the attention kernels as a negative window (minus the chunk's size).
 
 A layer with a temperature, a soft cap, a distance bias or a gate per feature hands the attention
@@ -18,9 +20,9 @@ kernels a score form (``kernels.attention.score_form``): all of it happens insid
 table over distances that is laid out once from the checkpoint's buckets.  Those kernels also
 take keys and values of different sizes.
 
-Kernels: bfloat16 with keys and values of one size that the tensor-core attention takes go
-through the framework's paged kernels (tcgen05 prompt tiles, TMA decode; the sink enters their
-final normalisation, the gate is one more kernel); every other shape, and the 32-bit path, runs
+Kernels: bfloat16 with key and value sizes that the tensor-core attention takes go through the
+framework's paged kernels (tcgen05 prompt tiles, TMA decode; the sink enters their final
+normalisation, the gate is one more kernel); every other shape, and the 32-bit path, runs
 on CUDA cores in 32-bit arithmetic with sink and gate inside the kernel.
 """
 from __future__ import annotations
@@ -58,8 +60,14 @@ def distance_buckets(rows: int, reach: float) -> list[int]:
             return out
 
 
+def half_split_order(dim: int, rotary_dim: int) -> list[int]:
+    """The features of a head with its rotating pairs (2i, 2i + 1) moved to (i, i + rotary_dim / 2)."""
+    return list(range(0, rotary_dim, 2)) + list(range(1, rotary_dim, 2)) + list(range(rotary_dim, dim))
+
+
 @register_mixer("gated_attention")
 class GatedAttention:
+    accepts_normed_rows = True      # its first product takes ``ops.NormedRows`` as x
     can_defer_output = True
 
     @staticmethod
@@ -82,6 +90,12 @@ class GatedAttention:
             out.append(TensorSpec(f"{prefix}.g", (spec.heads * spec.vdim, spec.hidden)))
         if spec.distance_bias is not None:
             out.append(TensorSpec(f"{prefix}.rel", (spec.distance_bias[0], spec.heads), "normal"))
+        if spec.biases:
+            out += [TensorSpec(f"{prefix}.{name}.b", (n,)) for name, n in (("q", nq), ("k", nk), ("v", nv))]
+        if spec.learned_sink:
+            out.append(TensorSpec(f"{prefix}.sink", (spec.heads,)))
+        if spec.value_mix is not None:
+            out.append(TensorSpec(f"{prefix}.vmix", (), "share"))
         return out
 
     def __init__(self, spec: GatedAttentionSpec, tensors, runtime: Runtime):
@@ -105,15 +119,34 @@ class GatedAttention:
             raise ValueError("an attention has a sliding window or a chunked mask, not both")
         if (spec.window is not None and spec.window < 1) or (spec.chunk is not None and spec.chunk < 1):
             raise ValueError("a window or a chunk holds at least one position")
+        if spec.value_mix not in (None, "first", "blend"):
+            raise ValueError(f"values are the first ones of the step or a blend with them, not {spec.value_mix!r}")
+        if (spec.biases or spec.value_mix) and (spec.qk_norm == "projection" or not spec.own_kv or self.keys_as_values):
+            raise ValueError("biases and mixed values go with keys and values of their own and without a norm over the projection")
+        if spec.learned_sink and not spec.sink:
+            raise ValueError("a learned sink is a sink")
         self.spec = spec
         self.runtime = runtime
         # what the attention kernels take as their window: W, 0 for none, -C for chunks of C
         self.mask = -spec.chunk if spec.chunk is not None else (spec.window or 0)
         self.nq, self.nk, self.nv = spec.heads * spec.dim, spec.kv_heads * spec.dim, spec.kv_heads * spec.vdim
+        self.position = POSITIONS.build(spec.position, {}, runtime) if spec.position is not None else None
+        self.pairing = getattr(self.position, "pairing", "half")
+        biases = {name: tensors[f"{name}.b"] for name in "qkv"} if spec.biases else {}
+        if self.pairing == "interleaved" and spec.qk_norm == "unit" and not self.keys_as_values:
+            # the features of every q and k head in another order, pairs (2i, 2i + 1) as (i, i + n/2): scores and
+            # a norm without a weight do not notice, and the kernels with half-split pairs take the layer
+            tensors = dict(tensors)
+            order = half_split_order(spec.dim, self.position.rotary_dim)
+            for name in ("q", "k") if spec.own_kv else ("q",):
+                tensors[name] = tensors[name].view(-1, spec.dim, spec.hidden)[:, order].reshape(tensors[name].shape)
+                if spec.biases:
+                    biases[name] = biases[name].view(-1, spec.dim)[:, order].reshape(-1)
+            self.pairing = "half"
         parts = [tensors["q"]] + ([tensors["k"]] + ([] if self.keys_as_values else [tensors["v"]]) if spec.own_kv else [])
         self.k_off, self.v_off = (self.nq, -1 if self.keys_as_values else self.nq + self.nk) if spec.own_kv else (-1, -1)
         # the kernel that norms head by head also serves the layers that norm nothing special
-        self.per_head = spec.qk_norm in ("head", "unit") or self.keys_as_values
+        self.per_head = spec.qk_norm in ("head", "unit") or self.keys_as_values or spec.biases or spec.value_mix is not None
         self.gate_off = sum(p.shape[0] for p in parts)
         if spec.head_gate or spec.element_gate:
             parts.append(tensors["g"])
@@ -121,6 +154,16 @@ class GatedAttention:
         if rows % 8:        # rows of the product's output start on 16 bytes, as the tensor-core kernels read q
             parts.append(torch.zeros((8 - rows % 8, spec.hidden), dtype=parts[0].dtype, device=parts[0].device))
         self.w_in = runtime.matrix(torch.cat(parts, dim=0))
+        self.b_in = self.b_rows = None          # biases of q, k and v; the same as long as the product's rows
+        if spec.biases:
+            b = torch.cat([biases[name].to(torch.float32) for name in "qkv"])
+            self.b_in = runtime.vector_f32(b)
+            self.b_rows = runtime.vector_f32(torch.cat([b, b.new_zeros(self.w_in.shape[0] - b.numel())]))
+        self.v_share = float(tensors["vmix"]) if spec.value_mix == "blend" else 0.0
+        self.sink = None
+        if spec.sink:
+            self.sink = (runtime.vector_f32(tensors["sink"]) if spec.learned_sink
+                         else torch.zeros(spec.heads, dtype=torch.float32, device=runtime.device))
         self.w_o = runtime.matrix(tensors["o"])
         self.q_weight = self.k_weight = None
         if spec.qk_norm == "unit":          # a norm without a weight: a weight of ones
@@ -128,8 +171,6 @@ class GatedAttention:
         elif spec.qk_norm is not None:
             self.q_weight = runtime.vector_f32(tensors["q.norm"])
             self.k_weight = runtime.vector_f32(tensors["k.norm"]) if spec.own_kv else None
-        self.position = POSITIONS.build(spec.position, {}, runtime) if spec.position is not None else None
-        self.pairing = getattr(self.position, "pairing", "half")
         ratio = spec.heads // spec.kv_heads
         # scores or outputs that the attention kernels work on themselves
         self.formed = (spec.temperature is not None or spec.soft_cap is not None or spec.distance_bias is not None
@@ -140,8 +181,7 @@ class GatedAttention:
             self.bias = runtime.vector_f32(tensors["rel"].to("cpu", torch.float32)[at].t())      # [heads, distances]
         # unit vectors times the root of their size: no product of two exceeds the size
         self.dot_bound = float(spec.dim) if spec.qk_norm == "unit" else math.inf
-        self.tensor_cores = (TENSOR_CORES and (self.formed or spec.dim == spec.vdim)
-                             and supports_tensor_cores(runtime.precision.act, spec.dim, ratio, spec.vdim))
+        self.tensor_cores = (TENSOR_CORES and supports_tensor_cores(runtime.precision.act, spec.dim, ratio, spec.vdim))
         # the tiled kernel that very wide groups fall to needs a tile list made on the host
         self.graph_safe = not (self.tensor_cores and ratio > 16)
         # rows laid out [q | k | v] with a norm per head and half-split pairs are what the decode
@@ -159,7 +199,8 @@ class GatedAttention:
 
     def activation_elements(self) -> int:
         s = self.spec
-        return 2 * self.nq + self.nk + self.nv + s.heads * (1 + 2 * s.vdim) + (s.heads * s.vdim if s.element_gate else 0)
+        kept = self.nv if s.value_mix is not None else 0
+        return kept + 2 * self.nq + self.nk + self.nv + s.heads * (1 + 2 * s.vdim) + (s.heads * s.vdim if s.element_gate else 0)
 
     def heads_forward(self, x, ctx, cache, out, scale: float = 1.0) -> None:
         """Everything in front of the output projection: the gated heads into the rows ``out`` (which may
@@ -171,7 +212,20 @@ class GatedAttention:
         if s.own_kv != bool(cache.writable):
             raise ValueError("an attention with keys and values of its own writes its own pages, one without reads another's")
         group = ctx.group(cache.group_key)
-        y = ops.linear(x, self.w_in)
+        fuses = self.fusable and decode_fuses_input(ctx, x.dtype, s.heads, s.kv_heads, s.dim, self.runtime.page_size)
+        plain = s.value_mix is None and not s.biases
+        blend = (ctx.shared["first_values"], self.v_share) if s.value_mix == "blend" else None
+        keep = None
+        if fuses and not plain and ops.skinny_ok(x, self.w_in):
+            # a handful of single tokens: biases and blended values come out of the product itself
+            y = ops.linear_blended(x, self.w_in, self.b_rows, None if blend is None else (*blend, self.v_off))
+            if s.value_mix == "first":
+                ctx.shared["first_values"] = y[:, self.v_off:self.v_off + self.nv]
+        else:
+            fuses = fuses and plain
+            y = ops.linear(x, self.w_in)
+            if s.value_mix == "first":
+                keep = ctx.shared["first_values"] = torch.empty((x.shape[0], self.nv), dtype=x.dtype, device=x.device)
         rot = self.position.rotation(ctx) if self.position is not None else None
         rotary_dim = self.position.rotary_dim if self.position is not None else 0
         gate = y[:, self.gate_off:self.gate_off + s.heads] if s.head_gate else None
@@ -184,25 +238,26 @@ class GatedAttention:
         elif scale != 1.0 or not out.is_contiguous():
             out = torch.empty(out.shape, dtype=out.dtype, device=out.device)
         raw = None
-        if self.fusable and decode_fuses_input(ctx, x.dtype, s.heads, s.kv_heads, s.dim, self.runtime.page_size):
+        if fuses:
             # a pure decode step: the attention kernel norms, rotates and stores q, k, v itself
             raw = (self.q_weight, self.k_weight, s.eps, rot, rotary_dim, group.slot_mapping)
         elif self.per_head:
             ops.head_norm_rope_cache(y, 0, max(self.k_off, 0), self.v_off, s.heads, s.kv_heads, s.dim, s.vdim,
                                      self.q_weight, self.k_weight, s.eps, rot, rotary_dim, self.pairing,
-                                     group.slot_mapping if s.own_kv else None, cache.k, cache.v, self.runtime.page_size)
+                                     group.slot_mapping if s.own_kv else None, cache.k, cache.v, self.runtime.page_size,
+                                     bias=self.b_in, keep=keep, blend=blend)
         else:
             ops.proj_norm_rope_cache(y, 0, self.k_off, self.v_off, s.heads, s.kv_heads, s.dim, s.vdim, self.q_weight,
                                      self.k_weight, s.eps, rot, rotary_dim, self.pairing,
                                      group.slot_mapping if s.own_kv else None, cache.k, cache.v, self.runtime.page_size)
         if self.tensor_cores:
-            paged_attention(y, y.stride(0), out, cache, group, ctx, s.heads, s.softmax_scale, self.mask, raw=raw, sink=s.sink,
+            paged_attention(y, y.stride(0), out, cache, group, ctx, s.heads, s.softmax_scale, self.mask, raw=raw, sink=self.sink,
                             form=form)
             if gate is not None:
                 ops.head_gate(out, gate, s.heads)
         else:
             ops.paged_attention_generic(y, y.stride(0), out, cache.k, cache.v, group.block_tables, ctx.token_slot,
-                                        ctx.positions, s.heads, s.softmax_scale, self.mask, sink=s.sink, gate=gate, form=form)
+                                        ctx.positions, s.heads, s.softmax_scale, self.mask, sink=self.sink, gate=gate, form=form)
         if out is not wanted:
             torch.mul(out, scale, out=wanted)
 

@@ -16,7 +16,9 @@ than those kernels' 256 features (a latent of 512, say) go to a tensor-core kern
 (``csrc/attention_latent.cu``: a block a token and 16 heads, a quarter of the value columns a warp).
 
 A layer without a query latent (``q_rank`` = 0) has one query projection ``q`` straight from the
-input; it rides in the same product as the key/value down-projection.  ``window`` reaches the
+input; it rides in the same product as the key/value down-projection, and so do the rows of a gate
+per head, whose sigmoid multiplies the heads behind W_h.  A layer without positions (``rot_dim`` = 0)
+caches the latent alone.  ``window`` reaches the
 attention kernels as it does for grouped-query attention.
 
 Per step: one product for both down-projections (their weights stacked), one kernel that norms
@@ -37,6 +39,7 @@ from .base import POSITIONS, Runtime, register_mixer
 
 @register_mixer("latent_attention")
 class LatentAttention:
+    accepts_normed_rows = True      # its first product takes ``ops.NormedRows`` as x
     can_defer_output = True         # ``forward(..., defer_output=True)`` may return ``ops.PendingLinear``
 
     @staticmethod
@@ -48,7 +51,8 @@ class LatentAttention:
                      TensorSpec(f"{prefix}.uq", (s.heads * (s.dim + s.rot_dim), s.q_rank))]
         else:
             query = [TensorSpec(f"{prefix}.q", (s.heads * (s.dim + s.rot_dim), s.hidden))]
-        return query + [
+        gate = [TensorSpec(f"{prefix}.g", (s.heads, s.hidden))] if s.head_gate else []
+        return query + gate + [
             TensorSpec(f"{prefix}.dkv", (s.kv_rank + s.rot_dim, s.hidden)),
             TensorSpec(f"{prefix}.dkv.norm", (s.kv_rank,), "norm"),
             TensorSpec(f"{prefix}.uk", (s.heads * s.dim, s.kv_rank)),
@@ -63,7 +67,13 @@ class LatentAttention:
             raise ValueError("a window holds at least one position")
         # the first product: [query latent | key/value latent | shared key part], or, without a
         # query latent, [queries | key/value latent | shared key part]
-        self.w_down = runtime.matrix(torch.cat([tensors["dq" if s.q_rank else "q"], tensors["dkv"]], dim=0))
+        parts = [tensors["dq" if s.q_rank else "q"], tensors["dkv"]]
+        self.gate_off = sum(p.shape[0] for p in parts)
+        if s.head_gate:         # with zero rows behind it, so that the product's rows start on 16 bytes
+            parts.append(tensors["g"])
+            rows = self.gate_off + s.heads
+            parts.append(torch.zeros((-rows % 8, s.hidden), dtype=parts[0].dtype, device=parts[0].device))
+        self.w_down = runtime.matrix(torch.cat(parts, dim=0))
         self.q_norm = runtime.vector_f32(tensors["dq.norm"]) if s.q_rank else None
         self.kv_norm = runtime.vector_f32(tensors["dkv.norm"])
         self.w_uq = runtime.matrix(tensors["uq"]) if s.q_rank else None
@@ -93,6 +103,8 @@ class LatentAttention:
         tokens = x.shape[0]
         group = ctx.group(cache.group_key)
         down = ops.linear(x, self.w_down)
+        gate = down[:, self.gate_off:self.gate_off + s.heads] if s.head_gate else None
+        down = down[:, :self.gate_off]
         rot = self.position.rotation(ctx) if self.position is not None else None
         slots = group.slot_mapping if cache.writable else None
         if s.q_rank:
@@ -106,14 +118,15 @@ class LatentAttention:
             ops.latent_prepare(down[:, nq:], None, self.kv_norm, s.eps, rot, self.rot_dims, self.pairing, slots, None,
                                cache.k, 0, s.kv_rank, s.rot_dim)
         q_att = torch.empty((tokens, s.heads, width), dtype=x.dtype, device=x.device)
-        ops.linear_per_head(q.unflatten(1, (s.heads, s.dim + s.rot_dim))[:, :, :s.dim], self.w_uk_t,
-                            q_att[:, :, :s.kv_rank])
-        ops.latent_query(q, rot, self.rot_dims, self.pairing, q_att, s.heads, s.dim, s.rot_dim, s.kv_rank)
+        ops.linears_batched(q.unflatten(1, (s.heads, s.dim + s.rot_dim))[:, :, :s.dim], self.w_uk_t,
+                            out=q_att[:, :, :s.kv_rank])
+        if width > s.kv_rank:       # a rotated part, or zeros up to the row's width
+            ops.latent_query(q, rot, self.rot_dims, self.pairing, q_att, s.heads, s.dim, s.rot_dim, s.kv_rank)
         mixed = torch.empty((tokens, s.heads * width), dtype=x.dtype, device=x.device)
         paged_attention(q_att.view(tokens, s.heads * width), s.heads * width, mixed, cache, group, ctx, s.heads,
                         s.softmax_scale, s.window or 0, value_dim=s.kv_rank)
         value = torch.empty((tokens, s.heads, s.vdim), dtype=x.dtype, device=x.device)
-        ops.linear_per_head(mixed.view(tokens, s.heads, width)[:, :, :s.kv_rank], self.w_uv, value)
+        ops.linears_batched(mixed.view(tokens, s.heads, width)[:, :, :s.kv_rank], self.w_uv, gate=gate, out=value)
         value = value.view(tokens, s.heads * s.vdim)
         if defer_output:
             return ops.linear_or_pending(value, self.w_o)

@@ -25,6 +25,7 @@ class RMSNorm:
     # comes back is ``ops.NormedRows`` (the row scale is applied by the product that reads it);
     # with more rows the vendor GEMM adds it into the 32-bit stream itself.
     accepts_pending = True
+    accepts_wide_delta = True       # ``delta`` may be 32-bit where the activations are not
 
     def __init__(self, spec: RMSNormSpec, tensors, runtime: Runtime):
         self.size, self.eps = spec.size, float(spec.eps)
@@ -45,16 +46,17 @@ class RMSNorm:
                                      self.eps, out)
         if isinstance(delta, (ops.PendingPairNorm, ops.PendingPostLayerNorm)):
             delta = delta.compute().to(self.act)        # no fused form with this norm: the addend, in the activation type
+        scaled = None
         if isinstance(delta, ops.PendingLinear):
             if ops.norm_fusable(delta, resid, self.weight):
                 return ops.linear_into_norm(delta, resid, self.weight, self.eps)
             if ops.accumulate_ok(delta, resid):
                 ops.linear_add_into(resid, delta)          # the sum rides in the vendor GEMM
-                delta = None
+                scaled, delta = delta.scaled, None         # rows that join with a factor: in the norm's pass
             else:
                 delta = delta.compute()
         out = torch.empty(resid.shape, dtype=self.act, device=resid.device)
-        return ops.add_rmsnorm(resid, delta, self.weight, self.eps, out)
+        return ops.add_rmsnorm(resid, delta, self.weight, self.eps, out, scaled=scaled)
 
     def rows_forward(self, resid: torch.Tensor, delta, rows: torch.Tensor) -> torch.Tensor:
         if isinstance(delta, ops.PendingPostNorm):
@@ -100,6 +102,8 @@ class LayerNorm:
         if isinstance(delta, ops.PendingLinear):
             if in_place and ops.accumulate_ok(delta, resid):
                 ops.linear_add_into(resid, delta)
+                if delta.scaled is not None:
+                    ops.add_scaled_rows(resid, *delta.scaled)
                 return None
             return delta.compute()
         if isinstance(delta, ops.PENDING):

@@ -80,7 +80,7 @@ class ParallelMixer:
         if defers:
             y = mixer.forward(x, ctx, cache, defer_output=True)
             if isinstance(y, ops.PendingLinear):
-                return ops.linear(y.x, y.w, out_dtype=torch.float32)
+                return y.compute(torch.float32)
         else:
             y = mixer.forward(x, ctx, cache)
         if isinstance(y, ops.PENDING):

@@ -69,12 +69,14 @@ def _register_builtin() -> None:
     from .config.fikudra import FikudraConfig
     from .config.nisotar import NisotarConfig
     from .config.katadra import KatadraConfig
+    from .config.sebevik import SebevikConfig
     register_architecture(Qwen3Config)
     register_architecture(ZasesunConfig)
     register_architecture(BalivikConfig)
     register_architecture(FikudraConfig)
     register_architecture(NisotarConfig)
     register_architecture(KatadraConfig)
+    register_architecture(SebevikConfig)
 
 
 _register_builtin()

@@ -217,7 +217,7 @@ def test_route_grouped_kernel(experts, top, groups, keep, shared):
     logits[0, :experts] -= 30.0                       # scores that all but vanish still give weights that sum to the scale
     logits[1, :experts] = 30.0                        # scores that are all 1 in 32-bit: a tie, any valid choice
     chosen = torch.empty((tokens, top), dtype=torch.int32, device=DEV)
-    weights, gate = ops.route_grouped(logits.to(DEV), experts, top, groups, keep, 2, 1.75, chosen=chosen)
+    weights, gate, _ = ops.route_grouped(logits.to(DEV), experts, top, groups, keep, 2, 1.75, chosen=chosen)
     router = {"experts": experts, "top": top, "scale": 1.75}
     if groups > 1 or keep != 1:
         router["groups"] = {"count": groups, "keep": keep}
