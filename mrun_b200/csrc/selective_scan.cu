@@ -16,7 +16,7 @@
 // read-outs are summed over the channel's lanes together: two exchanges halve the tokens a lane is in
 // charge of, so that lane l of the first four ends with token l's sum (three shuffles for four tokens).
 // The sum of a token is ((l0 + l1) + (l2 + l3)) + ... whatever its place, a step without a token has step 0
-// and leaves the state as it is (exp(0) S + 0), so a token's result has the same bits however its request was
+// and leaves the state as it is (decay 1, nothing written), so a token's result has the same bits however its request was
 // cut.  A step of single tokens has a smaller kernel with the same arithmetic.
 // grid: channel groups x segments; a segment of zero rows is padding.
 #include "common.cuh"
@@ -52,10 +52,6 @@ __device__ __forceinline__ float exp2_fast(float v) {
 }
 // What a decay's rate is multiplied by when it is loaded: the 16-bit path takes powers of two.
 template <typename TA> constexpr float RATE_UNIT = sizeof(TA) == 4 ? 1.f : 1.4426950408889634f;
-template <typename TA> __device__ __forceinline__ float decay_of(float v) {
-    if constexpr (sizeof(TA) == 4) return expf(v);
-    else return exp2_fast(v);
-}
 
 // W consecutive values as they lie in memory (W = 4: one 8- or 16-byte piece).
 template <typename TA, int W> struct Piece {
@@ -79,9 +75,13 @@ __device__ __forceinline__ float advance(float2 (&S)[NS / 2], const float2 (&rat
     float2 acc = both(0.f);
 #pragma unroll
     for (int i = 0; i < NS / 2; ++i) {
-        const float2 arg = __fmul2_rn(both(step), rate[i]);
-        const float2 decay = make_float2(decay_of<TA>(arg.x), decay_of<TA>(arg.y));
-        S[i] = __ffma2_rn(decay, S[i], __fmul2_rn(both(input), b[i]));
+        const float2 arg = __fmul2_rn(both(step), rate[i]), write = __fmul2_rn(both(input), b[i]);
+        if constexpr (sizeof(TA) == 4) {        // S + ((decay - 1) S + write): a decay next to one keeps its digits
+            const float2 loss = make_float2(expm1f(arg.x), expm1f(arg.y));
+            S[i] = __fadd2_rn(S[i], __ffma2_rn(loss, S[i], write));
+        } else {
+            S[i] = __ffma2_rn(make_float2(exp2_fast(arg.x), exp2_fast(arg.y)), S[i], write);
+        }
         acc = __ffma2_rn(S[i], c[i], acc);
     }
     return acc.x + acc.y;
