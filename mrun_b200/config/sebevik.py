@@ -75,7 +75,7 @@ class SebevikConfig:
         mixes = m.get("v_mix")
         if mixes is not None and not isinstance(mixes, bool):
             raise ConfigError(f"{mw}v_mix", f"must be true or false, got {mixes!r}")
-        if mixes and first is not None and first.kv_heads * first.vdim != kv_heads * vdim:
+        if mixes and first is not None and (first.kv_heads, first.vdim) != (kv_heads, vdim):
             raise ConfigError(f"{mw}v_mix", f"blends values of {kv_heads} x {vdim} with those of the first such layer, "
                                             f"{first.kv_heads} x {first.vdim}")
         window = None

@@ -239,7 +239,7 @@ selective_walk_kernel(const ScanArgs a) {
                     const float v = to_float(xs[i].v[k]);
                     step.x = softplus_f(ds[i].v[k] + a.dt_bias[ch]);
                     step.y = step.x * v;
-                    end = make_float2(a.skip[ch] * v, silu_f(to_float(zs[i].v[k])));
+                    end = make_float2(__fmul_rn(a.skip[ch], v), silu_f(to_float(zs[i].v[k])));
                 }
                 steps_of(s)[t * CB + c + k] = step;
                 ends_of(s)[t * CB + c + k] = end;
@@ -300,7 +300,7 @@ selective_single_kernel(const ScanArgs a) {
     store_lane<NS>(a, st, ch, l * NS, live, S);
     if (live && l == 0)
         ((TA*)a.out)[(size_t)q0 * a.ldo + ch] =
-            from_float<TA>((q + a.skip[ch] * v) * silu_f(to_float(((const TA*)a.z)[(size_t)q0 * a.ldz + ch])));
+            from_float<TA>((q + __fmul_rn(a.skip[ch], v)) * silu_f(to_float(((const TA*)a.z)[(size_t)q0 * a.ldz + ch])));
 }
 
 template <typename TA, int NS, int L>

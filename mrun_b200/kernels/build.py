@@ -215,7 +215,7 @@ COMMON_HEAD_DIMS = (16, 32, 48, 64, 80, 96, 128, 144, 256)      # the head sizes
 # (key size, value size) of the attentions with a score form among them
 COMMON_SCORED_DIMS = ((128, 128), (64, 64), (128, 64), (64, 128), (48, 16), (32, 80), (16, 16), (96, 48), (16, 48), (32, 16))
 # and of those whose values have another size and no score form
-COMMON_VALUE_DIMS = ((32, 16), (64, 128), (128, 64), (80, 48))
+COMMON_VALUE_DIMS = ((32, 16), (64, 128), (128, 64), (80, 48), (16, 48), (16, 64))
 
 
 def build_all() -> list[str]:
