@@ -3,7 +3,7 @@
 random weights and seeded synthetic token ids.
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--layers L] [--impl ours|reference]
-                    [--shape 8b|4b|32b] [--serve] [--design zasesun|balivik|fikudra|nisotar|katadra]
+                    [--shape 8b|4b|32b] [--serve] [--design zasesun|balivik|fikudra|nisotar|katadra|sebevik]
 
 A *step* is one decode step of a batch of 8 requests that each hold 1,024 tokens of context.
 ``value`` is decoded tokens per second over exactly K steps, timed on the device with CUDA events
@@ -29,6 +29,10 @@ depths, head counts and expert sizes.
 ``--design katadra`` measures the Katadra decoder (an attention with a soft cap, a distance bias and a
 gate per feature beside a time mixing, state-space mixers, dense feed-forwards, layer norms on branch
 outputs) beside the Nisotar decoder at equal widths, depths and head counts.
+``--design sebevik`` measures the Sebevik decoder (latent attention with a gate per head, attention under a
+sliding window with learned sinks and values shared between layers, selective state-space mixers, routed
+experts with identity experts and a shared expert) beside the Fikudra decoder at equal widths, depths,
+head counts and expert sizes.
 """
 from __future__ import annotations
 
@@ -540,9 +544,70 @@ def katadra_counts(cfg: dict, tokens: int):
     return flops + 2.0 * cfg["vocab"] * h, kv_bytes, state_bytes
 
 
+# Layer sizes for --design sebevik: (Sebevik sizes, the Fikudra sizes of equal width, depth, head counts and
+# expert sizes, from the table above).  Eight layers: latent attention with a dense feed-forward, attention
+# under a sliding window, a selective scan of twice the width with sixteen states a channel, then latent
+# attention, attention, two scans and attention, all but the first with a mixture of 8 experts and 4
+# identity experts in 4 groups of which 2 stay, 2 chosen, and a shared expert; keys and values of one size
+# (the tcgen05 and TMA attention kernels), all features rotated, the latent row 256 features wide.
+def _sebevik_sizes(width, heads, kv_heads, att_dim, kv_rank, window, dense_ff, experts, top, expert_ff, shared_ff, vocab):
+    lat = {"heads": heads, "dim": att_dim, "vdim": att_dim, "kv_rank": kv_rank, "scale": att_dim ** -0.5}
+    att = {"heads": heads, "kv_heads": kv_heads, "dim": att_dim, "vdim": att_dim, "scale": att_dim ** -0.5,
+           "mask": {"size": window}, "rot": {"base": 500000.0, "dims": att_dim}, "v_mix": True}
+    ssm = {"inner": 2 * width, "state": 16, "dt_rank": width // 16, "conv": 4}
+    moe = {"kind": "moe", "router": {"experts": experts, "identity": 4, "top": top, "groups": {"count": 4, "keep": 2}},
+           "expert": {"ff": expert_ff}, "shared": {"ff": shared_ff}}
+    order = "latent_attention attention mamba1 latent_attention attention mamba1 mamba1 attention".split()
+    return {"architecture": "Sebevik", "vocab": vocab, "width": width, "norm": {"eps": 1e-6},
+            "layers": [{"type": kind, "mixer": {"latent_attention": lat, "attention": att, "mamba1": ssm}[kind],
+                        "mlp": moe if i else {"kind": "dense", "ff": dense_ff}} for i, kind in enumerate(order)]}
+
+
+SEBEVIK_SIZES = {
+    "w2048": (_sebevik_sizes(2048, 16, 4, 128, 256, 512, 8192, 8, 2, 2048, 2048, 32768), FIKUDRA_SIZES["w2048"][0]),
+    "w4096": (_sebevik_sizes(4096, 32, 8, 128, 256, 512, 16384, 8, 2, 3072, 3072, 32768), FIKUDRA_SIZES["w4096"][0]),
+}
+
+
+def sebevik_counts(cfg: dict, tokens: int, context: int):
+    """(FLOPs of a prompt of ``tokens`` tokens as the design states them, bytes of cache rows a token decoded at
+    ``context`` reads divided by the context, bytes of one request's recurrent states) of a Sebevik
+    configuration over all layers: products count two FLOPs a weight and token (a routed layer as many of
+    its chosen experts as an even choice leaves beside the identity experts, and the shared one), the
+    latent attention its stated form (keys and values of every head from the latent), a scan the decay,
+    the update and the read-out of its state for every token."""
+    h, flops, kv_bytes, state_bytes = cfg["width"], 0.0, 0.0, 0
+    for layer in cfg["layers"]:
+        m, kind = layer["mixer"], layer["type"]
+        if kind == "mamba1":
+            params = m["inner"] * (3 * h + 2 * m["dt_rank"] + 2 * m["state"])
+            flops += 2.0 * tokens * 3 * m["inner"] * m["state"]
+            state_bytes += 4 * m["inner"] * m["state"]
+        elif kind == "latent_attention":
+            n, v = m["heads"] * m["dim"], m["heads"] * m["vdim"]
+            params = h * (n + v + m["kv_rank"] + m["heads"]) + m["kv_rank"] * (n + v)
+            flops += 2.0 * tokens * (tokens + 1) / 2.0 * (n + v)
+            kv_bytes += 2 * m["kv_rank"]
+        else:
+            n, v, window = m["heads"] * m["dim"], m["heads"] * m["vdim"], m["mask"]["size"]
+            params = h * (n + v + m["kv_heads"] * (m["dim"] + m["vdim"]))
+            seen = sum(min(i + 1, window) for i in range(tokens))
+            flops += 2.0 * seen * (n + v)
+            kv_bytes += 2 * m["kv_heads"] * (m["dim"] + m["vdim"]) * min(window, context) / context
+        mlp = layer["mlp"]
+        if mlp["kind"] == "dense":
+            params += 2 * h * mlp["ff"]
+        else:
+            r = mlp["router"]
+            ranked = r["experts"] + r["identity"]
+            params += h * (ranked + 1) + 3 * h * (r["top"] * r["experts"] / ranked * mlp["expert"]["ff"] + mlp["shared"]["ff"])
+        flops += 2.0 * tokens * params
+    return flops + 2.0 * cfg["vocab"] * h, kv_bytes, state_bytes
+
+
 def compare_designs(args, peaks: dict) -> int:
     """Prefill of 2,048 tokens and decode at batch 8 with 1,024-token contexts, the named design
-    beside Qwen3 (Fikudra: beside Balivik; Nisotar: beside Fikudra; Katadra: beside Nisotar) at equal sizes, each through
+    beside Qwen3 (Fikudra: beside Balivik; Nisotar and Sebevik: beside Fikudra; Katadra: beside Nisotar) at equal sizes, each through
     the same ``Executor.step`` and captured decode step."""
     import torch
     from mrun_b200 import Engine
@@ -551,20 +616,25 @@ def compare_designs(args, peaks: dict) -> int:
     from mrun_b200.config.fikudra import FikudraConfig
     from mrun_b200.config.katadra import KatadraConfig
     from mrun_b200.config.nisotar import NisotarConfig
+    from mrun_b200.config.sebevik import SebevikConfig
     from mrun_b200.engine import StepEntry
     context, batch = 1024, 8
     out = {}
     sampler = ClockSampler()
     sampler.start()
     size_sets = {"zasesun": DESIGN_SIZES, "balivik": BALIVIK_SIZES, "fikudra": FIKUDRA_SIZES,
-                 "nisotar": NISOTAR_SIZES, "katadra": KATADRA_SIZES}[args.design]
-    beside = {"fikudra": "balivik", "nisotar": "fikudra", "katadra": "nisotar"}.get(args.design, "qwen3")
+                 "nisotar": NISOTAR_SIZES, "katadra": KATADRA_SIZES, "sebevik": SEBEVIK_SIZES}[args.design]
+    beside = {"fikudra": "balivik", "nisotar": "fikudra", "katadra": "nisotar", "sebevik": "fikudra"}.get(args.design, "qwen3")
     for name in (args.sizes.split(",") if args.sizes else sorted(size_sets)):
         z_sizes, q_sizes = size_sets[name]
         row = {}
         for design in (args.design, beside):
             state_bytes = 0
-            if design == "katadra":
+            if design == "sebevik":
+                config = SebevikConfig.from_dict(z_sizes)
+                vocab, h = z_sizes["vocab"], z_sizes["width"]
+                flops, kv_bytes, state_bytes = sebevik_counts(z_sizes, PREFILL_TOKENS, context)
+            elif design == "katadra":
                 config = KatadraConfig.from_dict(z_sizes)
                 vocab, h = z_sizes["vocab"], z_sizes["width"]
                 flops, kv_bytes, state_bytes = katadra_counts(z_sizes, PREFILL_TOKENS)
@@ -573,7 +643,7 @@ def compare_designs(args, peaks: dict) -> int:
                 config = NisotarConfig.from_dict(sizes)
                 vocab, h = sizes["vocab"], sizes["width"]
                 flops, kv_bytes, state_bytes = nisotar_counts(sizes, PREFILL_TOKENS, context)
-            elif design == "fikudra" and args.design == "nisotar":
+            elif design == "fikudra" and args.design in ("nisotar", "sebevik"):
                 config = FikudraConfig.from_dict(q_sizes)
                 vocab, h = q_sizes["vocab"], q_sizes["width"]
                 flops, kv_bytes, state_bytes = fikudra_counts(q_sizes, PREFILL_TOKENS)
@@ -676,8 +746,8 @@ def main() -> int:
     parser.add_argument("--profiler-range", nargs="?", const="decode", default=None, choices=["decode", "prefill"],
                         help="bracket the timed decode steps (or the last timed prefill) with "
                              "cudaProfilerStart/Stop, for a profiler started with --profile-from-start off")
-    parser.add_argument("--design", choices=["zasesun", "balivik", "fikudra", "nisotar", "katadra"], default=None,
-                        help="instead of the default workload: the named design beside Qwen3 (fikudra: beside Balivik; nisotar: beside Fikudra; katadra: beside Nisotar) at equal sizes "
+    parser.add_argument("--design", choices=["zasesun", "balivik", "fikudra", "nisotar", "katadra", "sebevik"], default=None,
+                        help="instead of the default workload: the named design beside Qwen3 (fikudra: beside Balivik; nisotar: beside Fikudra; katadra: beside Nisotar; sebevik: beside Fikudra) at equal sizes "
                              "(prefill of 2,048 tokens, decode at batch 8)")
     parser.add_argument("--sizes", default=None, help="with --design: which of its size sets to run, comma separated")
     args = parser.parse_args()

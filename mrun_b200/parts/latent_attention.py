@@ -13,7 +13,8 @@ and W_h runs on the weighted latent.  The framework's paged attention kernels th
 this mixer unchanged (``heads`` query heads over one kv head whose K and V are the same pages);
 prefill, decode and mixed steps take the paths they take for grouped-query attention.  Rows wider
 than those kernels' 256 features (a latent of 512, say) go to a tensor-core kernel of their own
-(``csrc/attention_latent.cu``: a block a token and 16 heads, a quarter of the value columns a warp).
+(``csrc/attention_latent.cu``: a block a token and 16 heads, a quarter of the value columns a warp), and
+so do steps of single tokens with more than 16 heads (without a window).
 
 A layer without a query latent (``q_rank`` = 0) has one query projection ``q`` straight from the
 input; it rides in the same product as the key/value down-projection, and so do the rows of a gate
@@ -33,7 +34,7 @@ import torch
 from ..cache.needs import PagedLatent
 from ..config.spec import LatentAttentionSpec, TensorSpec
 from ..kernels import ops
-from ..kernels.attention import paged_attention, supports_tensor_cores
+from ..kernels.attention import latent_wide_ok, paged_attention, supports_tensor_cores
 from .base import POSITIONS, Runtime, register_mixer
 
 
@@ -88,8 +89,10 @@ class LatentAttention:
             raise ValueError(f"{self.rot_dims} rotating features do not fit the rotated part of {s.rot_dim}")
         # the cache row's width: a size the tensor-core attention kernels are built for
         self.width = -(-(s.kv_rank + s.rot_dim) // 16) * 16
-        # the tiled kernel that very wide groups fall to needs a tile list made on the host
-        self.graph_safe = not (supports_tensor_cores(runtime.precision.act, self.width, s.heads) and s.heads > 16)
+        # the tiled kernel that very wide groups fall to needs a tile list made on the host; without a
+        # window the single tokens of such groups have the kernel for wide rows
+        self.graph_safe = not (supports_tensor_cores(runtime.precision.act, self.width, s.heads) and s.heads > 16
+                               and (s.window is not None or not latent_wide_ok(runtime.precision.act, self.width, s.kv_rank)))
 
     def cache_need(self):
         return PagedLatent(self.width, self.spec.window)

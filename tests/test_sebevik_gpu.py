@@ -724,14 +724,14 @@ def test_greedy_generation_matches_plain(stiny, dtype):
 
 
 def test_captured_decode_steps_are_used():
-    """Every tiny model decodes captured, but for the one with more than sixteen heads over one latent."""
+    """Every tiny model decodes captured, the one with more than sixteen heads over one latent too."""
     from mrun_b200.parts import MIXERS
     safe = {}
     for name in STINY:
         for i, layer in enumerate(sconfig(name).to_spec().layers):
             w = {t.name[2:]: torch.zeros(t.shape) for t in MIXERS.tensor_specs(layer.mixer, "m")}
             safe[name, i] = MIXERS.build(layer.mixer, w, runtime("bfloat16")).graph_safe
-    assert [key for key, value in safe.items() if not value] == [("far", 0)]
+    assert all(safe.values())
 
 
 def test_command_line_random_then_run(tmp_path):
