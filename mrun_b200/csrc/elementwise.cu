@@ -23,11 +23,33 @@ __global__ void embed_kernel(const TW* __restrict__ table, const int* __restrict
     for (int h = threadIdx.x; h < hidden; h += blockDim.x) dst[h] = ok ? to_float(row[h]) : 0.f;
 }
 
+// Eight features a thread (a width that is a multiple of 8): a row is many threads' work, so that a step of a
+// few tokens is not one thread's chain of loads.
+template <typename TW>
+__global__ void __launch_bounds__(128)
+embed_vec_kernel(const TW* __restrict__ table, const int* __restrict__ ids, float* __restrict__ out, int hidden, int vocab) {
+    const int t = blockIdx.x, c = (blockIdx.y * 128 + threadIdx.x) * 8;
+    if (c >= hidden) return;
+    const int id = ids[t];
+    float v[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+    if (id >= 0 && id < vocab) Vec8<TW>::load(table + (size_t)id * hidden + c, v);
+    Vec8<float>::store(out + (size_t)t * hidden + c, v);
+}
+
 MRUN_API int mrun_embed(const void* table, int table_dtype, const int* ids, float* out, int tokens,
                         int hidden, int vocab, cudaStream_t stream) {
     MRUN_REQUIRE(tokens >= 0 && hidden > 0 && vocab > 0, "embed: bad sizes tokens=%d hidden=%d vocab=%d",
                  tokens, hidden, vocab);
     if (tokens == 0) return 0;
+    if (hidden % 8 == 0 && (((uintptr_t)table | (uintptr_t)out) & 15) == 0 && (table_dtype == MRUN_F32 || table_dtype == MRUN_BF16)) {
+        const dim3 grid(tokens, (hidden / 8 + 127) / 128);
+        if (table_dtype == MRUN_F32)
+            embed_vec_kernel<float><<<grid, 128, 0, stream>>>((const float*)table, ids, out, hidden, vocab);
+        else
+            embed_vec_kernel<__nv_bfloat16><<<grid, 128, 0, stream>>>((const __nv_bfloat16*)table, ids, out, hidden, vocab);
+        MRUN_CHECK_LAUNCH("embed");
+        return 0;
+    }
     if (table_dtype == MRUN_F32)
         embed_kernel<float><<<tokens, 256, 0, stream>>>((const float*)table, ids, out, hidden, vocab);
     else if (table_dtype == MRUN_BF16)

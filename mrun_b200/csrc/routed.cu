@@ -292,6 +292,82 @@ route_grouped_kernel(const float* __restrict__ logits, long ldz, int softmax, co
     }
 }
 
+// The same for at most 32 experts in all and groups ranked by their best one or two: a lane holds an expert, and
+// an expert's place in the order is the number of experts that come before it, so that no choice waits for
+// the one before.  The arithmetic of scores, sums and weights is the kernel's above.
+__global__ void __launch_bounds__(128)
+route_grouped_small_kernel(const float* __restrict__ logits, long ldz, int softmax, const float* __restrict__ correction,
+                           float* __restrict__ weights, float* __restrict__ identity_w, float* __restrict__ shared_w,
+                           int* __restrict__ chosen, int tokens, int experts, int total, int top, int groups, int keep,
+                           int group_top, int renormalize, float scale, const unsigned long long* __restrict__ in_sums,
+                           float in_inv_width, float in_eps) {
+    constexpr unsigned ALL = 0xffffffffu;
+    const int warp = threadIdx.x >> 5, e = threadIdx.x & 31;
+    const int t = blockIdx.x * 4 + warp;
+    if (t >= tokens) return;
+    const float* z = logits + (size_t)t * ldz;
+    const bool mine = e < total;
+    const float logit = mine ? z[e] : -INFINITY;
+    const float shared = shared_w ? z[total] : 0.f;
+    const unsigned long long square = in_sums ? in_sums[t] : 0ull;
+    float score;
+    if (softmax) {
+        const float largest = warp_max(logit);
+        score = mine ? expf(logit - largest) : 0.f;
+        score *= 1.f / warp_sum(score);
+    } else {
+        score = 1.f / (1.f + expf(-logit));
+    }
+    // a rank that is not a number, and the lanes without an expert, are never chosen
+    float rank = mine ? score + (correction ? correction[e] : 0.f) : -INFINITY;
+    if (!(rank > -INFINITY)) rank = -INFINITY;
+    const int size = total / groups, group = mine ? e / size : groups;
+    if (groups > 1) {
+        float first = -INFINITY, second = -INFINITY;
+        for (int i = 0; i < size; ++i) {
+            const float v = __shfl_sync(ALL, rank, min(group * size + i, 31));
+            second = fmaxf(second, fminf(first, v));
+            first = fmaxf(first, v);
+        }
+        const float best = group_top > 1 && size > 1 ? first + second : first;
+        int before = 0;
+        for (int g = 0; g < groups; ++g) {
+            const float v = __shfl_sync(ALL, best, g * size);
+            before += v > best || (v == best && g < group);
+        }
+        if (before >= keep) rank = -INFINITY;
+    }
+    int place = 0;
+    for (int i = 0; i < total; ++i) {
+        const float v = __shfl_sync(ALL, rank, i);
+        place += v > rank || (v == rank && i < e);
+    }
+    const bool taken = rank > -INFINITY && place < top;
+    float sum = 0.f, unchanged = 0.f;
+    const unsigned any = __ballot_sync(ALL, taken);
+    for (int k = 0; k < top; ++k) {
+        const unsigned who = __ballot_sync(ALL, taken && place == k);
+        const int from = who ? __ffs(who) - 1 : 0;
+        const float s = __shfl_sync(ALL, score, from);
+        if (!who) continue;
+        sum += s;
+        if (from >= experts) unchanged += s;
+    }
+    const float norm = renormalize ? scale / (sum + 1e-20f) : scale;
+    if (e < experts) weights[(size_t)t * experts + e] = taken ? score * norm : 0.f;
+    if (chosen) {
+        if (taken) chosen[(size_t)t * top + place] = e < experts ? e : -1;
+        for (int k = __popc(any) + e; k < top; k += 32) chosen[(size_t)t * top + k] = -1;
+    }
+    if (e == 0) {
+        if (shared_w) shared_w[t] = 1.f / (1.f + expf(-shared));
+        if (identity_w) {
+            const float row = in_sums ? rsqrtf(__ull2float_rn(square) * (1.f / 1073741824.f) * in_inv_width + in_eps) : 1.f;
+            identity_w[t] = unchanged * norm * row;
+        }
+    }
+}
+
 // u: row r at u + r * ldu, blocks * 2 * ff columns; act: row r at act + r * lda, blocks * ff
 // columns.  weights: per (row, block) when per_block (row r at weights + r * ldw), else one per row
 // (at weights + r * ldw), or null.
@@ -377,11 +453,18 @@ MRUN_API int mrun_route_grouped(const float* logits, long ldz, int score, const 
     MRUN_REQUIRE(ldz >= total + (shared_w ? 1 : 0), "route_grouped: the logits' row stride is below the row");
     MRUN_REQUIRE(identity == 0 || identity_w != nullptr, "route_grouped: identity experts without a place for their weight");
     if (tokens == 0) return 0;
+    const float in_inv_width = 1.f / (float)(in_width > 0 ? in_width : 1);
+    if (total <= 32 && group_top <= 2) {
+        route_grouped_small_kernel<<<(tokens + 3) / 4, 128, 0, stream>>>(logits, ldz, score == 0, correction, weights, identity_w,
+                                                                       shared_w, chosen, tokens, experts, total, top, groups, keep,
+                                                                       group_top, renormalize, scale, in_sums, in_inv_width, in_eps);
+        MRUN_CHECK_LAUNCH("route_grouped");
+        return 0;
+    }
     const size_t smem = 4 * (size_t)(total + groups) * sizeof(float);
     route_grouped_kernel<<<(tokens + 3) / 4, 128, smem, stream>>>(logits, ldz, score == 0, correction, weights, identity_w, shared_w,
                                                                 chosen, tokens, experts, total, top, groups, keep, group_top,
-                                                                renormalize, scale, in_sums, 1.f / (float)(in_width > 0 ? in_width : 1),
-                                                                in_eps);
+                                                                renormalize, scale, in_sums, in_inv_width, in_eps);
     MRUN_CHECK_LAUNCH("route_grouped");
     return 0;
 }

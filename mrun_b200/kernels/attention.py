@@ -242,6 +242,9 @@ def score_form(out: torch.Tensor, soft_cap: Optional[float] = None, temperature=
                      bias_len=0 if bias is None else bias.shape[1])
 
 
+# Rows of this many features and more decode on the kernel for wide latent rows (measured on B200 at 16 heads and
+# contexts of 1,024: 34 us a step against 40 at 192 features and 48 at 256; narrower rows lose or draw).
+LATENT_WIDE_DECODE = 192
 LATENT_WIDE_MAX_SPLITS = 32     # the most blocks one token's keys are dealt to by the kernel for wide latent rows
 
 
@@ -260,7 +263,7 @@ def paged_attention(q: torch.Tensor, q_stride: int, out: torch.Tensor, cache, gr
     ``q`` that is the projection's raw [q | k | v] rows.  ``value_dim``, for a cache whose rows
     are key and value at once (one tensor of pages, one kv head): how many of a row's first
     features the caller reads of the output; rows too wide for the per-head-size kernels, and single
-    tokens of more heads than the decode kernels take, then go to the kernel for wide latent rows.  ``sink`` (float32, a score a query head): one more term
+    tokens of wide rows or of more heads than the decode kernels take, then go to the kernel for wide latent rows.  ``sink`` (float32, a score a query head): one more term
     without a value in every softmax's denominator (it enters where a kernel normalises a finished row, after the
     pieces of split keys have been merged).  ``form``: a score form, whose output rows may be a
     column slice.  The values may have another size than the keys."""
@@ -270,7 +273,8 @@ def paged_attention(q: torch.Tensor, q_stride: int, out: torch.Tensor, cache, gr
     formed = ctypes.byref(form) if form is not None else _ptr(None)
     ratio = heads // kv_heads
     if (value_dim and cache.v is cache.k and kv_heads == 1 and window == 0 and raw is None and sink is None and form is None
-            and (not supports_tensor_cores(q.dtype, head_dim, ratio) or (ctx.all_decode and ratio > 16))
+            and (not supports_tensor_cores(q.dtype, head_dim, ratio)
+                 or (ctx.all_decode and (ratio > 16 or head_dim >= LATENT_WIDE_DECODE)))
             and latent_wide_ok(q.dtype, head_dim, value_dim)):
         ops._check(q, "q", torch.bfloat16, dense=False); ops._check(out, "out", torch.bfloat16)
         # few tokens and long contexts: every token's keys are dealt to several blocks, so that the

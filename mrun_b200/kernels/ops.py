@@ -1134,9 +1134,10 @@ def moe_sort(chosen: torch.Tensor, weights: torch.Tensor):
     if weights.shape[0] != tokens:
         raise KernelError(f"moe_sort: chosen {tuple(chosen.shape)} vs weights {tuple(weights.shape)}")
     dev = chosen.device
-    books = torch.zeros((3, experts), dtype=torch.int32, device=dev)          # counts, ends, cursor
-    source = torch.zeros(tokens * top, dtype=torch.int32, device=dev)
-    row_weight = torch.zeros(tokens * top, dtype=torch.float32, device=dev)
+    pairs = tokens * top
+    zeros = torch.zeros(3 * experts + 2 * pairs, dtype=torch.int32, device=dev)
+    books = zeros[:3 * experts].view(3, experts)                              # counts, ends, cursor
+    source, row_weight = zeros[3 * experts:3 * experts + pairs], zeros[3 * experts + pairs:].view(torch.float32)
     dest = torch.empty((tokens, top), dtype=torch.int32, device=dev)
     _lib.core().call("mrun_moe_sort", _ptr(chosen), _ptr(weights), _c_int(tokens), _c_int(experts), _c_int(top),
                      _ptr(books[0]), _ptr(books[1]), _ptr(books[2]), _ptr(source), _ptr(row_weight), _ptr(dest), _stream())
@@ -1517,7 +1518,7 @@ def selective_scan(x: torch.Tensor, z: torch.Tensor, dt: torch.Tensor, dt_bias: 
     """A state-space recurrence with a decay per channel and state over each request's tokens: step =
     softplus(dt + dt_bias); S <- exp(step * a) * S + step * x * b; y = (S . c + skip * x) * SiLU(z), from and into
     ``state`` (float32 [slots, inner, states]).  ``x``, ``z``: [tokens, inner]; ``b``, ``c``: [tokens, states] column
-    slices of one matrix; ``dt``: float32 [tokens, inner]; rows may be strided; ``a``: float32 [inner,
+    slices of one matrix, in 32-bit or, where every segment is a single token, in x's dtype; ``dt``: float32 [tokens, inner]; rows may be strided; ``a``: float32 [inner,
     states] (negative rates).  Returns dense rows of x's dtype."""
     ldx, ldz, ldb, lddt = _strided_rows(x, "x"), _strided_rows(z, "z"), _strided_rows(b, "b"), _strided_rows(dt, "dt")
     for name, t in (("dt_bias", dt_bias), ("a", a), ("skip", skip), ("state", state)):
@@ -1526,7 +1527,8 @@ def selective_scan(x: torch.Tensor, z: torch.Tensor, dt: torch.Tensor, dt_bias: 
     states = b.shape[1]
     if z.shape != x.shape or dt.shape != x.shape or dt.dtype != torch.float32 or c.shape != b.shape or b.shape[0] != tokens \
             or _strided_rows(c, "c") != ldb or a.shape != (inner, states) or dt_bias.numel() != inner or skip.numel() != inner \
-            or state.shape[1:] != (inner, states) or len({t.dtype for t in (x, z, b, c)}) != 1:
+            or state.shape[1:] != (inner, states) or z.dtype != x.dtype or c.dtype != b.dtype \
+            or b.dtype != (x.dtype if ctx.max_q_len == 1 else torch.float32):
         raise KernelError("selective_scan: sizes or types do not match")
     out = torch.empty((tokens, inner), dtype=x.dtype, device=x.device)
     _lib.core().call("mrun_selective_scan", _ptr(x), _c_long(ldx), _ptr(z), _c_long(ldz), _ptr(b), _ptr(c), _c_long(ldb),

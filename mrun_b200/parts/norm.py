@@ -65,10 +65,11 @@ class RMSNorm:
                                      self.eps, out, rows=rows)
         if isinstance(delta, (ops.PendingPairNorm, ops.PendingPostLayerNorm)):
             delta = delta.compute().to(self.act)
+        scaled = None
         if isinstance(delta, ops.PendingLinear):
-            delta = delta.compute()
+            scaled, delta = delta.scaled, ops.linear(delta.x, delta.w)
         out = torch.empty((rows.numel(), self.size), dtype=self.act, device=resid.device)
-        return ops.add_rmsnorm(resid, delta, self.weight, self.eps, out, rows=rows)
+        return ops.add_rmsnorm(resid, delta, self.weight, self.eps, out, rows=rows, scaled=scaled)
 
     def forward(self, x: torch.Tensor) -> torch.Tensor:
         return self.add_forward(x.to(torch.float32), None)

@@ -2,8 +2,8 @@
 :class:`SelectiveScanSpec`).
 
 One product makes [x | z]; ``ops.causal_conv`` runs the short convolution with its bias and SiLU over x, from and
-into the request's last inputs; one product of x makes [r | B | C], one of r the raw steps (32-bit output,
-as they enter the recurrence); ``ops.selective_scan`` forms steps and decays, walks each request's tokens
+into the request's last inputs; one product of x makes [r | B | C] (two where the step has more than single
+tokens, so that B and C come in 32-bit), one of r the raw steps (32-bit output, as they enter the recurrence); ``ops.selective_scan`` forms steps and decays, walks each request's tokens
 from the state it left (float32 [inner, state] per request) and applies the skip and the gate; the output
 projection follows.  r is padded with zero columns up to a size the decode GEMM takes.  The state and
 everything inside the recurrence are 32-bit in both precisions.
@@ -73,11 +73,14 @@ class SelectiveScan:
         xz = ops.linear(x, self.w_in)
         u = ops.causal_conv(xz[:, :s.inner], self.conv_weight, cache.states["conv"], ctx, residual=False, silu=True,
                             bias=self.conv_bias)
-        rbc = ops.linear(u, self.w_x)
-        dt = ops.linear(rbc[:, :self.rank], self.w_dt, out_dtype=torch.float32)
-        o = ops.selective_scan(u, xz[:, s.inner:2 * s.inner], dt, self.dt_bias, self.rates,
-                               rbc[:, self.rank:self.rank + s.state], rbc[:, self.rank + s.state:self.rank + 2 * s.state],
-                               self.skip, cache.states["state"], ctx)
+        if ctx.max_q_len == 1:
+            rbc = ops.linear(u, self.w_x)
+            r, bc = rbc[:, :self.rank], rbc[:, self.rank:]
+        else:
+            r, bc = ops.linear(u, self.w_x[:self.rank]), ops.linear(u, self.w_x[self.rank:], out_dtype=torch.float32)
+        dt = ops.linear(r, self.w_dt, out_dtype=torch.float32)
+        o = ops.selective_scan(u, xz[:, s.inner:2 * s.inner], dt, self.dt_bias, self.rates, bc[:, :s.state],
+                               bc[:, s.state:2 * s.state], self.skip, cache.states["state"], ctx)
         if defer_output:
             return ops.linear_or_pending(o, self.w_o)
         return ops.linear(o, self.w_o)
