@@ -9,9 +9,10 @@
 //
 // A lane holds NS states of one channel as pairs (packed 32-bit arithmetic), L lanes hold a channel.  Eight
 // warps of a block walk; eight others bring the input of the stage ahead and carry the finished rows of the
-// stage behind to memory.  Rows of x, z and dt are asked for two stages ahead and become (step, step * x)
-// and (skip * x, SiLU(z)), once an element; B and C, 32-bit rows, are copied two stages ahead into a ring of
-// three, the pairs of a lane side by side.  The roles meet at one barrier a stage.
+// stage behind to memory.  Rows of x, z and dt are asked for two stages ahead and become (step, step * x) in
+// shared memory and (skip * x, SiLU(z)) in the registers of the thread that later finishes the element; B and
+// C, 32-bit rows, are copied two stages ahead into a ring of three, the pairs of a lane side by side.  The
+// roles meet at one barrier a stage.  What bounds the walk is shared memory's bandwidth, then the exponentials.
 //
 // A walking lane's work is the exponential, one a state and token; so four tokens go side by side and their
 // read-outs are summed over the channel's lanes together: two exchanges halve the tokens a lane is in
@@ -168,8 +169,9 @@ template <int N> __device__ __forceinline__ void copies_wait() { asm volatile("c
 template <int NS, int L> constexpr int STAGE = NS * L <= 64 ? 32 : 16;          // tokens of a stage
 template <int L> constexpr int CHANNELS = WARPS * 32 / L;                        // channels of a block
 template <int NS, int L> constexpr size_t KEYED_BYTES = (size_t)STAGE<NS, L> * NS * L * 2 * sizeof(float);
-template <typename TA, int NS, int L> constexpr size_t ROW_BYTES = (size_t)STAGE<NS, L> * CHANNELS<L> * (4 * sizeof(float) + sizeof(TA));
-template <typename TA, int NS, int L> constexpr size_t SMEM = 3 * KEYED_BYTES<NS, L> + 2 * ROW_BYTES<TA, NS, L>;
+template <int L> constexpr int OUT_ROW = CHANNELS<L> + 4;      // four lanes' tokens lie in different banks
+template <int NS, int L> constexpr size_t ROW_BYTES = (size_t)STAGE<NS, L> * (2 * CHANNELS<L> + OUT_ROW<L>) * sizeof(float);
+template <int NS, int L> constexpr size_t SMEM = 3 * KEYED_BYTES<NS, L> + 2 * ROW_BYTES<NS, L>;
 
 // W: values a bringing thread moves at once (4 where sizes and addresses allow it, else 1).
 template <typename TA, int NS, int L, int W>
@@ -181,11 +183,10 @@ selective_walk_kernel(const ScanArgs a) {
     if (n_tok <= 0) return;
     const int block_ch = blockIdx.x * CB, tid = threadIdx.x;
     const int stages = (n_tok + TS - 1) / TS;
-    // a token's B and C: pair i as (b, b, c, c); then (step, step * x) and (skip * x, SiLU(z)) an element, finished rows
+    // a token's B and C: pair i as (b, b, c, c); then (step, step * x) an element; the walk's sums
     auto keyed_of = [&](int s) { return reinterpret_cast<float*>(smem_raw + (s % 3) * KEYED_BYTES<NS, L>); };
-    auto steps_of = [&](int s) { return reinterpret_cast<float2*>(smem_raw + 3 * KEYED_BYTES<NS, L> + (s & 1) * ROW_BYTES<TA, NS, L>); };
-    auto ends_of = [&](int s) { return steps_of(s) + TS * CB; };
-    auto out_of = [&](int s) { return reinterpret_cast<TA*>(ends_of(s) + TS * CB); };
+    auto steps_of = [&](int s) { return reinterpret_cast<float2*>(smem_raw + 3 * KEYED_BYTES<NS, L> + (s & 1) * ROW_BYTES<NS, L>); };
+    auto sums_of = [&](int s) { return reinterpret_cast<float*>(steps_of(s) + TS * CB); };
 
     if (tid < ROLE) {
         // ------------------------------------------------------------------------------ the walk
@@ -198,9 +199,8 @@ selective_walk_kernel(const ScanArgs a) {
         for (int s = 0; s < stages; ++s) {
             const int m = min(TS, n_tok - s * TS);
             const float2* steps = steps_of(s) + my;
-            const float2* ends = ends_of(s) + my + (l & 3) * CB;
             const float4* keyed = reinterpret_cast<const float4*>(keyed_of(s)) + l * (NS / 2);
-            TA* rows = out_of(s) + my + (l & 3) * CB;
+            float* sums = sums_of(s) + my + (l & 3) * OUT_ROW<L>;
             // four tokens at a time, the rows of the next four and their decays asked for before this four's
             // read-outs are exchanged (at the stage's end the last four again, unused)
             float2 b[4][NS / 2], c[4][NS / 2], d[4][NS / 2];
@@ -225,14 +225,13 @@ selective_walk_kernel(const ScanArgs a) {
                 float p[4];
 #pragma unroll
                 for (int j = 0; j < 4; ++j) p[j] = advance<TA, NS>(S, d[j], input[j], b[j], c[j]);
-                const float2 end = ends[t0 * CB];
                 rows_at(min(t0 + 4, TS - 4));
                 const float r0 = (odd ? p[1] : p[0]) + __shfl_xor_sync(0xffffffffu, odd ? p[0] : p[1], 1);
                 const float r1 = (odd ? p[3] : p[2]) + __shfl_xor_sync(0xffffffffu, odd ? p[2] : p[3], 1);
                 float q = (high ? r1 : r0) + __shfl_xor_sync(0xffffffffu, high ? r0 : r1, 2);
 #pragma unroll
                 for (int o = 4; o < L; o <<= 1) q += __shfl_xor_sync(0xffffffffu, q, o);
-                if (l < 4) rows[t0 * CB] = from_float<TA>((q + end.x) * end.y);
+                if (l < 4) sums[t0 * OUT_ROW<L>] = q;
             }
             stage_barrier();
         }
@@ -264,6 +263,7 @@ selective_walk_kernel(const ScanArgs a) {
     struct Rows {                                       // of one stage, as they lie in memory
         Piece<TA, W> x[ITEMS], z[ITEMS];
         Piece<float, W> dt[ITEMS];
+        float2 end[ITEMS][W];                           // (skip * x, SiLU(z)) of the stage settled last
     } even, odd;
     auto fetch = [&](int s, Rows& held) {
         if (s < stages) {
@@ -291,47 +291,47 @@ selective_walk_kernel(const ScanArgs a) {
         }
         copies_commit();                                // one group a stage, also an empty one
     };
-    auto settle = [&](int s, const Rows& held) {
+    auto settle = [&](int s, Rows& held) {
         if (s >= stages) return;
         const int left = n_tok - s * TS;
 #pragma unroll
         for (int i = 0; i < ITEMS; ++i) {
             const int t = t_first + i * ITEM_ROWS;
             if (t >= TS) continue;
-            float2 step[W], end[W];
+            float2 step[W];
             if (mine && t < left) {
 #pragma unroll
                 for (int k = 0; k < W; ++k) {
                     const float v = to_float(held.x[i].v[k]);
                     step[k].x = softplus_f<TA>(held.dt[i].v[k] + bias[k]);
                     step[k].y = step[k].x * v;
-                    end[k] = make_float2(__fmul_rn(skip[k], v), silu_f<TA>(to_float(held.z[i].v[k])));
+                    held.end[i][k] = make_float2(__fmul_rn(skip[k], v), silu_f<TA>(to_float(held.z[i].v[k])));
                 }
             } else {
 #pragma unroll
-                for (int k = 0; k < W; ++k) step[k] = end[k] = make_float2(0.f, 0.f);
+                for (int k = 0; k < W; ++k) step[k] = make_float2(0.f, 0.f);
             }
-            float2 *to = steps_of(s) + t * CB + c, *too = ends_of(s) + t * CB + c;
+            float2* to = steps_of(s) + t * CB + c;
             if constexpr (W == 4) {
 #pragma unroll
-                for (int k = 0; k < 4; k += 2) {
+                for (int k = 0; k < 4; k += 2)
                     *reinterpret_cast<float4*>(to + k) = make_float4(step[k].x, step[k].y, step[k + 1].x, step[k + 1].y);
-                    *reinterpret_cast<float4*>(too + k) = make_float4(end[k].x, end[k].y, end[k + 1].x, end[k + 1].y);
-                }
             } else {
                 to[0] = step[0];
-                too[0] = end[0];
             }
         }
     };
-    auto carry = [&](int s) {
+    auto carry = [&](int s, const Rows& held) {          // held: what stage s was settled from
         const int left = n_tok - s * TS;
 #pragma unroll
         for (int i = 0; i < ITEMS; ++i) {
             const int t = t_first + i * ITEM_ROWS;
             if (mine && t < TS && t < left) {
+                Piece<float, W> sum;
                 Piece<TA, W> row;
-                row.load(out_of(s) + t * CB + c);
+                sum.load(sums_of(s) + t * OUT_ROW<L> + c);
+#pragma unroll
+                for (int k = 0; k < W; ++k) row.v[k] = from_float<TA>((sum.v[k] + held.end[i][k].x) * held.end[i][k].y);
                 row.store(out + (size_t)(s * TS + i * ITEM_ROWS) * a.ldo);
             }
         }
@@ -343,19 +343,20 @@ selective_walk_kernel(const ScanArgs a) {
     copies_wait<1>();
     stage_barrier();
     for (int s = 0; s < stages; s += 2) {               // (the areas written here were walked before the last barrier)
-        if (s > 0) carry(s - 1);
+        if (s > 0) carry(s - 1, odd);
         fetch(s + 2, even);
         settle(s + 1, odd);
         copies_wait<1>();
         stage_barrier();
         if (s + 1 == stages) break;
-        carry(s);
+        carry(s, even);
         fetch(s + 3, odd);
         settle(s + 2, even);
         copies_wait<1>();
         stage_barrier();
     }
-    carry(stages - 1);
+    if (stages & 1) carry(stages - 1, even);
+    else carry(stages - 1, odd);
 }
 
 // A step in which every segment is a single token (or none).
@@ -400,7 +401,7 @@ int launch(const ScanArgs& a, int segments, int max_q_len, cudaStream_t stream) 
         MRUN_CHECK_LAUNCH("selective_scan");
         return 0;
     }
-    constexpr size_t smem = SMEM<TA, NS, L>, unit = 4 * sizeof(TA);
+    constexpr size_t smem = SMEM<NS, L>, unit = 4 * sizeof(TA);
     static_assert(smem <= 110 * 1024, "two blocks' stages must fit a multiprocessor's shared memory");
     const dim3 grid((a.inner + CHANNELS<L> - 1) / CHANNELS<L>, segments);
     auto on = [&](const void* p, long ld, size_t bytes) { return (uintptr_t)p % bytes == 0 && ld % 4 == 0; };
