@@ -394,6 +394,54 @@ MRUN_API int mrun_latent_query(const void* q, long ldq, int act_dtype, const flo
     return 0;
 }
 
+// ------------------------------------------------------------------------------------------
+// The latents of whole contexts, laid side by side: out[segment, j, :kv_rank] = the cached latent of the
+// segment's token j for j < seg_kv_len[segment], and zeros from there up to the next multiple of 128
+// rows (attention tiles read whole; keys that do not exist must not be patterns that are no numbers).
+// grid: rows x segments.
+// ------------------------------------------------------------------------------------------
+template <typename TA>
+__global__ void __launch_bounds__(64)
+latent_rows_kernel(const TA* __restrict__ cache, const int* __restrict__ block_tables, int max_blocks,
+                   const int* __restrict__ seg_slot, const int* __restrict__ seg_kv_len, TA* __restrict__ out, int rows,
+                   int page_size, int kv_rank, int width, int wide) {
+    const int j = blockIdx.x, seg = blockIdx.y, len = seg_kv_len[seg];
+    if (j >= ((len + 127) & ~127)) return;
+    TA* dst = out + ((size_t)seg * rows + j) * kv_rank;
+    const int page = j < len ? block_tables[(size_t)seg_slot[seg] * max_blocks + j / page_size] : -1;
+    const TA* src = cache + ((size_t)(page < 0 ? 0 : page) * page_size + j % page_size) * width;
+    if (wide) {
+        constexpr int N = 16 / sizeof(TA);
+        for (int c = threadIdx.x; c < kv_rank / N; c += 64)
+            reinterpret_cast<uint4*>(dst)[c] = page < 0 ? make_uint4(0, 0, 0, 0) : reinterpret_cast<const uint4*>(src)[c];
+    } else {
+        for (int c = threadIdx.x; c < kv_rank; c += 64) dst[c] = page < 0 ? from_float<TA>(0.f) : src[c];
+    }
+}
+
+// out: [segments, rows, kv_rank]; rows: at least every segment's length rounded up to a multiple of 128.
+MRUN_API int mrun_latent_rows(const void* cache, int act_dtype, const int* block_tables, int max_blocks, const int* seg_slot,
+                              const int* seg_kv_len, void* out, int segments, int rows, int page_size, int kv_rank, int width,
+                              cudaStream_t stream) {
+    MRUN_REQUIRE(segments >= 0 && segments <= 65535 && rows > 0 && rows % 128 == 0 && page_size > 0 && max_blocks > 0 && kv_rank > 0 &&
+                 width >= kv_rank, "latent_rows: bad sizes segments=%d rows=%d kv_rank=%d width=%d", segments, rows, kv_rank, width);
+    if (segments == 0) return 0;
+    const size_t unit = act_dtype == MRUN_F32 ? 4 : 2;
+    const int wide = kv_rank * unit % 16 == 0 && width * unit % 16 == 0 && (((uintptr_t)cache | (uintptr_t)out) & 15) == 0;
+    const dim3 grid(rows, segments);
+    if (act_dtype == MRUN_F32)
+        latent_rows_kernel<float><<<grid, 64, 0, stream>>>((const float*)cache, block_tables, max_blocks, seg_slot, seg_kv_len,
+                                                           (float*)out, rows, page_size, kv_rank, width, wide);
+    else if (act_dtype == MRUN_BF16)
+        latent_rows_kernel<__nv_bfloat16><<<grid, 64, 0, stream>>>((const __nv_bfloat16*)cache, block_tables, max_blocks, seg_slot,
+                                                                   seg_kv_len, (__nv_bfloat16*)out, rows, page_size, kv_rank, width,
+                                                                   wide);
+    else
+        return mrun_set_error("latent_rows: unknown dtype code %d", act_dtype);
+    MRUN_CHECK_LAUNCH("latent_rows");
+    return 0;
+}
+
 MRUN_API int mrun_post_norm_add(float* stream_rows, const float* branch, const float* w_post, float scale,
                                 float eps_post, const float* w_next, float eps_next, void* out, int act_dtype,
                                 const int* rows, int n_rows, int hidden, cudaStream_t stream) {

@@ -1016,6 +1016,23 @@ def latent_prepare(down: torch.Tensor, q_weight: Optional[torch.Tensor], kv_weig
                      _c_int(tokens), _c_int(q_rank), _c_int(kv_rank), _c_int(rot_dim), _c_int(width), _stream())
 
 
+def latent_rows(cache: torch.Tensor, block_tables: torch.Tensor, seg_slot: torch.Tensor, seg_kv_len: torch.Tensor, rows: int,
+                kv_rank: int) -> torch.Tensor:
+    """[segments, rows, kv_rank]: the cached latents (the first ``kv_rank`` features of ``cache``'s rows, [pages,
+    1, page_size, width]) of every segment's whole context, zeros from its length up to the next
+    multiple of 128 and nothing beyond.  ``rows``: a multiple of 128 that holds every context."""
+    _check(cache, "cache"); _check(block_tables, "block_tables", torch.int32)
+    _check(seg_slot, "seg_slot", torch.int32); _check(seg_kv_len, "seg_kv_len", torch.int32)
+    segments = seg_slot.numel()
+    if cache.dim() != 4 or cache.shape[1] != 1 or seg_kv_len.numel() != segments or cache.shape[3] < kv_rank:
+        raise KernelError(f"latent_rows: cache {tuple(cache.shape)}, {segments} segments, {seg_kv_len.numel()} lengths")
+    out = torch.empty((segments, rows, kv_rank), dtype=cache.dtype, device=cache.device)
+    _lib.core().call("mrun_latent_rows", _ptr(cache), dtype_code(cache.dtype), _ptr(block_tables), _c_int(block_tables.shape[1]),
+                     _ptr(seg_slot), _ptr(seg_kv_len), _ptr(out), _c_int(segments), _c_int(rows), _c_int(cache.shape[2]),
+                     _c_int(kv_rank), _c_int(cache.shape[3]), _stream())
+    return out
+
+
 def latent_query(q: torch.Tensor, rot: Optional[torch.Tensor], rot_dims: int, pairing: str, q_att: torch.Tensor,
                  heads: int, dim: int, rot_dim: int, kv_rank: int) -> None:
     """``q`` [tokens, heads * (dim + rot_dim)] (rows may be strided); fills ``q_att[t, h, kv_rank:]``

@@ -22,6 +22,15 @@ per head, whose sigmoid multiplies the heads behind W_h.  A layer without positi
 caches the latent alone.  ``window`` reaches the
 attention kernels as it does for grouped-query attention.
 
+**Steps with prompt portions** of a layer without positions and without a window, where the heads' plain keys
+and values are 64 or 128 features, make the keys and values after all (``_expanded``): the scores of a
+portion against its own context cost (dim + vdim) a key and head that way against 2 kv_rank, and the tcgen05
+kernel takes the shape.  The contexts' latents are gathered out of the pages, each segment's keys and
+values become one large page of scratch, and the paged kernels run over those.  Only while the contexts
+together are not much longer than the step (``EXPAND_ROWS`` times its rows), so that a long context is not
+projected up again for every portion of it; other steps, decode steps and the 32-bit path stay with the
+latent.
+
 Per step: one product for both down-projections (their weights stacked), one kernel that norms
 the two latents, rotates r and writes the cache row, the query up-projection, a per-head product
 with U_h^T, one kernel that rotates the queries' rotated parts into the query rows, attention, a
@@ -29,6 +38,7 @@ per-head product with W_h, the output projection (left pending for the norm afte
 """
 from __future__ import annotations
 
+import numpy as np
 import torch
 
 from ..cache.needs import PagedLatent
@@ -36,6 +46,17 @@ from ..config.spec import LatentAttentionSpec, TensorSpec
 from ..kernels import ops
 from ..kernels.attention import latent_wide_ok, paged_attention, supports_tensor_cores
 from .base import POSITIONS, Runtime, register_mixer
+
+
+EXPAND_ROWS = 4             # rows of scratch a step's row may bring with it where keys and values are made
+EXPAND_SEGMENTS = 8         # and the most segments (each is two products of its own)
+
+
+class _Pages:
+    """Scratch keys and values as the attention kernels take a cache: a page a segment."""
+
+    def __init__(self, k, v, table):
+        self.k, self.v, self.block_tables, self.max_blocks = k, v, table, 1
 
 
 @register_mixer("latent_attention")
@@ -70,9 +91,10 @@ class LatentAttention:
         # query latent, [queries | key/value latent | shared key part]
         parts = [tensors["dq" if s.q_rank else "q"], tensors["dkv"]]
         self.gate_off = sum(p.shape[0] for p in parts)
-        if s.head_gate:         # with zero rows behind it, so that the product's rows start on 16 bytes
+        if s.head_gate:
             parts.append(tensors["g"])
-            rows = self.gate_off + s.heads
+        if not s.q_rank:        # zero rows at the end: the queries in the product's rows start on 16 bytes
+            rows = sum(p.shape[0] for p in parts)
             parts.append(torch.zeros((-rows % 8, s.hidden), dtype=parts[0].dtype, device=parts[0].device))
         self.w_down = runtime.matrix(torch.cat(parts, dim=0))
         self.q_norm = runtime.vector_f32(tensors["dq.norm"]) if s.q_rank else None
@@ -94,12 +116,45 @@ class LatentAttention:
         self.graph_safe = not (supports_tensor_cores(runtime.precision.act, self.width, s.heads) and s.heads > 16
                                and (s.window is not None or not latent_wide_ok(runtime.precision.act, self.width, s.kv_rank)))
 
+        self.expandable = (runtime.precision.act == torch.bfloat16 and s.rot_dim == 0 and not s.q_rank and s.window is None
+                           and s.dim in (64, 128) and s.vdim in (64, 128))
+
+    def _scratch_rows(self, ctx) -> int:
+        """Rows of the scratch pages of a step whose keys and values are made, 0 for a step that keeps the latent."""
+        if not self.expandable or ctx.max_q_len == 1 or len(ctx.segments) > EXPAND_SEGMENTS:
+            return 0
+        rows = 128
+        while rows < ctx.max_kv_len:
+            rows *= 2
+        return rows if rows * len(ctx.segments) <= EXPAND_ROWS * max(128, ctx.num_tokens) else 0
+
+    def _expanded(self, q, ctx, cache, group, rows: int) -> torch.Tensor:
+        """The heads' outputs over keys and values made from the contexts' latents: [tokens, heads * vdim]."""
+        s, n = self.spec, len(ctx.segments)
+        latents = ops.latent_rows(cache.k, group.block_tables, ctx.seg_slot[:n], ctx.seg_kv_len[:n], rows, s.kv_rank)
+        k = torch.empty((n, s.heads, rows, s.dim), dtype=q.dtype, device=q.device)
+        v = torch.empty((n, s.heads, rows, s.vdim), dtype=q.dtype, device=q.device)
+        for i, seg in enumerate(ctx.segments):
+            used = -(-(seg.pos_start + seg.q_len) // 128) * 128
+            c = latents[i, :used].expand(s.heads, used, s.kv_rank)
+            torch.bmm(c, self.w_uk_t, out=k[i, :, :used])
+            torch.bmm(c, self.w_uv.transpose(1, 2), out=v[i, :, :used])
+        table = ctx.shared.get("segment_pages")
+        if table is None:           # state slot -> its segment's page
+            pages = np.full(group.block_tables.shape[0], -1, dtype=np.int32)
+            pages[[seg.slot for seg in ctx.segments]] = np.arange(n, dtype=np.int32)
+            table = ctx.shared["segment_pages"] = ctx.upload(pages).view(-1, 1)
+        scratch = _Pages(k, v, table)
+        out = torch.empty((q.shape[0], s.heads * s.vdim), dtype=q.dtype, device=q.device)
+        return paged_attention(q, q.stride(0), out, scratch, scratch, ctx, s.heads, s.softmax_scale, 0)
+
     def cache_need(self):
         return PagedLatent(self.width, self.spec.window)
 
     def activation_elements(self) -> int:
         s = self.spec
-        return s.q_rank + s.kv_rank + s.rot_dim + s.heads * (s.dim + s.rot_dim + 2 * self.width + s.vdim)
+        latent = s.q_rank + s.kv_rank + s.rot_dim + s.heads * (s.dim + s.rot_dim + 2 * self.width + s.vdim)
+        return latent + (EXPAND_ROWS * (s.kv_rank + s.heads * (s.dim + s.vdim)) if self.expandable else 0)
 
     def forward(self, x, ctx, cache, defer_output: bool = False):
         s, width = self.spec, self.width
@@ -120,6 +175,12 @@ class LatentAttention:
             q = down[:, :nq]
             ops.latent_prepare(down[:, nq:], None, self.kv_norm, s.eps, rot, self.rot_dims, self.pairing, slots, None,
                                cache.k, 0, s.kv_rank, s.rot_dim)
+        rows = self._scratch_rows(ctx)
+        if rows and cache.writable:
+            value = self._expanded(q, ctx, cache, group, rows)
+            if gate is not None:
+                ops.head_gate(value, gate, s.heads)
+            return ops.linear_or_pending(value, self.w_o) if defer_output else ops.linear(value, self.w_o)
         q_att = torch.empty((tokens, s.heads, width), dtype=x.dtype, device=x.device)
         ops.linears_batched(q.unflatten(1, (s.heads, s.dim + s.rot_dim))[:, :, :s.dim], self.w_uk_t,
                             out=q_att[:, :, :s.kv_rank])

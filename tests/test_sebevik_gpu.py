@@ -268,6 +268,46 @@ def test_latent_attention_alone(dtype, m, page):
                lambda h, _: plain.latent_attention(m, W, "m.", h, 1e-5), [part.cache_need()], rt)
 
 
+@pytest.mark.parametrize("expand", [4, 0])
+@pytest.mark.parametrize("dim, vdim, kv_rank, heads, page", [(64, 64, 80, 3, 16), (128, 128, 256, 2, 8), (128, 64, 40, 2, 4), (64, 128, 300, 5, 16)])
+def test_latent_attention_with_keys_and_values_made(dim, vdim, kv_rank, heads, page, expand, monkeypatch):
+    """Prompt portions whose keys and values are made from the contexts' latents, next to portions and single
+    tokens that stay with the latent: one request in one piece and cut, and several side by side."""
+    from mrun_b200.parts import MIXERS, latent_attention
+    monkeypatch.setattr(latent_attention, "EXPAND_ROWS", expand)
+    rt = runtime("bfloat16", page)
+    m = latent(heads, dim, vdim, kv_rank, 1.5 / dim)
+    spec = latent_spec(48, m)
+    w = random_tensors(MIXERS.tensor_specs(spec, "m"), "m", torch.Generator().manual_seed(dim + vdim), std=0.2)
+    part = MIXERS.build(spec, w, rt)
+    made = []
+    monkeypatch.setattr(part, "_expanded", lambda *a, inner=part._expanded: made.append(a[-1]) or inner(*a))
+    W = named(w, "m.")
+    total = 700
+    gen = torch.Generator().manual_seed(2)
+    x = torch.randn(total, 48, generator=gen).to(torch.bfloat16).float()
+    want = plain.latent_attention(m, W, "m.", x.double(), 1e-5)
+    for portions in ([total], [300, 400], [500, 1, 3, 2, 194], [128, 128, 127, 129, 188], [20, 40, 600, 5] + [1] * 35):
+        close(run_cut(part, rt, x, portions, pages=-(-total // page) + 2), want, "bfloat16", f"portions {portions[:6]}")
+    assert sorted(set(made)) == ([128, 256, 512, 1024] if expand else [])
+    made.clear()
+    lengths = {"a": 70, "b": 129, "c": 33, "d": 300, "e": 2}
+    rows = {r: torch.randn(n + 20, 48, generator=gen).to(torch.bfloat16).float() for r, n in lengths.items()}
+    book = Steps([part.cache_need()], rt, pages=1024 // page + 8, slots=5)
+    fed = {r: 0 for r in rows}
+    for sizes in ({"a": 60, "b": 120}, {"a": 10, "b": 9, "d": 300}, {"a": 1, "b": 1, "d": 1, "c": 33}, {"c": 7, "e": 2, "a": 9, "d": 1}):
+        def run(ctx, places):
+            h = torch.cat([rows[r][fed[r]:fed[r] + n] for r, n in sizes.items()]).to(DEV, torch.bfloat16)
+            return part.forward(h, ctx, book.caches[0]).float().cpu()
+        got, at = book.run([(r, [0] * n) for r, n in sizes.items()], run), 0
+        for r, n in sizes.items():
+            expected = plain.latent_attention(m, W, "m.", rows[r].double(), 1e-5)
+            fed[r] += n
+            close(got[at:at + n], expected[fed[r] - n:fed[r]], "bfloat16", f"{r} beside others", bound=4e-2)
+            at += n
+    assert bool(made) == bool(expand)
+
+
 def attention_spec(hidden, m, mix=None):
     from mrun_b200.config.sebevik import SebevikConfig
     from dataclasses import replace
